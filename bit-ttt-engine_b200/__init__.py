@@ -78,12 +78,12 @@ from .layers import (  # noqa: E402
 )
 
 from .model import (  # noqa: E402
-    BitLlama, BitLlamaConfig, QuantizedKVCache, attn_decode, tp_unique_id, ttt_update,
+    BitLlama, BitLlamaConfig, DeviceModel, LayeredLM, QuantizedKVCache, attn_decode, tp_unique_id, ttt_update,
 )
 from . import model  # noqa: E402,F401
 
 __all__ = [
-    "BitLlama", "BitLlamaConfig", "QuantizedKVCache", "attn_decode", "ttt_update",
+    "BitLlama", "BitLlamaConfig", "DeviceModel", "LayeredLM", "QuantizedKVCache", "attn_decode", "ttt_update",
     "lib", "lib_path", "check", "BitTTTError", "BitLinear", "PackedTensor", "Workspace",
     "act_quant", "pack_ternary", "unpack_ternary",
 ]

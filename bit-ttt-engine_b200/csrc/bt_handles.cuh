@@ -3,6 +3,7 @@
 
 #include <mutex>
 
+#include "bt_dense.cuh"
 #include "bt_model.cuh"
 
 struct bt_workspace {
@@ -36,6 +37,11 @@ struct bt_kv_cache {
     float* rope_cos = nullptr;   // device [max_seq, head_dim/2] for inv_freq_theta
     float* rope_sin = nullptr;
     int max_heads = 0;
+    // 16- or 32-bit cache (bt_kv_create_dense): rows of head_dim / v_dim values instead of the quantised ones
+    bool is_dense = false;
+    int64_t v_dim = 0;
+    bt::DenseKvView dense;
+    size_t dense_bytes(int64_t stride) const { return (size_t)batch * n_kv * max_seq * stride * (dense.f32 ? 4 : 2); }
 };
 
 namespace bt {

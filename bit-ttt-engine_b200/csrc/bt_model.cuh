@@ -32,7 +32,8 @@ cudaError_t launch_argmax(const float* logits, int batch, int vocab, int32_t* ou
 cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                  int batch, int hidden, int64_t vocab, float* logits, float* cand_val,
                                  int32_t* cand_idx, int* n_cand, int sm_count, cudaStream_t stream, bool pdl,
-                                 bool f16 = false);  // f16: w holds IEEE halves, not bf16
+                                 bool f16 = false,   // f16: w holds IEEE halves, not bf16
+                                 int ld = 0);        // row stride of w (multiple of 8, zero beyond hidden); 0: hidden
 // Reduces the candidates to the greedy pick per token and advances the positions.
 cudaError_t launch_pick(const float* cand_val, const int32_t* cand_idx, int n_cand, int batch, int32_t* out,
                         int32_t* pos, int n_pos, cudaStream_t stream, bool pdl);
@@ -41,7 +42,7 @@ int lm_head_max_candidates(int sm_count);
 // Tensor-core lm_head for batches above 8 (tcgen05, bf16 x (bf16 hi + bf16 lo), f32 accumulate).
 size_t lm_head_tc_weight_bytes(int64_t vocab, int hidden);
 size_t lm_head_tc_act_bytes(int hidden);
-cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, void* tiles, cudaStream_t stream);
+cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, void* tiles, cudaStream_t stream, int ld = 0);
 cudaError_t launch_lm_head_tc(const void* wtiles, const float* h, const float* norm_w, float eps, int batch, int hidden,
                               int64_t vocab, void* btiles, float* logits, unsigned int* err, int sm_count,
                               cudaStream_t stream, bool w_f16 = false);  // w_f16: the weight tiles hold IEEE halves

@@ -330,10 +330,10 @@ template <int B, bool F16>
 __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16* __restrict__ w,
                                                             const float* __restrict__ h,
                                                             const float* __restrict__ norm_w, float eps,
-                                                            int hidden, int64_t vocab, float* __restrict__ logits,
+                                                            int hidden, int ld, int64_t vocab, float* __restrict__ logits,
                                                             float* __restrict__ cand_val,
                                                             int32_t* __restrict__ cand_idx) {
-    extern __shared__ float xs[];  // [B][hidden]
+    extern __shared__ float xs[];  // [B][ld], zero beyond hidden
     __shared__ double red_d[32];
     __shared__ float best_v[8][B];
     __shared__ int best_i[8][B];
@@ -347,13 +347,14 @@ __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16*
         double ss = 0.0;
         for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
             const float v = h[(int64_t)b * hidden + c];
-            xs[b * hidden + c] = v;
+            xs[b * ld + c] = v;
             ss = fma((double)v, (double)v, ss);
         }
         ss = block_sum_d(ss, red_d);
         const float denom = sqrtf(__fadd_rn((float)(ss / (double)hidden), eps));
         for (int c = threadIdx.x; c < hidden; c += blockDim.x)
-            xs[b * hidden + c] = __fmul_rn(__fdiv_rn(xs[b * hidden + c], denom), norm_w[c]);
+            xs[b * ld + c] = __fmul_rn(__fdiv_rn(xs[b * ld + c], denom), norm_w[c]);
+        for (int c = hidden + threadIdx.x; c < ld; c += blockDim.x) xs[b * ld + c] = 0.0f;
     }
     __syncthreads();
     float bv[B];
@@ -361,12 +362,12 @@ __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16*
 #pragma unroll
     for (int b = 0; b < B; ++b) { bv[b] = -INFINITY; bi[b] = -1; }
     for (int64_t v = warp_global; v < vocab; v += warps_total) {
-        const uint4* wr = reinterpret_cast<const uint4*>(w + v * hidden);
+        const uint4* wr = reinterpret_cast<const uint4*>(w + v * ld);
         float acc[B];
 #pragma unroll
         for (int b = 0; b < B; ++b) acc[b] = 0.0f;
 #pragma unroll 4
-        for (int c8 = lane; c8 < hidden / 8; c8 += 32) {
+        for (int c8 = lane; c8 < ld / 8; c8 += 32) {
             const uint4 pk = wr[c8];
             const uint32_t u[4] = {pk.x, pk.y, pk.z, pk.w};
             float wf[8];
@@ -374,8 +375,8 @@ __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16*
             for (int j = 0; j < 4; ++j) unpack16<F16>(u[j], wf[2 * j], wf[2 * j + 1]);
 #pragma unroll
             for (int b = 0; b < B; ++b) {
-                const float4 x0 = *reinterpret_cast<const float4*>(xs + b * hidden + c8 * 8);
-                const float4 x1 = *reinterpret_cast<const float4*>(xs + b * hidden + c8 * 8 + 4);
+                const float4 x0 = *reinterpret_cast<const float4*>(xs + b * ld + c8 * 8);
+                const float4 x1 = *reinterpret_cast<const float4*>(xs + b * ld + c8 * 8 + 4);
                 acc[b] = fmaf(wf[0], x0.x, acc[b]);
                 acc[b] = fmaf(wf[1], x0.y, acc[b]);
                 acc[b] = fmaf(wf[2], x0.z, acc[b]);
@@ -522,31 +523,32 @@ int lm_head_max_candidates(int sm_count) { return sm_count * 4; }
 
 template <int B, bool F16>
 static cudaError_t launch_lm_head_fused_bt(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
-                                           int hidden, int64_t vocab, float* logits, float* cand_val,
+                                           int hidden, int ld, int64_t vocab, float* logits, float* cand_val,
                                            int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl) {
-    const size_t smem = (size_t)B * hidden * sizeof(float);
+    const size_t smem = (size_t)B * ld * sizeof(float);
     static PerDeviceOnce once;
     cudaError_t ce = once.run([] { return cudaFuncSetAttribute(lm_head_fused_kernel<B, F16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); });
     if (ce != cudaSuccess) return ce;
     if (smem > 200 * 1024) return cudaErrorInvalidConfiguration;
-    return launch_pdl(lm_head_fused_kernel<B, F16>, dim3(grid), dim3(256), smem, stream, pdl, w, h, norm_w, eps, hidden,
+    return launch_pdl(lm_head_fused_kernel<B, F16>, dim3(grid), dim3(256), smem, stream, pdl, w, h, norm_w, eps, hidden, ld,
                       vocab, logits, cand_val, cand_idx);
 }
 template <int B>
 static cudaError_t launch_lm_head_fused_b(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
-                                          int hidden, int64_t vocab, float* logits, float* cand_val,
+                                          int hidden, int ld, int64_t vocab, float* logits, float* cand_val,
                                           int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl, bool f16) {
-    return f16 ? launch_lm_head_fused_bt<B, true>(w, h, norm_w, eps, hidden, vocab, logits, cand_val, cand_idx, grid, stream, pdl)
-               : launch_lm_head_fused_bt<B, false>(w, h, norm_w, eps, hidden, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
+    return f16 ? launch_lm_head_fused_bt<B, true>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl)
+               : launch_lm_head_fused_bt<B, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
 }
 
 cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                  int batch, int hidden, int64_t vocab, float* logits, float* cand_val,
-                                 int32_t* cand_idx, int* n_cand, int sm_count, cudaStream_t stream, bool pdl, bool f16) {
-    if (hidden % 8 != 0 || batch < 1) return cudaErrorInvalidValue;
+                                 int32_t* cand_idx, int* n_cand, int sm_count, cudaStream_t stream, bool pdl, bool f16, int ld) {
+    if (ld == 0) ld = hidden;
+    if (ld % 8 != 0 || ld < hidden || batch < 1) return cudaErrorInvalidValue;
     // one grid size for every group of tokens, so that the candidate rows share a stride
     const int per_pass = batch > 4 ? 8 : 4;  // tokens per pass over the weights
-    const size_t smem_max = (size_t)(batch < per_pass ? batch : per_pass) * hidden * sizeof(float);
+    const size_t smem_max = (size_t)(batch < per_pass ? batch : per_pass) * ld * sizeof(float);
     int per_sm = (int)((200 * 1024) / (smem_max + 2048));
     per_sm = per_sm > 4 ? 4 : (per_sm < 1 ? 1 : per_sm);
     const int grid = sm_count * per_sm;
@@ -559,14 +561,14 @@ cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const f
         int32_t* ci = cand_idx + (size_t)b0 * grid;
         cudaError_t e;
         switch (bc) {
-            case 1: e = launch_lm_head_fused_b<1>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 2: e = launch_lm_head_fused_b<2>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 3: e = launch_lm_head_fused_b<3>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 4: e = launch_lm_head_fused_b<4>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 5: e = launch_lm_head_fused_b<5>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 6: e = launch_lm_head_fused_b<6>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 7: e = launch_lm_head_fused_b<7>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            default: e = launch_lm_head_fused_b<8>(w, hb, norm_w, eps, hidden, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 1: e = launch_lm_head_fused_b<1>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 2: e = launch_lm_head_fused_b<2>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 3: e = launch_lm_head_fused_b<3>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 4: e = launch_lm_head_fused_b<4>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 5: e = launch_lm_head_fused_b<5>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 6: e = launch_lm_head_fused_b<6>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 7: e = launch_lm_head_fused_b<7>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            default: e = launch_lm_head_fused_b<8>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
         }
         if (e != cudaSuccess) return e;
     }

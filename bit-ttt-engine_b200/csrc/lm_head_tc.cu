@@ -38,10 +38,10 @@ __device__ __host__ __forceinline__ int64_t tile_off(int row, int c, int chunk) 
 }
 
 // row-major bf16 [vocab, hidden] -> tiles [row_set][k_chunk][16 KB]
-__global__ void lm_retile_kernel(const __nv_bfloat16* __restrict__ w, int64_t vocab, int hidden,
+__global__ void lm_retile_kernel(const __nv_bfloat16* __restrict__ w, int64_t vocab, int hidden, int ld,
                                  __nv_bfloat16* __restrict__ tiles) {
     const int64_t row_sets = (vocab + kRows - 1) / kRows;
-    const int chunks = hidden / kChunk;
+    const int chunks = (hidden + kChunk - 1) / kChunk;
     const int64_t total = row_sets * chunks * (kRows * kChunk);
     for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
         const int64_t tile = i / (kRows * kChunk);
@@ -50,7 +50,7 @@ __global__ void lm_retile_kernel(const __nv_bfloat16* __restrict__ w, int64_t vo
         const int64_t rs = tile / chunks;
         const int kc = (int)(tile % chunks);
         const int64_t v = rs * kRows + row;
-        const __nv_bfloat16 val = v < vocab ? w[v * hidden + kc * kChunk + c] : __float2bfloat16_rn(0.0f);
+        const __nv_bfloat16 val = v < vocab && kc * kChunk + c < hidden ? w[v * ld + kc * kChunk + c] : __float2bfloat16_rn(0.0f);
         *reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<uint8_t*>(tiles) + tile * kATile + tile_off(row, c, kChunk)) = val;
     }
 }
@@ -73,8 +73,8 @@ __global__ void __launch_bounds__(256) lm_prep_kernel(const float* __restrict__ 
     ss = 0.0;
     for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += red[w];
     const float denom = sqrtf(__fadd_rn((float)(ss / (double)hidden), eps));
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-        const float v = real ? __fmul_rn(__fdiv_rn(hr[c], denom), norm_w[c]) : 0.0f;
+    for (int c = threadIdx.x; c < (hidden + kChunk - 1) / kChunk * kChunk; c += blockDim.x) {
+        const float v = real && c < hidden ? __fmul_rn(__fdiv_rn(hr[c], denom), norm_w[c]) : 0.0f;
         uint8_t* tile = btiles + (int64_t)(c / kChunk) * kBTile;
         if (f16) {
             const __half hi = __float2half_rn(v);
@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(kThreads, 1) lm_head_tc_kernel(const uint8_t* 
     uint64_t* acc_empty = acc_full + 1;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int chunks = hidden / kChunk;
+    const int chunks = (hidden + kChunk - 1) / kChunk;
     const int64_t row_sets = (vocab + kRows - 1) / kRows;
 
     if (threadIdx.x == 0) {
@@ -191,13 +191,12 @@ __global__ void __launch_bounds__(kThreads, 1) lm_head_tc_kernel(const uint8_t* 
 }  // namespace
 
 size_t lm_head_tc_weight_bytes(int64_t vocab, int hidden) {
-    return (size_t)((vocab + kRows - 1) / kRows) * (hidden / kChunk) * kATile;
+    return (size_t)((vocab + kRows - 1) / kRows) * ((hidden + kChunk - 1) / kChunk) * kATile;
 }
-size_t lm_head_tc_act_bytes(int hidden) { return (size_t)(hidden / kChunk) * kBTile; }
+size_t lm_head_tc_act_bytes(int hidden) { return (size_t)((hidden + kChunk - 1) / kChunk) * kBTile; }
 
-cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, void* tiles, cudaStream_t stream) {
-    if (hidden % kChunk != 0) return cudaErrorInvalidValue;
-    lm_retile_kernel<<<1184, 256, 0, stream>>>(w, vocab, hidden, reinterpret_cast<__nv_bfloat16*>(tiles));
+cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, void* tiles, cudaStream_t stream, int ld) {
+    lm_retile_kernel<<<1184, 256, 0, stream>>>(w, vocab, hidden, ld ? ld : hidden, reinterpret_cast<__nv_bfloat16*>(tiles));
     return cudaGetLastError();
 }
 
@@ -205,7 +204,6 @@ cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, 
 cudaError_t launch_lm_head_tc(const void* wtiles, const float* h, const float* norm_w, float eps, int batch, int hidden,
                               int64_t vocab, void* btiles, float* logits, unsigned int* err, int sm_count,
                               cudaStream_t stream, bool w_f16) {
-    if (hidden % kChunk != 0) return cudaErrorInvalidValue;
     const size_t smem = (size_t)kStages * (kATile + kBTile) + 256;
     static PerDeviceOnce once;
     cudaError_t ce = once.run([smem] { return cudaFuncSetAttribute(lm_head_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); });

@@ -5,9 +5,8 @@
 #include <string.h>
 
 #include <new>
-#include <vector>
 
-#include "bt_handles.cuh"
+#include "bt_model_impl.cuh"
 
 using namespace bt;
 
@@ -28,105 +27,25 @@ __global__ void f32_to_16bit_kernel(const float* __restrict__ in, __nv_bfloat16*
         else out[i] = __float2bfloat16_rn(in[i]);
     }
 }
+
+// staged through a bounded f32 buffer, converted on the device
+bt_status upload_16bit(const float* host, int64_t n_elem, __nv_bfloat16* dst, bool f16) {
+    const int64_t chunk = 16 << 20;
+    float* tmp = nullptr;
+    BT_CUDA_TRY(cudaMalloc(reinterpret_cast<void**>(&tmp), (size_t)(n_elem < chunk ? n_elem : chunk) * sizeof(float)));
+    for (int64_t off = 0; off < n_elem; off += chunk) {
+        const int64_t n = n_elem - off < chunk ? n_elem - off : chunk;
+        cudaError_t e = cudaMemcpy(tmp, host + off, (size_t)n * sizeof(float), cudaMemcpyHostToDevice);
+        if (e == cudaSuccess) {
+            f32_to_16bit_kernel<<<1184, 256>>>(tmp, dst + off, n, f16);
+            e = cudaDeviceSynchronize();
+        }
+        if (e != cudaSuccess) { cudaFree(tmp); return set_error(BT_ERR_CUDA, "uploading a table: %s", cudaGetErrorString(e)); }
+    }
+    cudaFree(tmp);
+    return BT_OK;
+}
 }  // namespace bt
-
-namespace {
-
-constexpr float kRmsEps = 1e-5f;  // model/block.rs:10, model/llama.rs:13
-
-struct HostLinear {
-    std::vector<uint8_t> packed;  // [n_out, k_in/4, n_bases]
-    int64_t n_out = 0, k_in = 0;
-    int n_bases = 1;
-    float scales[8] = {0};
-    bool set = false;
-};
-
-struct Layer {
-    HostLinear host[9];
-    bt_linear* qkv = nullptr;
-    bt_linear* o = nullptr;
-    bt_linear* gate_up_il = nullptr;   // gate/up interleaved by 8 rows (fused SwiGLU epilogue; SwiGLU row kernel)
-    bt_linear* down = nullptr;
-    bt_linear* ttt_down = nullptr;
-    bt_linear* ttt_up = nullptr;
-    float* norm1 = nullptr;
-    float* norm2 = nullptr;
-    bt_kv_cache* kv = nullptr;
-    float* w_state = nullptr;  // [max_batch, d, d]
-};
-
-}  // namespace
-
-struct bt_model {
-    bt_model_config cfg{};
-    int device = 0;
-    int sm_count = 0;
-    int head_dim = 0, d_small = 0, qkv_dim = 0;
-    int tp = 1;                      // tensor-parallel degree
-    int nh_l = 0, nkv_l = 0, i_l = 0;  // this rank's query heads, KV heads, MLP columns
-    void* comm = nullptr;            // NCCL communicator when tp > 1
-    void* peer = nullptr;            // peer-memory exchange (CUDA IPC inboxes) when the ranks have set it up
-    int32_t* acc_i32 = nullptr;      // [max_batch, hidden] accumulators of a row-parallel projection
-    bool finalized = false;
-    bool multi_basis = false;        // a projection has several bases: the step runs quantiser and product kernels separately
-    std::vector<Layer> layers;
-    __nv_bfloat16* embed = nullptr;   // 16-bit storage: bf16, or IEEE half when embed_f16
-    __nv_bfloat16* lm_head = nullptr;
-    bool embed_f16 = false, head_f16 = false;
-    float* norm_f = nullptr;
-    float* inv_freq = nullptr;
-    float* rope_cos = nullptr;   // [max_pos, head_dim/2]
-    float* rope_sin = nullptr;
-    // activations
-    int32_t* tokens = nullptr;
-    int32_t* pos = nullptr;
-    float* h = nullptr;
-    int8_t* q = nullptr;
-    int64_t q_stride = 0;
-    float* sx = nullptr;
-    int32_t* qsum = nullptr;
-    float* qkv = nullptr;
-    float* att = nullptr;
-    float* gu = nullptr;
-    float* feat = nullptr;
-    float* z = nullptr;
-    float* xn = nullptr;
-    float* logits = nullptr;
-    int32_t* next = nullptr;
-    float* act = nullptr;            // [max_batch, intermediate] silu(gate)*up
-    float* xt = nullptr;             // [max_batch, max(hidden, intermediate)] transformed rows (batches above 8)
-    int8_t* qtc = nullptr;           // activations in the tensor-core product's layout (batches above 8)
-    void* lm_tiles = nullptr;        // lm_head in tensor-core tile order (batches above 8, hidden % 64 == 0)
-    void* lm_btiles = nullptr;       // normalised hidden states as bf16 hi|lo tiles
-    float* lm_gather = nullptr;      // tensor parallelism: the ranks' vocabulary slices of the logits, [tp][batch][vl]
-    int64_t vl = 0;                  // rows of the head per rank (multiple of 128)
-    unsigned int* absmax = nullptr;  // [num_layers][2][max_batch] max|x| cells of the fused path
-    float* cand_val = nullptr;
-    int32_t* cand_idx = nullptr;
-    int32_t* tokens_pinned = nullptr;
-    int32_t* next_pinned = nullptr;
-    float* trace = nullptr;          // inspection aid: per-layer intermediate tensors of a step (caller's device buffer)
-    int trace_rows = 0;              // rows per tensor the trace buffer was sized for
-    // prefill scratch (allocated at the first bt_model_prefill, for pf_rows = sequences x tokens of a chunk)
-    int pf_rows = 0;
-    int32_t* pf_tokens = nullptr;
-    float* pf_h = nullptr;
-    float* pf_qkv = nullptr;
-    float* pf_att = nullptr;
-    float* pf_gu = nullptr;
-    float* pf_act = nullptr;         // silu(gate)*up rows, only while a trace is recorded
-    int pf_act_rows = 0;
-    int8_t* pf_qtc = nullptr;
-    float* pf_sx = nullptr;
-    int32_t* pf_qsum = nullptr;
-    std::vector<int32_t> pf_host;
-    unsigned int* err_pinned = nullptr;  // tensor parallel: the device error word as read after a step
-    int host_pos = 0;
-    int64_t ternary_bytes = 0;
-    cudaStream_t stream = nullptr;
-    cudaGraphExec_t graphs[65] = {nullptr};
-};
 
 namespace {
 
@@ -208,6 +127,7 @@ void trace_widths(const bt_model* m, int64_t (&w)[TR_SLOTS]) {
     w[TR_H_OUT] = H;
 }
 int64_t trace_layer_floats(const bt_model* m, int rows) {
+    if (m->lay) return (int64_t)m->cfg.hidden_dim * rows;  // the residual stream after the layer
     int64_t w[TR_SLOTS], n = 0;
     trace_widths(m, w);
     for (int i = 0; i < TR_SLOTS; ++i) n += w[i] * rows;
@@ -223,7 +143,7 @@ cudaError_t trace_copy(const bt_model* m, int layer, int slot, const float* src,
     return cudaMemcpyAsync(dst, src, (size_t)rows * w[slot] * sizeof(float), cudaMemcpyDeviceToDevice, s);
 }
 
-bt_status enqueue_head(bt_model* m, int batch, cudaStream_t s, bool fused_launches);
+bt_status enqueue_head(bt_model* m, int rows, cudaStream_t s, bool fused_launches, bool advance = true);
 
 bt_status enqueue_step_fused(bt_model* m, int batch, cudaStream_t s) {
     const bt_model_config& c = m->cfg;
@@ -321,7 +241,8 @@ bt_status enqueue_step_fused(bt_model* m, int batch, cudaStream_t s) {
 // logits = lm_head(norm(h))  (model/llama.rs:256-266), greedy pick, position advance.  Under tensor parallelism with
 // an NCCL communicator every rank computes the vocabulary rows rank * vl .. (the weights stay replicated in memory,
 // the reading and the arithmetic are split), the slices are all-gathered and every rank picks from the full row.
-bt_status enqueue_head(bt_model* m, int batch, cudaStream_t s, bool fused_launches) {
+// advance: the positions move on (a decode step); a prefill sets them itself.
+bt_status enqueue_head(bt_model* m, int batch, cudaStream_t s, bool fused_launches, bool advance) {
     const bt_model_config& c = m->cfg;
     const int H = c.hidden_dim, B = c.max_batch;
     unsigned int* err = device_error_word(m->device);
@@ -350,17 +271,17 @@ bt_status enqueue_head(bt_model* m, int batch, cudaStream_t s, bool fused_launch
         return BT_OK;
     }
     if (tc) {
-        BT_CUDA_TRY(launch_lm_head_tc(m->lm_tiles, m->h, m->norm_f, kRmsEps, batch, H, c.vocab_size, m->lm_btiles, m->logits,
+        BT_CUDA_TRY(launch_lm_head_tc(m->lm_tiles, m->h, m->norm_f, m->rms_eps, batch, H, c.vocab_size, m->lm_btiles, m->logits,
                                       err, sm, s, m->head_f16));
         BT_CUDA_TRY(launch_argmax(m->logits, batch, c.vocab_size, m->next, s));
-        advance_pos_kernel<<<1, 64, 0, s>>>(m->pos, B);
+        if (advance) advance_pos_kernel<<<1, 64, 0, s>>>(m->pos, B);
         BT_CUDA_TRY(cudaGetLastError());
         return BT_OK;
     }
     int n_cand = 0;
-    BT_CUDA_TRY(launch_lm_head_fused(m->lm_head, m->h, m->norm_f, kRmsEps, batch, H, c.vocab_size, m->logits,
-                                     m->cand_val, m->cand_idx, &n_cand, sm, s, fused_launches, m->head_f16));
-    BT_CUDA_TRY(launch_pick(m->cand_val, m->cand_idx, n_cand, batch, m->next, m->pos, B, s, fused_launches));
+    BT_CUDA_TRY(launch_lm_head_fused(m->lm_head, m->h, m->norm_f, m->rms_eps, batch, H, c.vocab_size, m->logits,
+                                     m->cand_val, m->cand_idx, &n_cand, sm, s, fused_launches, m->head_f16, m->head_ld));
+    BT_CUDA_TRY(launch_pick(m->cand_val, m->cand_idx, n_cand, batch, m->next, m->pos, advance ? B : 0, s, fused_launches));
     return BT_OK;
 }
 
@@ -580,6 +501,7 @@ extern "C" bt_status bt_model_set_linear_bases(bt_model* m, int layer, bt_weight
                                                int64_t n_out, int64_t k_in, int n_bases, const float* scales_host) {
     if (!m || !packed_host || !scales_host) return set_error(BT_ERR_ARG, "bt_model_set_linear: null pointer");
     if (m->finalized) return set_error(BT_ERR_ARG, "bt_model_set_linear: model already finalized");
+    if (m->lay) return set_error(BT_ERR_ARG, "bt_model_set_linear: a layer-list model takes its weights through bt_model_set_layer_tensor");
     if (layer < 0 || layer >= m->cfg.num_layers || (int)kind < 0 || (int)kind > 8)
         return set_error(BT_ERR_ARG, "bt_model_set_linear: layer %d / kind %d out of range", layer, (int)kind);
     if (n_bases < 1 || n_bases > 8) return set_error(BT_ERR_ARG, "bt_model_set_linear: n_bases %d outside 1..8", n_bases);
@@ -621,6 +543,7 @@ extern "C" bt_status bt_model_set_tensor_typed(bt_model* m, bt_tensor_kind kind,
     if (!m || !data) return set_error(BT_ERR_ARG, "bt_model_set_tensor: null pointer");
     if (storage != BT_BF16 && storage != BT_F16) return set_error(BT_ERR_ARG, "bt_model_set_tensor: storage must be BT_BF16 or BT_F16");
     if (m->finalized) return set_error(BT_ERR_ARG, "bt_model_set_tensor: model already finalized");
+    if (m->lay) return layered_set_tensor(m, kind, data, n_elem, storage);
     const bt_model_config& c = m->cfg;
     DeviceGuard guard(m->device);
     const int64_t H = c.hidden_dim, VH = (int64_t)c.vocab_size * H;
@@ -629,21 +552,7 @@ extern "C" bt_status bt_model_set_tensor_typed(bt_model* m, bt_tensor_kind kind,
         __nv_bfloat16** dst = kind == BT_T_EMBED ? &m->embed : &m->lm_head;
         (kind == BT_T_EMBED ? m->embed_f16 : m->head_f16) = storage == BT_F16;
         if (!*dst) BT_CUDA_TRY(dev_alloc(dst, (size_t)VH));
-        // staged through a bounded f32 buffer, converted on the device
-        const int64_t chunk = 16 << 20;
-        float* tmp = nullptr;
-        BT_CUDA_TRY(dev_alloc(&tmp, (size_t)(VH < chunk ? VH : chunk)));
-        for (int64_t off = 0; off < VH; off += chunk) {
-            const int64_t n = VH - off < chunk ? VH - off : chunk;
-            cudaError_t e = cudaMemcpy(tmp, data + off, (size_t)n * sizeof(float), cudaMemcpyHostToDevice);
-            if (e == cudaSuccess) {
-                f32_to_16bit_kernel<<<1184, 256>>>(tmp, *dst + off, n, storage == BT_F16);
-                e = cudaDeviceSynchronize();
-            }
-            if (e != cudaSuccess) { cudaFree(tmp); return set_error(BT_ERR_CUDA, "bt_model_set_tensor: %s", cudaGetErrorString(e)); }
-        }
-        cudaFree(tmp);
-        return BT_OK;
+        return upload_16bit(data, VH, *dst, storage == BT_F16);
     }
     if (n_elem != H) return set_error(BT_ERR_SHAPE, "bt_model_set_tensor: norm weight has %lld elements, %lld expected", (long long)n_elem, (long long)H);
     float** dst = nullptr;
@@ -660,6 +569,13 @@ extern "C" bt_status bt_model_set_tensor_typed(bt_model* m, bt_tensor_kind kind,
 extern "C" bt_status bt_model_finalize(bt_model* m) {
     if (!m) return set_error(BT_ERR_ARG, "bt_model_finalize: null handle");
     if (m->finalized) return BT_OK;
+    if (m->lay) {
+        DeviceGuard guard(m->device);
+        bt_status st = layered_finalize(m);
+        if (st != BT_OK) return st;
+        m->finalized = true;
+        return bt_model_reset(m);
+    }
     const bt_model_config& c = m->cfg;
     DeviceGuard guard(m->device);
     if (!m->embed || !m->lm_head || !m->norm_f) return set_error(BT_ERR_ARG, "bt_model_finalize: embedding, lm_head or final norm missing");
@@ -740,6 +656,7 @@ extern "C" bt_status bt_model_finalize(bt_model* m) {
     BT_CUDA_TRY(cudaMallocHost(reinterpret_cast<void**>(&m->err_pinned), sizeof(unsigned int)));
     *m->err_pinned = 0;
     BT_CUDA_TRY(cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking));
+    m->head_rows = B;
     m->finalized = true;
     return bt_model_reset(m);
 }
@@ -750,6 +667,7 @@ extern "C" bt_status bt_model_destroy(bt_model* m) {
     cudaDeviceSynchronize();
     for (auto& g : m->graphs)
         if (g && g != reinterpret_cast<cudaGraphExec_t>(uintptr_t(1))) cudaGraphExecDestroy(g);  // 1 = "ran eagerly once" sentinel
+    if (m->lay) layered_destroy(m);
     for (auto& L : m->layers) {
         bt_linear_destroy(L.qkv); bt_linear_destroy(L.o); bt_linear_destroy(L.gate_up_il); bt_linear_destroy(L.down);
         bt_linear_destroy(L.ttt_down); bt_linear_destroy(L.ttt_up);
@@ -779,6 +697,7 @@ extern "C" bt_status bt_model_reset(bt_model* m) {
         if (L.kv) { bt_status st = bt_kv_reset(L.kv); if (st != BT_OK) return st; }
         if (L.w_state) BT_CUDA_TRY(cudaMemset(L.w_state, 0, (size_t)m->cfg.max_batch * m->d_small * m->d_small * sizeof(float)));
     }
+    if (m->lay) { bt_status st = layered_reset(m); if (st != BT_OK) return st; }
     BT_CUDA_TRY(cudaMemset(m->pos, 0, (size_t)m->cfg.max_batch * sizeof(int32_t)));
     BT_CUDA_TRY(cudaDeviceSynchronize());  // the clears are done before a step on another stream can start
     m->host_pos = 0;
@@ -798,6 +717,10 @@ extern "C" bt_status bt_model_tp_resync(bt_model* m) {
 namespace {
 
 bt_status enqueue_any(bt_model* m, int batch, cudaStream_t s) {
+    if (m->lay) {
+        bt_status st = layered_step(m, batch, s);
+        return st != BT_OK ? st : enqueue_head(m, batch, s, batch <= 8);
+    }
     if (m->multi_basis) return enqueue_step_generic(m, batch, s);
     return batch <= 8 ? enqueue_step_fused(m, batch, s) : enqueue_step(m, batch, s);
 }
@@ -805,7 +728,7 @@ bt_status enqueue_any(bt_model* m, int batch, cudaStream_t s) {
 bt_status run_step(bt_model* m, int batch, cudaStream_t s) {
     if (m->tp > 1 && !m->comm && !tp_peer_ready(m->peer))
         return set_error(BT_ERR_NCCL, "tensor-parallel model used before bt_model_tp_init / bt_model_tp_peer_import");
-    if (m->cfg.arch == 1 && m->host_pos >= m->cfg.max_position_embeddings)
+    if (m->cfg.arch != 0 && m->host_pos >= m->cfg.max_position_embeddings)
         return set_error(BT_ERR_SHAPE, "position %d reaches max_position_embeddings %d", m->host_pos, m->cfg.max_position_embeddings);
     // first call at a batch size runs eagerly (it also sets kernel attributes); the second
     // is captured into a graph that later calls replay
@@ -889,6 +812,7 @@ namespace {
 constexpr int kPrefillRowsMax = 2048;  // rows (sequences x tokens) one prefill chunk works on
 
 bt_status prefill_buffers(bt_model* m, int rows) {
+    if (m->lay) return layered_prefill_buffers(m, rows);
     if (rows <= m->pf_rows) return BT_OK;
     const bt_model_config& c = m->cfg;
     const int64_t H = c.hidden_dim, I = m->i_l;
@@ -916,6 +840,7 @@ bt_status prefill_buffers(bt_model* m, int rows) {
 // (model/block.rs:87-134 applied to a [batch, n, hidden] input, cache semantics of model/llama.rs:495-498).
 bt_status enqueue_prefill_chunk(bt_model* m, int batch, int n, int past, int ttt_chunk, cudaStream_t s) {
     const bt_model_config& c = m->cfg;
+    if (m->lay) return layered_prefill(m, batch, n, s);
     const int H = c.hidden_dim, I = m->i_l, M = batch * n;
     unsigned int* err = device_error_word(m->device);
     const int sm = m->sm_count;
@@ -987,15 +912,21 @@ bt_status enqueue_prefill_chunk(bt_model* m, int batch, int n, int past, int ttt
 
 }  // namespace
 
-extern "C" bt_status bt_model_prefill(bt_model* m, const int32_t* tokens_host, int batch, int n_tokens, int ttt_chunk,
-                                      float* logits_host, int32_t* next_host) {
+namespace {
+
+// Prefill with the logits of chosen tokens: want[0 .. n_want) are token indices (the same for every sequence),
+// logits_host [batch][n_want][vocab].  next_host: the greedy id of the last token, which must then be the one wanted.
+bt_status prefill_impl(bt_model* m, const int32_t* tokens_host, int batch, int n_tokens, int ttt_chunk, const int32_t* want,
+                       int n_want, float* logits_host, int32_t* next_host) {
     if (!m || !m->finalized || !tokens_host) return set_error(BT_ERR_ARG, "bt_model_prefill: null pointer or model not finalized");
     if (batch < 1 || batch > m->cfg.max_batch) return set_error(BT_ERR_SHAPE, "bt_model_prefill: batch %d outside 1..%d", batch, m->cfg.max_batch);
     if (n_tokens < 1) return set_error(BT_ERR_SHAPE, "bt_model_prefill: no tokens");
     if (m->tp > 1) return set_error(BT_ERR_ARG, "bt_model_prefill: tensor-parallel models prefill token by token (bt_model_forward_one)");
     if (ttt_chunk < 1 || ttt_chunk > 64) return set_error(BT_ERR_ARG, "bt_model_prefill: ttt_chunk %d outside 1..64", ttt_chunk);
+    for (int i = 0; i < n_want; ++i)
+        if (want[i] < 0 || want[i] >= n_tokens) return set_error(BT_ERR_SHAPE, "bt_model_prefill: wanted token %d outside 0..%d", want[i], n_tokens - 1);
     const bt_model_config& c = m->cfg;
-    if (c.arch == 1 && m->host_pos + n_tokens > c.max_position_embeddings)
+    if (c.arch != 0 && m->host_pos + n_tokens > c.max_position_embeddings)
         return set_error(BT_ERR_SHAPE, "position %d reaches max_position_embeddings %d", m->host_pos + n_tokens, c.max_position_embeddings);
     DeviceGuard guard(m->device);
     cudaStream_t s = m->stream;
@@ -1008,7 +939,7 @@ extern "C" bt_status bt_model_prefill(bt_model* m, const int32_t* tokens_host, i
     if (per < 1) return set_error(BT_ERR_NOMEM, "bt_model_prefill: the trace buffer holds fewer rows than sequences");
     bt_status st = prefill_buffers(m, batch * per);
     if (st != BT_OK) return st;
-    if (m->trace && m->pf_act_rows < batch * per) {
+    if (m->trace && !m->lay && m->pf_act_rows < batch * per) {
         BT_CUDA_TRY(cudaDeviceSynchronize());
         cudaFree(m->pf_act);
         m->pf_act = nullptr;
@@ -1016,7 +947,8 @@ extern "C" bt_status bt_model_prefill(bt_model* m, const int32_t* tokens_host, i
         m->pf_act_rows = batch * per;
     }
     const int H = c.hidden_dim, past0 = m->host_pos;
-    int last_n = 0;
+    struct Pick { int row; int64_t dst; };
+    std::vector<Pick> picks;
     for (int c0 = 0; c0 < n_tokens; c0 += per) {
         const int n = n_tokens - c0 < per ? n_tokens - c0 : per;
         m->pf_host.resize((size_t)batch * n);
@@ -1026,31 +958,47 @@ extern "C" bt_status bt_model_prefill(bt_model* m, const int32_t* tokens_host, i
         set_pos_kernel<<<1, 64, 0, s>>>(m->pos, c.max_batch, past0 + c0);
         BT_CUDA_TRY(cudaGetLastError());
         if ((st = enqueue_prefill_chunk(m, batch, n, past0 + c0, ttt_chunk, s)) != BT_OK) return st;
+        // the wanted tokens of this chunk: their hidden states move into the decode buffers, through the head in groups
+        picks.clear();
+        for (int b = 0; b < batch; ++b)
+            for (int i = 0; i < n_want; ++i)
+                if (want[i] >= c0 && want[i] < c0 + n) picks.push_back({b * n + want[i] - c0, (int64_t)b * n_want + i});
+        for (size_t p0 = 0; p0 < picks.size(); p0 += (size_t)m->head_rows) {
+            const int cnt = (int)(picks.size() - p0 < (size_t)m->head_rows ? picks.size() - p0 : (size_t)m->head_rows);
+            for (int i = 0, run; i < cnt; i += run) {  // runs of neighbouring rows in one copy
+                for (run = 1; i + run < cnt && picks[p0 + i + run].row == picks[p0 + i].row + run; ++run) {}
+                BT_CUDA_TRY(cudaMemcpyAsync(m->h + (size_t)i * H, m->pf_h + (size_t)picks[p0 + i].row * H, (size_t)run * H * sizeof(float), cudaMemcpyDeviceToDevice, s));
+            }
+            if ((st = enqueue_head(m, cnt, s, false, false)) != BT_OK) return st;
+            const size_t vb = (size_t)c.vocab_size * sizeof(float);
+            for (int i = 0, run; logits_host && i < cnt; i += run) {
+                for (run = 1; i + run < cnt && picks[p0 + i + run].dst == picks[p0 + i].dst + run; ++run) {}
+                BT_CUDA_TRY(cudaMemcpyAsync(logits_host + picks[p0 + i].dst * c.vocab_size, m->logits + (size_t)i * c.vocab_size, run * vb, cudaMemcpyDeviceToHost, s));
+            }
+        }
         BT_CUDA_TRY(cudaStreamSynchronize(s));  // pf_host is reused by the next chunk
-        last_n = n;
-    }
-    // logits of the last token of every sequence: its hidden state moves into the decode buffers
-    BT_CUDA_TRY(cudaMemcpy2DAsync(m->h, (size_t)H * sizeof(float), m->pf_h + (size_t)(last_n - 1) * H, (size_t)last_n * H * sizeof(float),
-                                  (size_t)H * sizeof(float), (size_t)batch, cudaMemcpyDeviceToDevice, s));
-    if (m->lm_tiles && batch > 8) {
-        BT_CUDA_TRY(launch_lm_head_tc(m->lm_tiles, m->h, m->norm_f, kRmsEps, batch, H, c.vocab_size, m->lm_btiles, m->logits,
-                                      device_error_word(m->device), m->sm_count, s, m->head_f16));
-        BT_CUDA_TRY(launch_argmax(m->logits, batch, c.vocab_size, m->next, s));
-    } else {
-        int n_cand = 0;
-        BT_CUDA_TRY(launch_lm_head_fused(m->lm_head, m->h, m->norm_f, kRmsEps, batch, H, c.vocab_size, m->logits,
-                                         m->cand_val, m->cand_idx, &n_cand, m->sm_count, s, false, m->head_f16));
-        BT_CUDA_TRY(launch_pick(m->cand_val, m->cand_idx, n_cand, batch, m->next, m->pos, 0, s, false));
     }
     set_pos_kernel<<<1, 64, 0, s>>>(m->pos, c.max_batch, past0 + n_tokens);
     BT_CUDA_TRY(cudaGetLastError());
     m->host_pos = past0 + n_tokens;
-    if (logits_host)
-        BT_CUDA_TRY(cudaMemcpyAsync(logits_host, m->logits, (size_t)batch * c.vocab_size * sizeof(float), cudaMemcpyDeviceToHost, s));
-    BT_CUDA_TRY(cudaMemcpyAsync(m->next_pinned, m->next, (size_t)batch * sizeof(int32_t), cudaMemcpyDeviceToHost, s));
+    if (next_host) BT_CUDA_TRY(cudaMemcpyAsync(m->next_pinned, m->next, (size_t)batch * sizeof(int32_t), cudaMemcpyDeviceToHost, s));
     BT_CUDA_TRY(cudaStreamSynchronize(s));
     if (next_host) memcpy(next_host, m->next_pinned, (size_t)batch * sizeof(int32_t));
     return BT_OK;
+}
+
+}  // namespace
+
+extern "C" bt_status bt_model_prefill(bt_model* m, const int32_t* tokens_host, int batch, int n_tokens, int ttt_chunk,
+                                      float* logits_host, int32_t* next_host) {
+    const int32_t last = n_tokens - 1;
+    return prefill_impl(m, tokens_host, batch, n_tokens, ttt_chunk, &last, n_tokens < 1 ? 0 : 1, logits_host, next_host);
+}
+
+extern "C" bt_status bt_model_prefill_logits(bt_model* m, const int32_t* tokens_host, int batch, int n_tokens, int ttt_chunk,
+                                             const int32_t* want_host, int n_want, float* logits_host) {
+    if (n_want < 0 || (n_want > 0 && (!want_host || !logits_host))) return set_error(BT_ERR_ARG, "bt_model_prefill_logits: null pointer");
+    return prefill_impl(m, tokens_host, batch, n_tokens, ttt_chunk, want_host, n_want, logits_host, nullptr);
 }
 
 extern "C" const float* bt_model_logits(bt_model* m) { return m ? m->logits : nullptr; }
@@ -1061,6 +1009,7 @@ extern "C" float* bt_model_ttt_state(bt_model* m, int layer) {
     return m->layers[(size_t)layer].w_state;
 }
 extern "C" bt_kv_cache* bt_model_kv_cache(bt_model* m, int layer) {
+    if (m && m->lay) return layered_kv(m, layer);
     if (!m || layer < 0 || layer >= (int)m->layers.size()) return nullptr;
     return m->layers[(size_t)layer].kv;
 }
@@ -1080,6 +1029,7 @@ extern "C" int64_t bt_model_ternary_bytes(const bt_model* m) { return m ? m->ter
 
 extern "C" bt_status bt_model_enqueue_products(bt_model* m, int batch, int as_in_step, void* stream, int* n_launches) {
     if (!m || !m->finalized) return set_error(BT_ERR_ARG, "bt_model_enqueue_products: model not finalized");
+    if (m->lay) return set_error(BT_ERR_ARG, "bt_model_enqueue_products: the model has no ternary products");
     if (batch < 1 || batch > m->cfg.max_batch) return set_error(BT_ERR_SHAPE, "batch %d outside 1..%d", batch, m->cfg.max_batch);
     DeviceGuard guard(m->device);
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
@@ -1127,6 +1077,7 @@ extern "C" bt_status bt_model_enqueue_products(bt_model* m, int batch, int as_in
 
 extern "C" int bt_model_launches_per_step(const bt_model* m, int batch) {
     if (!m) return 0;
+    if (m->lay) return m->finalized ? layered_launches(m, batch) : 0;
     // kernels of this library only: NCCL's own kernels (all-reduce, all-gather) are not counted
     const bool split_head = m->tp > 1 && m->comm && m->lm_gather;  // the head's rows cut over the ranks
     if (batch <= 8) {
@@ -1153,7 +1104,7 @@ extern "C" int bt_model_launches_per_step(const bt_model* m, int batch) {
 
 extern "C" bt_status bt_model_seek(bt_model* m, int pos) {
     if (!m || !m->finalized) return set_error(BT_ERR_ARG, "bt_model_seek: model not finalized");
-    if (pos < 0 || (m->cfg.arch == 1 && pos >= m->cfg.max_position_embeddings))
+    if (pos < 0 || (m->cfg.arch != 0 && pos >= m->cfg.max_position_embeddings))
         return set_error(BT_ERR_SHAPE, "bt_model_seek: position %d outside [0, %d)", pos, m->cfg.max_position_embeddings);
     DeviceGuard guard(m->device);
     BT_CUDA_TRY(cudaDeviceSynchronize());

@@ -1,6 +1,7 @@
 // extern "C" entry points for the TTT fast-weight update, the Q8 KV cache and decode
 // attention.
 #include <math.h>
+#include <string.h>
 
 #include <new>
 #include <vector>
@@ -73,9 +74,86 @@ extern "C" bt_status bt_kv_create(bt_kv_cache** out, int64_t batch, int64_t n_kv
     return bt_kv_reset(c);
 }
 
+extern "C" bt_status bt_kv_create_dense(bt_kv_cache** out, int64_t batch, int64_t n_kv_heads, int64_t k_dim, int64_t v_dim,
+                                        int64_t max_seq_len, bt_dtype dtype, int device) {
+    if (!out) return set_error(BT_ERR_ARG, "bt_kv_create_dense: null out pointer");
+    *out = nullptr;
+    if (batch < 1 || n_kv_heads < 1 || max_seq_len < 1 || k_dim < 1 || v_dim < 1)
+        return set_error(BT_ERR_SHAPE, "bt_kv_create_dense: bad shape");
+    if (dtype != BT_BF16 && dtype != BT_F32) return set_error(BT_ERR_ARG, "bt_kv_create_dense: dtype must be BT_BF16 or BT_F32");
+    if (bt_device_count() <= device || device < 0) return set_error(BT_ERR_DEVICE, "bt_kv_create_dense: no CUDA device %d", device);
+    DeviceGuard guard(device);
+    if (!guard.ok) return set_error(BT_ERR_DEVICE, "cannot select device %d", device);
+    bt_kv_cache* c = new (std::nothrow) bt_kv_cache();
+    if (!c) return set_error(BT_ERR_NOMEM, "host allocation failed");
+    c->device = device;
+    c->batch = batch; c->n_kv = n_kv_heads; c->head_dim = k_dim; c->v_dim = v_dim; c->max_seq = max_seq_len;
+    c->is_dense = true;
+    DenseKvView& d = c->dense;
+    d.max_seq = (int)max_seq_len;
+    d.f32 = dtype == BT_F32;
+    d.k_stride = (int)((k_dim + 7) / 8 * 8);
+    d.v_stride = (int)((v_dim + 7) / 8 * 8);
+    cudaError_t e = cudaMalloc(&d.k, c->dense_bytes(d.k_stride));
+    if (e == cudaSuccess) e = cudaMalloc(&d.v, c->dense_bytes(d.v_stride));
+    if (e != cudaSuccess) {
+        bt_kv_destroy(c);
+        return set_error(BT_ERR_NOMEM, "bt_kv_create_dense: %s", cudaGetErrorString(e));
+    }
+    *out = c;
+    return bt_kv_reset(c);
+}
+
+namespace {
+// rows [0, t_len) of sequence b between host f32 [n_kv, t_len, dim] and the cache's padded rows
+bt_status dense_rows(bt_kv_cache* c, int64_t b, int64_t t_len, float* k_host, float* v_host, bool store) {
+    if (!c || !c->is_dense) return set_error(BT_ERR_ARG, "bt_kv_*_dense: null handle or a quantised cache");
+    if (b < 0 || b >= c->batch || t_len < 0 || t_len > c->max_seq)
+        return set_error(BT_ERR_SHAPE, "bt_kv_*_dense: sequence %lld / length %lld out of range", (long long)b, (long long)t_len);
+    DeviceGuard guard(c->device);
+    BT_CUDA_TRY(cudaDeviceSynchronize());
+    for (int which = 0; which < 2; ++which) {
+        float* host = which ? v_host : k_host;
+        if (!host) continue;
+        const int64_t stride = which ? c->dense.v_stride : c->dense.k_stride, dim = which ? c->v_dim : c->head_dim;
+        const size_t es = c->dense.f32 ? 4 : 2;
+        uint8_t* base = reinterpret_cast<uint8_t*>(which ? c->dense.v : c->dense.k);
+        std::vector<uint8_t> tmp((size_t)t_len * stride * es, 0);
+        for (int64_t h = 0; h < c->n_kv; ++h) {
+            uint8_t* dev = base + (size_t)((b * c->n_kv + h) * c->max_seq) * stride * es;
+            if (!store) BT_CUDA_TRY(cudaMemcpy(tmp.data(), dev, tmp.size(), cudaMemcpyDeviceToHost));
+            for (int64_t t = 0; t < t_len; ++t)
+                for (int64_t j = 0; j < dim; ++j) {
+                    float& hv = host[(h * t_len + t) * dim + j];
+                    uint8_t* p = tmp.data() + (t * stride + j) * es;
+                    if (store) {
+                        if (es == 4) memcpy(p, &hv, 4);
+                        else { const __nv_bfloat16 q = __float2bfloat16_rn(hv); memcpy(p, &q, 2); }
+                    } else if (es == 4) memcpy(&hv, p, 4);
+                    else { __nv_bfloat16 q; memcpy(&q, p, 2); hv = __bfloat162float(q); }
+                }
+            if (store) BT_CUDA_TRY(cudaMemcpy(dev, tmp.data(), tmp.size(), cudaMemcpyHostToDevice));
+        }
+    }
+    return BT_OK;
+}
+}  // namespace
+
+extern "C" bt_status bt_kv_export_dense(bt_kv_cache* c, int64_t b, int64_t t_len, float* k_host, float* v_host) {
+    return dense_rows(c, b, t_len, k_host, v_host, false);
+}
+extern "C" bt_status bt_kv_import_dense(bt_kv_cache* c, int64_t b, int64_t t_len, const float* k_host, const float* v_host) {
+    return dense_rows(c, b, t_len, const_cast<float*>(k_host), const_cast<float*>(v_host), true);
+}
+
 extern "C" bt_status bt_kv_reset(bt_kv_cache* c) {
     if (!c) return set_error(BT_ERR_ARG, "bt_kv_reset: null handle");
     DeviceGuard guard(c->device);
+    if (c->is_dense) {
+        BT_CUDA_TRY(cudaMemset(c->dense.k, 0, c->dense_bytes(c->dense.k_stride)));
+        BT_CUDA_TRY(cudaMemset(c->dense.v, 0, c->dense_bytes(c->dense.v_stride)));
+        return BT_OK;
+    }
     const size_t rows = (size_t)c->batch * c->n_kv * c->max_seq;
     BT_CUDA_TRY(cudaMemset(c->view.k_q, 128, rows * c->head_dim));
     BT_CUDA_TRY(cudaMemset(c->view.v_q, 128, rows * c->head_dim));
@@ -89,13 +167,14 @@ extern "C" bt_status bt_kv_destroy(bt_kv_cache* c) {
     DeviceGuard guard(c->device);
     cudaFree(c->view.k_q); cudaFree(c->view.v_q); cudaFree(c->view.k_s); cudaFree(c->view.v_s);
     cudaFree(c->inv_freq); cudaFree(c->rope_cos); cudaFree(c->rope_sin);
+    cudaFree(c->dense.k); cudaFree(c->dense.v);
     delete c;
     return BT_OK;
 }
 
 extern "C" bt_status bt_kv_export(bt_kv_cache* c, int64_t b, int64_t t_len, uint8_t* k_q_host, float* k_s_host,
                                   uint8_t* v_q_host, float* v_s_host) {
-    if (!c) return set_error(BT_ERR_ARG, "bt_kv_export: null handle");
+    if (!c || c->is_dense) return set_error(BT_ERR_ARG, "bt_kv_export: null handle or a cache that is not Q8");
     if (b < 0 || b >= c->batch || t_len < 0 || t_len > c->max_seq)
         return set_error(BT_ERR_SHAPE, "bt_kv_export: sequence %lld / length %lld out of range", (long long)b, (long long)t_len);
     DeviceGuard guard(c->device);
@@ -113,7 +192,7 @@ extern "C" bt_status bt_kv_export(bt_kv_cache* c, int64_t b, int64_t t_len, uint
 
 extern "C" bt_status bt_kv_import(bt_kv_cache* c, int64_t b, int64_t t_len, const uint8_t* k_q_host, const float* k_s_host,
                                   const uint8_t* v_q_host, const float* v_s_host) {
-    if (!c) return set_error(BT_ERR_ARG, "bt_kv_import: null handle");
+    if (!c || c->is_dense) return set_error(BT_ERR_ARG, "bt_kv_import: null handle or a cache that is not Q8");
     if (b < 0 || b >= c->batch || t_len < 0 || t_len > c->max_seq)
         return set_error(BT_ERR_SHAPE, "bt_kv_import: sequence %lld / length %lld out of range", (long long)b, (long long)t_len);
     DeviceGuard guard(c->device);
@@ -131,7 +210,7 @@ extern "C" bt_status bt_kv_import(bt_kv_cache* c, int64_t b, int64_t t_len, cons
 
 extern "C" bt_status bt_kv_append(bt_kv_cache* c, const float* k_dev, const float* v_dev, const int32_t* pos_dev,
                                   int64_t batch, void* stream) {
-    if (!c || !k_dev || !v_dev || !pos_dev) return set_error(BT_ERR_ARG, "bt_kv_append: null pointer");
+    if (!c || c->is_dense || !k_dev || !v_dev || !pos_dev) return set_error(BT_ERR_ARG, "bt_kv_append: null pointer");
     if (batch < 1 || batch > c->batch) return set_error(BT_ERR_SHAPE, "bt_kv_append: batch %lld exceeds the cache's %lld", (long long)batch, (long long)c->batch);
     DeviceGuard guard(c->device);
     if (!guard.ok) return set_error(BT_ERR_DEVICE, "cannot select device %d", c->device);
@@ -142,7 +221,7 @@ extern "C" bt_status bt_kv_append(bt_kv_cache* c, const float* k_dev, const floa
 
 extern "C" bt_status bt_attn_decode(bt_kv_cache* c, const float* qkv_dev, const int32_t* pos_dev, int64_t batch,
                                     int64_t n_heads, double rope_theta, float* out_dev, void* stream) {
-    if (!c || !qkv_dev || !pos_dev || !out_dev) return set_error(BT_ERR_ARG, "bt_attn_decode: null pointer");
+    if (!c || c->is_dense || !qkv_dev || !pos_dev || !out_dev) return set_error(BT_ERR_ARG, "bt_attn_decode: null pointer");
     if (batch < 1 || batch > c->batch) return set_error(BT_ERR_SHAPE, "bt_attn_decode: batch %lld exceeds the cache's %lld", (long long)batch, (long long)c->batch);
     const int64_t rep = n_heads / c->n_kv;
     if (n_heads % c->n_kv != 0 || !(rep == 1 || rep == 2 || rep == 4 || rep == 8) || n_heads > c->max_heads)

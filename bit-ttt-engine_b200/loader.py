@@ -213,21 +213,28 @@ def weights_from_tensors(tensors: dict, cfg: BitLlamaConfig) -> SyntheticWeights
     return w
 
 
-def load_checkpoint(path: str):
-    """(config, weights) from a model directory (config.json + *.safetensors) or from a single
-    .safetensors file with config.json beside it."""
+def read_checkpoint(path: str):
+    """(config dictionary, tensors) of a model directory (config.json + *.safetensors) or of a single .safetensors
+    file with config.json beside it."""
     directory = path if os.path.isdir(path) else os.path.dirname(os.path.abspath(path))
     cfg_path = os.path.join(directory, "config.json")
     if not os.path.exists(cfg_path):
         raise CheckpointError(f"{cfg_path} is missing")
     with open(cfg_path, "r", encoding="utf-8") as f:
-        cfg = config_from_dict(json.load(f))
+        cfg = json.load(f)
     files = [path] if os.path.isfile(path) else sorted(glob.glob(os.path.join(directory, "*.safetensors")))
     if not files:
         raise CheckpointError(f"no .safetensors file in {directory}")
     tensors = {}
     for fp in files:
         tensors.update(read_safetensors(fp))
+    return cfg, tensors
+
+
+def load_checkpoint(path: str):
+    """(config, weights) of a ternary Llama / TTT checkpoint."""
+    d, tensors = read_checkpoint(path)
+    cfg = config_from_dict(d)
     return cfg, weights_from_tensors(tensors, cfg)
 
 
@@ -266,8 +273,20 @@ def save_checkpoint(directory: str, w: SyntheticWeights, hf_names: bool = True, 
         json.dump(d, f, indent=1)
 
 
-def load_model(path: str, max_batch: int = 1, device: int = 0):
-    """`Llama::load_auto` for the decode path: read the checkpoint and build the device model."""
+def load_model(path: str, max_batch: int = 1, device: int = 0, dtype: str | None = None, max_seq_len: int | None = None):
+    """`Llama::load_auto` for the decode path: read the checkpoint, choose the model class by its config.json
+    (`architecture` names a layer-list design, layered.py; otherwise a ternary Llama / TTT model) and build the device
+    model.  dtype ("bfloat16" or "float32") and max_seq_len (positions the caches hold) matter to layer-list models."""
+    from .layered import DESIGNS, build_layered
+    d, tensors = read_checkpoint(path)
+    design = d.get("architecture")
+    if design is not None:
+        if design not in DESIGNS:
+            raise CheckpointError(f"config: unknown architecture {design!r} (known: {', '.join(sorted(DESIGNS))})")
+        return build_layered(DESIGNS[design](d), tensors, max_batch=max_batch, device=device, dtype=dtype or "bfloat16",
+                             max_seq_len=max_seq_len)
+    if dtype == "float32":
+        raise CheckpointError("ternary models quantise their activations to 8 bits: there is no 32-bit form of them")
     from .synthetic import build_model
-    cfg, w = load_checkpoint(path)
-    return build_model(w, max_batch=max_batch, device=device)
+    cfg = config_from_dict(d)
+    return build_model(weights_from_tensors(tensors, cfg), max_batch=max_batch, device=device)

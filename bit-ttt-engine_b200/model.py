@@ -7,12 +7,16 @@ from dataclasses import dataclass
 
 import numpy as np
 
-from . import check, lib
+from . import BT_BF16, BT_F32, check, lib
 from .layers import _ptr, _stream_ptr, _torch
 
 ARCH_TTT, ARCH_LLAMA = 0, 1
 (W_Q, W_K, W_V, W_O, W_GATE, W_UP, W_DOWN, W_TTT_DOWN, W_TTT_UP) = range(9)
-(T_EMBED, T_LM_HEAD, T_NORM_F, T_NORM1, T_NORM2) = range(5)
+(T_EMBED, T_LM_HEAD, T_NORM_F, T_NORM1, T_NORM2, T_POS) = range(6)
+MIX_ATTENTION, MIX_SSM = 0, 1
+MLP_NONE, MLP_DENSE_RELU2 = 0, 1
+(LT_NORM1, LT_NORM2, LT_Q, LT_K, LT_V, LT_O, LT_Q_NORM, LT_K_NORM, LT_SINK, LT_VMIX, LT_SSM_IN, LT_SSM_CONV,
+ LT_SSM_CONV_B, LT_SSM_DT_BIAS, LT_SSM_A_LOG, LT_SSM_D, LT_SSM_NORM, LT_SSM_O, LT_MLP_UP, LT_MLP_DOWN) = range(20)
 
 
 class _CModelConfig(C.Structure):
@@ -21,6 +25,20 @@ class _CModelConfig(C.Structure):
                 ("intermediate_dim", C.c_int), ("inner_lr", C.c_float), ("rope_theta", C.c_double),
                 ("max_position_embeddings", C.c_int), ("max_batch", C.c_int),
                 ("tp_rank", C.c_int), ("tp_size", C.c_int)]
+
+
+class _CLayerConfig(C.Structure):
+    _fields_ = [("mixer", C.c_int), ("heads", C.c_int), ("vdim", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int),
+                ("qk_norm", C.c_int), ("sink", C.c_int), ("v_mix", C.c_int), ("scale", C.c_float),
+                ("softcap", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_double),
+                ("state", C.c_int), ("groups", C.c_int), ("conv_taps", C.c_int), ("norm_groups", C.c_int),
+                ("mlp", C.c_int), ("ff", C.c_int)]
+
+
+class _CLayersConfig(C.Structure):
+    _fields_ = [("vocab_size", C.c_int), ("width", C.c_int), ("num_layers", C.c_int), ("max_positions", C.c_int),
+                ("max_seq_len", C.c_int), ("max_batch", C.c_int), ("norm_eps", C.c_float),
+                ("norm_one_plus", C.c_int), ("dtype", C.c_int)]
 
 
 def _bind():
@@ -60,6 +78,16 @@ def _bind():
     L.bt_model_trace_floats.argtypes = [vp, i32]
     L.bt_model_set_trace.argtypes = [vp, vp, i32]
     L.bt_model_prefill.argtypes = [vp, vp, i32, i32, i32, vp, vp]
+    L.bt_model_prefill_logits.argtypes = [vp, vp, i32, i32, i32, vp, i32, vp]
+    L.bt_kv_create_dense.argtypes = [C.POINTER(vp), i64, i64, i64, i64, i64, i32, i32]
+    L.bt_kv_export_dense.argtypes = [vp, i64, i64, vp, vp]
+    L.bt_kv_import_dense.argtypes = [vp, i64, i64, vp, vp]
+    L.bt_model_create_layers.argtypes = [C.POINTER(vp), C.POINTER(_CLayersConfig), C.POINTER(_CLayerConfig), i32]
+    L.bt_model_set_layer_tensor.argtypes = [vp, i32, i32, vp, i64]
+    L.bt_model_recurrent_state.restype = vp
+    L.bt_model_recurrent_state.argtypes = [vp, i32, C.POINTER(i64)]
+    L.bt_model_conv_ring.restype = vp
+    L.bt_model_conv_ring.argtypes = [vp, i32, C.POINTER(i64)]
     L.bt_model_ternary_bytes.restype = i64
     L.bt_model_ternary_bytes.argtypes = [vp]
     L.bt_tp_unique_id.argtypes = [vp]
@@ -174,7 +202,100 @@ class BitLlamaConfig:
     max_position_embeddings: int = 2048
 
 
-class BitLlama:
+class DeviceModel:
+    """What every model behind `bt_model` shares: the step, the prefill, positions, caches' reset, results.
+    Subclasses create the handle (`_h`) and hand over configuration and weights."""
+
+    _L, _h, cfg, max_batch, device = None, None, None, 1, 0
+
+    def finalize(self):
+        check(self._L.bt_model_finalize(self._h))
+
+    def reset_kv_cache(self):
+        check(self._L.bt_model_reset(self._h))
+
+    def seek(self, pos: int):
+        """Continue from position `pos` with the caches as they are in device memory."""
+        check(self._L.bt_model_seek(self._h, pos))
+
+    @property
+    def current_pos(self) -> int:
+        return self._L.bt_model_pos(self._h)
+
+    def forward_one(self, tokens, want_logits: bool = True):
+        """tokens: host ints [batch].  Returns (logits np [batch, vocab] or None, next ids)."""
+        tokens = np.ascontiguousarray(tokens, np.int32).reshape(-1)
+        b = tokens.size
+        logits = np.empty((b, self.cfg.vocab_size), np.float32) if want_logits else None
+        nxt = np.empty(b, np.int32)
+        check(self._L.bt_model_forward_one(self._h, tokens.ctypes.data, b,
+                                           logits.ctypes.data if want_logits else None, nxt.ctypes.data))
+        return logits, nxt
+
+    def prefill(self, tokens, ttt_chunk: int = 1, want_logits: bool = True):
+        """tokens: host ints [batch, n_tokens].  Batched prefill, equivalent to n_tokens forward_one calls
+        (model/llama.rs:495-498); returns (logits of the last token np [batch, vocab] or None, next ids)."""
+        tokens = np.ascontiguousarray(tokens, np.int32)
+        if tokens.ndim == 1:
+            tokens = tokens[None, :]
+        b, n = tokens.shape
+        logits = np.empty((b, self.cfg.vocab_size), np.float32) if want_logits else None
+        nxt = np.empty(b, np.int32)
+        check(self._L.bt_model_prefill(self._h, tokens.ctypes.data, b, n, ttt_chunk,
+                                       logits.ctypes.data if want_logits else None, nxt.ctypes.data))
+        return logits, nxt
+
+    def prefill_logits(self, tokens, want, ttt_chunk: int = 1) -> np.ndarray:
+        """Prefill that returns the logits of chosen tokens: tokens host ints [n] or [batch, n], want = indices into
+        the n tokens.  Returns np [batch, len(want), vocab] (without the batch axis for 1-d tokens)."""
+        tokens = np.ascontiguousarray(tokens, np.int32)
+        t2 = tokens[None, :] if tokens.ndim == 1 else tokens
+        want = np.ascontiguousarray(want, np.int32).reshape(-1)
+        logits = np.empty((t2.shape[0], want.size, self.cfg.vocab_size), np.float32)
+        check(self._L.bt_model_prefill_logits(self._h, t2.ctypes.data, t2.shape[0], t2.shape[1], ttt_chunk,
+                                              want.ctypes.data, want.size, logits.ctypes.data))
+        return logits[0] if tokens.ndim == 1 else logits
+
+    def generate(self, tokens, max_new: int) -> np.ndarray:
+        """Greedy generation from a fresh cache: prompts [batch, n] (or [n]) in, [batch, max_new] ids out - the loop of
+        the reference's command line (model/llama.rs:494-527) with the prompt as one batched prefill."""
+        tokens = np.ascontiguousarray(tokens, np.int32)
+        self.reset_kv_cache()
+        _, ids = self.prefill(tokens, want_logits=False)
+        out = [ids]
+        while len(out) < max_new:
+            _, ids = self.forward_one(ids, want_logits=False)
+            out.append(ids)
+        out = np.stack(out[:max_new], axis=1)
+        return out[0] if tokens.ndim == 1 else out
+
+    def step_dev(self, tokens_dev):
+        """Device-resident step on torch's current stream; results stay on the device."""
+        check(self._L.bt_model_step_dev(self._h, _ptr(tokens_dev), tokens_dev.numel(),
+                                        _stream_ptr(tokens_dev.device.index)))
+
+    def launches_per_step(self, batch: int) -> int:
+        return self._L.bt_model_launches_per_step(self._h, batch)
+
+    def next_dev(self):
+        torch = _torch()
+        return _wrap_dev(self._L.bt_model_next(self._h), (self.max_batch,), torch.int32, self.device)
+
+    def logits_dev(self):
+        torch = _torch()
+        return _wrap_dev(self._L.bt_model_logits(self._h), (self.max_batch, self.cfg.vocab_size),
+                         torch.float32, self.device)
+
+    def __del__(self):
+        try:
+            if getattr(self, "_h", None):
+                self._L.bt_model_destroy(self._h)
+                self._h = None
+        except Exception:
+            pass
+
+
+class BitLlama(DeviceModel):
     """model/llama.rs:37-272: load weights, forward_one, reset_kv_cache."""
 
     def __init__(self, cfg: BitLlamaConfig, max_batch: int = 1, device: int = 0, tp_rank: int = 0,
@@ -203,9 +324,6 @@ class BitLlama:
         instead of bf16."""
         data = np.ascontiguousarray(data, np.float32)
         check(self._L.bt_model_set_tensor_typed(self._h, kind, layer, data.ctypes.data, data.size, 4 if f16 else 1))
-
-    def finalize(self):
-        check(self._L.bt_model_finalize(self._h))
 
     def tp_init(self, unique_id: bytes):
         """Joins the tensor-parallel communicator (collective); unique_id from tp_unique_id() of rank 0."""
@@ -241,48 +359,9 @@ class BitLlama:
         """Back to the NCCL exchange (every rank must call it)."""
         check(self._L.bt_model_tp_peer_import(self._h, None))
 
-    def reset_kv_cache(self):
-        check(self._L.bt_model_reset(self._h))
-
-    def seek(self, pos: int):
-        """Continue from position `pos` with the caches as they are in device memory."""
-        check(self._L.bt_model_seek(self._h, pos))
-
-    @property
-    def current_pos(self) -> int:
-        return self._L.bt_model_pos(self._h)
-
     @property
     def ternary_bytes(self) -> int:
         return self._L.bt_model_ternary_bytes(self._h)
-
-    def forward_one(self, tokens, want_logits: bool = True):
-        """tokens: host ints [batch].  Returns (logits np [batch, vocab] or None, next ids)."""
-        tokens = np.ascontiguousarray(tokens, np.int32).reshape(-1)
-        b = tokens.size
-        logits = np.empty((b, self.cfg.vocab_size), np.float32) if want_logits else None
-        nxt = np.empty(b, np.int32)
-        check(self._L.bt_model_forward_one(self._h, tokens.ctypes.data, b,
-                                           logits.ctypes.data if want_logits else None, nxt.ctypes.data))
-        return logits, nxt
-
-    def prefill(self, tokens, ttt_chunk: int = 1, want_logits: bool = True):
-        """tokens: host ints [batch, n_tokens].  Batched prefill, equivalent to n_tokens forward_one calls
-        (model/llama.rs:495-498); returns (logits of the last token np [batch, vocab] or None, next ids)."""
-        tokens = np.ascontiguousarray(tokens, np.int32)
-        if tokens.ndim == 1:
-            tokens = tokens[None, :]
-        b, n = tokens.shape
-        logits = np.empty((b, self.cfg.vocab_size), np.float32) if want_logits else None
-        nxt = np.empty(b, np.int32)
-        check(self._L.bt_model_prefill(self._h, tokens.ctypes.data, b, n, ttt_chunk,
-                                       logits.ctypes.data if want_logits else None, nxt.ctypes.data))
-        return logits, nxt
-
-    def step_dev(self, tokens_dev):
-        """Device-resident step on torch's current stream; results stay on the device."""
-        check(self._L.bt_model_step_dev(self._h, _ptr(tokens_dev), tokens_dev.numel(),
-                                        _stream_ptr(tokens_dev.device.index)))
 
     def set_trace(self, on: bool = True, rows: int = 0) -> None:
         """Keep the per-layer intermediate tensors of the following steps (see read_trace).
@@ -326,18 +405,6 @@ class BitLlama:
         n = C.c_int(0)
         check(self._L.bt_model_enqueue_products(self._h, batch, int(as_in_step), _stream_ptr(self.device), C.byref(n)))
         return n.value
-
-    def launches_per_step(self, batch: int) -> int:
-        return self._L.bt_model_launches_per_step(self._h, batch)
-
-    def next_dev(self):
-        torch = _torch()
-        return _wrap_dev(self._L.bt_model_next(self._h), (self.max_batch,), torch.int32, self.device)
-
-    def logits_dev(self):
-        torch = _torch()
-        return _wrap_dev(self._L.bt_model_logits(self._h), (self.max_batch, self.cfg.vocab_size),
-                         torch.float32, self.device)
 
     def ttt_state(self, layer: int):
         torch = _torch()
@@ -416,13 +483,118 @@ class BitLlama:
         return QuantizedKVCache(c.max_position_embeddings, self.max_batch, c.n_kv_heads // max(self.tp_size, 1),
                                 c.hidden_dim // c.n_heads, self.device, _borrowed=p)
 
-    def __del__(self):
-        try:
-            if getattr(self, "_h", None):
-                self._L.bt_model_destroy(self._h)
-                self._h = None
-        except Exception:
-            pass
+
+class LayeredLM(DeviceModel):
+    """A decoder given as a list of layers (layered.py): dense projections, a mixer per layer, caches and recurrent
+    states per layer behind the same step, prefill and pick as `BitLlama`.  dtype "bfloat16" or "float32"."""
+
+    def __init__(self, cfg, max_batch: int = 1, device: int = 0, dtype: str = "bfloat16", max_seq_len: int | None = None):
+        self._L = _bind()
+        self.cfg, self.max_batch, self.device, self.dtype = cfg, max_batch, device, dtype
+        self.max_seq_len = min(max_seq_len or cfg.max_positions, cfg.max_positions)
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"dtype {dtype!r} is neither bfloat16 nor float32")
+        cc = _CLayersConfig(cfg.vocab_size, cfg.width, len(cfg.layers), cfg.max_positions, self.max_seq_len, max_batch,
+                            cfg.norm_eps, int(cfg.norm_one_plus), BT_F32 if dtype == "float32" else BT_BF16)
+        lc = (_CLayerConfig * len(cfg.layers))(*[_CLayerConfig(*[getattr(layer, name) for name, _ in _CLayerConfig._fields_])
+                                                 for layer in cfg.layers])
+        self._h = C.c_void_p()
+        check(self._L.bt_model_create_layers(C.byref(self._h), C.byref(cc), lc, device))
+
+    def set_tensor(self, kind: int, data: np.ndarray):
+        data = np.ascontiguousarray(data, np.float32)
+        check(self._L.bt_model_set_tensor(self._h, kind, 0, data.ctypes.data, data.size))
+
+    def set_layer_tensor(self, layer: int, kind: int, data: np.ndarray):
+        data = np.ascontiguousarray(data, np.float32)
+        check(self._L.bt_model_set_layer_tensor(self._h, layer, kind, data.ctypes.data, data.size))
+
+    def set_trace(self, on: bool = True, rows: int = 0) -> None:
+        """Keep the residual stream after every layer of the following steps (rows: see BitLlama.set_trace)."""
+        torch = _torch()
+        if on:
+            self._trace_rows = max(rows, self.max_batch)
+            n = self._L.bt_model_trace_floats(self._h, self._trace_rows)
+            self._trace = torch.zeros(n, dtype=torch.float32, device=f"cuda:{self.device}")
+            check(self._L.bt_model_set_trace(self._h, _ptr(self._trace), self._trace_rows))
+        else:
+            check(self._L.bt_model_set_trace(self._h, None, 0))
+
+    def read_trace(self, rows: int) -> np.ndarray:
+        """[layers, rows, width] of the last traced step or prefill (rows ordered [sequence][token])."""
+        torch = _torch()
+        torch.cuda.synchronize(self.device)
+        return self._trace.cpu().numpy().reshape(len(self.cfg.layers), self._trace_rows, self.cfg.width)[:, :rows].copy()
+
+    def kv_rows(self, layer: int, b: int, t_len: int):
+        """Cached keys and values of one sequence, f32 [kv_heads, t_len, dim] and [kv_heads, t_len, vdim]."""
+        p = self._L.bt_model_kv_cache(self._h, layer)
+        c = self.cfg.layers[layer]
+        k = np.zeros((c.kv_heads, t_len, c.dim), np.float32)
+        v = np.zeros((c.kv_heads, t_len, c.vdim), np.float32)
+        check(self._L.bt_kv_export_dense(p, b, t_len, k.ctypes.data, v.ctypes.data))
+        return k, v
+
+    def load_kv_rows(self, layer: int, b: int, k: np.ndarray, v: np.ndarray) -> None:
+        k, v = np.ascontiguousarray(k, np.float32), np.ascontiguousarray(v, np.float32)
+        check(self._L.bt_kv_import_dense(self._L.bt_model_kv_cache(self._h, layer), b, k.shape[1], k.ctypes.data, v.ctypes.data))
+
+    def recurrent_state(self, layer: int):
+        """(state, convolution ring) of a recurrent layer as device views, None for attention layers."""
+        torch = _torch()
+        n, r = C.c_int64(0), C.c_int64(0)
+        p = self._L.bt_model_recurrent_state(self._h, layer, C.byref(n))
+        q = self._L.bt_model_conv_ring(self._h, layer, C.byref(r))
+        if not p:
+            return None
+        c = self.cfg.layers[layer]
+        inner = c.heads * c.vdim
+        return (_wrap_dev(p, (self.max_batch, c.heads, c.vdim, n.value // (self.max_batch * inner)), torch.float32, self.device),
+                _wrap_dev(q, (self.max_batch, c.conv_taps, inner + 2 * c.groups * c.state), torch.float32, self.device))
+
+    def save_memory(self, path: str) -> None:
+        """Caches, recurrent states and the position to a safetensors file, so that the sequences can be resumed without
+        a second prefill (the counterpart of BitLlama.save_memory)."""
+        from .loader import write_safetensors
+        torch = _torch()
+        torch.cuda.synchronize(self.device)
+        t_len, tensors = self.current_pos, {"position": np.array([self.current_pos], np.int32)}
+        for li in range(len(self.cfg.layers)):
+            st = self.recurrent_state(li)
+            if st is not None:
+                tensors[f"state_{li}"], tensors[f"conv_{li}"] = st[0].cpu().numpy(), st[1].cpu().numpy()
+            elif t_len > 0:
+                rows = [self.kv_rows(li, b, t_len) for b in range(self.max_batch)]
+                tensors[f"kv_{li}.k"], tensors[f"kv_{li}.v"] = (np.stack([r[j] for r in rows]) for j in (0, 1))
+        write_safetensors(path, tensors)
+
+    def load_memory(self, path: str) -> None:
+        from .loader import CheckpointError, read_safetensors
+        torch = _torch()
+        tensors = read_safetensors(path)
+        t_len = int(np.array(tensors["position"]).reshape(-1)[0])
+        if not 0 <= t_len < self.max_seq_len:
+            raise CheckpointError(f"{path}: position {t_len} outside 0..{self.max_seq_len - 1}")
+        torch.cuda.synchronize(self.device)
+        for li, c in enumerate(self.cfg.layers):
+            st = self.recurrent_state(li)
+            names = (f"state_{li}", f"conv_{li}") if st is not None else (f"kv_{li}.k", f"kv_{li}.v")
+            if st is None and t_len == 0:
+                continue
+            want = [tuple(x.shape) for x in st] if st is not None else \
+                [(self.max_batch, c.kv_heads, t_len, d) for d in (c.dim, c.vdim)]
+            for name, shape in zip(names, want):
+                if name not in tensors or tuple(tensors[name].shape) != shape:
+                    raise CheckpointError(f"{path}: {name} is missing or not of shape {shape}")
+            data = [np.array(tensors[n], np.float32) for n in names]
+            if st is not None:
+                for dst, a in zip(st, data):
+                    dst.copy_(torch.from_numpy(a).to(dst.device))
+            else:
+                for b in range(self.max_batch):
+                    self.load_kv_rows(li, b, data[0][b], data[1][b])
+        torch.cuda.synchronize(self.device)
+        self.seek(t_len)
 
 
 def tp_unique_id() -> bytes:

@@ -204,6 +204,14 @@ bt_status bt_kv_export(bt_kv_cache* cache, int64_t b, int64_t t_len, uint8_t* k_
  * continues decoding at t_len.  Synchronous. */
 bt_status bt_kv_import(bt_kv_cache* cache, int64_t b, int64_t t_len, const uint8_t* k_q_host,
                        const float* k_s_host, const uint8_t* v_q_host, const float* v_s_host);
+/* An unquantised cache (no reference counterpart) for models with dense projections: rows of k_dim / v_dim values in
+ * BT_BF16 or BT_F32 per (sequence, KV head, position).  reset and destroy are shared with the Q8 form; the entry points
+ * that speak Q8 refuse it.  export / import move positions [0, t_len) of sequence b as f32 [n_kv, t_len, dim]
+ * (either may be NULL); synchronous. */
+bt_status bt_kv_create_dense(bt_kv_cache** out, int64_t batch, int64_t n_kv_heads, int64_t k_dim, int64_t v_dim,
+                             int64_t max_seq_len, bt_dtype dtype, int device);
+bt_status bt_kv_export_dense(bt_kv_cache* cache, int64_t b, int64_t t_len, float* k_host, float* v_host);
+bt_status bt_kv_import_dense(bt_kv_cache* cache, int64_t b, int64_t t_len, const float* k_host, const float* v_host);
 /* QuantizedKVCache::append (RE/layers/kv_cache.rs:50-92) on its own, one new token per sequence:
  * k_dev, v_dev [batch, n_kv_heads, head_dim] f32 (keys already rotated, as the caller at
  * RE/layers/attention.rs:180-196 passes them) are quantised (RE/layers/kv_cache.rs:95-119) into row
@@ -254,7 +262,8 @@ typedef enum {
     BT_T_LM_HEAD,     /* [vocab, hidden], dense (RE/model/llama.rs:23) */
     BT_T_NORM_F,      /* [hidden] */
     BT_T_NORM1,       /* per layer [hidden] */
-    BT_T_NORM2
+    BT_T_NORM2,
+    BT_T_POS          /* [max_positions, width], learned positions of a layer-list model */
 } bt_tensor_kind;
 
 /* BitLlama::load (RE/model/llama.rs:37-158) split into create / set_* / finalize so that
@@ -360,6 +369,77 @@ bt_kv_cache* bt_model_kv_cache(bt_model* m, int layer);
  * Not available on tensor-parallel models (BT_ERR_ARG). */
 bt_status bt_model_prefill(bt_model* m, const int32_t* tokens_host, int batch, int n_tokens, int ttt_chunk,
                            float* logits_host, int32_t* next_host);
+
+/* The same with the logits of chosen tokens: want_host[n_want] are indices into the n_tokens new ones (the same for
+ * every sequence); logits_host [batch][n_want][vocab].  n_want may be 0. */
+bt_status bt_model_prefill_logits(bt_model* m, const int32_t* tokens_host, int batch, int n_tokens, int ttt_chunk,
+                                  const int32_t* want_host, int n_want, float* logits_host);
+
+/* ---- models given as a list of layers (no reference counterpart) ---------------------------------------------------
+ * A decoder with dense 16-bit projections whose layers each name a mixer (softmax attention or a state-space recurrence)
+ * and, optionally, a dense feed-forward.  Every sublayer reads the residual stream x as it is and adds its normed
+ * output: x <- x + rmsnorm(sublayer(x)) * norm.  It is a bt_model like the others: set tensors, finalize, then
+ * bt_model_prefill / bt_model_forward_one / bt_model_step_dev / bt_model_reset / bt_model_set_trace (the trace then
+ * holds [rows, width] per layer, the residual stream after it).  Constants are parameters of the layer, so that one
+ * mechanism can be switched off or shared by another design. */
+typedef enum { BT_MIX_ATTENTION = 0, BT_MIX_SSM = 1 } bt_mixer_kind;
+typedef enum { BT_MLP_NONE = 0, BT_MLP_DENSE_RELU2 = 1 } bt_mlp_kind; /* W_down relu(W_up x)^2 */
+
+typedef struct {
+    int mixer;            /* bt_mixer_kind */
+    int heads;            /* query heads / heads of the recurrence */
+    int vdim;             /* value size per head */
+    /* attention: scores (q . k) * scale, then softcap * tanh(score / softcap), softmax over positions <= own */
+    int kv_heads;
+    int dim;              /* query / key size per head */
+    int qk_norm;          /* RMS norm over the whole query and the whole key projection, plain weights */
+    int sink;             /* a learned exp(sink_h) in the softmax denominator */
+    int v_mix;            /* v <- (1 - vmix) v + vmix v_first in every such layer but the first, v_first its values */
+    float scale;
+    float softcap;        /* 0: none */
+    float q_temp_coef;    /* q *= 1 + coef * ln(floor((p + 1) / every) + 1); 0: none */
+    double q_temp_every;
+    /* recurrence: S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x; dt = softplus(. + dt_bias); causal convolution
+     * and silu in front of x, B, C; y * silu(z), RMS norm in norm_groups equal parts, output projection */
+    int state;            /* 1..256 */
+    int groups;           /* B and C are shared by heads / groups heads */
+    int conv_taps;
+    int norm_groups;
+    /* feed-forward */
+    int mlp;              /* bt_mlp_kind */
+    int ff;
+} bt_layer_config;
+
+typedef struct {
+    int vocab_size;
+    int width;
+    int num_layers;
+    int max_positions;    /* rows of the learned position table; 0: none */
+    int max_seq_len;      /* positions the caches hold (<= max_positions when there is a table) */
+    int max_batch;        /* 1..64 */
+    float norm_eps;
+    int norm_one_plus;    /* the layer norms and the final norm multiply by 1 + w */
+    int dtype;            /* BT_BF16: bf16 products with f32 accumulation and a bf16 cache; BT_F32: 32-bit throughout */
+} bt_layers_config;
+
+bt_status bt_model_create_layers(bt_model** out, const bt_layers_config* cfg, const bt_layer_config* layers, int device);
+
+typedef enum {
+    BT_LT_NORM1 = 0, BT_LT_NORM2,                                /* [width] */
+    BT_LT_Q, BT_LT_K, BT_LT_V, BT_LT_O,                          /* [out, in] */
+    BT_LT_Q_NORM, BT_LT_K_NORM, BT_LT_SINK, BT_LT_VMIX,          /* [heads dim], [kv_heads dim], [heads], scalar */
+    BT_LT_SSM_IN,                                                /* [2 heads vdim + 2 groups state + heads, width]: z x B C dt */
+    BT_LT_SSM_CONV, BT_LT_SSM_CONV_B,                            /* [channels, taps], last column = current token; [channels] */
+    BT_LT_SSM_DT_BIAS, BT_LT_SSM_A_LOG, BT_LT_SSM_D,             /* [heads] */
+    BT_LT_SSM_NORM, BT_LT_SSM_O,                                 /* [heads vdim]; [width, heads vdim] */
+    BT_LT_MLP_UP, BT_LT_MLP_DOWN                                 /* [ff, width]; [width, ff] */
+} bt_layer_tensor;
+/* Matrices are kept in bf16 (f32 models compute with exactly those values), vectors in f32. */
+bt_status bt_model_set_layer_tensor(bt_model* m, int layer, bt_layer_tensor kind, const float* data_host, int64_t n_elem);
+/* Recurrent state of one layer (NULL for attention layers): f32 [max_batch, heads, vdim, state_pad] and the ring of the
+ * convolution's last inputs, f32 [max_batch, taps, channels], slot = position % taps.  Sizes in floats. */
+float* bt_model_recurrent_state(bt_model* m, int layer, int64_t* n_floats);
+float* bt_model_conv_ring(bt_model* m, int layer, int64_t* n_floats);
 
 /* Inspection aid: the tensors between the calls of BitLlamaBlock::forward (RE/model/block.rs:87-134).
  * While a trace buffer is set, every decode step runs launch by launch (no graph replay) and copies, per layer,

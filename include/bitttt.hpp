@@ -163,9 +163,12 @@ private:
 class BitLlama {
 public:
     BitLlama(const bt_model_config& cfg, int device) { check(bt_model_create(&h_, &cfg, device)); }
+    // a model given as a list of layers: weights through set_tensor and set_layer_tensor
+    BitLlama(const bt_layers_config& cfg, const bt_layer_config* layers, int device) { check(bt_model_create_layers(&h_, &cfg, layers, device)); }
     BitLlama(const BitLlama&) = delete;
     BitLlama& operator=(const BitLlama&) = delete;
     ~BitLlama() { if (h_) bt_model_destroy(h_); }
+    void set_layer_tensor(int layer, bt_layer_tensor kind, const float* data, int64_t n_elem) { check(bt_model_set_layer_tensor(h_, layer, kind, data, n_elem)); }
     void set_linear(int layer, bt_weight_kind kind, const uint8_t* packed, int64_t n_out, int64_t k_in, int n_bases, const float* scales) {
         check(bt_model_set_linear_bases(h_, layer, kind, packed, n_out, k_in, n_bases, scales));
     }
@@ -180,6 +183,10 @@ public:
     // the CLI's prefill loop (RE/model/llama.rs:495-498) as one batched call
     void prefill(const int32_t* tokens, int batch, int n_tokens, float* logits, int32_t* next, int ttt_chunk = 1) {
         check(bt_model_prefill(h_, tokens, batch, n_tokens, ttt_chunk, logits, next));
+    }
+    // the same with the logits of chosen tokens, [batch][n_want][vocab]
+    void prefill_logits(const int32_t* tokens, int batch, int n_tokens, const int32_t* want, int n_want, float* logits, int ttt_chunk = 1) {
+        check(bt_model_prefill_logits(h_, tokens, batch, n_tokens, ttt_chunk, want, n_want, logits));
     }
     bt_model* handle() const { return h_; }
 

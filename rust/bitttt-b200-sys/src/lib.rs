@@ -59,6 +59,43 @@ pub mod ffi {
         pub tp_size: c_int,
     }
 
+    #[repr(C)]
+    #[derive(Clone, Copy, Debug)]
+    pub struct bt_layer_config {
+        pub mixer: c_int,
+        pub heads: c_int,
+        pub vdim: c_int,
+        pub kv_heads: c_int,
+        pub dim: c_int,
+        pub qk_norm: c_int,
+        pub sink: c_int,
+        pub v_mix: c_int,
+        pub scale: c_float,
+        pub softcap: c_float,
+        pub q_temp_coef: c_float,
+        pub q_temp_every: c_double,
+        pub state: c_int,
+        pub groups: c_int,
+        pub conv_taps: c_int,
+        pub norm_groups: c_int,
+        pub mlp: c_int,
+        pub ff: c_int,
+    }
+
+    #[repr(C)]
+    #[derive(Clone, Copy, Debug)]
+    pub struct bt_layers_config {
+        pub vocab_size: c_int,
+        pub width: c_int,
+        pub num_layers: c_int,
+        pub max_positions: c_int,
+        pub max_seq_len: c_int,
+        pub max_batch: c_int,
+        pub norm_eps: c_float,
+        pub norm_one_plus: c_int,
+        pub dtype: c_int,
+    }
+
     pub type bt_weight_kind = c_int; // BT_W_Q = 0 .. BT_W_TTT_UP = 8
     pub type bt_tensor_kind = c_int; // BT_T_EMBED = 0 .. BT_T_NORM2 = 4
 
@@ -101,6 +138,12 @@ pub mod ffi {
                             v_q_host: *mut u8, v_s_host: *mut c_float) -> bt_status;
         pub fn bt_kv_import(cache: *mut bt_kv_cache, b: i64, t_len: i64, k_q_host: *const u8, k_s_host: *const c_float,
                             v_q_host: *const u8, v_s_host: *const c_float) -> bt_status;
+        pub fn bt_kv_create_dense(out: *mut *mut bt_kv_cache, batch: i64, n_kv_heads: i64, k_dim: i64, v_dim: i64,
+                                  max_seq_len: i64, dtype: bt_dtype, device: c_int) -> bt_status;
+        pub fn bt_kv_export_dense(cache: *mut bt_kv_cache, b: i64, t_len: i64, k_host: *mut c_float,
+                                  v_host: *mut c_float) -> bt_status;
+        pub fn bt_kv_import_dense(cache: *mut bt_kv_cache, b: i64, t_len: i64, k_host: *const c_float,
+                                  v_host: *const c_float) -> bt_status;
         pub fn bt_kv_append(cache: *mut bt_kv_cache, k_dev: *const c_float, v_dev: *const c_float, pos_dev: *const i32,
                             batch: i64, stream: *mut c_void) -> bt_status;
         pub fn bt_attn_decode(cache: *mut bt_kv_cache, qkv_dev: *const c_float, pos_dev: *const i32, batch: i64, n_heads: i64,
@@ -135,6 +178,15 @@ pub mod ffi {
         pub fn bt_model_seek(m: *mut bt_model, pos: c_int) -> bt_status;
         pub fn bt_model_ttt_state(m: *mut bt_model, layer: c_int) -> *mut c_float;
         pub fn bt_model_kv_cache(m: *mut bt_model, layer: c_int) -> *mut bt_kv_cache;
+        pub fn bt_model_prefill_logits(m: *mut bt_model, tokens_host: *const i32, batch: c_int, n_tokens: c_int,
+                                       ttt_chunk: c_int, want_host: *const i32, n_want: c_int,
+                                       logits_host: *mut c_float) -> bt_status;
+        pub fn bt_model_create_layers(out: *mut *mut bt_model, cfg: *const bt_layers_config, layers: *const bt_layer_config,
+                                      device: c_int) -> bt_status;
+        pub fn bt_model_set_layer_tensor(m: *mut bt_model, layer: c_int, kind: c_int, data_host: *const c_float,
+                                         n_elem: i64) -> bt_status;
+        pub fn bt_model_recurrent_state(m: *mut bt_model, layer: c_int, n_floats: *mut i64) -> *mut c_float;
+        pub fn bt_model_conv_ring(m: *mut bt_model, layer: c_int, n_floats: *mut i64) -> *mut c_float;
         pub fn bt_model_trace_floats(m: *const bt_model, rows: c_int) -> i64;
         pub fn bt_model_set_trace(m: *mut bt_model, trace_dev: *mut c_float, rows: c_int) -> bt_status;
         pub fn bt_model_ternary_bytes(m: *const bt_model) -> i64;
