@@ -352,6 +352,168 @@ def run_cpu_cases(bt, device):
                               "model (quantised pipeline) on the host cores"}), flush=True)
 
 
+def layered_bench_config(lay, size):
+    """Layers of the sizes a real model has: four attention layers with a feed-forward and four recurrent layers."""
+    w, h, kv, d, ff, sh, groups = {"2048": (2048, 32, 4, 64, 5632, 64, 1), "4096": (4096, 32, 8, 128, 14336, 128, 8)}[size]
+    att = lay.LayerConfig(lay.MIX_ATTENTION, h, d, kv_heads=kv, dim=d, qk_norm=1, sink=1, v_mix=1, scale=d ** -0.5, softcap=30.0,
+                          q_temp_coef=0.1, q_temp_every=1024, mlp=lay.MLP_DENSE_RELU2, ff=ff)
+    rec = lay.LayerConfig(lay.MIX_SSM, sh, 64, state=128, groups=groups, conv_taps=4, norm_groups=groups)
+    return lay.LayersConfig(32000, w, 4096, 1e-5, True, [rec, att] * 4)
+
+
+def layered_bench_tensors(lay, cfg):
+    """Random values of sensible size; every matrix is cut from one block (the device copies stay distinct)."""
+    rng = np.random.default_rng(5)
+    block = (rng.normal(0, 1, 1 << 22)).astype(np.float32)
+    out = {}
+    for name, shape, _, _ in lay.tensor_shapes(cfg):
+        n = int(np.prod(shape, dtype=np.int64))
+        if len(shape) == 2 and "conv" not in name:
+            out[name] = (np.resize(block, n) / np.float32(np.sqrt(shape[1]) if name not in ("embed", "pos") else 1.0)).reshape(shape)
+        elif name.endswith("A_log"):
+            out[name] = rng.uniform(-3, 0, shape).astype(np.float32)
+        elif name.endswith(("q.norm", "k.norm", "mix.norm")):
+            out[name] = np.ones(shape, np.float32)
+        elif name.endswith("vmix"):
+            out[name] = np.float32(0.3)
+        else:
+            out[name] = np.resize(0.1 * block, n).reshape(shape)
+    return out
+
+
+def graph_us(torch, fn, reps=10):
+    """Microseconds of one call of `fn`, replayed as a CUDA graph (three replays as warm-up)."""
+    fn()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    side = torch.cuda.Stream()
+    with torch.cuda.stream(side):
+        with torch.cuda.graph(g, stream=side):
+            fn()
+    for _ in range(3):
+        g.replay()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(reps):
+        g.replay()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) * 1e3 / reps
+
+
+def run_layered(bt, device, context):
+    """--layered: the layer-list design beside the ternary model of the same width.  Per size one line for each model:
+    decode rate at batch 1 and 64, prefill rate, and per kind of kernel microseconds, achieved rate and its share of the
+    measured roofline (weights and states larger than L2 rotate through the layers)."""
+    import torch
+    lay = importlib.import_module("bit-ttt-engine_b200.layered")
+    syn = importlib.import_module("bit-ttt-engine_b200.synthetic")
+    hbm, bf16_tf, kind = measured_peaks()
+    tm = Timer(torch, None, 1, torch.device(f"cuda:{device}"))
+    rng = np.random.default_rng(3)
+    fma_tf = 148 * 128 * 2 * 1.965e9 / 1e12  # f32 FMA units at the nominal clock
+    for size in ("2048", "4096"):
+        cfg = layered_bench_config(lay, size)
+        t = layered_bench_tensors(lay, cfg)
+        W = cfg.width
+        sampler = ClockSampler(device)
+        sampler.start()
+        line = {"layered": "gufotar", "width": W, "layers": len(cfg.layers), "context": context, "dtype": "bf16", "data": "synthetic", "peak_kind": kind}
+        att, rec = cfg.layers[1], cfg.layers[0]
+        inner, ch = rec.heads * rec.vdim, rec.heads * rec.vdim + 2 * rec.groups * rec.state
+        n_in = {"att": att.heads * att.dim + att.kv_heads * (att.dim + att.vdim), "rec": inner + ch + rec.heads}
+        params = 4 * W * (n_in["att"] + att.heads * att.vdim + 2 * att.ff + n_in["rec"] + inner)
+        part_params = {1: 4 * W * (n_in["att"] + n_in["rec"]), 4: 4 * W * (att.heads * att.vdim + inner), 8: 4 * W * att.ff, 16: 4 * W * att.ff}
+        names = {1: "input projections", 2: "mixers", 4: "output projections", 8: "up", 16: "down", 32: "norms"}
+        for B in (1, 64):
+            m = lay.build_layered(cfg, t, max_batch=B, max_seq_len=context + 256, device=device)
+            prompt = rng.integers(0, cfg.vocab_size, size=(B, context)).astype(np.int32)
+            m.prefill(prompt[:, :64], want_logits=False)
+            m.reset_kv_cache()
+            m.prefill(prompt[:, :2048 // B], want_logits=False)
+            m.reset_kv_cache()
+            torch.cuda.synchronize()
+            t0 = time.perf_counter()
+            m.prefill(prompt, want_logits=False)
+            dt = time.perf_counter() - t0
+            ms, _ = time_decode(m, cfg, B, 64, 4, context, tm, rng)
+            kv_bytes = 4 * B * 2 * att.kv_heads * (context + 1) * (att.dim + att.vdim)
+            state_bytes = 4 * B * 2 * 4 * inner * rec.state
+            parts = {}
+            for part, name in names.items():
+                us = graph_us(torch, lambda: m.enqueue_parts(B, 1, part))
+                byts = 2 * part_params[part] if part in part_params else (kv_bytes + state_bytes if part == 2 else 0)
+                parts[name] = {"us": us, "GBps": byts / us / 1e3, "hbm_frac": byts / us / 1e3 / hbm}
+            line[f"batch{B}"] = {"decode_tokens_per_s": B * 64 / (ms * 1e-3), "ms_per_step": ms / 64, "prefill_tokens_per_s": B * context / dt,
+                                 "weight_GB": 2 * params / 1e9, "decode_kernels_per_step": parts, "launches_per_step": m.launches_per_step(B)}
+            if B == 1:
+                # a prefill chunk of 2048 tokens: the launches of each kind alone
+                n = min(2048, context)
+                m.seek(0)
+                pre = {}
+                for part, name in names.items():
+                    us = graph_us(torch, lambda: m.enqueue_parts(1, n, part), reps=3)
+                    fl = 2.0 * n * part_params[part] if part in part_params else 0
+                    pre[name] = {"us": us, "TFLOPs": fl / us / 1e6, "tensor_frac": fl / us / 1e6 / bf16_tf}
+                line["prefill_chunk_kernels"] = {"tokens": n, **pre}
+            del m
+            # the two mixers apart: models of one kind of layer
+            for what, layers in (("attention", [att] * 4), ("recurrence", [rec] * 4)):
+                c2 = lay.LayersConfig(64, W, cfg.max_positions, 1e-5, True, layers)
+                m = lay.build_layered(c2, layered_bench_tensors(lay, c2), max_batch=B, max_seq_len=context + 256, device=device)
+                n = min(2048 // B, context)
+                m.prefill(rng.integers(0, 64, size=(B, n)).astype(np.int32), want_logits=False)
+                pre_us = None
+                if B == 1:
+                    m.seek(0)
+                    pre_us = graph_us(torch, lambda: m.enqueue_parts(1, n, 2), reps=3) / 4
+                m.seek(context)
+                us = graph_us(torch, lambda: m.enqueue_parts(B, 1, 2)) / 4
+                byts = (kv_bytes if what == "attention" else state_bytes) / 4
+                d = {"decode_us_per_layer": us, "hbm_frac": byts / us / 1e3 / hbm}
+                if pre_us:
+                    fl = 2.0 * n * n / 2 * att.heads * (att.dim + att.vdim) if what == "attention" else 5.0 * n * inner * rec.state
+                    d.update(prefill_us_per_layer=pre_us, prefill_TFLOPs=fl / pre_us / 1e6)
+                    d["prefill_frac"] = fl / pre_us / 1e6 / (bf16_tf if what == "attention" else fma_tf)
+                line[f"batch{B}"][what] = d
+                del m
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+        del t
+        # ---- the ternary model of the same width ----
+        line = {"layered": "ternary model beside it", "width": W, "context": context}
+        shape = "8b" if size == "4096" else "tinyllama"
+        for B in (1, 64):
+            tcfg, _, m = build_8b(bt, syn, B, context + 256, device=device, num_layers=8, shape=shape)
+            pf = fill_context(m, tcfg, B, context, rng, tm)
+            ms, _ = time_decode(m, tcfg, B, 64, 4, context, tm, rng)
+            us, n_l = time_products(m, B, True, torch)
+            us_att, att_bytes = time_attention(bt, tcfg, B, context, torch)
+            line[f"batch{B}"] = {"decode_tokens_per_s": B * 64 / (ms * 1e-3), "ms_per_step": ms / 64, "prefill_tokens_per_s": pf["tokens_per_s"],
+                                 "products_us_per_step": us, "products_hbm_frac": product_bytes(tcfg, syn, m, B) / us / 1e3 / hbm,
+                                 "attention_us_per_layer": us_att, "attention_hbm_frac": att_bytes / us_att / 1e3 / hbm}
+            del m
+        # like kernels: a ternary product over 2048 tokens; the fast-weight update on as many bytes of state as the recurrence
+        n, k = tcfg.intermediate_dim, W
+        lin = bt.BitLinear.from_packed(rng.integers(0, 256, size=(n, k // 4), dtype=np.uint8), [0.016], n, k, device=device)
+        x = torch.randn(2048, k, device="cuda").bfloat16()
+        us = graph_us(torch, lambda: lin.forward(x))
+        line["ternary_product_2048_tokens"] = {"us": us, "int8_TOPs": 2.0 * 2048 * n * k / us / 1e6,
+                                               "frac_of_2x_bf16_peak": 2.0 * 2048 * n * k / us / 1e6 / (2 * bf16_tf)}
+        for B, tl in ((1, 1), (64, 1), (1, 2048)):
+            states = B * inner * rec.state // 4096
+            w = torch.zeros(states, 64, 64, device="cuda")
+            f = torch.randn(states, tl, 64, device="cuda")
+            us = graph_us(torch, lambda: bt.ttt_update(w, f, 0.01, 16 if tl > 1 else 1), reps=3)
+            byts = states * (2 * 64 * 64 * 4 + 2 * tl * 64 * 4)
+            line[f"fast_weight_update_{states}_states_{tl}_tokens"] = {
+                "us": us, "hbm_frac": byts / us / 1e3 / hbm, "TFLOPs": 4.0 * tl * states * 4096 / us / 1e6,
+                "fma_frac": 4.0 * tl * states * 4096 / us / 1e6 / fma_tf}
+            del w, f
+        print(json.dumps(line), flush=True)
+
+
 def run_reference_arm(args, rank):
     """--impl reference: the reference's CPU implementation of the path.  The reference is a
     Rust workspace with no Rust toolchain available here, so the timed code is the CPU port
@@ -573,6 +735,9 @@ def main():
     ap.add_argument("--sweep", action="store_true",
                     help="BitLinear shape sweep (K,N in {4096x4096, 4096x14336, 14336x4096, 4096x128256}, "
                          "M in {1, 8, 64, 512, 4096}, bf16 activations) plus the TTT update: one JSON line per point")
+    ap.add_argument("--layered", action="store_true",
+                    help="the layer-list design (attention and recurrent layers, bf16) beside the ternary model at two widths: "
+                         "prefill and decode rates and per-kernel roofline shares, one JSON line per model and width")
     ap.add_argument("--profile-case", type=int, default=0, metavar="BATCH",
                     help="small case for a profiler, not a benchmark: --layers blocks of the 8B shape, BATCH sequences, "
                          "the context filled by the batched prefill, then 3 decode steps; prints a line marked profile_case")
@@ -604,6 +769,9 @@ def main():
     syn = importlib.import_module("bit-ttt-engine_b200.synthetic")
     if args.sweep:
         run_sweep(bt, local_rank)
+        return
+    if args.layered:
+        run_layered(bt, local_rank, args.context)
         return
 
     if args.profile_case:

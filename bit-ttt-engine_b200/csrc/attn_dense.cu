@@ -30,20 +30,9 @@ __device__ __forceinline__ float to_cache<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 to_cache<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
-// eight consecutive cache values as they are loaded (16 or 32 bytes), and widened
+// eight consecutive cache values as they are loaded
 template <typename T>
 struct Raw8;
-template <>
-struct Raw8<__nv_bfloat16> {
-    uint4 u;
-    __device__ __forceinline__ void load(const __nv_bfloat16* p) { u = *reinterpret_cast<const uint4*>(p); }
-    __device__ __forceinline__ void zero() { u = make_uint4(0, 0, 0, 0); }
-    __device__ __forceinline__ void widen(float (&v)[8]) const {
-        const uint32_t q[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-        for (int j = 0; j < 4; ++j) { v[2 * j] = __uint_as_float(q[j] << 16); v[2 * j + 1] = __uint_as_float(q[j] & 0xffff0000u); }
-    }
-};
 template <>
 struct Raw8<float> {
     float4 a, b;
@@ -112,9 +101,70 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const DenseAttn a) {
     }
 }
 
+// The end of a span kernel: every CTA of the cluster holds (maximum, sum, un-normed output [h][c] at o_s[h * W + c]) of
+// its span for nr heads; rank 0 reads them all, adds the sink and writes the rows of `head0 ..`.
+__device__ __forceinline__ void merge_spans(const DenseAttn& a, float* m_s, float* l_s, float* o_s, int W, int nr, int head0,
+                                            int64_t r, int split, int splits, int threads, const ActOut& out) {
+    cg::cluster_group cluster = cg::this_cluster();
+    if (splits > 1) cluster.sync(); else __syncthreads();
+    if (split == 0) {
+        for (int i = threadIdx.x; i < nr * a.dv; i += threads) {
+            const int h = i / a.dv, c = i - h * a.dv, head = head0 + h;
+            float ms[8], ls[8], os[8];
+#pragma unroll
+            for (int s = 0; s < 8; ++s) {  // all remote reads in flight together
+                ms[s] = -INFINITY; ls[s] = os[s] = 0.0f;
+                if (s < splits) {
+                    ms[s] = *(splits > 1 ? cluster.map_shared_rank(m_s, s) + h : m_s + h);
+                    ls[s] = *(splits > 1 ? cluster.map_shared_rank(l_s, s) + h : l_s + h);
+                    os[s] = *(splits > 1 ? cluster.map_shared_rank(o_s, s) + h * W + c : o_s + h * W + c);
+                }
+            }
+            const float sink = a.sink ? a.sink[head] : -INFINITY;
+            float m = sink;
+#pragma unroll
+            for (int s = 0; s < 8; ++s) m = fmaxf(m, ms[s]);
+            float den = a.sink ? expf(sink - m) : 0.0f, num = 0.0f;
+#pragma unroll
+            for (int s = 0; s < 8; ++s) {
+                const float f = expf(ms[s] - m);  // an empty span: exp(-inf) = 0
+                den = fmaf(ls[s], f, den);
+                num = fmaf(os[s], f, num);
+            }
+            const float v = num / den;
+            const int col = head * a.dv + c;
+            if (out.tiles) *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, col, out.m_pad)) = __float2bfloat16_rn(v);
+            else out.rows[r * out.ld + col] = v;
+        }
+    }
+    if (splits > 1) cluster.sync();  // no CTA leaves while its sums are being read
+}
+// spans per query position: enough CTAs for the device, no span below 64 positions
+int span_splits(const DenseAttn& a, int64_t groups) {
+    int splits = 1;
+    while (splits < 8 && groups * splits * 2 <= 2ll * a.sm_count && splits * 64 < a.kv.max_seq) splits *= 2;
+    return splits;
+}
+template <typename... KArgs, typename... Args>
+cudaError_t launch_spans(void (*kernel)(KArgs...), dim3 grid, int threads, size_t smem, cudaStream_t s, bool pdl, Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3((unsigned)threads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = grid.x; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
+}
+
 // ---------------------------------------------------------------------------------------
 // one query position per CTA group: (row, KV head, up to 8 of its query heads), the positions cut into spans over the
-// CTAs of a cluster
+// CTAs of a cluster.  This form computes in f32 on the FMA units (32-bit models).
 // ---------------------------------------------------------------------------------------
 // A CTA takes its span in tiles of 128 positions.  Scores: four lanes share a key (pieces of 8 dimensions in turn), two
 // keys per lane, all heads of the group on the widened key.  Softmax: a warp per head over the tile.  Values: LPV lanes
@@ -295,56 +345,21 @@ __global__ void __launch_bounds__(kSpanThreads) attn_span_kernel(const DenseAttn
         for (int w = 0; w < 8; ++w) v += o_s[w * NR * W + i];
         o_s[i] = v;  // row 0 of the eight: read and written by this thread only
     }
-    cg::cluster_group cluster = cg::this_cluster();
-    if (splits > 1) cluster.sync(); else __syncthreads();
-    if (split == 0) {
-        for (int i = threadIdx.x; i < nr * dv; i += kSpanThreads) {
-            const int h = i / dv, c = i - h * dv, head = g * rep + h0 + h;
-            const float sink = a.sink ? a.sink[head] : -INFINITY;
-            float m = sink;
-            for (int s = 0; s < splits; ++s) m = fmaxf(m, *(splits > 1 ? cluster.map_shared_rank(m_s, s) + h : m_s + h));
-            float den = a.sink ? expf(sink - m) : 0.0f, num = 0.0f;
-            for (int s = 0; s < splits; ++s) {
-                const float* ms = splits > 1 ? cluster.map_shared_rank(m_s, s) : m_s;
-                const float* ls = splits > 1 ? cluster.map_shared_rank(l_s, s) : l_s;
-                const float* os = splits > 1 ? cluster.map_shared_rank(o_s, s) : o_s;
-                const float f = expf(ms[h] - m);  // an empty span: exp(-inf) = 0
-                den = fmaf(ls[h], f, den);
-                num = fmaf(os[h * W + c], f, num);
-            }
-            const float v = num / den;
-            const int col = head * dv + c;
-            if (out.tiles) *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, col, out.m_pad)) = __float2bfloat16_rn(v);
-            else out.rows[r * out.ld + col] = v;
-        }
-    }
-    if (splits > 1) cluster.sync();  // no CTA leaves while its sums are being read
+    merge_spans(a, m_s, l_s, o_s, W, nr, g * rep + h0, r, split, splits, kSpanThreads, out);
 }
 
 template <typename T, int NR, int LPV>
 cudaError_t span_launch(const DenseAttn& a, bool prepared, const ActOut& out, cudaStream_t s, bool pdl) {
     const int rep = a.heads / a.n_kv, hchunks = (rep + NR - 1) / NR;
     const int64_t groups = (int64_t)a.n_kv * hchunks * a.batch * a.q_rows;
-    int splits = 1;
-    while (splits < 8 && groups * splits * 2 <= 2ll * a.sm_count && splits * 64 < a.kv.max_seq) splits *= 2;
+    const int splits = span_splits(a, groups);
     const size_t smem = ((size_t)NR * a.kv.k_stride + NR * kSpanTile + 24 + 64 + (size_t)8 * NR * LPV * 8) * sizeof(float);
     static PerDeviceOnce once;
     cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_span_kernel<T, NR, LPV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); });
     if (e != cudaSuccess) return e;
     if (smem > 100 * 1024) return cudaErrorInvalidConfiguration;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3((unsigned)splits, (unsigned)(a.n_kv * hchunks), (unsigned)(a.batch * a.q_rows));
-    cfg.blockDim = dim3(kSpanThreads);
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = s;
-    cudaLaunchAttribute attr[2];
-    attr[0].id = cudaLaunchAttributeClusterDimension;
-    attr[0].val.clusterDim.x = (unsigned)splits; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
-    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[1].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = pdl ? 2 : 1;
-    return cudaLaunchKernelEx(&cfg, attn_span_kernel<T, NR, LPV>, a, prepared, splits, out);
+    return launch_spans(attn_span_kernel<T, NR, LPV>, dim3((unsigned)splits, (unsigned)(a.n_kv * hchunks), (unsigned)(a.batch * a.q_rows)),
+                        kSpanThreads, smem, s, pdl, a, prepared, splits, out);
 }
 template <typename T, int NR>
 cudaError_t span_launch_v(const DenseAttn& a, bool prepared, const ActOut& out, cudaStream_t s, bool pdl) {
@@ -368,28 +383,238 @@ cudaError_t span_launch_r(const DenseAttn& a, bool prepared, const ActOut& out, 
 // Rows in shared memory are padded by 16 bytes, so that the eight rows of an ldmatrix fall into different banks.
 constexpr int kTileQ = 64, kTileKeys = 64, kTileThreads = 128;
 
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool live) {
-    const int n = live ? 16 : 0;  // the rest of the 16 bytes is zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack2(float lo, float hi) {
-    __nv_bfloat162 p = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<uint32_t*>(&p);
-}
 // cap * tanh(x / cap) with tanh(u) = 1 - 2 / (e^2u + 1): absolute error of the order of 1e-7 cap
 __device__ __forceinline__ float soft_cap(float x, float two_over_cap, float cap) {
     return cap - __fdividef(2.0f * cap, __expf(x * two_over_cap) + 1.0f);
+}
+
+// ---------------------------------------------------------------------------------------
+// one query position per CTA group on the tensor cores (bf16 cache, decode)
+// ---------------------------------------------------------------------------------------
+// The heads of a group are the rows of the products: rows 0-7 the queries' (softmax weights') bf16 values, rows 8-15 what
+// bf16 left over of them, so that the sum of the two accumulator rows carries 16 significand bits.  Every warp walks its
+// own blocks of 16 positions with its own copy ring, maximum and sums - no CTA barrier inside - and the first blocks are
+// requested before the wait on the projection in front (only the block of the new token has to come after it).
+constexpr int kMmaThreads = 128, kMmaWarps = 4;
+template <int DK, int DV>
+struct MmaCfg {
+    static constexpr int kStages = DK + DV <= 128 ? 4 : (DK + DV <= 256 ? 3 : 2);
+    static constexpr int KS = DK * 2 + 16, VS = DV * 2 + 16;   // bytes per row
+    static constexpr int kStage = 16 * (KS + VS);
+    static constexpr int kRing = kMmaWarps * kStages * kStage;
+    static constexpr int kMerge = kMmaWarps * 8 * DV * 4;       // the warps' outputs, in the ring's place
+    static constexpr size_t kSmem = (size_t)(kRing > kMerge ? kRing : kMerge) + 16 * KS + (64 + 2 * 8 + 2 * kMmaWarps * 8) * 4;
+};
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseAttn a, bool prepared, int splits, const ActOut out) {
+    using Cfg = MmaCfg<DK, DV>;
+    constexpr int S = Cfg::kStages, KS = Cfg::KS, VS = Cfg::VS;
+    extern __shared__ __align__(16) uint8_t tsm[];
+    uint8_t* q_sm = tsm + (Cfg::kRing > Cfg::kMerge ? Cfg::kRing : Cfg::kMerge);   // [16][KS]: 8 rows hi, 8 rows lo
+    float* red = reinterpret_cast<float*>(q_sm + 16 * KS);  // 64
+    float* m_s = red + 64;                                   // [8]
+    float* l_s = m_s + 8;                                    // [8]
+    float* mw_s = l_s + 8;                                   // [4 warps][8]
+    float* lw_s = mw_s + kMmaWarps * 8;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int dk = a.dk, dv = a.dv, ks = a.kv.k_stride, vs = a.kv.v_stride;
+    const int nk = (ks + 15) / 16, nv = (vs + 15) / 16;
+    const int rep = a.heads / a.n_kv, hchunks = (rep + 7) / 8;
+    const int g = blockIdx.y / hchunks, h0 = (blockIdx.y % hchunks) * 8;
+    const int nr = min(8, rep - h0);
+    const int64_t r = blockIdx.z;
+    const int b = (int)(r / a.q_rows), split = blockIdx.x;
+    const int nq = a.heads * dk, nkw = a.n_kv * dk, nvw = a.n_kv * dv;
+    // positions move on long before the kernel in front of this one: they may be read ahead of the wait
+    const int p = a.pos[b] + (int)(r % a.q_rows);
+    const int total = min(p + 1, a.kv.max_seq);
+    const int span = ((total + splits - 1) / splits + 15) / 16 * 16;
+    const int t0 = min(split * span, total), t1 = min(t0 + span, total);
+    __nv_bfloat16* kc = reinterpret_cast<__nv_bfloat16*>(a.kv.k) + ((int64_t)b * a.n_kv + g) * a.kv.max_seq * ks;
+    __nv_bfloat16* vc = reinterpret_cast<__nv_bfloat16*>(a.kv.v) + ((int64_t)b * a.n_kv + g) * a.kv.max_seq * vs;
+    const int blocks = (t1 - t0 + 15) / 16;
+    const bool owner = !prepared && t1 == p + 1 && t0 < t1;    // appends the new token
+    const uint32_t ring = ptx::smem_u32(tsm) + warp * S * Cfg::kStage;
+    const int kp = nk * 2, vp = nv * 2;                          // 16-byte pieces per row
+    auto load = [&](int i) {                                     // this warp's i-th block
+        const int blk = warp + i * kMmaWarps;
+        if (blk < blocks) {
+            const int base = t0 + blk * 16;
+            const uint32_t st = ring + (i % S) * Cfg::kStage;
+            for (int e = lane; e < 16 * kp; e += 32) {
+                const int row = e / kp, c = e - row * kp;
+                const bool live = base + row < t1 && c * 8 < ks;
+                ptx::cp16(st + row * KS + c * 16, live ? kc + (int64_t)(base + row) * ks + c * 8 : kc, live);
+            }
+            for (int e = lane; e < 16 * vp; e += 32) {
+                const int row = e / vp, c = e - row * vp;
+                const bool live = base + row < t1 && c * 8 < vs;
+                ptx::cp16(st + 16 * KS + row * VS + c * 16, live ? vc + (int64_t)(base + row) * vs + c * 8 : vc, live);
+            }
+        }
+    };
+    auto is_new = [&](int i) { return owner && warp + i * kMmaWarps == blocks - 1; };
+    auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+    if (prepared) { ptx::pdl_wait(); }                           // the cache rows come from the kernel in front
+#pragma unroll
+    for (int i = 0; i < S - 1; ++i) { if (!is_new(i)) load(i); commit(); }
+    if (!prepared) ptx::pdl_wait();
+    ptx::pdl_launch_dependents();
+
+    // ---- queries as bf16 hi | lo rows, zero beyond the heads and sizes in use ----
+    float inv_q = 1.0f, inv_k = 1.0f;
+    const float* row = a.qkv + r * a.ld;
+    if (!prepared) {
+        qk_sums(a, row, red, inv_q, inv_k);
+        inv_q *= temperature(a.temp_coef, a.temp_every, p);
+    }
+    const int kw = nk * 16;
+    for (int i = threadIdx.x; i < 8 * kw; i += kMmaThreads) {
+        const int h = i / kw, c = i - h * kw;
+        float v = 0.0f;
+        if (h < nr && c < dk) {
+            const int head = g * rep + h0 + h, s = head * dk + c;
+            v = prepared ? reinterpret_cast<const float*>(a.q_buf)[(r * a.heads + head) * ks + c]
+                         : row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f);
+        }
+        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+        *reinterpret_cast<__nv_bfloat16*>(q_sm + h * KS + c * 2) = hi;
+        *reinterpret_cast<__nv_bfloat16*>(q_sm + (8 + h) * KS + c * 2) = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+    if (owner) {  // (head chunks of one KV head write the same values)
+        for (int c = threadIdx.x; c < ks; c += kMmaThreads) {
+            const int s = g * dk + c;
+            kc[(int64_t)p * ks + c] = __float2bfloat16_rn(c < dk ? row[nq + s] * inv_k * (a.k_norm ? a.k_norm[s] : 1.0f) : 0.0f);
+        }
+        for (int c = threadIdx.x; c < vs; c += kMmaThreads) {
+            const int s = g * dv + c;
+            float v = 0.0f;
+            if (c < dv) {
+                v = row[nq + nkw + s];
+                if (a.v_first_out) a.v_first_out[r * nvw + s] = v;
+                if (a.v_first_in) v = (1.0f - a.v_lambda) * v + a.v_lambda * a.v_first_in[r * nvw + s];
+            }
+            vc[(int64_t)p * vs + c] = __float2bfloat16_rn(v);
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < S - 1; ++i)
+        if (is_new(i)) { load(i); commit(); }
+
+    float o[DV / 8][4];
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[i][j] = 0.0f;
+    float m_run = -INFINITY, l_run = 0.0f;
+    const float two_over_cap = a.softcap > 0.0f ? 2.0f / a.softcap : 0.0f;
+    const uint32_t q_addr = ptx::smem_u32(q_sm) + (lane & 15) * KS + (lane >> 4) * 16;
+    constexpr bool kQRegs = DK <= 128;
+    uint32_t qf[kQRegs ? DK / 16 : 1][4];
+    if (kQRegs) {
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk)
+            if (kk < nk) ptx::ldsm4(qf[kQRegs ? kk : 0], q_addr + kk * 32);
+    }
+    for (int i = 0; warp + i * kMmaWarps < blocks; ++i) {
+        if (is_new(i)) asm volatile("cp.async.wait_group 0;" ::: "memory");
+        else asm volatile("cp.async.wait_group %0;" ::"n"(S - 2) : "memory");
+        __syncwarp();
+        load(i + S - 1);  // into the slot of the block before this one
+        commit();
+        const uint32_t kb = ring + (i % S) * Cfg::kStage, vb = kb + 16 * KS;
+        float s[2][4] = {};
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk)
+            if (kk < nk) {
+                uint32_t kf[4];
+                ptx::ldsm4(kf, kb + ((lane & 7) + ((lane >> 4) << 3)) * KS + kk * 32 + ((lane >> 3) & 1) * 16);
+                if (!kQRegs) ptx::ldsm4(qf[0], q_addr + kk * 32);
+                ptx::mma_bf16(s[0], qf[kQRegs ? kk : 0], kf[0], kf[1]);
+                ptx::mma_bf16(s[1], qf[kQRegs ? kk : 0], kf[2], kf[3]);
+            }
+        // head = lane / 4; positions 2 (lane % 4) + {0, 1} of both halves
+        const int key0 = t0 + (warp + i * kMmaWarps) * 16 + (lane & 3) * 2;
+        float x[4], mx = m_run;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            x[j] = (s[j >> 1][j & 1] + s[j >> 1][2 + (j & 1)]) * a.scale;
+            if (a.softcap > 0.0f) x[j] = soft_cap(x[j], two_over_cap, a.softcap);
+            if (key0 + (j >> 1) * 8 + (j & 1) >= t1) x[j] = -INFINITY;
+            mx = fmaxf(mx, x[j]);
+        }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float al = __expf(m_run - mx);
+        m_run = mx;
+        l_run *= al;
+        uint32_t pf[4];
+#pragma unroll
+        for (int j = 0; j < 4; j += 2) {
+            const float e0 = __expf(x[j] - mx), e1 = __expf(x[j + 1] - mx);
+            l_run += e0 + e1;
+            const uint32_t hi = ptx::pack2(e0, e1);
+            pf[j] = hi;                                                                          // rows 0-7: hi
+            pf[j + 1] = ptx::pack2(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));  // rows 8-15: the rest
+        }
+#pragma unroll
+        for (int n2 = 0; n2 < DV / 16; ++n2)
+            if (n2 < nv) {
+                uint32_t vf[4];
+                ptx::ldsm4t(vf, vb + ((lane & 7) + ((lane >> 3) & 1) * 8) * VS + n2 * 32 + (lane >> 4) * 16);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) { o[2 * n2][j] *= al; o[2 * n2 + 1][j] *= al; }
+                ptx::mma_bf16(o[2 * n2], pf, vf[0], vf[1]);
+                ptx::mma_bf16(o[2 * n2 + 1], pf, vf[2], vf[3]);
+            }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    l_run += __shfl_xor_sync(0xffffffffu, l_run, 1);
+    l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
+    if ((lane & 3) == 0) { mw_s[warp * 8 + (lane >> 2)] = m_run; lw_s[warp * 8 + (lane >> 2)] = l_run; }
+    __syncthreads();  // the ring is free on every warp
+    float* o_w = reinterpret_cast<float*>(tsm);  // [4 warps][8][DV]
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) o_w[(warp * 8 + (lane >> 2)) * DV + i * 8 + (lane & 3) * 2 + j] = o[i][j] + o[i][2 + j];
+    __syncthreads();
+    for (int i = threadIdx.x; i < nr * DV; i += kMmaThreads) {
+        const int h = i / DV;
+        float m = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < kMmaWarps; ++w) m = fmaxf(m, mw_s[w * 8 + h]);
+        float v = 0.0f, l = 0.0f;
+#pragma unroll
+        for (int w = 0; w < kMmaWarps; ++w) {
+            const float f = mw_s[w * 8 + h] == -INFINITY ? 0.0f : __expf(mw_s[w * 8 + h] - m);
+            v = fmaf(o_w[w * 8 * DV + i], f, v);
+            l = fmaf(lw_s[w * 8 + h], f, l);
+        }
+        o_w[i] = v;  // warp 0's slice: read and written by this thread only
+        if (i == h * DV) { m_s[h] = m; l_s[h] = l; }
+    }
+    merge_spans(a, m_s, l_s, o_w, DV, nr, g * rep + h0, r, split, splits, kMmaThreads, out);
+}
+
+template <int DK, int DV>
+cudaError_t span_mma_launch(const DenseAttn& a, bool prepared, const ActOut& out, cudaStream_t s, bool pdl) {
+    const int hchunks = (a.heads / a.n_kv + 7) / 8;
+    const int splits = span_splits(a, (int64_t)a.n_kv * hchunks * a.batch * a.q_rows);
+    constexpr size_t smem = MmaCfg<DK, DV>::kSmem;
+    static PerDeviceOnce once;
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_span_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); });
+    if (e != cudaSuccess) return e;
+    return launch_spans(attn_span_mma_kernel<DK, DV>, dim3((unsigned)splits, (unsigned)(a.n_kv * hchunks), (unsigned)(a.batch * a.q_rows)),
+                        kMmaThreads, smem, s, pdl, a, prepared, splits, out);
+}
+template <int DK>
+cudaError_t span_mma_launch_v(const DenseAttn& a, bool prepared, const ActOut& out, cudaStream_t s, bool pdl) {
+    if (a.kv.v_stride <= 64) return span_mma_launch<DK, 64>(a, prepared, out, s, pdl);
+    if (a.kv.v_stride <= 128) return span_mma_launch<DK, 128>(a, prepared, out, s, pdl);
+    return span_mma_launch<DK, 256>(a, prepared, out, s, pdl);
 }
 
 template <int DK, int DV>  // upper bounds of the (padded) head sizes
@@ -414,19 +639,19 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
     for (int i = threadIdx.x; i < kTileQ * qpieces; i += kTileThreads) {
         const int r = i / qpieces, c = i - r * qpieces;
         const bool live = r < rows && c * 8 < ks;
-        cp16(q_sm + r * KS + c * 16, live ? qg + (int64_t)r * a.heads * ks + c * 8 : qg, live);
+        ptx::cp16(q_sm + r * KS + c * 16, live ? qg + (int64_t)r * a.heads * ks + c * 8 : qg, live);
     }
     auto load = [&](int kt, int bufi) {
         const int base = kt * kTileKeys;
         for (int i = threadIdx.x; i < kTileKeys * qpieces; i += kTileThreads) {
             const int r = i / qpieces, c = i - r * qpieces;
             const bool live = base + r <= last && c * 8 < ks;
-            cp16(k_sm + (bufi * kTileKeys + r) * KS + c * 16, live ? kg + (int64_t)(base + r) * ks + c * 8 : kg, live);
+            ptx::cp16(k_sm + (bufi * kTileKeys + r) * KS + c * 16, live ? kg + (int64_t)(base + r) * ks + c * 8 : kg, live);
         }
         for (int i = threadIdx.x; i < kTileKeys * vpieces; i += kTileThreads) {
             const int r = i / vpieces, c = i - r * vpieces;
             const bool live = base + r <= last && c * 8 < vs;
-            cp16(v_sm + (bufi * kTileKeys + r) * VS + c * 16, live ? vg + (int64_t)(base + r) * vs + c * 8 : vg, live);
+            ptx::cp16(v_sm + (bufi * kTileKeys + r) * VS + c * 16, live ? vg + (int64_t)(base + r) * vs + c * 8 : vg, live);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -461,13 +686,13 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         for (int kk = 0; kk < DK / 16; ++kk)
             if (kk < nk) {
                 uint32_t qa[4];
-                ldsm4(qa, q_addr + kk * 32);
+                ptx::ldsm4(qa, q_addr + kk * 32);
 #pragma unroll
                 for (int n2 = 0; n2 < kTileKeys / 16; ++n2) {  // 16 keys: two n-tiles
                     uint32_t kf[4];
-                    ldsm4(kf, kb + (n2 * 16 + (lane & 7) + ((lane >> 4) << 3)) * KS + kk * 32 + ((lane >> 3) & 1) * 16);
-                    mma_bf16(s[2 * n2], qa, kf[0], kf[1]);
-                    mma_bf16(s[2 * n2 + 1], qa, kf[2], kf[3]);
+                    ptx::ldsm4(kf, kb + (n2 * 16 + (lane & 7) + ((lane >> 4) << 3)) * KS + kk * 32 + ((lane >> 3) & 1) * 16);
+                    ptx::mma_bf16(s[2 * n2], qa, kf[0], kf[1]);
+                    ptx::mma_bf16(s[2 * n2 + 1], qa, kf[2], kf[3]);
                 }
             }
         const int key0 = kt * kTileKeys + (lane & 3) * 2;
@@ -508,18 +733,18 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
 #pragma unroll
             for (int f = 0; f < 4; ++f) {
                 const float x = s[2 * k2 + (f >> 1)][(f & 1) * 2], y = s[2 * k2 + (f >> 1)][(f & 1) * 2 + 1];
-                hi[f] = pack2(x, y);
-                lo[f] = pack2(x - __uint_as_float(hi[f] << 16), y - __uint_as_float(hi[f] & 0xffff0000u));
+                hi[f] = ptx::pack2(x, y);
+                lo[f] = ptx::pack2(x - __uint_as_float(hi[f] << 16), y - __uint_as_float(hi[f] & 0xffff0000u));
             }
 #pragma unroll
             for (int n2 = 0; n2 < DV / 16; ++n2)
                 if (n2 < nv) {
                     uint32_t vf[4];
-                    ldsm4t(vf, vb + (k2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + n2 * 32 + (lane >> 4) * 16);
-                    mma_bf16(o[2 * n2], hi, vf[0], vf[1]);
-                    mma_bf16(o[2 * n2], lo, vf[0], vf[1]);
-                    mma_bf16(o[2 * n2 + 1], hi, vf[2], vf[3]);
-                    mma_bf16(o[2 * n2 + 1], lo, vf[2], vf[3]);
+                    ptx::ldsm4t(vf, vb + (k2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + n2 * 32 + (lane >> 4) * 16);
+                    ptx::mma_bf16(o[2 * n2], hi, vf[0], vf[1]);
+                    ptx::mma_bf16(o[2 * n2], lo, vf[0], vf[1]);
+                    ptx::mma_bf16(o[2 * n2 + 1], hi, vf[2], vf[3]);
+                    ptx::mma_bf16(o[2 * n2 + 1], lo, vf[2], vf[3]);
                 }
         }
         __syncthreads();  // before the buffer is refilled
@@ -550,7 +775,7 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
             const int col = head * dv + c;
             const float x = o[i][2 * q] * f[q], y = o[i][2 * q + 1] * f[q];
             if ((dv & 1) == 0) {
-                *reinterpret_cast<uint32_t*>(out.tiles + dense_off(r, col, out.m_pad)) = pack2(x, y);
+                *reinterpret_cast<uint32_t*>(out.tiles + dense_off(r, col, out.m_pad)) = ptx::pack2(x, y);
             } else {
                 *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, col, out.m_pad)) = __float2bfloat16_rn(x);
                 if (c + 1 < dv) *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, col + 1, out.m_pad)) = __float2bfloat16_rn(y);
@@ -576,7 +801,7 @@ cudaError_t tile_launch_v(const DenseAttn& a, const ActOut& out, cudaStream_t s)
 
 }  // namespace
 
-int attn_max_vdim() { return 256; }
+int attn_max_dim() { return 256; }
 
 cudaError_t launch_attn_prep(const DenseAttn& a, cudaStream_t s) {
     const unsigned grid = (unsigned)(a.batch * a.q_rows);
@@ -587,8 +812,11 @@ cudaError_t launch_attn_prep(const DenseAttn& a, cudaStream_t s) {
 }
 
 cudaError_t launch_attn_span(const DenseAttn& a, bool prepared, const ActOut& out, cudaStream_t s, bool pdl) {
-    if (a.kv.v_stride > 256 || (!prepared && a.q_rows != 1) || (prepared && a.q_bf16)) return cudaErrorInvalidValue;
-    return a.kv.f32 ? span_launch_r<float>(a, prepared, out, s, pdl) : span_launch_r<__nv_bfloat16>(a, prepared, out, s, pdl);
+    if (a.kv.k_stride > 256 || a.kv.v_stride > 256 || (!prepared && a.q_rows != 1) || (prepared && a.q_bf16)) return cudaErrorInvalidValue;
+    if (a.kv.f32) return span_launch_r<float>(a, prepared, out, s, pdl);
+    if (a.kv.k_stride <= 64) return span_mma_launch_v<64>(a, prepared, out, s, pdl);
+    if (a.kv.k_stride <= 128) return span_mma_launch_v<128>(a, prepared, out, s, pdl);
+    return span_mma_launch_v<256>(a, prepared, out, s, pdl);
 }
 
 bool attn_tile_fits(const DenseAttn& a) { return !a.kv.f32 && a.kv.k_stride <= 256 && a.kv.v_stride <= 256; }

@@ -137,7 +137,7 @@ cudaError_t launch_attn_span(const DenseAttn& a, bool prepared, const ActOut& ou
 // Tiles of query positions on the tensor cores (bf16 cache, prepared bf16 queries)
 bool attn_tile_fits(const DenseAttn& a);
 cudaError_t launch_attn_tile(const DenseAttn& a, const ActOut& out, cudaStream_t s);
-int attn_max_vdim();
+int attn_max_dim();  // of query/key and of value heads
 
 // ---------------------------------------------------------------------------------------
 // State-space recurrence (per head: S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x)
@@ -156,12 +156,14 @@ struct SsmArgs {
     int state_pad = 0;
     const int32_t* pos = nullptr;
     int batch = 1, q_rows = 1;
-    float* conv_out = nullptr;     // prefill: [rows, channels] after convolution and silu
+    float* conv_out = nullptr;     // prefill: x | B | C of the rows after convolution and silu
     float* y = nullptr;            // [rows, inner] (S^T C + D x) * silu(z)
     int sm_count = 0;
 };
 int ssm_state_pad(int state);     // 0: not supported
 cudaError_t launch_ssm_step(const SsmArgs& a, cudaStream_t s, bool pdl);     // q_rows == 1
-cudaError_t launch_ssm_prefill(const SsmArgs& a, cudaStream_t s);
+int64_t ssm_conv_floats(const SsmArgs& a);  // floats per row that conv_out needs
+// bf16: 64 tokens at a time on the tensor cores, convolution outputs in bf16; else token by token in f32
+cudaError_t launch_ssm_prefill(const SsmArgs& a, bool bf16, cudaStream_t s);
 
 }  // namespace bt

@@ -566,65 +566,73 @@ __global__ void __launch_bounds__(512) embed_pos_kernel(const int32_t* __restric
     }
 }
 
+// NC: groups of eight columns per thread; the whole row is requested before anything is computed.
+template <int NC>
 __global__ void __launch_bounds__(512) row_op_kernel(const RowArgs a) {
     __shared__ float red[33];
-    ptx::pdl_wait();
-    ptx::pdl_launch_dependents();
+    extern __shared__ float inv_g[];
     const int64_t row = blockIdx.x;
     const int k = a.k, kp = dense_kpad(k);
+    float v[NC][8], w[NC][8], h[NC][8];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) get8(a.w, (i * blockDim.x + threadIdx.x) * 8, k, true, w[i]);
+    ptx::pdl_wait();
+    ptx::pdl_launch_dependents();
     const float* y = a.y + row * a.ld;
     const bool vec = (reinterpret_cast<uintptr_t>(y) & 15) == 0;
-    if (a.op == ROW_RESNORM || a.groups == 1) {
+    const bool parts = a.op == ROW_GROUPNORM && a.groups > 1;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+        const int c0 = (i * blockDim.x + threadIdx.x) * 8;
+        get8(y, c0, k, vec, v[i]);
+        if (a.op == ROW_RESNORM) get8(a.h_in + row * k, c0, k, (k & 3) == 0, h[i]);
+    }
+    float inv = 0.0f;
+    if (!parts) {
         float ss = 0.0f;
-        for (int c0 = threadIdx.x * 8; c0 < k; c0 += blockDim.x * 8) {
-            float v[8];
-            get8(y, c0, k, vec, v);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
-        }
+        for (int i = 0; i < NC; ++i)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss = fmaf(v[i][j], v[i][j], ss);
         ss = block_sum(ss, red);
-        const float inv = 1.0f / sqrtf(ss / (float)k + a.eps);
-        for (int c0 = threadIdx.x * 8; c0 < kp; c0 += blockDim.x * 8) {
-            float v[8], w[8], h[8];
-            get8(y, c0, k, vec, v);
-            get8(a.w, c0, k, true, w);
-            if (a.op == ROW_RESNORM) {
-                get8(a.h_in + row * k, c0, k, (k & 3) == 0, h);
-#pragma unroll
-                for (int j = 0; j < 8; ++j) {
-                    v[j] = fmaf(v[j] * inv, w[j], h[j]);
-                    if (c0 + j < k) a.h_out[row * k + c0 + j] = v[j];
-                }
-            } else {
-#pragma unroll
-                for (int j = 0; j < 8; ++j) v[j] = v[j] * inv * w[j];
-            }
-            put8(a.act, row, c0, k, v);
-        }
+        inv = 1.0f / sqrtf(ss / (float)k + a.eps);
     } else {
-        // equal parts, a warp per part for the sums, then the whole row
-        extern __shared__ float inv_g[];
+        // equal parts, a warp per part for the sums
         const int part = k / a.groups, nw = blockDim.x >> 5;
         for (int g = threadIdx.x >> 5; g < a.groups; g += nw) {
             float ss = 0.0f;
-            for (int c = threadIdx.x & 31; c < part; c += 32) { const float v = y[g * part + c]; ss = fmaf(v, v, ss); }
+            for (int c = threadIdx.x & 31; c < part; c += 32) { const float x = y[g * part + c]; ss = fmaf(x, x, ss); }
             ss = warp_sum(ss);
             if ((threadIdx.x & 31) == 0) inv_g[g] = 1.0f / sqrtf(ss / (float)part + a.eps);
         }
         __syncthreads();
-        for (int c0 = threadIdx.x * 8; c0 < kp; c0 += blockDim.x * 8) {
-            float v[8], w[8];
-            get8(y, c0, k, vec, v);
-            get8(a.w, c0, k, true, w);
+    }
 #pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = c0 + j < k ? v[j] * inv_g[(c0 + j) / part] * w[j] : 0.0f;
-            put8(a.act, row, c0, k, v);
+    for (int i = 0; i < NC; ++i) {
+        const int c0 = (i * blockDim.x + threadIdx.x) * 8;
+        if (c0 >= kp) break;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            if (parts) v[i][j] = c0 + j < k ? v[i][j] * inv_g[(c0 + j) / (k / a.groups)] * w[i][j] : 0.0f;
+            else v[i][j] = a.op == ROW_RESNORM ? fmaf(v[i][j] * inv, w[i][j], h[i][j]) : v[i][j] * inv * w[i][j];
         }
+        if (a.op == ROW_RESNORM) {
+            float* o = a.h_out + row * k;
+            if ((k & 3) == 0 && c0 + 8 <= k) {
+                *reinterpret_cast<float4*>(o + c0) = make_float4(v[i][0], v[i][1], v[i][2], v[i][3]);
+                *reinterpret_cast<float4*>(o + c0 + 4) = make_float4(v[i][4], v[i][5], v[i][6], v[i][7]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    if (c0 + j < k) o[c0 + j] = v[i][j];
+            }
+        }
+        put8(a.act, row, c0, k, v[i]);
     }
 }
 
 unsigned row_threads(int k) {
-    const int t = ((k + 7) / 8 + 31) / 32 * 32;
+    const int t = (dense_kpad(k) / 8 + 31) / 32 * 32;
     return (unsigned)(t < 64 ? 64 : (t > 512 ? 512 : t));
 }
 
@@ -709,7 +717,12 @@ cudaError_t launch_embed_pos(const int32_t* tokens, const __nv_bfloat16* table, 
 cudaError_t launch_row_op(const RowArgs& a, cudaStream_t s, bool pdl) {
     const size_t smem = a.op == ROW_GROUPNORM && a.groups > 1 ? (size_t)a.groups * sizeof(float) : 0;
     if (smem > 40 * 1024) return cudaErrorInvalidConfiguration;
-    return launch_pdl(row_op_kernel, dim3((unsigned)a.rows), dim3(row_threads(a.k)), smem, s, pdl, a);
+    const dim3 grid((unsigned)a.rows), block(row_threads(a.k));
+    const int nc = (dense_kpad(a.k) / 8 + (int)block.x - 1) / (int)block.x;
+    if (nc <= 1) return launch_pdl(row_op_kernel<1>, grid, block, smem, s, pdl, a);
+    if (nc <= 2) return launch_pdl(row_op_kernel<2>, grid, block, smem, s, pdl, a);
+    if (nc <= 4) return launch_pdl(row_op_kernel<4>, grid, block, smem, s, pdl, a);
+    return nc <= 8 ? launch_pdl(row_op_kernel<8>, grid, block, smem, s, pdl, a) : cudaErrorInvalidConfiguration;
 }
 
 }  // namespace bt

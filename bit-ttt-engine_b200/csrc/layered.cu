@@ -206,10 +206,13 @@ cudaError_t trace_stream(const bt_model* m, int layer, const float* h, int rows,
     return cudaMemcpyAsync(m->trace + (size_t)layer * m->trace_rows * W, h, (size_t)rows * W * sizeof(float), cudaMemcpyDeviceToDevice, s);
 }
 
+// The launches of a pass by what they do; a pass can be asked for some of them only (measurement aid).
+enum Part : int { PART_IN = 1, PART_CORE = 2, PART_O = 4, PART_UP = 8, PART_DOWN = 16, PART_ROWS = 32, PART_ALL = 63 };
+
 // One decode step for a few sequences: four or five dependent launches per attention layer, three per recurrent one.
 // A sublayer's output norm and the residual sum are the prologue of the next projection, which reads the old stream
 // and the un-normed output and leaves the new stream in the other buffer.
-bt_status step_fused(bt_model* m, int batch, cudaStream_t s) {
+bt_status step_fused(bt_model* m, int batch, cudaStream_t s, int parts = PART_ALL) {
     Layered* L = m->lay;
     RowBuffers& r = L->dec;
     const int W = L->c.width, sm = m->sm_count;
@@ -217,8 +220,9 @@ bt_status step_fused(bt_model* m, int batch, cudaStream_t s) {
     float* cur = m->h;
     float* other = L->h2;
     const float* pending = nullptr;  // norm weight of the sublayer whose output waits in r.y
-    BT_CUDA_TRY(launch_embed_pos(m->tokens, m->embed, L->pos_table, m->pos, batch, 1, W, m->cfg.vocab_size, L->c.max_positions, cur, ActOut(), s, true));
-    auto from_stream = [&](const DenseLin& lin, float* out, int act) -> cudaError_t {
+    if (parts & PART_ROWS)
+        BT_CUDA_TRY(launch_embed_pos(m->tokens, m->embed, L->pos_table, m->pos, batch, 1, W, m->cfg.vocab_size, L->c.max_positions, cur, ActOut(), s, true));
+    auto from_stream = [&](int part, const DenseLin& lin, float* out, int act) -> cudaError_t {
         DenseIn in;
         if (pending) {
             in.kind = DPRO_RESNORM; in.x = r.y; in.ld = W; in.w = pending; in.eps = eps; in.h = cur; in.h_out = other;
@@ -227,30 +231,31 @@ bt_status step_fused(bt_model* m, int batch, cudaStream_t s) {
         } else {
             in.x = cur; in.ld = W;
         }
+        if (!(parts & part)) return cudaSuccess;
         return launch_dense_stream(lin, in, batch, out, lin.n, act, sm, s, true);
     };
     RowArgs res;  // the residual sum on its own
     res.op = ROW_RESNORM; res.y = r.y; res.ld = W; res.eps = eps; res.rows = batch; res.k = W;
     for (size_t li = 0; li < L->layers.size(); ++li) {
         LayLayer& l = L->layers[li];
-        BT_CUDA_TRY(from_stream(l.in, r.proj, DACT_NONE));
+        BT_CUDA_TRY(from_stream(PART_IN, l.in, r.proj, DACT_NONE));
         DenseIn o;
         o.x = r.mix; o.ld = l.inner();
         if (l.c.mixer == BT_MIX_ATTENTION) {
             ActOut att;
             att.rows = r.mix; att.ld = l.inner();
-            BT_CUDA_TRY(launch_attn_span(attn_args(m, l, r, batch, 1), false, att, s, true));
+            if (parts & PART_CORE) BT_CUDA_TRY(launch_attn_span(attn_args(m, l, r, batch, 1), false, att, s, true));
         } else {
-            BT_CUDA_TRY(launch_ssm_step(ssm_args(m, l, r, batch, 1), s, true));
+            if (parts & PART_CORE) BT_CUDA_TRY(launch_ssm_step(ssm_args(m, l, r, batch, 1), s, true));
             o.kind = DPRO_GROUPNORM; o.w = l.vec[BT_LT_SSM_NORM]; o.eps = eps; o.groups = l.c.norm_groups;
         }
-        BT_CUDA_TRY(launch_dense_stream(l.o, o, batch, r.y, W, DACT_NONE, sm, s, true));
+        if (parts & PART_O) BT_CUDA_TRY(launch_dense_stream(l.o, o, batch, r.y, W, DACT_NONE, sm, s, true));
         pending = l.vec[BT_LT_NORM1];
         if (l.c.mlp != BT_MLP_NONE) {
-            BT_CUDA_TRY(from_stream(l.up, r.ff, DACT_RELU2));
+            BT_CUDA_TRY(from_stream(PART_UP, l.up, r.ff, DACT_RELU2));
             DenseIn d;
             d.x = r.ff; d.ld = l.c.ff;
-            BT_CUDA_TRY(launch_dense_stream(l.down, d, batch, r.y, W, DACT_NONE, sm, s, true));
+            if (parts & PART_DOWN) BT_CUDA_TRY(launch_dense_stream(l.down, d, batch, r.y, W, DACT_NONE, sm, s, true));
             pending = l.vec[BT_LT_NORM2];
         }
         if (m->trace) {  // the stream after the layer, into the trace only
@@ -260,14 +265,15 @@ bt_status step_fused(bt_model* m, int batch, cudaStream_t s) {
         }
     }
     res.w = pending; res.h_in = cur; res.h_out = m->h;  // in place when the stream is there already
-    BT_CUDA_TRY(launch_row_op(res, s, true));
+    if (parts & PART_ROWS) BT_CUDA_TRY(launch_row_op(res, s, true));
     return BT_OK;
 }
 
 // `n` new tokens for each of `batch` sequences, every stage its own kernel over all rows: tcgen05 products of bf16
 // activations (f32 models: f32 products), attention by tiles of query positions.  The stream ends in h.
 constexpr int kTileRowsMin = 16;  // new tokens per sequence from which the tile kernel pays
-bt_status forward_rows(bt_model* m, const int32_t* tokens, float* h, RowBuffers& r, int batch, int n, cudaStream_t s) {
+bt_status forward_rows(bt_model* m, const int32_t* tokens, float* h, RowBuffers& r, int batch, int n, cudaStream_t s,
+                       int parts = PART_ALL) {
     Layered* L = m->lay;
     const int W = L->c.width, sm = m->sm_count, M = batch * n;
     const float eps = L->c.norm_eps;
@@ -277,21 +283,24 @@ bt_status forward_rows(bt_model* m, const int32_t* tokens, float* h, RowBuffers&
     auto tiled = [&](uint8_t* t) { ActOut o; o.tiles = t; o.m_pad = mp; return o; };
     auto plain = [&](float* p, int64_t ld) { ActOut o; o.rows = p; o.ld = ld; return o; };
     const ActOut xa = f32 ? ActOut() : tiled(r.xt);
-    auto product = [&](const DenseLin& lin, const uint8_t* xt, const float* x, float* out, uint8_t* ot, int act) -> cudaError_t {
+    auto product = [&](int part, const DenseLin& lin, const uint8_t* xt, const float* x, float* out, uint8_t* ot, int act) -> cudaError_t {
+        if (!(parts & part)) return cudaSuccess;
         return f32 ? launch_dense_f32(lin, x, lin.k, M, out, lin.n, act, s)
                    : launch_dense_tc(lin, xt, M, out, lin.n, ot, act, r.scratch, err, sm, s);
     };
     RowArgs res;
     res.op = ROW_RESNORM; res.y = r.y; res.ld = W; res.eps = eps; res.rows = M; res.k = W; res.h_in = h; res.h_out = h; res.act = xa;
-    BT_CUDA_TRY(launch_embed_pos(tokens, m->embed, L->pos_table, m->pos, batch, n, W, m->cfg.vocab_size, L->c.max_positions, h, xa, s, false));
+    if (parts & PART_ROWS)
+        BT_CUDA_TRY(launch_embed_pos(tokens, m->embed, L->pos_table, m->pos, batch, n, W, m->cfg.vocab_size, L->c.max_positions, h, xa, s, false));
     for (size_t li = 0; li < L->layers.size(); ++li) {
         LayLayer& l = L->layers[li];
-        BT_CUDA_TRY(product(l.in, r.xt, h, r.proj, nullptr, DACT_NONE));
+        BT_CUDA_TRY(product(PART_IN, l.in, r.xt, h, r.proj, nullptr, DACT_NONE));
         const float* mixed = r.mix;
         if (l.c.mixer == BT_MIX_ATTENTION) {
             DenseAttn a = attn_args(m, l, r, batch, n);
             const ActOut out = f32 ? plain(r.mix, l.inner()) : tiled(r.mt);
-            if (n >= kTileRowsMin && attn_tile_fits(a)) {
+            if (!(parts & PART_CORE)) {
+            } else if (n >= kTileRowsMin && attn_tile_fits(a)) {
                 a.q_bf16 = true;
                 BT_CUDA_TRY(launch_attn_prep(a, s));
                 BT_CUDA_TRY(launch_attn_tile(a, out, s));
@@ -303,22 +312,22 @@ bt_status forward_rows(bt_model* m, const int32_t* tokens, float* h, RowBuffers&
             }
         } else {
             SsmArgs a = ssm_args(m, l, r, batch, n);
-            BT_CUDA_TRY(n == 1 ? launch_ssm_step(a, s, false) : launch_ssm_prefill(a, s));
+            if (parts & PART_CORE) BT_CUDA_TRY(n == 1 ? launch_ssm_step(a, s, false) : launch_ssm_prefill(a, !f32, s));
             RowArgs g;
             g.op = ROW_GROUPNORM; g.y = r.mix; g.ld = l.inner(); g.w = l.vec[BT_LT_SSM_NORM]; g.eps = eps; g.groups = l.c.norm_groups;
             g.rows = M; g.k = l.inner();
             g.act = f32 ? plain(r.proj, l.inner()) : tiled(r.mt);  // the projection rows are used up
-            BT_CUDA_TRY(launch_row_op(g, s, false));
+            if (parts & PART_ROWS) BT_CUDA_TRY(launch_row_op(g, s, false));
             mixed = r.proj;
         }
-        BT_CUDA_TRY(product(l.o, r.mt, mixed, r.y, nullptr, DACT_NONE));
+        BT_CUDA_TRY(product(PART_O, l.o, r.mt, mixed, r.y, nullptr, DACT_NONE));
         res.w = l.vec[BT_LT_NORM1];
-        BT_CUDA_TRY(launch_row_op(res, s, false));
+        if (parts & PART_ROWS) BT_CUDA_TRY(launch_row_op(res, s, false));
         if (l.c.mlp != BT_MLP_NONE) {
-            BT_CUDA_TRY(product(l.up, r.xt, h, r.ff, f32 ? nullptr : r.ft, DACT_RELU2));
-            BT_CUDA_TRY(product(l.down, r.ft, r.ff, r.y, nullptr, DACT_NONE));
+            BT_CUDA_TRY(product(PART_UP, l.up, r.xt, h, r.ff, f32 ? nullptr : r.ft, DACT_RELU2));
+            BT_CUDA_TRY(product(PART_DOWN, l.down, r.ft, r.ff, r.y, nullptr, DACT_NONE));
             res.w = l.vec[BT_LT_NORM2];
-            BT_CUDA_TRY(launch_row_op(res, s, false));
+            if (parts & PART_ROWS) BT_CUDA_TRY(launch_row_op(res, s, false));
         }
         BT_CUDA_TRY(trace_stream(m, (int)li, h, M, s));
     }
@@ -396,7 +405,7 @@ bt_status layered_finalize(bt_model* m) {
             L->max_q = std::max(L->max_q, l.c.heads * l.kv->dense.k_stride);
             L->max_v = std::max(L->max_v, l.v_width());
         } else {
-            L->max_channels = std::max(L->max_channels, l.channels());
+            L->max_channels = std::max(L->max_channels, (int)ssm_conv_floats(ssm_args(m, l, L->dec, 1, 1)));
             BT_CUDA_TRY(dev_alloc(&l.state, (size_t)B * l.inner() * l.state_pad()));
             BT_CUDA_TRY(dev_alloc(&l.ring, (size_t)B * l.c.conv_taps * l.channels()));
         }
@@ -474,6 +483,16 @@ bt_kv_cache* layered_kv(bt_model* m, int layer) {
 
 using namespace bt;
 
+extern "C" bt_status bt_model_enqueue_parts(bt_model* m, int batch, int n_tokens, int parts, void* stream) {
+    if (!m || !m->lay || !m->finalized) return set_error(BT_ERR_ARG, "bt_model_enqueue_parts: not a finalized layer-list model");
+    if (batch < 1 || batch > m->cfg.max_batch || n_tokens < 1 || (n_tokens > 1 && (int64_t)batch * n_tokens > m->pf_rows))
+        return set_error(BT_ERR_SHAPE, "bt_model_enqueue_parts: %d sequences of %d tokens (prefill that many first)", batch, n_tokens);
+    DeviceGuard guard(m->device);
+    cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+    if (n_tokens > 1) return forward_rows(m, m->pf_tokens, m->pf_h, m->lay->pf, batch, n_tokens, s, parts);
+    return step_is_fused(m, batch) ? step_fused(m, batch, s, parts) : forward_rows(m, m->tokens, m->h, m->lay->dec, batch, 1, s, parts);
+}
+
 extern "C" bt_status bt_model_create_layers(bt_model** out, const bt_layers_config* cfg, const bt_layer_config* layers, int device) {
     if (!out || !cfg || !layers) return set_error(BT_ERR_ARG, "bt_model_create_layers: null pointer");
     *out = nullptr;
@@ -489,9 +508,10 @@ extern "C" bt_status bt_model_create_layers(bt_model** out, const bt_layers_conf
         const bt_layer_config& l = layers[i];
         if (l.heads < 1 || l.vdim < 1) return set_error(BT_ERR_SHAPE, "bt_model_create_layers: layer %d: no heads", i);
         if (l.mixer == BT_MIX_ATTENTION) {
-            if (l.kv_heads < 1 || l.heads % l.kv_heads != 0 || l.dim < 1 || l.dim > 1024)
+            if (l.kv_heads < 1 || l.heads % l.kv_heads != 0 || l.dim < 1)
                 return set_error(BT_ERR_SHAPE, "bt_model_create_layers: layer %d: %d query heads over %d KV heads of size %d", i, l.heads, l.kv_heads, l.dim);
-            if (l.vdim > attn_max_vdim()) return set_error(BT_ERR_SHAPE, "bt_model_create_layers: layer %d: value heads of %d, at most %d", i, l.vdim, attn_max_vdim());
+            if (l.vdim > attn_max_dim() || l.dim > attn_max_dim())
+                return set_error(BT_ERR_SHAPE, "bt_model_create_layers: layer %d: key and value heads of %d and %d, at most %d", i, l.dim, l.vdim, attn_max_dim());
             if (l.q_temp_coef != 0.0f && !(l.q_temp_every > 0.0)) return set_error(BT_ERR_ARG, "bt_model_create_layers: layer %d: q_temp_every must be positive", i);
             if (l.v_mix) {
                 if (v_width && v_width != l.kv_heads * l.vdim) return set_error(BT_ERR_SHAPE, "bt_model_create_layers: layer %d: value mixing between layers of different value size", i);

@@ -31,16 +31,51 @@ __device__ __forceinline__ float conv_silu(const SsmArgs& a, const float* x_row,
 // ---------------------------------------------------------------------------------------
 // convolution of the new tokens (prefill)
 // ---------------------------------------------------------------------------------------
+// Output columns: x | B | C.  PAD: bf16, every head's x and every group's B and C padded to a multiple of 8 (zeros), so that
+// each starts on a 16-byte boundary.
 constexpr int kConvTokens = 8;
+__host__ __device__ inline int pad8(int n) { return (n + 7) / 8 * 8; }
+__host__ __device__ inline int conv_cols(const SsmArgs& a) { return a.heads * pad8(a.vdim) + 2 * a.groups * pad8(a.state); }
+template <bool PAD>
 __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a, int channels) {
-    const int ch = blockIdx.x * blockDim.x + threadIdx.x;
-    if (ch >= channels) return;
+    const int col = blockIdx.x * blockDim.x + threadIdx.x;
+    const int cols = PAD ? conv_cols(a) : channels;
+    if (col >= cols) return;
+    int ch = col;
+    if (PAD) {
+        const int vp = pad8(a.vdim), np = pad8(a.state), xw = a.heads * vp;
+        if (col < xw) {
+            const int h = col / vp, c = col - h * vp;
+            ch = c < a.vdim ? h * a.vdim + c : -1;
+        } else {
+            const int q = (col - xw) / np, c = (col - xw) - q * np;  // group of B, then group of C
+            ch = c < a.state ? a.heads * a.vdim + q * a.state + c : -1;
+        }
+    }
     const int b = blockIdx.z, i0 = blockIdx.y * kConvTokens, i1 = min(i0 + kConvTokens, a.q_rows);
     const int inner = a.heads * a.vdim, p0 = a.pos[b];
     const float* ring = a.ring + (int64_t)b * a.taps * channels;
     for (int i = i0; i < i1; ++i) {
         const int64_t r = (int64_t)b * a.q_rows + i;
-        a.conv_out[r * channels + ch] = conv_silu(a, a.proj + r * a.ld + inner, ring, channels, ch, i, p0 + i);
+        const float v = ch >= 0 ? conv_silu(a, a.proj + r * a.ld + inner, ring, channels, ch, i, p0 + i) : 0.0f;
+        if (PAD) reinterpret_cast<__nv_bfloat16*>(a.conv_out)[r * cols + col] = __float2bfloat16_rn(v);
+        else a.conv_out[r * channels + ch] = v;
+    }
+}
+
+// The last inputs of the convolution stay behind for the next tokens: a CTA keeps its x channels, the group's B and C
+// channels are kept by its first head.
+__device__ __forceinline__ void keep_inputs(const SsmArgs& a, float* ring, int channels, int b, int head, int v0, int vc, int p0) {
+    const int N = a.state, inner = a.heads * a.vdim, g = head / (a.heads / a.groups);
+    const int xch = head * a.vdim + v0, bch = inner + g * N, cch = inner + (a.groups + g) * N;
+    const int keep = min(a.q_rows, a.taps);
+    const bool owns_bc = head % (a.heads / a.groups) == 0 && v0 == 0;
+    const int nch = vc + (owns_bc ? 2 * N : 0);
+    for (int e = threadIdx.x; e < keep * nch; e += blockDim.x) {
+        const int k = e / nch, c = e - k * nch;
+        const int ch = c < vc ? xch + c : (c < vc + N ? bch + c - vc : cch + c - vc - N);
+        const int i = a.q_rows - keep + k;
+        ring[(int64_t)((p0 + i) % a.taps) * channels + ch] = a.proj[((int64_t)b * a.q_rows + i) * a.ld + inner + ch];
     }
 }
 
@@ -72,44 +107,56 @@ __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmArgs a, int chan
     const int xch = head * a.vdim + v0, bch = inner + g * N, cch = inner + (a.groups + g) * N;
     float* ring = a.ring + (int64_t)b * a.taps * channels;
     const float a_neg = -expf(a.a_log[head]), bias = a.dt_bias[head], dskip = a.d[head];
-    if (STEP) ptx::pdl_wait();
-    if (STEP) ptx::pdl_launch_dependents();
+    // everything the kernel in front does not write may be requested ahead of the wait on it
     const int p0 = a.pos[b];
     float4 s[NJ];
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
-        s[j] = live && p0 > 0 ? *reinterpret_cast<const float4*>(state + 16 * j + 4 * ln) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s[j] = live ? *reinterpret_cast<const float4*>(state + 16 * j + 4 * ln) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (p0 <= 0)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) s[j] = make_float4(0.f, 0.f, 0.f, 0.f);
 
     for (int i0 = 0; i0 < a.q_rows; i0 += TT) {
         const int n = min(TT, a.q_rows - i0);
         const int64_t r0 = (int64_t)b * a.q_rows + i0;
-        __syncthreads();
-        for (int e = threadIdx.x; e < n * NP; e += 256) {
-            const int t = e / NP, c = e - t * NP;
-            float vb = 0.0f, vcx = 0.0f;
-            if (c < N) {
-                if (STEP) {
-                    const float* xr = a.proj + r0 * a.ld + inner;
-                    vb = conv_silu(a, xr, ring, channels, bch + c, 0, p0);
-                    vcx = conv_silu(a, xr, ring, channels, cch + c, 0, p0);
-                } else {
-                    vb = a.conv_out[(r0 + t) * channels + bch + c];
-                    vcx = a.conv_out[(r0 + t) * channels + cch + c];
+        if (STEP) {
+            // one channel per thread and turn: B, C, then x and z
+            const float* xr = a.proj + r0 * a.ld + inner;
+            bool waited = false;
+            for (int e = threadIdx.x; e < 2 * NP + 128; e += 256) {
+                const int c = e < NP ? e : (e < 2 * NP ? e - NP : (e - 2 * NP) & 63);
+                const bool is_z = e >= 2 * NP + 64;
+                const int ch = e < NP ? bch + c : (e < 2 * NP ? cch + c : xch + c);
+                const bool used = c < (e < 2 * NP ? N : vc);
+                float hist = 0.0f, wl = 0.0f;
+                if (used && !is_z) {  // the taps on earlier inputs
+                    hist = a.conv_b[ch];
+                    wl = a.conv_w[(int64_t)ch * a.taps + a.taps - 1];
+#pragma unroll 4
+                    for (int back = a.taps - 1; back > 0; --back) {
+                        const int q = p0 - back;
+                        if (q >= 0) hist = fmaf(a.conv_w[(int64_t)ch * a.taps + a.taps - 1 - back], ring[(int64_t)(q % a.taps) * channels + ch], hist);
+                    }
                 }
+                if (!waited) { ptx::pdl_wait(); ptx::pdl_launch_dependents(); waited = true; }
+                float v = 0.0f;
+                if (used) v = is_z ? silu_f(xr[ch - inner]) : silu_f(fmaf(wl, xr[ch], hist));
+                (e < NP ? b_s : (e < 2 * NP ? c_s : (is_z ? z_s : x_s)))[c] = v;
             }
-            b_s[e] = vb;
-            c_s[e] = vcx;
-        }
-        for (int e = threadIdx.x; e < n * 64; e += 256) {
-            const int t = e >> 6, c = e & 63;
-            float vx = 0.0f, vz = 0.0f;
-            if (c < vc) {
-                vx = STEP ? conv_silu(a, a.proj + r0 * a.ld + inner, ring, channels, xch + c, 0, p0)
-                          : a.conv_out[(r0 + t) * channels + xch + c];
-                vz = silu_f(a.proj[(r0 + t) * a.ld + xch + c]);
+            if (!waited) { ptx::pdl_wait(); ptx::pdl_launch_dependents(); }
+        } else {
+            __syncthreads();
+            for (int e = threadIdx.x; e < n * NP; e += 256) {
+                const int t = e / NP, c = e - t * NP;
+                b_s[e] = c < N ? a.conv_out[(r0 + t) * channels + bch + c] : 0.0f;
+                c_s[e] = c < N ? a.conv_out[(r0 + t) * channels + cch + c] : 0.0f;
             }
-            x_s[e] = vx;
-            z_s[e] = vz;
+            for (int e = threadIdx.x; e < n * 64; e += 256) {
+                const int t = e >> 6, c = e & 63;
+                x_s[e] = c < vc ? a.conv_out[(r0 + t) * channels + xch + c] : 0.0f;
+                z_s[e] = c < vc ? silu_f(a.proj[(r0 + t) * a.ld + xch + c]) : 0.0f;
+            }
         }
         if (threadIdx.x < n) {
             const float dt = softplus_f(a.proj[(r0 + threadIdx.x) * a.ld + inner + channels + head] + bias);
@@ -140,16 +187,7 @@ __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmArgs a, int chan
     if (live)
 #pragma unroll
         for (int j = 0; j < NJ; ++j) *reinterpret_cast<float4*>(state + 16 * j + 4 * ln) = s[j];
-    // the last inputs of the convolution: this CTA's x channels; the group's B and C channels by its first head
-    const int keep = min(a.q_rows, a.taps);
-    const bool owns_bc = head % (a.heads / a.groups) == 0 && blockIdx.y == 0;
-    const int nch = vc + (owns_bc ? 2 * N : 0);
-    for (int e = threadIdx.x; e < keep * nch; e += 256) {
-        const int k = e / nch, c = e - k * nch;
-        const int ch = c < vc ? xch + c : (c < vc + N ? bch + c - vc : cch + c - vc - N);
-        const int i = a.q_rows - keep + k;
-        ring[(int64_t)((p0 + i) % a.taps) * channels + ch] = a.proj[((int64_t)b * a.q_rows + i) * a.ld + inner + ch];
-    }
+    keep_inputs(a, ring, channels, b, head, v0, vc, p0);
 }
 
 template <int NJ, bool STEP>
@@ -172,6 +210,266 @@ cudaError_t scan_launch_n(const SsmArgs& a, cudaStream_t s, bool pdl) {
     return cudaErrorInvalidValue;
 }
 
+// ---------------------------------------------------------------------------------------
+// recurrence, 64 tokens at a time on the tensor cores (prefill of bf16 models)
+// ---------------------------------------------------------------------------------------
+// With c_t the running sum of the decays' logarithms inside a chunk, the recurrence over the chunk is
+//   y_t = exp(c_t) C_t S + sum_{s <= t} (C_t . B_s) exp(c_t - c_s) dt_s x_s,   S <- exp(c_last) S + sum_s B_s (exp(c_last - c_s) dt_s x_s)^T.
+// B, C and x are bf16 (convolution outputs); every f32 factor enters its product as bf16 hi + lo (16 significand bits):
+// the state, the weights of the pairs (t, s) and the scaled x.  The state itself, the sums and all decays stay f32.
+// A CTA owns 64 columns of one head and walks the chunks in order; the next chunk is copied while one is computed.
+// Eight warps: state tiles of 16 elements x (64 / WP) columns each; outputs: 16 tokens x 32 columns each.
+constexpr int kChunk = 64;
+template <int NP>
+struct ChunkCfg {
+    static constexpr int WN = NP / 16 < 8 ? NP / 16 : 8, WP = 8 / WN < 4 ? 8 / WN : 4;   // warps over state rows / columns
+    static constexpr int TN = NP / 16 / WN, TP = 8 / WP;                                  // 16-row tiles, 8-column tiles per warp
+    static constexpr int NS = NP * 2 + 16, PS = 64 * 2 + 16;                              // bytes per shared-memory row
+    static constexpr int kIn = kChunk * (2 * NS + PS);                                    // B, C, x of a chunk
+    static constexpr int kStages = NP <= 128 ? 2 : 1;
+    static constexpr size_t kSmem = (size_t)kStages * kIn + 2 * NP * PS + 2 * kChunk * PS + 3 * kChunk * 4;
+};
+
+template <int NP>
+__global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int channels) {
+    using Cfg = ChunkCfg<NP>;
+    constexpr int NS = Cfg::NS, PS = Cfg::PS, TN = Cfg::TN, TP = Cfg::TP;
+    extern __shared__ __align__(16) uint8_t csm[];
+    uint8_t* s_hi = csm + Cfg::kStages * Cfg::kIn;   // state [NP][64] hi, lo
+    uint8_t* s_lo = s_hi + NP * PS;
+    uint8_t* w_hi = s_lo + NP * PS;                  // scaled x [64][64] hi, lo
+    uint8_t* w_lo = w_hi + kChunk * PS;
+    float* dt_s = reinterpret_cast<float*>(w_lo + kChunk * PS);
+    float* cum_s = dt_s + kChunk;
+    float* wt_s = cum_s + kChunk;                    // exp(c_last - c_t) dt_t
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.x, v0 = blockIdx.y * 64, b = blockIdx.z;
+    const int vc = min(64, a.vdim - v0), inner = a.heads * a.vdim, g = head / (a.heads / a.groups);
+    const int vp = pad8(a.vdim), np = pad8(a.state), cols = conv_cols(a);
+    const __nv_bfloat16* in = reinterpret_cast<const __nv_bfloat16*>(a.conv_out) + (int64_t)b * a.q_rows * cols;
+    const int xcol = head * vp + v0, bcol = a.heads * vp + g * np, ccol = bcol + a.groups * np;
+    const int xlive = min(64, vp - v0);
+    const float a_neg = -expf(a.a_log[head]), bias = a.dt_bias[head], dskip = a.d[head];
+    const int p0 = a.pos[b];
+    float* ring = a.ring + (int64_t)b * a.taps * channels;
+    float* state = a.s + (((int64_t)b * a.heads + head) * a.vdim + v0) * a.state_pad;
+    const int wn = warp % Cfg::WN, wp = warp / Cfg::WN;
+    const bool s_live = wp < Cfg::WP;
+    const int tt = warp & 3, ph = (warp >> 2) * 32;  // output tile: tokens 16 tt .., columns ph ..
+
+    float st[TN][TP][4];  // (n = g / g + 8 of the tile, p = 2 t, 2 t + 1)
+#pragma unroll
+    for (int i = 0; i < TN; ++i)
+#pragma unroll
+        for (int k = 0; k < TP; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int n = (wn * TN + i) * 16 + (lane >> 2) + (e >> 1) * 8, p = (wp * TP + k) * 8 + (lane & 3) * 2 + (e & 1);
+                st[i][k][e] = s_live && p < vc && p0 > 0 ? state[(int64_t)p * a.state_pad + n] : 0.0f;
+            }
+
+    auto load = [&](int t0, int buf) {
+        const uint32_t dst = ptx::smem_u32(csm) + buf * Cfg::kIn;
+        constexpr int NQ = NP / 8;
+        for (int e = threadIdx.x; e < kChunk * (2 * NQ + 8); e += 256) {
+            const int t = e / (2 * NQ + 8), q = e - t * (2 * NQ + 8);
+            const __nv_bfloat16* row = in + (int64_t)(t0 + t) * cols;
+            const bool tok = t0 + t < a.q_rows;
+            if (q < NQ) {
+                const bool live = tok && q * 8 < np;
+                ptx::cp16(dst + t * NS + q * 16, live ? row + bcol + q * 8 : in, live);
+            } else if (q < 2 * NQ) {
+                const bool live = tok && (q - NQ) * 8 < np;
+                ptx::cp16(dst + kChunk * NS + t * NS + (q - NQ) * 16, live ? row + ccol + (q - NQ) * 8 : in, live);
+            } else {
+                const bool live = tok && (q - 2 * NQ) * 8 < xlive;
+                ptx::cp16(dst + 2 * kChunk * NS + t * PS + (q - 2 * NQ) * 16, live ? row + xcol + (q - 2 * NQ) * 8 : in, live);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    auto raw_dt = [&](int t0) {  // threads 0-63: this chunk's step-size projections
+        const int t = t0 + (int)threadIdx.x;
+        return threadIdx.x < kChunk && t < a.q_rows ? a.proj[((int64_t)b * a.q_rows + t) * a.ld + inner + channels + head] : 0.0f;
+    };
+    load(0, 0);
+    float dt_raw = raw_dt(0);
+
+    int buf = 0;
+    for (int t0 = 0; t0 < a.q_rows; t0 += kChunk) {
+        const int n = min(kChunk, a.q_rows - t0);
+        // ---- step sizes and running decay; the state as hi | lo for the products ----
+        if (threadIdx.x < kChunk) dt_s[threadIdx.x] = (int)threadIdx.x < n ? softplus_f(dt_raw + bias) : 0.0f;
+        dt_raw = raw_dt(t0 + kChunk);
+        if (s_live)
+#pragma unroll
+            for (int i = 0; i < TN; ++i)
+#pragma unroll
+                for (int k = 0; k < TP; ++k)
+#pragma unroll
+                    for (int e = 0; e < 4; e += 2) {
+                        const int o = ((wn * TN + i) * 16 + (lane >> 2) + (e >> 1) * 8) * PS + ((wp * TP + k) * 8 + (lane & 3) * 2) * 2;
+                        const uint32_t hi = ptx::pack2(st[i][k][e], st[i][k][e + 1]);
+                        *reinterpret_cast<uint32_t*>(s_hi + o) = hi;
+                        *reinterpret_cast<uint32_t*>(s_lo + o) = ptx::pack2(st[i][k][e] - __uint_as_float(hi << 16), st[i][k][e + 1] - __uint_as_float(hi & 0xffff0000u));
+                    }
+        __syncthreads();
+        if (warp == 0) {
+            float c0 = a_neg * dt_s[2 * lane], c1 = a_neg * dt_s[2 * lane + 1];
+            float sum = c0 + c1;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float up = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += up;
+            }
+            const float last = __shfl_sync(0xffffffffu, sum, 31);
+            const float before = sum - (c0 + c1);
+            cum_s[2 * lane] = before + c0;
+            cum_s[2 * lane + 1] = sum;
+            wt_s[2 * lane] = expf(last - (before + c0)) * dt_s[2 * lane];
+            wt_s[2 * lane + 1] = expf(last - sum) * dt_s[2 * lane + 1];
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (Cfg::kStages == 2 && t0 + kChunk < a.q_rows) load(t0 + kChunk, buf ^ 1);
+        uint8_t* bt = csm + buf * Cfg::kIn;
+        uint8_t* xt = bt + 2 * kChunk * NS;
+        const uint32_t b_sm = ptx::smem_u32(bt), c_sm = b_sm + kChunk * NS, x_sm = b_sm + 2 * kChunk * NS;
+        // ---- x scaled for the state update ----
+        for (int e = threadIdx.x; e < kChunk * 32; e += 256) {
+            const int t = e >> 5, o = t * PS + (e & 31) * 4;
+            const uint32_t u = *reinterpret_cast<const uint32_t*>(xt + o);
+            const float w = wt_s[t], lo = __uint_as_float(u << 16) * w, hi = __uint_as_float(u & 0xffff0000u) * w;
+            const uint32_t h = ptx::pack2(lo, hi);
+            *reinterpret_cast<uint32_t*>(w_hi + o) = h;
+            *reinterpret_cast<uint32_t*>(w_lo + o) = ptx::pack2(lo - __uint_as_float(h << 16), hi - __uint_as_float(h & 0xffff0000u));
+        }
+        // ---- outputs: 16 tokens x 32 columns per warp ----
+        float y[4][4] = {};
+        if (tt * 16 < n) {
+            const uint32_t c_addr = c_sm + (tt * 16 + (lane & 15)) * NS + (lane >> 4) * 16;
+            float gm[8][4] = {};
+#pragma unroll
+            for (int kk = 0; kk < NP / 16; ++kk) {
+                uint32_t ca[4];
+                ptx::ldsm4(ca, c_addr + kk * 32);
+                const uint32_t srow = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PS + (ph + (lane >> 4) * 8) * 2;
+#pragma unroll
+                for (int k2 = 0; k2 < 2; ++k2) {
+                    uint32_t f[4];
+                    ptx::ldsm4t(f, ptx::smem_u32(s_hi) + srow + k2 * 32);
+                    ptx::mma_bf16(y[2 * k2], ca, f[0], f[1]);
+                    ptx::mma_bf16(y[2 * k2 + 1], ca, f[2], f[3]);
+                    ptx::ldsm4t(f, ptx::smem_u32(s_lo) + srow + k2 * 32);
+                    ptx::mma_bf16(y[2 * k2], ca, f[0], f[1]);
+                    ptx::mma_bf16(y[2 * k2 + 1], ca, f[2], f[3]);
+                }
+#pragma unroll
+                for (int s2 = 0; s2 < 4; ++s2)  // pairs with earlier tokens only
+                    if (s2 <= tt) {
+                        uint32_t f[4];
+                        ptx::ldsm4(f, b_sm + (s2 * 16 + (lane & 7) + ((lane >> 4) << 3)) * NS + kk * 32 + ((lane >> 3) & 1) * 16);
+                        ptx::mma_bf16(gm[2 * s2], ca, f[0], f[1]);
+                        ptx::mma_bf16(gm[2 * s2 + 1], ca, f[2], f[3]);
+                    }
+            }
+            const int ta = tt * 16 + (lane >> 2), tb = ta + 8;
+            const float ca_ = cum_s[ta], cb_ = cum_s[tb];
+            const float ea = expf(ca_), eb = expf(cb_);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { y[i][0] *= ea; y[i][1] *= ea; y[i][2] *= eb; y[i][3] *= eb; }
+#pragma unroll
+            for (int s2 = 0; s2 < 4; ++s2)
+                if (s2 <= tt) {
+                    uint32_t hi[4], lo[4];
+#pragma unroll
+                    for (int f = 0; f < 4; ++f) {  // A operand: rows ta, tb; pairs 2 (lane % 4) + {0, 1} of both halves
+                        const int q = 2 * s2 + (f >> 1), sa = s2 * 16 + (f >> 1) * 8 + (lane & 3) * 2;
+                        const int row = (f & 1) ? tb : ta;
+                        const float cr = (f & 1) ? cb_ : ca_;
+                        const float w0 = sa <= row ? gm[q][(f & 1) * 2] * expf(cr - cum_s[sa]) * dt_s[sa] : 0.0f;
+                        const float w1 = sa + 1 <= row ? gm[q][(f & 1) * 2 + 1] * expf(cr - cum_s[sa + 1]) * dt_s[sa + 1] : 0.0f;
+                        hi[f] = ptx::pack2(w0, w1);
+                        lo[f] = ptx::pack2(w0 - __uint_as_float(hi[f] << 16), w1 - __uint_as_float(hi[f] & 0xffff0000u));
+                    }
+#pragma unroll
+                    for (int k2 = 0; k2 < 2; ++k2) {
+                        uint32_t f[4];
+                        ptx::ldsm4t(f, x_sm + (s2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PS + (ph + k2 * 16 + (lane >> 4) * 8) * 2);
+                        ptx::mma_bf16(y[2 * k2], hi, f[0], f[1]);
+                        ptx::mma_bf16(y[2 * k2], lo, f[0], f[1]);
+                        ptx::mma_bf16(y[2 * k2 + 1], hi, f[2], f[3]);
+                        ptx::mma_bf16(y[2 * k2 + 1], lo, f[2], f[3]);
+                    }
+                }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int t = (e >> 1) ? tb : ta, c = ph + i * 8 + (lane & 3) * 2 + (e & 1);
+                    if (t < n && c < vc) {
+                        const int64_t r = (int64_t)b * a.q_rows + t0 + t;
+                        const float x = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(xt + t * PS + c * 2));
+                        a.y[r * inner + head * a.vdim + v0 + c] = fmaf(dskip, x, y[i][e]) * silu_f(a.proj[r * a.ld + head * a.vdim + v0 + c]);
+                    }
+                }
+        }
+        __syncthreads();  // scaled x complete, state copy and outputs done
+        // ---- state ----
+        if (s_live) {
+            const float dec = expf(cum_s[kChunk - 1]);
+#pragma unroll
+            for (int i = 0; i < TN; ++i)
+#pragma unroll
+                for (int k = 0; k < TP; ++k)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) st[i][k][e] *= dec;
+#pragma unroll
+            for (int kk = 0; kk < kChunk / 16; ++kk)
+                if (kk * 16 < n) {
+                    const uint32_t wrow = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PS + (wp * TP * 8 + (lane >> 4) * 8) * 2;
+#pragma unroll
+                    for (int i = 0; i < TN; ++i) {
+                        uint32_t af[4];
+                        ptx::ldsm4t(af, b_sm + (kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * NS + ((wn * TN + i) * 16 + ((lane >> 3) & 1) * 8) * 2);
+#pragma unroll
+                        for (int k2 = 0; k2 < TP / 2; ++k2) {
+                            uint32_t f[4];
+                            ptx::ldsm4t(f, ptx::smem_u32(w_hi) + wrow + k2 * 32);
+                            ptx::mma_bf16(st[i][2 * k2], af, f[0], f[1]);
+                            ptx::mma_bf16(st[i][2 * k2 + 1], af, f[2], f[3]);
+                            ptx::ldsm4t(f, ptx::smem_u32(w_lo) + wrow + k2 * 32);
+                            ptx::mma_bf16(st[i][2 * k2], af, f[0], f[1]);
+                            ptx::mma_bf16(st[i][2 * k2 + 1], af, f[2], f[3]);
+                        }
+                    }
+                }
+        }
+        __syncthreads();
+        if (Cfg::kStages == 1) { if (t0 + kChunk < a.q_rows) load(t0 + kChunk, 0); } else buf ^= 1;
+    }
+#pragma unroll
+    for (int i = 0; i < TN; ++i)
+#pragma unroll
+        for (int k = 0; k < TP; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int n = (wn * TN + i) * 16 + (lane >> 2) + (e >> 1) * 8, p = (wp * TP + k) * 8 + (lane & 3) * 2 + (e & 1);
+                if (s_live && p < vc) state[(int64_t)p * a.state_pad + n] = st[i][k][e];
+            }
+    keep_inputs(a, ring, channels, b, head, v0, vc, p0);
+}
+
+template <int NP>
+cudaError_t chunk_launch(const SsmArgs& a, cudaStream_t s) {
+    static PerDeviceOnce once;
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(ssm_chunk_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ChunkCfg<NP>::kSmem); });
+    if (e != cudaSuccess) return e;
+    ssm_chunk_kernel<NP><<<dim3((unsigned)a.heads, (unsigned)((a.vdim + 63) / 64), (unsigned)a.batch), 256, ChunkCfg<NP>::kSmem, s>>>(
+        a, a.heads * a.vdim + 2 * a.groups * a.state);
+    return cudaGetLastError();
+}
+
 }  // namespace
 
 int ssm_state_pad(int state) {
@@ -186,12 +484,27 @@ cudaError_t launch_ssm_step(const SsmArgs& a, cudaStream_t s, bool pdl) {
     return scan_launch_n<true>(a, s, pdl);
 }
 
-cudaError_t launch_ssm_prefill(const SsmArgs& a, cudaStream_t s) {
-    const int channels = a.heads * a.vdim + 2 * a.groups * a.state;
-    ssm_conv_kernel<<<dim3((unsigned)((channels + 255) / 256), (unsigned)((a.q_rows + kConvTokens - 1) / kConvTokens), (unsigned)a.batch), 256, 0, s>>>(a, channels);
+int64_t ssm_conv_floats(const SsmArgs& a) {  // per row, for either form
+    const int64_t plain = a.heads * (int64_t)a.vdim + 2ll * a.groups * a.state, padded = (conv_cols(a) + 1) / 2;
+    return plain > padded ? plain : padded;
+}
+
+cudaError_t launch_ssm_prefill(const SsmArgs& a, bool bf16, cudaStream_t s) {
+    const int channels = a.heads * a.vdim + 2 * a.groups * a.state, cols = bf16 ? conv_cols(a) : channels;
+    const dim3 grid((unsigned)((cols + 255) / 256), (unsigned)((a.q_rows + kConvTokens - 1) / kConvTokens), (unsigned)a.batch);
+    if (bf16) ssm_conv_kernel<true><<<grid, 256, 0, s>>>(a, channels);
+    else ssm_conv_kernel<false><<<grid, 256, 0, s>>>(a, channels);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
-    return scan_launch_n<false>(a, s, false);
+    if (!bf16) return scan_launch_n<false>(a, s, false);
+    switch (a.state_pad) {
+        case 16: return chunk_launch<16>(a, s);
+        case 32: return chunk_launch<32>(a, s);
+        case 64: return chunk_launch<64>(a, s);
+        case 128: return chunk_launch<128>(a, s);
+        case 256: return chunk_launch<256>(a, s);
+    }
+    return cudaErrorInvalidValue;
 }
 
 }  // namespace bt

@@ -88,7 +88,7 @@ def write_safetensors(path: str, tensors: dict, metadata: dict | None = None) ->
     if metadata:
         header["__metadata__"] = {str(k): str(v) for k, v in metadata.items()}
     for name, arr in tensors.items():
-        arr = np.ascontiguousarray(arr)
+        arr = np.asarray(arr, order="C")  # keeps a scalar a scalar
         if arr.dtype not in _NAMES:
             raise CheckpointError(f"tensor {name}: dtype {arr.dtype} cannot be stored")
         blob = arr.tobytes()

@@ -84,6 +84,7 @@ def _bind():
     L.bt_kv_import_dense.argtypes = [vp, i64, i64, vp, vp]
     L.bt_model_create_layers.argtypes = [C.POINTER(vp), C.POINTER(_CLayersConfig), C.POINTER(_CLayerConfig), i32]
     L.bt_model_set_layer_tensor.argtypes = [vp, i32, i32, vp, i64]
+    L.bt_model_enqueue_parts.argtypes = [vp, i32, i32, i32, vp]
     L.bt_model_recurrent_state.restype = vp
     L.bt_model_recurrent_state.argtypes = [vp, i32, C.POINTER(i64)]
     L.bt_model_conv_ring.restype = vp
@@ -508,6 +509,12 @@ class LayeredLM(DeviceModel):
     def set_layer_tensor(self, layer: int, kind: int, data: np.ndarray):
         data = np.ascontiguousarray(data, np.float32)
         check(self._L.bt_model_set_layer_tensor(self._h, layer, kind, data.ctypes.data, data.size))
+
+    PART_IN, PART_CORE, PART_O, PART_UP, PART_DOWN, PART_ROWS = 1, 2, 4, 8, 16, 32
+
+    def enqueue_parts(self, batch: int, n_tokens: int, parts: int) -> None:
+        """Measurement aid: some of the launches of a step or of a prefill chunk already run (bt_model_enqueue_parts)."""
+        check(self._L.bt_model_enqueue_parts(self._h, batch, n_tokens, parts, _stream_ptr(self.device)))
 
     def set_trace(self, on: bool = True, rows: int = 0) -> None:
         """Keep the residual stream after every layer of the following steps (rows: see BitLlama.set_trace)."""

@@ -436,6 +436,11 @@ typedef enum {
 } bt_layer_tensor;
 /* Matrices are kept in bf16 (f32 models compute with exactly those values), vectors in f32. */
 bt_status bt_model_set_layer_tensor(bt_model* m, int layer, bt_layer_tensor kind, const float* data_host, int64_t n_elem);
+/* Measurement aid: enqueues some of the launches of a decode step (n_tokens = 1) or of a prefill chunk already run
+ * (n_tokens > 1), on whatever the buffers hold: parts is a sum of 1 = mixers' input projections, 2 = attention and
+ * recurrence, 4 = their output projections, 8 = feed-forward up, 16 = down, 32 = embedding, norms and residual sums.
+ * Positions stay; recurrent states and the cache rows at the current positions do not. */
+bt_status bt_model_enqueue_parts(bt_model* m, int batch, int n_tokens, int parts, void* stream);
 /* Recurrent state of one layer (NULL for attention layers): f32 [max_batch, heads, vdim, state_pad] and the ring of the
  * convolution's last inputs, f32 [max_batch, taps, channels], slot = position % taps.  Sizes in floats. */
 float* bt_model_recurrent_state(bt_model* m, int layer, int64_t* n_floats);

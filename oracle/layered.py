@@ -72,20 +72,20 @@ def causal_attention(q, k, v, scale, cap, sinks, flaw=None):
 
 
 def attention_mixer(x, w, cfg, eps, v_first, flaw=None):
-    """x [T, width] -> (mixed [T, width], v as projected [T, G, dv]).  v_first: the first value-mixing layer's
+    """x [T, width] -> (mixed [T, width], v as projected [T, G dv]).  v_first: the first value-mixing layer's
     projected values, or None in that layer and in layers without value mixing."""
     t = x.shape[0]
     H, G, d, dv = cfg["heads"], cfg["kv_heads"], cfg["dim"], cfg["vdim"]
     q = rms_norm(x @ w["q"].T, w["q.norm"], eps)  # over all heads at once
     k = rms_norm(x @ w["k"].T, w["k.norm"], eps)
-    v = (x @ w["v"].T).reshape(t, G, dv)
+    v = x @ w["v"].T
     if flaw != "no_temperature":
         q = q * query_temperature(np.arange(t), cfg["q_temp"]["coef"], cfg["q_temp"]["every"]).astype(q.dtype)[:, None]
     mixed = v
     if v_first is not None and flaw != "no_value_mix":
         lam = w["vmix"]
         mixed = (1.0 - lam) * v + lam * v_first
-    o = causal_attention(q.reshape(t, H, d), k.reshape(t, G, d), mixed, cfg["scale"], cfg["softcap"], w["sink"], flaw)
+    o = causal_attention(q.reshape(t, H, d), k.reshape(t, G, d), mixed.reshape(t, G, dv), cfg["scale"], cfg["softcap"], w["sink"], flaw)
     return o.reshape(t, H * dv) @ w["o"].T, v
 
 

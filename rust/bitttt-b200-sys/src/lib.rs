@@ -185,6 +185,8 @@ pub mod ffi {
                                       device: c_int) -> bt_status;
         pub fn bt_model_set_layer_tensor(m: *mut bt_model, layer: c_int, kind: c_int, data_host: *const c_float,
                                          n_elem: i64) -> bt_status;
+        pub fn bt_model_enqueue_parts(m: *mut bt_model, batch: c_int, n_tokens: c_int, parts: c_int,
+                                      stream: *mut c_void) -> bt_status;
         pub fn bt_model_recurrent_state(m: *mut bt_model, layer: c_int, n_floats: *mut i64) -> *mut c_float;
         pub fn bt_model_conv_ring(m: *mut bt_model, layer: c_int, n_floats: *mut i64) -> *mut c_float;
         pub fn bt_model_trace_floats(m: *const bt_model, rows: c_int) -> i64;
