@@ -53,7 +53,9 @@ __device__ __forceinline__ float temperature(float coef, double every, int pos) 
 __device__ __forceinline__ void qk_sums(const DenseAttn& a, const float* row, float* red, float& inv_q, float& inv_k) {
     const int nq = a.heads * a.dk, nk = a.n_kv * a.dk;
     float sq = 0.0f, sk = 0.0f;
+#pragma unroll 16
     for (int c = threadIdx.x; c < nq; c += blockDim.x) sq = fmaf(row[c], row[c], sq);
+#pragma unroll 8
     for (int c = threadIdx.x; c < nk; c += blockDim.x) sk = fmaf(row[nq + c], row[nq + c], sk);
     sq = warp_sum(sq);
     sk = warp_sum(sk);
@@ -77,27 +79,34 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const DenseAttn a) {
     float inv_q, inv_k;
     qk_sums(a, row, red, inv_q, inv_k);
     inv_q *= temperature(a.temp_coef, a.temp_every, p);
-    for (int i = threadIdx.x; i < a.heads * ks; i += blockDim.x) {
-        const int h = i / ks, c = i - h * ks, s = h * dk + c;
-        const float v = c < dk ? row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f) : 0.0f;
-        if (QBF16) reinterpret_cast<__nv_bfloat16*>(a.q_buf)[r * a.heads * ks + i] = __float2bfloat16_rn(v);
-        else reinterpret_cast<float*>(a.q_buf)[r * a.heads * ks + i] = v;
-    }
-    if (p < 0 || p >= a.kv.max_seq) return;
-    for (int i = threadIdx.x; i < a.n_kv * ks; i += blockDim.x) {
-        const int g = i / ks, c = i - g * ks, s = g * dk + c;
-        const float v = c < dk ? row[nq + s] * inv_k * (a.k_norm ? a.k_norm[s] : 1.0f) : 0.0f;
-        reinterpret_cast<T*>(a.kv.k)[(((int64_t)b * a.n_kv + g) * a.kv.max_seq + p) * ks + c] = to_cache<T>(v);
-    }
-    for (int i = threadIdx.x; i < a.n_kv * vs; i += blockDim.x) {
-        const int g = i / vs, c = i - g * vs, s = g * dv + c;
-        float v = 0.0f;
-        if (c < dv) {
-            v = row[nq + nk + s];
-            if (a.v_first_out) a.v_first_out[r * nv + s] = v;
-            if (a.v_first_in) v = (1.0f - a.v_lambda) * v + a.v_lambda * a.v_first_in[r * nv + s];
+    // a warp per head and turn
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int h = warp; h < a.heads; h += 8)
+        for (int c = lane; c < ks; c += 32) {
+            const int s = h * dk + c;
+            const float v = c < dk ? row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f) : 0.0f;
+            const int64_t o = (r * a.heads + h) * ks + c;
+            if (QBF16) reinterpret_cast<__nv_bfloat16*>(a.q_buf)[o] = __float2bfloat16_rn(v);
+            else reinterpret_cast<float*>(a.q_buf)[o] = v;
         }
-        reinterpret_cast<T*>(a.kv.v)[(((int64_t)b * a.n_kv + g) * a.kv.max_seq + p) * vs + c] = to_cache<T>(v);
+    if (p < 0 || p >= a.kv.max_seq) return;
+    for (int g = warp; g < a.n_kv; g += 8) {
+        const int64_t at = ((int64_t)b * a.n_kv + g) * a.kv.max_seq + p;
+        for (int c = lane; c < ks; c += 32) {
+            const int s = g * dk + c;
+            const float v = c < dk ? row[nq + s] * inv_k * (a.k_norm ? a.k_norm[s] : 1.0f) : 0.0f;
+            reinterpret_cast<T*>(a.kv.k)[at * ks + c] = to_cache<T>(v);
+        }
+        for (int c = lane; c < vs; c += 32) {
+            const int s = g * dv + c;
+            float v = 0.0f;
+            if (c < dv) {
+                v = row[nq + nk + s];
+                if (a.v_first_out) a.v_first_out[r * nv + s] = v;
+                if (a.v_first_in) v = (1.0f - a.v_lambda) * v + a.v_lambda * a.v_first_in[r * nv + s];
+            }
+            reinterpret_cast<T*>(a.kv.v)[at * vs + c] = to_cache<T>(v);
+        }
     }
 }
 
@@ -383,10 +392,31 @@ cudaError_t span_launch_r(const DenseAttn& a, bool prepared, const ActOut& out, 
 // Rows in shared memory are padded by 16 bytes, so that the eight rows of an ldmatrix fall into different banks.
 constexpr int kTileQ = 64, kTileKeys = 64, kTileThreads = 128;
 
-// cap * tanh(x / cap) with tanh(u) = 1 - 2 / (e^2u + 1): absolute error of the order of 1e-7 cap
-__device__ __forceinline__ float soft_cap(float x, float two_over_cap, float cap) {
-    return cap - __fdividef(2.0f * cap, __expf(x * two_over_cap) + 1.0f);
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// A raw score in units of ln 2, so that its exponential is one ex2: s * scale, or capped: cap * tanh(s * scale / cap) with
+// tanh(u) = 1 - 2 / (e^2u + 1), whose absolute error is of the order of 1e-7 cap.
+struct ScoreMap {
+    float k, cap2;  // factor on the raw score; 2 cap / ln 2, 0: no cap
+    __device__ __forceinline__ ScoreMap(float scale, float cap) {
+        const float log2e = 1.4426950408889634f;
+        k = cap > 0.0f ? scale / cap * (2.0f * log2e) : scale * log2e;
+        cap2 = cap > 0.0f ? 2.0f * cap * log2e : 0.0f;
+    }
+    __device__ __forceinline__ float operator()(float s) const {
+        const float u = s * k;
+        return cap2 > 0.0f ? fmaf(-cap2, rcp(ex2(u) + 1.0f), 0.5f * cap2) : u;
+    }
+};
+constexpr float kLn2 = 0.6931471805599453f;
 
 // ---------------------------------------------------------------------------------------
 // one query position per CTA group on the tensor cores (bf16 cache, decode)
@@ -396,6 +426,8 @@ __device__ __forceinline__ float soft_cap(float x, float two_over_cap, float cap
 // own blocks of 16 positions with its own copy ring, maximum and sums - no CTA barrier inside - and the first blocks are
 // requested before the wait on the projection in front (only the block of the new token has to come after it).
 constexpr int kMmaThreads = 128, kMmaWarps = 4;
+template <int V>
+struct Const { static constexpr int value = V; };
 template <int DK, int DV>
 struct MmaCfg {
     static constexpr int kStages = DK + DV <= 128 ? 4 : (DK + DV <= 256 ? 3 : 2);
@@ -403,7 +435,9 @@ struct MmaCfg {
     static constexpr int kStage = 16 * (KS + VS);
     static constexpr int kRing = kMmaWarps * kStages * kStage;
     static constexpr int kMerge = kMmaWarps * 8 * DV * 4;       // the warps' outputs, in the ring's place
-    static constexpr size_t kSmem = (size_t)(kRing > kMerge ? kRing : kMerge) + 16 * KS + (64 + 2 * 8 + 2 * kMmaWarps * 8) * 4;
+    static constexpr size_t kBase = (size_t)(kRing > kMerge ? kRing : kMerge) + 16 * KS + (64 + 2 * kMmaWarps * 8) * 4;
+    static constexpr size_t kSpan = (8 * DV + 16) * 4;          // a span's outputs, maxima and sums
+    static constexpr size_t smem(int splits) { return kBase + splits * kSpan; }
 };
 
 template <int DK, int DV>
@@ -413,10 +447,11 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
     extern __shared__ __align__(16) uint8_t tsm[];
     uint8_t* q_sm = tsm + (Cfg::kRing > Cfg::kMerge ? Cfg::kRing : Cfg::kMerge);   // [16][KS]: 8 rows hi, 8 rows lo
     float* red = reinterpret_cast<float*>(q_sm + 16 * KS);  // 64
-    float* m_s = red + 64;                                   // [8]
-    float* l_s = m_s + 8;                                    // [8]
-    float* mw_s = l_s + 8;                                   // [4 warps][8]
+    float* mw_s = red + 64;                                  // [4 warps][8]
     float* lw_s = mw_s + kMmaWarps * 8;
+    float* span_s = lw_s + kMmaWarps * 8;                    // rank 0: [splits][8 maxima, 8 sums, 8 x DV outputs]
+    cg::cluster_group cluster = cg::this_cluster();
+    if (splits > 1) cluster.barrier_arrive();                // every CTA of the cluster runs before one writes to another
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int dk = a.dk, dv = a.dv, ks = a.kv.k_stride, vs = a.kv.v_stride;
     const int nk = (ks + 15) / 16, nv = (vs + 15) / 16;
@@ -437,21 +472,26 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
     const bool owner = !prepared && t1 == p + 1 && t0 < t1;    // appends the new token
     const uint32_t ring = ptx::smem_u32(tsm) + warp * S * Cfg::kStage;
     const int kp = nk * 2, vp = nv * 2;                          // 16-byte pieces per row
+    // 16 rows of `stride` elements; FULL: the template's size, whose piece count is a constant
+    auto copy_rows = [&](auto full, uint32_t dst, int dst_stride, const __nv_bfloat16* src, int stride, int pieces_rt, int base) {
+        constexpr int kFull = decltype(full)::value;
+        const int pieces = kFull ? kFull : pieces_rt;
+#pragma unroll 8
+        for (int e = lane; e < 16 * pieces; e += 32) {
+            const int row = e / pieces, c = e - row * pieces;
+            const bool live = base + row < t1 && (kFull || c * 8 < stride);
+            ptx::cp16(dst + row * dst_stride + c * 16, live ? src + (int64_t)(base + row) * stride + c * 8 : src, live);
+        }
+    };
     auto load = [&](int i) {                                     // this warp's i-th block
         const int blk = warp + i * kMmaWarps;
         if (blk < blocks) {
             const int base = t0 + blk * 16;
             const uint32_t st = ring + (i % S) * Cfg::kStage;
-            for (int e = lane; e < 16 * kp; e += 32) {
-                const int row = e / kp, c = e - row * kp;
-                const bool live = base + row < t1 && c * 8 < ks;
-                ptx::cp16(st + row * KS + c * 16, live ? kc + (int64_t)(base + row) * ks + c * 8 : kc, live);
-            }
-            for (int e = lane; e < 16 * vp; e += 32) {
-                const int row = e / vp, c = e - row * vp;
-                const bool live = base + row < t1 && c * 8 < vs;
-                ptx::cp16(st + 16 * KS + row * VS + c * 16, live ? vc + (int64_t)(base + row) * vs + c * 8 : vc, live);
-            }
+            if (ks == DK) copy_rows(Const<DK / 8>(), st, KS, kc, ks, 0, base);
+            else copy_rows(Const<0>(), st, KS, kc, ks, kp, base);
+            if (vs == DV) copy_rows(Const<DV / 8>(), st + 16 * KS, VS, vc, vs, 0, base);
+            else copy_rows(Const<0>(), st + 16 * KS, VS, vc, vs, vp, base);
         }
     };
     auto is_new = [&](int i) { return owner && warp + i * kMmaWarps == blocks - 1; };
@@ -470,17 +510,23 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
         inv_q *= temperature(a.temp_coef, a.temp_every, p);
     }
     const int kw = nk * 16;
-    for (int i = threadIdx.x; i < 8 * kw; i += kMmaThreads) {
-        const int h = i / kw, c = i - h * kw;
-        float v = 0.0f;
-        if (h < nr && c < dk) {
-            const int head = g * rep + h0 + h, s = head * dk + c;
-            v = prepared ? reinterpret_cast<const float*>(a.q_buf)[(r * a.heads + head) * ks + c]
-                         : row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f);
+    for (int c = threadIdx.x; c < kw; c += kMmaThreads) {
+        float v[8];
+#pragma unroll
+        for (int h = 0; h < 8; ++h) {  // all heads requested together
+            v[h] = 0.0f;
+            if (h < nr && c < dk) {
+                const int head = g * rep + h0 + h, s = head * dk + c;
+                v[h] = prepared ? reinterpret_cast<const float*>(a.q_buf)[(r * a.heads + head) * ks + c]
+                                : row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f);
+            }
         }
-        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-        *reinterpret_cast<__nv_bfloat16*>(q_sm + h * KS + c * 2) = hi;
-        *reinterpret_cast<__nv_bfloat16*>(q_sm + (8 + h) * KS + c * 2) = __float2bfloat16_rn(v - __bfloat162float(hi));
+#pragma unroll
+        for (int h = 0; h < 8; ++h) {
+            const __nv_bfloat16 hi = __float2bfloat16_rn(v[h]);
+            *reinterpret_cast<__nv_bfloat16*>(q_sm + h * KS + c * 2) = hi;
+            *reinterpret_cast<__nv_bfloat16*>(q_sm + (8 + h) * KS + c * 2) = __float2bfloat16_rn(v[h] - __bfloat162float(hi));
+        }
     }
     if (owner) {  // (head chunks of one KV head write the same values)
         for (int c = threadIdx.x; c < ks; c += kMmaThreads) {
@@ -509,7 +555,7 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[i][j] = 0.0f;
     float m_run = -INFINITY, l_run = 0.0f;
-    const float two_over_cap = a.softcap > 0.0f ? 2.0f / a.softcap : 0.0f;
+    const ScoreMap score(a.scale, a.softcap);
     const uint32_t q_addr = ptx::smem_u32(q_sm) + (lane & 15) * KS + (lane >> 4) * 16;
     constexpr bool kQRegs = DK <= 128;
     uint32_t qf[kQRegs ? DK / 16 : 1][4];
@@ -540,20 +586,19 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
         float x[4], mx = m_run;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            x[j] = (s[j >> 1][j & 1] + s[j >> 1][2 + (j & 1)]) * a.scale;
-            if (a.softcap > 0.0f) x[j] = soft_cap(x[j], two_over_cap, a.softcap);
+            x[j] = score(s[j >> 1][j & 1] + s[j >> 1][2 + (j & 1)]);
             if (key0 + (j >> 1) * 8 + (j & 1) >= t1) x[j] = -INFINITY;
             mx = fmaxf(mx, x[j]);
         }
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        const float al = __expf(m_run - mx);
+        const float al = ex2(m_run - mx);
         m_run = mx;
         l_run *= al;
         uint32_t pf[4];
 #pragma unroll
         for (int j = 0; j < 4; j += 2) {
-            const float e0 = __expf(x[j] - mx), e1 = __expf(x[j + 1] - mx);
+            const float e0 = ex2(x[j] - mx), e1 = ex2(x[j + 1] - mx);
             l_run += e0 + e1;
             const uint32_t hi = ptx::pack2(e0, e1);
             pf[j] = hi;                                                                          // rows 0-7: hi
@@ -573,7 +618,7 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     l_run += __shfl_xor_sync(0xffffffffu, l_run, 1);
     l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
-    if ((lane & 3) == 0) { mw_s[warp * 8 + (lane >> 2)] = m_run; lw_s[warp * 8 + (lane >> 2)] = l_run; }
+    if ((lane & 3) == 0) { mw_s[warp * 8 + (lane >> 2)] = m_run * kLn2; lw_s[warp * 8 + (lane >> 2)] = l_run; }
     __syncthreads();  // the ring is free on every warp
     float* o_w = reinterpret_cast<float*>(tsm);  // [4 warps][8][DV]
 #pragma unroll
@@ -581,6 +626,13 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
 #pragma unroll
         for (int j = 0; j < 2; ++j) o_w[(warp * 8 + (lane >> 2)) * DV + i * 8 + (lane & 3) * 2 + j] = o[i][j] + o[i][2 + j];
     __syncthreads();
+    // this span's sums go straight to the CTA that finishes them
+    float* dst = span_s + split * (Cfg::kSpan / 4);
+    if (splits > 1) {
+        cluster.barrier_wait();
+        dst = cluster.map_shared_rank(dst, 0);
+    }
+#pragma unroll 4
     for (int i = threadIdx.x; i < nr * DV; i += kMmaThreads) {
         const int h = i / DV;
         float m = -INFINITY;
@@ -593,19 +645,38 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
             v = fmaf(o_w[w * 8 * DV + i], f, v);
             l = fmaf(lw_s[w * 8 + h], f, l);
         }
-        o_w[i] = v;  // warp 0's slice: read and written by this thread only
-        if (i == h * DV) { m_s[h] = m; l_s[h] = l; }
+        dst[16 + i] = v;
+        if (i == h * DV) { dst[h] = m; dst[8 + h] = l; }
     }
-    merge_spans(a, m_s, l_s, o_w, DV, nr, g * rep + h0, r, split, splits, kMmaThreads, out);
+    if (splits > 1) cluster.sync(); else __syncthreads();
+    if (split != 0) return;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < nr * dv; i += kMmaThreads) {
+        const int h = i / dv, c = i - h * dv, head = g * rep + h0 + h;
+        const float sink = a.sink ? a.sink[head] : -INFINITY;
+        float m = sink;
+        for (int s = 0; s < splits; ++s) m = fmaxf(m, span_s[s * (Cfg::kSpan / 4) + h]);
+        float den = a.sink ? expf(sink - m) : 0.0f, num = 0.0f;
+        for (int s = 0; s < splits; ++s) {
+            const float* e = span_s + s * (Cfg::kSpan / 4);
+            const float f = expf(e[h] - m);  // an empty span: exp(-inf) = 0
+            den = fmaf(e[8 + h], f, den);
+            num = fmaf(e[16 + h * DV + c], f, num);
+        }
+        const float v = num / den;
+        const int col = head * dv + c;
+        if (out.tiles) *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, col, out.m_pad)) = __float2bfloat16_rn(v);
+        else out.rows[r * out.ld + col] = v;
+    }
 }
 
 template <int DK, int DV>
 cudaError_t span_mma_launch(const DenseAttn& a, bool prepared, const ActOut& out, cudaStream_t s, bool pdl) {
     const int hchunks = (a.heads / a.n_kv + 7) / 8;
     const int splits = span_splits(a, (int64_t)a.n_kv * hchunks * a.batch * a.q_rows);
-    constexpr size_t smem = MmaCfg<DK, DV>::kSmem;
+    const size_t smem = MmaCfg<DK, DV>::smem(splits);
     static PerDeviceOnce once;
-    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_span_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); });
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_span_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MmaCfg<DK, DV>::smem(8)); });
     if (e != cudaSuccess) return e;
     return launch_spans(attn_span_mma_kernel<DK, DV>, dim3((unsigned)splits, (unsigned)(a.n_kv * hchunks), (unsigned)(a.batch * a.q_rows)),
                         kMmaThreads, smem, s, pdl, a, prepared, splits, out);
@@ -664,7 +735,7 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         for (int j = 0; j < 4; ++j) o[i][j] = 0.0f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
     const int row_a = past + q0 + warp * 16 + (lane >> 2);  // positions of this lane's two query rows: row_a, row_a + 8
-    const float two_over_cap = a.softcap > 0.0f ? 2.0f / a.softcap : 0.0f;
+    const ScoreMap score(a.scale, a.softcap);
     const uint32_t q_addr = q_sm + (warp * 16 + (lane & 15)) * KS + (lane >> 4) * 16;
 
     for (int kt = 0; kt < key_tiles; ++kt) {
@@ -702,8 +773,7 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         for (int i = 0; i < kTileKeys / 8; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                float x = s[i][j] * a.scale;
-                if (a.softcap > 0.0f) x = soft_cap(x, two_over_cap, a.softcap);
+                float x = score(s[i][j]);
                 if (mask && key0 + i * 8 + (j & 1) > row_a + (j >> 1) * 8) x = -INFINITY;
                 s[i][j] = x;
                 mx[j >> 1] = fmaxf(mx[j >> 1], x);
@@ -713,7 +783,7 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         for (int q = 0; q < 2; ++q) {
             mx[q] = fmaxf(mx[q], __shfl_xor_sync(0xffffffffu, mx[q], 1));
             mx[q] = fmaxf(mx[q], __shfl_xor_sync(0xffffffffu, mx[q], 2));
-            al[q] = __expf(m_run[q] - mx[q]);  // position 0 is visible to every row, so mx is finite after the first tile
+            al[q] = ex2(m_run[q] - mx[q]);  // position 0 is visible to every row, so mx is finite after the first tile
             m_run[q] = mx[q];
             l_run[q] *= al[q];
         }
@@ -721,7 +791,7 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         for (int i = 0; i < kTileKeys / 8; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const float e = __expf(s[i][j] - mx[j >> 1]);
+                const float e = ex2(s[i][j] - mx[j >> 1]);
                 s[i][j] = e;
                 l_run[j >> 1] += e;
             }
@@ -754,12 +824,13 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
     for (int q = 0; q < 2; ++q) {
         l_run[q] += __shfl_xor_sync(0xffffffffu, l_run[q], 1);
         l_run[q] += __shfl_xor_sync(0xffffffffu, l_run[q], 2);
-        float m = m_run[q], den = l_run[q];
+        const float m_nat = m_run[q] * kLn2;
+        float m = m_nat, den = l_run[q];
         f[q] = 1.0f;
         if (a.sink) {
             const float sk = a.sink[head];
             m = fmaxf(m, sk);
-            f[q] = expf(m_run[q] - m);
+            f[q] = expf(m_nat - m);
             den = den * f[q] + expf(sk - m);
         }
         f[q] /= den;

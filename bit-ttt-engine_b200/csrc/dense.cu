@@ -456,7 +456,7 @@ int tc_tokens(const DenseLin& lin, int64_t m, int sm_count) {
     if (m <= 128) return 128;
     const int64_t rs = lin.n_pad / kTcRows;
     const int64_t w256 = (rs * ((m + 255) / 256) + sm_count - 1) / sm_count * 2, w128 = (rs * ((m + 127) / 128) + sm_count - 1) / sm_count;
-    return w128 < w256 ? 128 : 256;
+    return 4 * w128 < 3 * w256 ? 128 : 256;  // the smaller tile reads its operands twice as often
 }
 int tc_splits(const DenseLin& lin, int64_t m, int sm_count) {
     if (m > 128) return 1;
@@ -564,6 +564,40 @@ __global__ void __launch_bounds__(512) embed_pos_kernel(const int32_t* __restric
         }
         put8(act, row, c0, hidden, v);
     }
+}
+
+// Norm in equal parts of a multiple of eight columns: a warp per part and turn, the part in registers.
+template <int NI>
+__global__ void __launch_bounds__(256) group_norm_kernel(const RowArgs a, int part) {
+    const int64_t row = blockIdx.x;
+    const int k = a.k, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    ptx::pdl_wait();
+    ptx::pdl_launch_dependents();
+    const float* y = a.y + row * a.ld;
+    const bool vec = (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+    for (int g = warp; g < a.groups; g += 8) {
+        float v[NI][8];
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) get8(y + g * part, (i * 32 + lane) * 8, part, vec, v[i]);
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss = fmaf(v[i][j], v[i][j], ss);
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)part + a.eps);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c0 = (i * 32 + lane) * 8;
+            if (c0 >= part) break;
+            float w[8];
+            get8(a.w + g * part, c0, part, true, w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[i][j] = v[i][j] * inv * w[j];
+            put8(a.act, row, g * part + c0, k, v[i]);
+        }
+    }
+    const float zero[8] = {};
+    for (int c0 = k + (int)threadIdx.x * 8; c0 < dense_kpad(k); c0 += 256 * 8) put8(a.act, row, c0, k, zero);
 }
 
 // NC: groups of eight columns per thread; the whole row is requested before anything is computed.
@@ -717,7 +751,19 @@ cudaError_t launch_embed_pos(const int32_t* tokens, const __nv_bfloat16* table, 
 cudaError_t launch_row_op(const RowArgs& a, cudaStream_t s, bool pdl) {
     const size_t smem = a.op == ROW_GROUPNORM && a.groups > 1 ? (size_t)a.groups * sizeof(float) : 0;
     if (smem > 40 * 1024) return cudaErrorInvalidConfiguration;
-    const dim3 grid((unsigned)a.rows), block(row_threads(a.k));
+    if (a.op == ROW_GROUPNORM && a.groups > 1) {
+        const int part = a.k / a.groups;
+        if (part % 8 == 0 && part <= 2048) {
+            const dim3 grid((unsigned)a.rows);
+            if (part <= 256) return launch_pdl(group_norm_kernel<1>, grid, dim3(256), 0, s, pdl, a, part);
+            if (part <= 1024) return launch_pdl(group_norm_kernel<4>, grid, dim3(256), 0, s, pdl, a, part);
+            return launch_pdl(group_norm_kernel<8>, grid, dim3(256), 0, s, pdl, a, part);
+        }
+    }
+    // many rows: fewer threads with more of the row each, so that more rows share an SM
+    unsigned threads = row_threads(a.k);
+    if (a.rows > 64) threads = threads > 256 ? (threads / 4 + 31) / 32 * 32 : (threads > 128 ? (threads / 2 + 31) / 32 * 32 : threads);
+    const dim3 grid((unsigned)a.rows), block(threads);
     const int nc = (dense_kpad(a.k) / 8 + (int)block.x - 1) / (int)block.x;
     if (nc <= 1) return launch_pdl(row_op_kernel<1>, grid, block, smem, s, pdl, a);
     if (nc <= 2) return launch_pdl(row_op_kernel<2>, grid, block, smem, s, pdl, a);

@@ -10,6 +10,7 @@ namespace bt {
 namespace {
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+__device__ __forceinline__ float silu_fast(float v) { return __fdividef(v, 1.0f + __expf(-v)); }  // where the result is rounded to bf16
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
 
 // Input of the convolution at position p - back, for a token at row r (i-th new token, position p): from the projection
@@ -55,11 +56,41 @@ __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmArgs a, int chan
     const int b = blockIdx.z, i0 = blockIdx.y * kConvTokens, i1 = min(i0 + kConvTokens, a.q_rows);
     const int inner = a.heads * a.vdim, p0 = a.pos[b];
     const float* ring = a.ring + (int64_t)b * a.taps * channels;
-    for (int i = i0; i < i1; ++i) {
+    auto put = [&](int i, float v) {
         const int64_t r = (int64_t)b * a.q_rows + i;
-        const float v = ch >= 0 ? conv_silu(a, a.proj + r * a.ld + inner, ring, channels, ch, i, p0 + i) : 0.0f;
         if (PAD) reinterpret_cast<__nv_bfloat16*>(a.conv_out)[r * cols + col] = __float2bfloat16_rn(v);
         else a.conv_out[r * channels + ch] = v;
+    };
+    const float* x = a.proj + (int64_t)b * a.q_rows * a.ld + inner + ch;
+    if (ch < 0) {
+        for (int i = i0; i < i1; ++i) put(i, 0.0f);
+    } else if (a.taps <= 4) {
+        // the inputs of the block and the three before it in registers
+        float w[4], v[kConvTokens + 3];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j] = j < a.taps ? a.conv_w[(int64_t)ch * a.taps + a.taps - 1 - j] : 0.0f;  // by distance back
+#pragma unroll
+        for (int j = 0; j < kConvTokens + 3; ++j) {
+            const int i = i0 + j - 3;
+            v[j] = i >= 0 && i < i1 ? x[(int64_t)i * a.ld] : 0.0f;
+        }
+        if (i0 == 0)
+#pragma unroll
+            for (int j = 0; j < 3; ++j) {
+                const int q = p0 + j - 3;
+                if (q >= 0 && 3 - j < a.taps) v[j] = ring[(int64_t)(q % a.taps) * channels + ch];
+            }
+        const float bias = a.conv_b[ch];
+#pragma unroll
+        for (int j = 0; j < kConvTokens; ++j)
+            if (i0 + j < i1) {
+                float s = bias;
+#pragma unroll
+                for (int k = 3; k >= 0; --k) s = fmaf(w[k], v[j + 3 - k], s);
+                put(i0 + j, PAD ? silu_fast(s) : silu_f(s));
+            }
+    } else {
+        for (int i = i0; i < i1; ++i) put(i, conv_silu(a, a.proj + ((int64_t)b * a.q_rows + i) * a.ld + inner, ring, channels, ch, i, p0 + i));
     }
 }
 
@@ -218,20 +249,21 @@ cudaError_t scan_launch_n(const SsmArgs& a, cudaStream_t s, bool pdl) {
 // B, C and x are bf16 (convolution outputs); every f32 factor enters its product as bf16 hi + lo (16 significand bits):
 // the state, the weights of the pairs (t, s) and the scaled x.  The state itself, the sums and all decays stay f32.
 // A CTA owns 64 columns of one head and walks the chunks in order; the next chunk is copied while one is computed.
-// Eight warps: state tiles of 16 elements x (64 / WP) columns each; outputs: 16 tokens x 32 columns each.
-constexpr int kChunk = 64;
+// Sixteen warps as 4 x 4 over (16 tokens) x (16 earlier tokens | 16 columns): each makes its tile of pair weights, leaves it
+// in shared memory and then its tile of outputs; the state is cut over the warps by rows of 16 elements and columns.
+constexpr int kChunk = 64, kChunkThreads = 512;
 template <int NP>
 struct ChunkCfg {
-    static constexpr int WN = NP / 16 < 8 ? NP / 16 : 8, WP = 8 / WN < 4 ? 8 / WN : 4;   // warps over state rows / columns
+    static constexpr int WN = NP / 16 < 8 ? NP / 16 : 8, WP = 16 / WN < 4 ? 16 / WN : 4;  // warps over state rows / columns
     static constexpr int TN = NP / 16 / WN, TP = 8 / WP;                                  // 16-row tiles, 8-column tiles per warp
     static constexpr int NS = NP * 2 + 16, PS = 64 * 2 + 16;                              // bytes per shared-memory row
     static constexpr int kIn = kChunk * (2 * NS + PS);                                    // B, C, x of a chunk
     static constexpr int kStages = NP <= 128 ? 2 : 1;
-    static constexpr size_t kSmem = (size_t)kStages * kIn + 2 * NP * PS + 2 * kChunk * PS + 3 * kChunk * 4;
+    static constexpr size_t kSmem = (size_t)kStages * kIn + 2 * NP * PS + 4 * kChunk * PS + 3 * kChunk * 4;
 };
 
 template <int NP>
-__global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int channels) {
+__global__ void __launch_bounds__(kChunkThreads, 1) ssm_chunk_kernel(const SsmArgs a, int channels) {
     using Cfg = ChunkCfg<NP>;
     constexpr int NS = Cfg::NS, PS = Cfg::PS, TN = Cfg::TN, TP = Cfg::TP;
     extern __shared__ __align__(16) uint8_t csm[];
@@ -239,7 +271,9 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
     uint8_t* s_lo = s_hi + NP * PS;
     uint8_t* w_hi = s_lo + NP * PS;                  // scaled x [64][64] hi, lo
     uint8_t* w_lo = w_hi + kChunk * PS;
-    float* dt_s = reinterpret_cast<float*>(w_lo + kChunk * PS);
+    uint8_t* m_hi = w_lo + kChunk * PS;              // pair weights [64][64] hi, lo
+    uint8_t* m_lo = m_hi + kChunk * PS;
+    float* dt_s = reinterpret_cast<float*>(m_lo + kChunk * PS);
     float* cum_s = dt_s + kChunk;
     float* wt_s = cum_s + kChunk;                    // exp(c_last - c_t) dt_t
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -255,7 +289,7 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
     float* state = a.s + (((int64_t)b * a.heads + head) * a.vdim + v0) * a.state_pad;
     const int wn = warp % Cfg::WN, wp = warp / Cfg::WN;
     const bool s_live = wp < Cfg::WP;
-    const int tt = warp & 3, ph = (warp >> 2) * 32;  // output tile: tokens 16 tt .., columns ph ..
+    const int tt = warp >> 2, qq = warp & 3;         // tokens 16 tt ..; earlier tokens / columns 16 qq ..
 
     float st[TN][TP][4];  // (n = g / g + 8 of the tile, p = 2 t, 2 t + 1)
 #pragma unroll
@@ -271,7 +305,7 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
     auto load = [&](int t0, int buf) {
         const uint32_t dst = ptx::smem_u32(csm) + buf * Cfg::kIn;
         constexpr int NQ = NP / 8;
-        for (int e = threadIdx.x; e < kChunk * (2 * NQ + 8); e += 256) {
+        for (int e = threadIdx.x; e < kChunk * (2 * NQ + 8); e += kChunkThreads) {
             const int t = e / (2 * NQ + 8), q = e - t * (2 * NQ + 8);
             const __nv_bfloat16* row = in + (int64_t)(t0 + t) * cols;
             const bool tok = t0 + t < a.q_rows;
@@ -298,9 +332,18 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
     int buf = 0;
     for (int t0 = 0; t0 < a.q_rows; t0 += kChunk) {
         const int n = min(kChunk, a.q_rows - t0);
-        // ---- step sizes and running decay; the state as hi | lo for the products ----
+        const int ta = tt * 16 + (lane >> 2), tb = ta + 8;  // this lane's tokens
+        // ---- step sizes and running decay; the state as hi | lo for the products; the gates are requested ----
         if (threadIdx.x < kChunk) dt_s[threadIdx.x] = (int)threadIdx.x < n ? softplus_f(dt_raw + bias) : 0.0f;
         dt_raw = raw_dt(t0 + kChunk);
+        float z[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int t = (e >> 1) ? tb : ta, c = qq * 16 + i * 8 + (lane & 3) * 2 + (e & 1);
+                z[i][e] = t < n && c < vc ? a.proj[((int64_t)b * a.q_rows + t0 + t) * a.ld + head * a.vdim + v0 + c] : 0.0f;
+            }
         if (s_live)
 #pragma unroll
             for (int i = 0; i < TN; ++i)
@@ -313,9 +356,15 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
                         *reinterpret_cast<uint32_t*>(s_hi + o) = hi;
                         *reinterpret_cast<uint32_t*>(s_lo + o) = ptx::pack2(st[i][k][e] - __uint_as_float(hi << 16), st[i][k][e + 1] - __uint_as_float(hi & 0xffff0000u));
                     }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
+        if (Cfg::kStages == 2 && t0 + kChunk < a.q_rows) load(t0 + kChunk, buf ^ 1);
+        uint8_t* bt = csm + buf * Cfg::kIn;
+        uint8_t* xt = bt + 2 * kChunk * NS;
+        const uint32_t b_sm = ptx::smem_u32(bt), c_sm = b_sm + kChunk * NS, x_sm = b_sm + 2 * kChunk * NS;
+        // ---- running sums of the decays' logarithms, while the other warps multiply ----
         if (warp == 0) {
-            float c0 = a_neg * dt_s[2 * lane], c1 = a_neg * dt_s[2 * lane + 1];
+            const float c0 = a_neg * dt_s[2 * lane], c1 = a_neg * dt_s[2 * lane + 1];
             float sum = c0 + c1;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -329,14 +378,34 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
             wt_s[2 * lane] = expf(last - (before + c0)) * dt_s[2 * lane];
             wt_s[2 * lane + 1] = expf(last - sum) * dt_s[2 * lane + 1];
         }
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();
-        if (Cfg::kStages == 2 && t0 + kChunk < a.q_rows) load(t0 + kChunk, buf ^ 1);
-        uint8_t* bt = csm + buf * Cfg::kIn;
-        uint8_t* xt = bt + 2 * kChunk * NS;
-        const uint32_t b_sm = ptx::smem_u32(bt), c_sm = b_sm + kChunk * NS, x_sm = b_sm + 2 * kChunk * NS;
-        // ---- x scaled for the state update ----
-        for (int e = threadIdx.x; e < kChunk * 32; e += 256) {
+        // ---- C S (16 tokens x 16 columns) and C B^T (16 x 16 pairs) ----
+        float y[2][4] = {}, gm[2][4] = {};
+        const bool live = tt * 16 < n, pairs = live && qq <= tt;
+        if (live) {
+            const uint32_t c_addr = c_sm + (tt * 16 + (lane & 15)) * NS + (lane >> 4) * 16;
+            const uint32_t b_addr = b_sm + (qq * 16 + (lane & 7) + ((lane >> 4) << 3)) * NS + ((lane >> 3) & 1) * 16;
+            const uint32_t s_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * PS + (qq * 16 + (lane >> 4) * 8) * 2;
+            const uint32_t sh = ptx::smem_u32(s_hi) + s_off, sl = ptx::smem_u32(s_lo) + s_off;
+#pragma unroll
+            for (int kk = 0; kk < NP / 16; ++kk) {
+                uint32_t ca[4], f[4];
+                ptx::ldsm4(ca, c_addr + kk * 32);
+                ptx::ldsm4t(f, sh + kk * 16 * PS);
+                ptx::mma_bf16(y[0], ca, f[0], f[1]);
+                ptx::mma_bf16(y[1], ca, f[2], f[3]);
+                ptx::ldsm4t(f, sl + kk * 16 * PS);
+                ptx::mma_bf16(y[0], ca, f[0], f[1]);
+                ptx::mma_bf16(y[1], ca, f[2], f[3]);
+                if (pairs) {
+                    ptx::ldsm4(f, b_addr + kk * 32);
+                    ptx::mma_bf16(gm[0], ca, f[0], f[1]);
+                    ptx::mma_bf16(gm[1], ca, f[2], f[3]);
+                }
+            }
+        }
+        __syncthreads();  // running sums
+        // ---- x scaled for the state update; pair weights ----
+        for (int e = threadIdx.x; e < kChunk * 32; e += kChunkThreads) {
             const int t = e >> 5, o = t * PS + (e & 31) * 4;
             const uint32_t u = *reinterpret_cast<const uint32_t*>(xt + o);
             const float w = wt_s[t], lo = __uint_as_float(u << 16) * w, hi = __uint_as_float(u & 0xffff0000u) * w;
@@ -344,77 +413,52 @@ __global__ void __launch_bounds__(256, 1) ssm_chunk_kernel(const SsmArgs a, int 
             *reinterpret_cast<uint32_t*>(w_hi + o) = h;
             *reinterpret_cast<uint32_t*>(w_lo + o) = ptx::pack2(lo - __uint_as_float(h << 16), hi - __uint_as_float(h & 0xffff0000u));
         }
-        // ---- outputs: 16 tokens x 32 columns per warp ----
-        float y[4][4] = {};
-        if (tt * 16 < n) {
-            const uint32_t c_addr = c_sm + (tt * 16 + (lane & 15)) * NS + (lane >> 4) * 16;
-            float gm[8][4] = {};
+        const float cum_a = cum_s[ta], cum_b = cum_s[tb];
+        if (pairs)
 #pragma unroll
-            for (int kk = 0; kk < NP / 16; ++kk) {
-                uint32_t ca[4];
-                ptx::ldsm4(ca, c_addr + kk * 32);
-                const uint32_t srow = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PS + (ph + (lane >> 4) * 8) * 2;
+            for (int i = 0; i < 2; ++i)
 #pragma unroll
-                for (int k2 = 0; k2 < 2; ++k2) {
-                    uint32_t f[4];
-                    ptx::ldsm4t(f, ptx::smem_u32(s_hi) + srow + k2 * 32);
-                    ptx::mma_bf16(y[2 * k2], ca, f[0], f[1]);
-                    ptx::mma_bf16(y[2 * k2 + 1], ca, f[2], f[3]);
-                    ptx::ldsm4t(f, ptx::smem_u32(s_lo) + srow + k2 * 32);
-                    ptx::mma_bf16(y[2 * k2], ca, f[0], f[1]);
-                    ptx::mma_bf16(y[2 * k2 + 1], ca, f[2], f[3]);
+                for (int e = 0; e < 4; e += 2) {
+                    const int s0 = qq * 16 + i * 8 + (lane & 3) * 2, row = e ? tb : ta;
+                    const float cr = e ? cum_b : cum_a;
+                    const float w0 = s0 <= row ? gm[i][e] * __expf(cr - cum_s[s0]) * dt_s[s0] : 0.0f;
+                    const float w1 = s0 + 1 <= row ? gm[i][e + 1] * __expf(cr - cum_s[s0 + 1]) * dt_s[s0 + 1] : 0.0f;
+                    const uint32_t hi = ptx::pack2(w0, w1);
+                    *reinterpret_cast<uint32_t*>(m_hi + row * PS + s0 * 2) = hi;
+                    *reinterpret_cast<uint32_t*>(m_lo + row * PS + s0 * 2) = ptx::pack2(w0 - __uint_as_float(hi << 16), w1 - __uint_as_float(hi & 0xffff0000u));
                 }
+        __syncthreads();
+        // ---- outputs ----
+        if (live) {
+            const float ea = __expf(cum_a), eb = __expf(cum_b);
 #pragma unroll
-                for (int s2 = 0; s2 < 4; ++s2)  // pairs with earlier tokens only
-                    if (s2 <= tt) {
-                        uint32_t f[4];
-                        ptx::ldsm4(f, b_sm + (s2 * 16 + (lane & 7) + ((lane >> 4) << 3)) * NS + kk * 32 + ((lane >> 3) & 1) * 16);
-                        ptx::mma_bf16(gm[2 * s2], ca, f[0], f[1]);
-                        ptx::mma_bf16(gm[2 * s2 + 1], ca, f[2], f[3]);
-                    }
-            }
-            const int ta = tt * 16 + (lane >> 2), tb = ta + 8;
-            const float ca_ = cum_s[ta], cb_ = cum_s[tb];
-            const float ea = expf(ca_), eb = expf(cb_);
-#pragma unroll
-            for (int i = 0; i < 4; ++i) { y[i][0] *= ea; y[i][1] *= ea; y[i][2] *= eb; y[i][3] *= eb; }
+            for (int i = 0; i < 2; ++i) { y[i][0] *= ea; y[i][1] *= ea; y[i][2] *= eb; y[i][3] *= eb; }
+            const uint32_t m_off = (tt * 16 + (lane & 15)) * PS + (lane >> 4) * 16;
+            const uint32_t mh = ptx::smem_u32(m_hi) + m_off, ml = ptx::smem_u32(m_lo) + m_off;
+            const uint32_t x_addr = x_sm + ((lane & 7) + ((lane >> 3) & 1) * 8) * PS + (qq * 16 + (lane >> 4) * 8) * 2;
 #pragma unroll
             for (int s2 = 0; s2 < 4; ++s2)
                 if (s2 <= tt) {
-                    uint32_t hi[4], lo[4];
-#pragma unroll
-                    for (int f = 0; f < 4; ++f) {  // A operand: rows ta, tb; pairs 2 (lane % 4) + {0, 1} of both halves
-                        const int q = 2 * s2 + (f >> 1), sa = s2 * 16 + (f >> 1) * 8 + (lane & 3) * 2;
-                        const int row = (f & 1) ? tb : ta;
-                        const float cr = (f & 1) ? cb_ : ca_;
-                        const float w0 = sa <= row ? gm[q][(f & 1) * 2] * expf(cr - cum_s[sa]) * dt_s[sa] : 0.0f;
-                        const float w1 = sa + 1 <= row ? gm[q][(f & 1) * 2 + 1] * expf(cr - cum_s[sa + 1]) * dt_s[sa + 1] : 0.0f;
-                        hi[f] = ptx::pack2(w0, w1);
-                        lo[f] = ptx::pack2(w0 - __uint_as_float(hi[f] << 16), w1 - __uint_as_float(hi[f] & 0xffff0000u));
-                    }
-#pragma unroll
-                    for (int k2 = 0; k2 < 2; ++k2) {
-                        uint32_t f[4];
-                        ptx::ldsm4t(f, x_sm + (s2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PS + (ph + k2 * 16 + (lane >> 4) * 8) * 2);
-                        ptx::mma_bf16(y[2 * k2], hi, f[0], f[1]);
-                        ptx::mma_bf16(y[2 * k2], lo, f[0], f[1]);
-                        ptx::mma_bf16(y[2 * k2 + 1], hi, f[2], f[3]);
-                        ptx::mma_bf16(y[2 * k2 + 1], lo, f[2], f[3]);
-                    }
+                    uint32_t hi[4], lo[4], f[4];
+                    ptx::ldsm4(hi, mh + s2 * 32);
+                    ptx::ldsm4(lo, ml + s2 * 32);
+                    ptx::ldsm4t(f, x_addr + s2 * 16 * PS);
+                    ptx::mma_bf16(y[0], hi, f[0], f[1]);
+                    ptx::mma_bf16(y[1], hi, f[2], f[3]);
+                    ptx::mma_bf16(y[0], lo, f[0], f[1]);
+                    ptx::mma_bf16(y[1], lo, f[2], f[3]);
                 }
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+            for (int i = 0; i < 2; ++i)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const int t = (e >> 1) ? tb : ta, c = ph + i * 8 + (lane & 3) * 2 + (e & 1);
+                    const int t = (e >> 1) ? tb : ta, c = qq * 16 + i * 8 + (lane & 3) * 2 + (e & 1);
                     if (t < n && c < vc) {
-                        const int64_t r = (int64_t)b * a.q_rows + t0 + t;
                         const float x = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(xt + t * PS + c * 2));
-                        a.y[r * inner + head * a.vdim + v0 + c] = fmaf(dskip, x, y[i][e]) * silu_f(a.proj[r * a.ld + head * a.vdim + v0 + c]);
+                        a.y[((int64_t)b * a.q_rows + t0 + t) * inner + head * a.vdim + v0 + c] = fmaf(dskip, x, y[i][e]) * silu_fast(z[i][e]);
                     }
                 }
         }
-        __syncthreads();  // scaled x complete, state copy and outputs done
         // ---- state ----
         if (s_live) {
             const float dec = expf(cum_s[kChunk - 1]);
@@ -465,7 +509,7 @@ cudaError_t chunk_launch(const SsmArgs& a, cudaStream_t s) {
     static PerDeviceOnce once;
     cudaError_t e = once.run([] { return cudaFuncSetAttribute(ssm_chunk_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ChunkCfg<NP>::kSmem); });
     if (e != cudaSuccess) return e;
-    ssm_chunk_kernel<NP><<<dim3((unsigned)a.heads, (unsigned)((a.vdim + 63) / 64), (unsigned)a.batch), 256, ChunkCfg<NP>::kSmem, s>>>(
+    ssm_chunk_kernel<NP><<<dim3((unsigned)a.heads, (unsigned)((a.vdim + 63) / 64), (unsigned)a.batch), kChunkThreads, ChunkCfg<NP>::kSmem, s>>>(
         a, a.heads * a.vdim + 2 * a.groups * a.state);
     return cudaGetLastError();
 }
