@@ -41,9 +41,11 @@ struct Raw8<float> {
     __device__ __forceinline__ void widen(float (&v)[8]) const { v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w; }
 };
 
-__device__ __forceinline__ float temperature(float coef, double every, int pos) {
-    if (coef == 0.0f) return 1.0f;
-    return 1.0f + coef * logf((float)floor((double)(pos + 1) / every) + 1.0f);
+__device__ __forceinline__ float temperature(const DenseAttn& a, int pos) {
+    if (a.temp_coef == 0.0f) return 1.0f;
+    const float steps = a.temp_every_int > 0 ? (float)((unsigned)(pos + 1) / (unsigned)a.temp_every_int)
+                                             : (float)floor((double)(pos + 1) / a.temp_every);
+    return 1.0f + a.temp_coef * logf(steps + 1.0f);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -78,10 +80,11 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const DenseAttn a) {
     const int nq = a.heads * dk, nk = a.n_kv * dk, nv = a.n_kv * dv;
     float inv_q, inv_k;
     qk_sums(a, row, red, inv_q, inv_k);
-    inv_q *= temperature(a.temp_coef, a.temp_every, p);
+    inv_q *= temperature(a, p);
     // a warp per head and turn
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int h = warp; h < a.heads; h += 8)
+#pragma unroll 4
         for (int c = lane; c < ks; c += 32) {
             const int s = h * dk + c;
             const float v = c < dk ? row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f) : 0.0f;
@@ -92,6 +95,7 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const DenseAttn a) {
     if (p < 0 || p >= a.kv.max_seq) return;
     for (int g = warp; g < a.n_kv; g += 8) {
         const int64_t at = ((int64_t)b * a.n_kv + g) * a.kv.max_seq + p;
+#pragma unroll 4
         for (int c = lane; c < ks; c += 32) {
             const int s = g * dk + c;
             const float v = c < dk ? row[nq + s] * inv_k * (a.k_norm ? a.k_norm[s] : 1.0f) : 0.0f;
@@ -214,7 +218,7 @@ __global__ void __launch_bounds__(kSpanThreads) attn_span_kernel(const DenseAttn
         const float* row = a.qkv + r * a.ld;
         float inv_q, inv_k;
         qk_sums(a, row, red, inv_q, inv_k);
-        inv_q *= temperature(a.temp_coef, a.temp_every, p);
+        inv_q *= temperature(a, p);
         for (int i = threadIdx.x; i < NR * ks; i += kSpanThreads) {
             const int h = i / ks, c = i - h * ks, s = (g * rep + h0 + h) * dk + c;
             q_s[i] = (h < nr && c < dk) ? row[s] * inv_q * (a.q_norm ? a.q_norm[s] : 1.0f) : 0.0f;
@@ -476,7 +480,7 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
     auto copy_rows = [&](auto full, uint32_t dst, int dst_stride, const __nv_bfloat16* src, int stride, int pieces_rt, int base) {
         constexpr int kFull = decltype(full)::value;
         const int pieces = kFull ? kFull : pieces_rt;
-#pragma unroll 8
+#pragma unroll 4
         for (int e = lane; e < 16 * pieces; e += 32) {
             const int row = e / pieces, c = e - row * pieces;
             const bool live = base + row < t1 && (kFull || c * 8 < stride);
@@ -497,7 +501,7 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
     auto is_new = [&](int i) { return owner && warp + i * kMmaWarps == blocks - 1; };
     auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
     if (prepared) { ptx::pdl_wait(); }                           // the cache rows come from the kernel in front
-#pragma unroll
+#pragma unroll 1
     for (int i = 0; i < S - 1; ++i) { if (!is_new(i)) load(i); commit(); }
     if (!prepared) ptx::pdl_wait();
     ptx::pdl_launch_dependents();
@@ -507,7 +511,7 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
     const float* row = a.qkv + r * a.ld;
     if (!prepared) {
         qk_sums(a, row, red, inv_q, inv_k);
-        inv_q *= temperature(a.temp_coef, a.temp_every, p);
+        inv_q *= temperature(a, p);
     }
     const int kw = nk * 16;
     for (int c = threadIdx.x; c < kw; c += kMmaThreads) {
@@ -545,7 +549,7 @@ __global__ void __launch_bounds__(kMmaThreads) attn_span_mma_kernel(const DenseA
         }
     }
     __syncthreads();
-#pragma unroll
+#pragma unroll 1
     for (int i = 0; i < S - 1; ++i)
         if (is_new(i)) { load(i); commit(); }
 

@@ -118,6 +118,7 @@ struct DenseAttn {
     float eps = 0.f;
     float temp_coef = 0.f;          // q *= 1 + coef * ln(floor((pos + 1) / every) + 1)
     double temp_every = 1.0;
+    int temp_every_int = 0;         // the same where it is a whole number, else 0
     float v_lambda = 0.f;           // v = (1 - lambda) v + lambda v_first, when v_first_in is set
     const float* v_first_in = nullptr;
     float* v_first_out = nullptr;   // the projected v of the new tokens is kept here for later layers

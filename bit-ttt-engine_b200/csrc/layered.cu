@@ -169,6 +169,7 @@ DenseAttn attn_args(const bt_model* m, const LayLayer& l, const RowBuffers& r, i
     a.eps = m->lay->c.norm_eps;
     a.temp_coef = c.q_temp_coef;
     a.temp_every = c.q_temp_every;
+    a.temp_every_int = c.q_temp_every >= 1.0 && c.q_temp_every < 1e9 && c.q_temp_every == floor(c.q_temp_every) ? (int)c.q_temp_every : 0;
     a.v_lambda = l.vmix;
     a.v_first_in = l.v_target ? r.v_first : nullptr;
     a.v_first_out = l.v_source ? r.v_first : nullptr;

@@ -120,10 +120,10 @@ def layer_mix(cfg, t, tokens):
     return x + y
 
 
-@pytest.mark.parametrize("on", ["none", "qk_norm", "sink", "softcap", "q_temp", "plain_norm"])
+@pytest.mark.parametrize("on", ["none", "qk_norm", "sink", "softcap", "q_temp", "q_temp_fraction", "plain_norm"])
 def test_attention_mechanisms_alone(bt, on):
     c = lay.LayerConfig(A, 4, 24, kv_heads=2, dim=16, qk_norm=int(on == "qk_norm"), sink=int(on == "sink"), scale=0.5,
-                        softcap=1.5 if on == "softcap" else 0.0, q_temp_coef=0.7 if on == "q_temp" else 0.0, q_temp_every=9)
+                        softcap=1.5 if on == "softcap" else 0.0, q_temp_coef=0.7 if on.startswith("q_temp") else 0.0, q_temp_every=8.5 if on == "q_temp_fraction" else 9)
     cfg = lay.LayersConfig(50, 64, 120, 1e-5, on != "plain_norm", [c])
     t = make_tensors(cfg, seed=9)
     tokens = np.random.default_rng(9).integers(0, 50, 70).astype(np.int32)
