@@ -326,13 +326,15 @@ __device__ __forceinline__ void unpack16(uint32_t u, float& lo, float& hi) {
 // hidden vector itself, sum of squares in f64) and a running arg-max per CTA, so that the greedy pick does
 // not need a pass over all logits.  Ties keep the larger index (model/llama.rs:510-515).  HBM-bound on W:
 // one warp per output row, 16-byte loads, x in shared memory, f32 accumulation.
-template <int B, bool F16>
+// PAD: rows of w (and xs) are `ld_pad` apart instead of `hidden`.
+template <int B, bool F16, bool PAD>
 __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16* __restrict__ w,
                                                             const float* __restrict__ h,
                                                             const float* __restrict__ norm_w, float eps,
-                                                            int hidden, int ld, int64_t vocab, float* __restrict__ logits,
+                                                            int hidden, int ld_pad, int64_t vocab, float* __restrict__ logits,
                                                             float* __restrict__ cand_val,
                                                             int32_t* __restrict__ cand_idx) {
+    const int ld = PAD ? ld_pad : hidden;
     extern __shared__ float xs[];  // [B][ld], zero beyond hidden
     __shared__ double red_d[32];
     __shared__ float best_v[8][B];
@@ -354,7 +356,8 @@ __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16*
         const float denom = sqrtf(__fadd_rn((float)(ss / (double)hidden), eps));
         for (int c = threadIdx.x; c < hidden; c += blockDim.x)
             xs[b * ld + c] = __fmul_rn(__fdiv_rn(xs[b * ld + c], denom), norm_w[c]);
-        for (int c = hidden + threadIdx.x; c < ld; c += blockDim.x) xs[b * ld + c] = 0.0f;
+        if (PAD)
+            for (int c = hidden + threadIdx.x; c < ld; c += blockDim.x) xs[b * ld + c] = 0.0f;
     }
     __syncthreads();
     float bv[B];
@@ -521,24 +524,27 @@ cudaError_t launch_argmax(const float* logits, int batch, int vocab, int32_t* ou
 
 int lm_head_max_candidates(int sm_count) { return sm_count * 4; }
 
-template <int B, bool F16>
+template <int B, bool F16, bool PAD>
 static cudaError_t launch_lm_head_fused_bt(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                            int hidden, int ld, int64_t vocab, float* logits, float* cand_val,
                                            int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl) {
     const size_t smem = (size_t)B * ld * sizeof(float);
     static PerDeviceOnce once;
-    cudaError_t ce = once.run([] { return cudaFuncSetAttribute(lm_head_fused_kernel<B, F16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); });
+    cudaError_t ce = once.run([] { return cudaFuncSetAttribute(lm_head_fused_kernel<B, F16, PAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); });
     if (ce != cudaSuccess) return ce;
     if (smem > 200 * 1024) return cudaErrorInvalidConfiguration;
-    return launch_pdl(lm_head_fused_kernel<B, F16>, dim3(grid), dim3(256), smem, stream, pdl, w, h, norm_w, eps, hidden, ld,
+    return launch_pdl(lm_head_fused_kernel<B, F16, PAD>, dim3(grid), dim3(256), smem, stream, pdl, w, h, norm_w, eps, hidden, ld,
                       vocab, logits, cand_val, cand_idx);
 }
 template <int B>
 static cudaError_t launch_lm_head_fused_b(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                           int hidden, int ld, int64_t vocab, float* logits, float* cand_val,
                                           int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl, bool f16) {
-    return f16 ? launch_lm_head_fused_bt<B, true>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl)
-               : launch_lm_head_fused_bt<B, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
+    if (ld != hidden)  // bf16 tables only
+        return f16 ? cudaErrorInvalidValue
+                   : launch_lm_head_fused_bt<B, false, true>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
+    return f16 ? launch_lm_head_fused_bt<B, true, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl)
+               : launch_lm_head_fused_bt<B, false, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
 }
 
 cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
