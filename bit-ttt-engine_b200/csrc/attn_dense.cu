@@ -692,23 +692,37 @@ cudaError_t span_mma_launch_v(const DenseAttn& a, bool prepared, const ActOut& o
     return span_mma_launch<DK, 256>(a, prepared, out, s, pdl);
 }
 
-template <int DK, int DV>  // upper bounds of the (padded) head sizes
-__global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn a, const ActOut out) {
+// LATENT: keys and values are bf16 rows expanded from the latents, the last key columns the rotated part all heads share.
+struct LatentTile {
+    const __nv_bfloat16* kv = nullptr;  // [sequence][kv_rows][heads k_main | heads v_stride]
+    int64_t kv_ld = 0, kv_seq = 0;      // elements between positions and between sequences
+    int k_main = 0;                     // columns of a head's own key part
+    const uint8_t* rot = nullptr;       // tiled latent cache
+    int64_t rot_seq = 0;
+    int rot_col = 0, seq_pad = 0, b0 = 0;
+    const float* gate = nullptr;        // output gates of the rows
+    int64_t gate_ld = 0;
+};
+template <int DK, int DV, bool LATENT>  // upper bounds of the (padded) head sizes
+__global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn a, const LatentTile lt, const ActOut out) {
     extern __shared__ __align__(16) uint8_t tsm[];
     constexpr int KS = DK * 2 + 16, VS = DV * 2 + 16;  // bytes per row
     const uint32_t q_sm = ptx::smem_u32(tsm);
     const uint32_t k_sm = q_sm + kTileQ * KS, v_sm = k_sm + 2 * kTileKeys * KS;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int qt = gridDim.x - 1 - blockIdx.x;  // the longest first
-    const int head = blockIdx.y, b = blockIdx.z, g = head / (a.heads / a.n_kv);
+    const int head = blockIdx.y, b = blockIdx.z + (LATENT ? lt.b0 : 0), g = LATENT ? 0 : head / (a.heads / a.n_kv);
     const int ks = a.kv.k_stride, vs = a.kv.v_stride;
     const int nk = (ks + 15) / 16, nv = (vs + 15) / 16;  // 16-wide steps in use
     const int past = a.pos[b], q0 = qt * kTileQ, rows = min(kTileQ, a.q_rows - q0);
     const int last = past + q0 + rows - 1;               // last position any row of this tile sees
     const int key_tiles = last / kTileKeys + 1;
     const __nv_bfloat16* qg = reinterpret_cast<const __nv_bfloat16*>(a.q_buf) + (((int64_t)b * a.q_rows + q0) * a.heads + head) * ks;
-    const __nv_bfloat16* kg = reinterpret_cast<const __nv_bfloat16*>(a.kv.k) + ((int64_t)b * a.n_kv + g) * a.kv.max_seq * ks;
-    const __nv_bfloat16* vg = reinterpret_cast<const __nv_bfloat16*>(a.kv.v) + ((int64_t)b * a.n_kv + g) * a.kv.max_seq * vs;
+    const __nv_bfloat16* kg = LATENT ? lt.kv + blockIdx.z * lt.kv_seq + head * lt.k_main
+                                     : reinterpret_cast<const __nv_bfloat16*>(a.kv.k) + ((int64_t)b * a.n_kv + g) * a.kv.max_seq * ks;
+    const __nv_bfloat16* vg = LATENT ? lt.kv + blockIdx.z * lt.kv_seq + a.heads * lt.k_main + head * vs
+                                     : reinterpret_cast<const __nv_bfloat16*>(a.kv.v) + ((int64_t)b * a.n_kv + g) * a.kv.max_seq * vs;
+    const int64_t k_ld = LATENT ? lt.kv_ld : ks, v_ld = LATENT ? lt.kv_ld : vs;
 
     const int qpieces = nk * 2, vpieces = nv * 2;        // 16-byte pieces per row
     for (int i = threadIdx.x; i < kTileQ * qpieces; i += kTileThreads) {
@@ -721,12 +735,14 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         for (int i = threadIdx.x; i < kTileKeys * qpieces; i += kTileThreads) {
             const int r = i / qpieces, c = i - r * qpieces;
             const bool live = base + r <= last && c * 8 < ks;
-            ptx::cp16(k_sm + (bufi * kTileKeys + r) * KS + c * 16, live ? kg + (int64_t)(base + r) * ks + c * 8 : kg, live);
+            const void* src = kg + (int64_t)(base + r) * k_ld + c * 8;
+            if (LATENT && c * 8 >= lt.k_main) src = lt.rot + b * lt.rot_seq + dense_off(base + r, lt.rot_col + c * 8 - lt.k_main, lt.seq_pad);
+            ptx::cp16(k_sm + (bufi * kTileKeys + r) * KS + c * 16, live ? src : kg, live);
         }
         for (int i = threadIdx.x; i < kTileKeys * vpieces; i += kTileThreads) {
             const int r = i / vpieces, c = i - r * vpieces;
             const bool live = base + r <= last && c * 8 < vs;
-            ptx::cp16(v_sm + (bufi * kTileKeys + r) * VS + c * 16, live ? vg + (int64_t)(base + r) * vs + c * 8 : vg, live);
+            ptx::cp16(v_sm + (bufi * kTileKeys + r) * VS + c * 16, live ? vg + (int64_t)(base + r) * v_ld + c * 8 : vg, live);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -838,6 +854,8 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
             den = den * f[q] + expf(sk - m);
         }
         f[q] /= den;
+        const int lr = warp * 16 + (lane >> 2) + q * 8;
+        if (LATENT && lt.gate && lr < rows) f[q] /= 1.0f + expf(-lt.gate[((int64_t)b * a.q_rows + q0 + lr) * lt.gate_ld + head]);
     }
     const int dv = a.dv;
 #pragma unroll
@@ -858,21 +876,29 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
         }
 }
 
-template <int DK, int DV>
-cudaError_t tile_launch(const DenseAttn& a, const ActOut& out, cudaStream_t s) {
+template <int DK, int DV, bool LATENT>
+cudaError_t tile_launch(const DenseAttn& a, const LatentTile& lt, const ActOut& out, cudaStream_t s) {
     constexpr size_t smem = (size_t)kTileQ * (DK * 2 + 16) + 2 * kTileKeys * (DK * 2 + 16 + DV * 2 + 16);
     static PerDeviceOnce once;
-    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_tile_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); });
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_tile_kernel<DK, DV, LATENT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); });
     if (e != cudaSuccess) return e;
-    attn_tile_kernel<DK, DV><<<dim3((unsigned)((a.q_rows + kTileQ - 1) / kTileQ), (unsigned)a.heads, (unsigned)a.batch), kTileThreads, smem, s>>>(a, out);
+    attn_tile_kernel<DK, DV, LATENT><<<dim3((unsigned)((a.q_rows + kTileQ - 1) / kTileQ), (unsigned)a.heads, (unsigned)a.batch), kTileThreads, smem, s>>>(a, lt, out);
     return cudaGetLastError();
 }
-template <int DK>
-cudaError_t tile_launch_v(const DenseAttn& a, const ActOut& out, cudaStream_t s) {
-    if (a.kv.v_stride <= 64) return tile_launch<DK, 64>(a, out, s);
-    if (a.kv.v_stride <= 128) return tile_launch<DK, 128>(a, out, s);
-    return tile_launch<DK, 256>(a, out, s);
+template <int DK, bool LATENT>
+cudaError_t tile_launch_v(const DenseAttn& a, const LatentTile& lt, const ActOut& out, cudaStream_t s) {
+    if (a.kv.v_stride <= 64) return tile_launch<DK, 64, LATENT>(a, lt, out, s);
+    if (a.kv.v_stride <= 128) return tile_launch<DK, 128, LATENT>(a, lt, out, s);
+    return tile_launch<DK, 256, LATENT>(a, lt, out, s);
 }
+template <bool LATENT>
+cudaError_t tile_launch_k(const DenseAttn& a, const LatentTile& lt, const ActOut& out, cudaStream_t s) {
+    if (a.kv.k_stride <= 64) return tile_launch_v<64, LATENT>(a, lt, out, s);
+    if (a.kv.k_stride <= 128) return tile_launch_v<128, LATENT>(a, lt, out, s);
+    if (LATENT && a.kv.k_stride <= 192) return tile_launch_v<192, LATENT>(a, lt, out, s);
+    return tile_launch_v<256, LATENT>(a, lt, out, s);
+}
+int pad8(int n) { return (n + 7) / 8 * 8; }
 
 }  // namespace
 
@@ -898,9 +924,24 @@ bool attn_tile_fits(const DenseAttn& a) { return !a.kv.f32 && a.kv.k_stride <= 2
 
 cudaError_t launch_attn_tile(const DenseAttn& a, const ActOut& out, cudaStream_t s) {
     if (!attn_tile_fits(a) || !a.q_bf16 || !out.tiles) return cudaErrorInvalidValue;
-    if (a.kv.k_stride <= 64) return tile_launch_v<64>(a, out, s);
-    if (a.kv.k_stride <= 128) return tile_launch_v<128>(a, out, s);
-    return tile_launch_v<256>(a, out, s);
+    return tile_launch_k<false>(a, LatentTile(), out, s);
+}
+
+bool latent_tile_fits(const LatentAttn& a) { return !a.kv.f32 && pad8(a.dim) + pad8(a.rot) <= 256 && pad8(a.vdim) <= 256; }
+
+cudaError_t launch_latent_tile(const LatentAttn& l, const __nv_bfloat16* kv16, int64_t kv_rows, int b0, int nb, const ActOut& out, cudaStream_t s) {
+    if (!latent_tile_fits(l) || !l.q_buf || !out.tiles) return cudaErrorInvalidValue;
+    DenseAttn a;
+    a.q_buf = l.q_buf; a.q_bf16 = true;
+    a.scale = l.scale; a.pos = l.pos; a.batch = nb; a.q_rows = l.q_rows; a.heads = l.heads; a.n_kv = l.heads;
+    a.kv.k_stride = pad8(l.dim) + pad8(l.rot); a.kv.v_stride = pad8(l.vdim); a.kv.max_seq = l.kv.max_seq;
+    a.dk = a.kv.k_stride; a.dv = l.vdim;
+    LatentTile t;
+    t.kv = kv16; t.k_main = pad8(l.dim); t.kv_ld = (int64_t)l.heads * (t.k_main + a.kv.v_stride); t.kv_seq = kv_rows * t.kv_ld;
+    t.rot = reinterpret_cast<const uint8_t*>(l.kv.rows); t.rot_seq = l.kv.seq_bytes(); t.rot_col = dense_kpad(l.rank); t.seq_pad = l.kv.seq_pad; t.b0 = b0;
+    t.gate = l.gate ? l.proj + l.heads * (l.dim + l.rot) + l.rank + l.rot : nullptr;
+    t.gate_ld = l.ld;
+    return tile_launch_k<true>(a, t, out, s);
 }
 
 }  // namespace bt

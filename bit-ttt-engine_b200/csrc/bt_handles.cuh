@@ -41,6 +41,8 @@ struct bt_kv_cache {
     bool is_dense = false;
     int64_t v_dim = 0;
     bt::DenseKvView dense;
+    bool is_latent = false;  // bt_kv_create_latent: is_dense as well
+    bt::LatentView latent;
     size_t dense_bytes(int64_t stride) const { return (size_t)batch * n_kv * max_seq * stride * (dense.f32 ? 4 : 2); }
 };
 

@@ -33,7 +33,8 @@ cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const f
                                  int batch, int hidden, int64_t vocab, float* logits, float* cand_val,
                                  int32_t* cand_idx, int* n_cand, int sm_count, cudaStream_t stream, bool pdl,
                                  bool f16 = false,   // f16: w holds IEEE halves, not bf16
-                                 int ld = 0);        // row stride of w (multiple of 8, zero beyond hidden); 0: hidden
+                                 int ld = 0,         // row stride of w (multiple of 8, zero beyond hidden); 0: hidden
+                                 float cap = 0.f);   // logits <- cap * tanh(logits / cap); 0: none
 // Reduces the candidates to the greedy pick per token and advances the positions.
 cudaError_t launch_pick(const float* cand_val, const int32_t* cand_idx, int n_cand, int batch, int32_t* out,
                         int32_t* pos, int n_pos, cudaStream_t stream, bool pdl);
@@ -45,7 +46,8 @@ size_t lm_head_tc_act_bytes(int hidden);
 cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, void* tiles, cudaStream_t stream, int ld = 0);
 cudaError_t launch_lm_head_tc(const void* wtiles, const float* h, const float* norm_w, float eps, int batch, int hidden,
                               int64_t vocab, void* btiles, float* logits, unsigned int* err, int sm_count,
-                              cudaStream_t stream, bool w_f16 = false);  // w_f16: the weight tiles hold IEEE halves
+                              cudaStream_t stream, bool w_f16 = false,   // w_f16: the weight tiles hold IEEE halves
+                              float cap = 0.f);                          // logits <- cap * tanh(logits / cap); 0: none
 
 // Q8 KV cache of one layer: u8 data [batch, n_kv, max_seq, head_dim] and f32 scales
 // [batch, n_kv, max_seq] for K and V (layers/kv_cache.rs:14-24).

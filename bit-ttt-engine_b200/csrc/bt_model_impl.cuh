@@ -58,6 +58,7 @@ struct bt_model {
     bool embed_f16 = false, head_f16 = false;
     float* norm_f = nullptr;
     float rms_eps = kRmsEps;
+    float logit_cap = 0.f;           // logits <- cap * tanh(logits / cap); 0: none
     int head_ld = 0;                 // row stride of lm_head (0: hidden)
     int head_rows = 0;               // rows the head's buffers (h, logits, next) hold; >= max_batch
     bt::Layered* lay = nullptr;      // arch 2: per-layer mixers with dense projections (layered.cu)
@@ -122,9 +123,10 @@ bt_status layered_reset(bt_model* m);
 bt_status layered_set_tensor(bt_model* m, bt_tensor_kind kind, const float* data, int64_t n_elem, bt_dtype storage);
 bt_status layered_step(bt_model* m, int batch, cudaStream_t s);          // up to the residual stream in m->h
 bt_status layered_prefill_buffers(bt_model* m, int rows);
-bt_status layered_prefill(bt_model* m, int batch, int n, cudaStream_t s);  // up to the residual stream in m->pf_h
+bt_status layered_prefill(bt_model* m, int batch, int n, int past, cudaStream_t s);  // up to the residual stream in m->pf_h
 int layered_launches(const bt_model* m, int batch);
-bt_kv_cache* layered_kv(bt_model* m, int layer);
+int layered_runs(const bt_model* m);
+bt_kv_cache* layered_kv(bt_model* m, int run);
 // f32 host values -> 16-bit device storage (model.cu)
 bt_status upload_16bit(const float* host, int64_t n, __nv_bfloat16* dst, bool f16);
 }  // namespace bt

@@ -333,7 +333,7 @@ __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16*
                                                             const float* __restrict__ norm_w, float eps,
                                                             int hidden, int ld_pad, int64_t vocab, float* __restrict__ logits,
                                                             float* __restrict__ cand_val,
-                                                            int32_t* __restrict__ cand_idx) {
+                                                            int32_t* __restrict__ cand_idx, float cap) {
     const int ld = PAD ? ld_pad : hidden;
     extern __shared__ float xs[];  // [B][ld], zero beyond hidden
     __shared__ double red_d[32];
@@ -392,7 +392,8 @@ __global__ void __launch_bounds__(256) lm_head_fused_kernel(const __nv_bfloat16*
         }
 #pragma unroll
         for (int b = 0; b < B; ++b) {
-            const float r = warp_sum(acc[b]);
+            float r = warp_sum(acc[b]);
+            if (PAD && cap > 0.0f) r = cap * tanhf(r / cap);
             if (lane == 0) logits[(int64_t)b * vocab + v] = r;
             if (r >= bv[b]) { bv[b] = r; bi[b] = (int)v; }  // v increases: ties keep the later index
         }
@@ -527,29 +528,29 @@ int lm_head_max_candidates(int sm_count) { return sm_count * 4; }
 template <int B, bool F16, bool PAD>
 static cudaError_t launch_lm_head_fused_bt(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                            int hidden, int ld, int64_t vocab, float* logits, float* cand_val,
-                                           int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl) {
+                                           int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl, float cap) {
     const size_t smem = (size_t)B * ld * sizeof(float);
     static PerDeviceOnce once;
     cudaError_t ce = once.run([] { return cudaFuncSetAttribute(lm_head_fused_kernel<B, F16, PAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); });
     if (ce != cudaSuccess) return ce;
     if (smem > 200 * 1024) return cudaErrorInvalidConfiguration;
     return launch_pdl(lm_head_fused_kernel<B, F16, PAD>, dim3(grid), dim3(256), smem, stream, pdl, w, h, norm_w, eps, hidden, ld,
-                      vocab, logits, cand_val, cand_idx);
+                      vocab, logits, cand_val, cand_idx, cap);
 }
 template <int B>
 static cudaError_t launch_lm_head_fused_b(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                           int hidden, int ld, int64_t vocab, float* logits, float* cand_val,
-                                          int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl, bool f16) {
-    if (ld != hidden)  // bf16 tables only
+                                          int32_t* cand_idx, int grid, cudaStream_t stream, bool pdl, bool f16, float cap) {
+    if (ld != hidden || cap > 0.0f)  // bf16 tables only
         return f16 ? cudaErrorInvalidValue
-                   : launch_lm_head_fused_bt<B, false, true>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
-    return f16 ? launch_lm_head_fused_bt<B, true, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl)
-               : launch_lm_head_fused_bt<B, false, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl);
+                   : launch_lm_head_fused_bt<B, false, true>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl, cap);
+    return f16 ? launch_lm_head_fused_bt<B, true, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl, cap)
+               : launch_lm_head_fused_bt<B, false, false>(w, h, norm_w, eps, hidden, ld, vocab, logits, cand_val, cand_idx, grid, stream, pdl, cap);
 }
 
 cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const float* norm_w, float eps,
                                  int batch, int hidden, int64_t vocab, float* logits, float* cand_val,
-                                 int32_t* cand_idx, int* n_cand, int sm_count, cudaStream_t stream, bool pdl, bool f16, int ld) {
+                                 int32_t* cand_idx, int* n_cand, int sm_count, cudaStream_t stream, bool pdl, bool f16, int ld, float cap) {
     if (ld == 0) ld = hidden;
     if (ld % 8 != 0 || ld < hidden || batch < 1) return cudaErrorInvalidValue;
     // one grid size for every group of tokens, so that the candidate rows share a stride
@@ -567,14 +568,14 @@ cudaError_t launch_lm_head_fused(const __nv_bfloat16* w, const float* h, const f
         int32_t* ci = cand_idx + (size_t)b0 * grid;
         cudaError_t e;
         switch (bc) {
-            case 1: e = launch_lm_head_fused_b<1>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 2: e = launch_lm_head_fused_b<2>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 3: e = launch_lm_head_fused_b<3>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 4: e = launch_lm_head_fused_b<4>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 5: e = launch_lm_head_fused_b<5>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 6: e = launch_lm_head_fused_b<6>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            case 7: e = launch_lm_head_fused_b<7>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
-            default: e = launch_lm_head_fused_b<8>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16); break;
+            case 1: e = launch_lm_head_fused_b<1>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            case 2: e = launch_lm_head_fused_b<2>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            case 3: e = launch_lm_head_fused_b<3>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            case 4: e = launch_lm_head_fused_b<4>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            case 5: e = launch_lm_head_fused_b<5>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            case 6: e = launch_lm_head_fused_b<6>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            case 7: e = launch_lm_head_fused_b<7>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
+            default: e = launch_lm_head_fused_b<8>(w, hb, norm_w, eps, hidden, ld, vocab, lb, cv, ci, grid, stream, pdl, f16, cap); break;
         }
         if (e != cudaSuccess) return e;
     }

@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(256) lm_prep_kernel(const float* __restrict__ 
 __global__ void __launch_bounds__(kThreads, 1) lm_head_tc_kernel(const uint8_t* __restrict__ wtiles,
                                                                  const uint8_t* __restrict__ btiles, int64_t vocab,
                                                                  int hidden, int m, float* __restrict__ logits,
-                                                                 unsigned int* err, bool w_f16) {
+                                                                 unsigned int* err, bool w_f16, float cap) {
     extern __shared__ __align__(128) uint8_t smem[];
     uint8_t* stage_base = smem;  // kStages x (A tile | B tile)
     uint64_t* full = reinterpret_cast<uint64_t*>(stage_base + (size_t)kStages * (kATile + kBTile));
@@ -174,8 +174,11 @@ __global__ void __launch_bounds__(kThreads, 1) lm_head_tc_kernel(const uint8_t* 
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
                     const int token = c0 + j;
-                    if (token < m && v < vocab)
-                        logits[(int64_t)token * vocab + v] = __fadd_rn(__uint_as_float(hi[j]), __uint_as_float(lo[j]));
+                    if (token < m && v < vocab) {
+                        float r = __fadd_rn(__uint_as_float(hi[j]), __uint_as_float(lo[j]));
+                        if (cap > 0.0f) r = cap * tanhf(r / cap);
+                        logits[(int64_t)token * vocab + v] = r;
+                    }
                 }
             }
             ptx::tc_fence_before();
@@ -203,7 +206,7 @@ cudaError_t launch_lm_retile(const __nv_bfloat16* w, int64_t vocab, int hidden, 
 // logits for up to 64 tokens per pass; h: [batch, hidden] residual stream (RMSNorm applied here)
 cudaError_t launch_lm_head_tc(const void* wtiles, const float* h, const float* norm_w, float eps, int batch, int hidden,
                               int64_t vocab, void* btiles, float* logits, unsigned int* err, int sm_count,
-                              cudaStream_t stream, bool w_f16) {
+                              cudaStream_t stream, bool w_f16, float cap) {
     const size_t smem = (size_t)kStages * (kATile + kBTile) + 256;
     static PerDeviceOnce once;
     cudaError_t ce = once.run([smem] { return cudaFuncSetAttribute(lm_head_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); });
@@ -216,7 +219,7 @@ cudaError_t launch_lm_head_tc(const void* wtiles, const float* h, const float* n
                                                  reinterpret_cast<uint8_t*>(btiles), w_f16);
         lm_head_tc_kernel<<<grid, kThreads, smem, stream>>>(reinterpret_cast<const uint8_t*>(wtiles),
                                                            reinterpret_cast<const uint8_t*>(btiles), vocab, hidden, bc,
-                                                           logits + (size_t)b0 * vocab, err, w_f16);
+                                                           logits + (size_t)b0 * vocab, err, w_f16, cap);
     }
     return cudaGetLastError();
 }

@@ -272,7 +272,7 @@ bt_status enqueue_head(bt_model* m, int batch, cudaStream_t s, bool fused_launch
     }
     if (tc) {
         BT_CUDA_TRY(launch_lm_head_tc(m->lm_tiles, m->h, m->norm_f, m->rms_eps, batch, H, c.vocab_size, m->lm_btiles, m->logits,
-                                      err, sm, s, m->head_f16));
+                                      err, sm, s, m->head_f16, m->logit_cap));
         BT_CUDA_TRY(launch_argmax(m->logits, batch, c.vocab_size, m->next, s));
         if (advance) advance_pos_kernel<<<1, 64, 0, s>>>(m->pos, B);
         BT_CUDA_TRY(cudaGetLastError());
@@ -280,7 +280,7 @@ bt_status enqueue_head(bt_model* m, int batch, cudaStream_t s, bool fused_launch
     }
     int n_cand = 0;
     BT_CUDA_TRY(launch_lm_head_fused(m->lm_head, m->h, m->norm_f, m->rms_eps, batch, H, c.vocab_size, m->logits,
-                                     m->cand_val, m->cand_idx, &n_cand, sm, s, fused_launches, m->head_f16, m->head_ld));
+                                     m->cand_val, m->cand_idx, &n_cand, sm, s, fused_launches, m->head_f16, m->head_ld, m->logit_cap));
     BT_CUDA_TRY(launch_pick(m->cand_val, m->cand_idx, n_cand, batch, m->next, m->pos, advance ? B : 0, s, fused_launches));
     return BT_OK;
 }
@@ -840,7 +840,7 @@ bt_status prefill_buffers(bt_model* m, int rows) {
 // (model/block.rs:87-134 applied to a [batch, n, hidden] input, cache semantics of model/llama.rs:495-498).
 bt_status enqueue_prefill_chunk(bt_model* m, int batch, int n, int past, int ttt_chunk, cudaStream_t s) {
     const bt_model_config& c = m->cfg;
-    if (m->lay) return layered_prefill(m, batch, n, s);
+    if (m->lay) return layered_prefill(m, batch, n, past, s);
     const int H = c.hidden_dim, I = m->i_l, M = batch * n;
     unsigned int* err = device_error_word(m->device);
     const int sm = m->sm_count;
@@ -1014,7 +1014,7 @@ extern "C" bt_kv_cache* bt_model_kv_cache(bt_model* m, int layer) {
     return m->layers[(size_t)layer].kv;
 }
 extern "C" int64_t bt_model_trace_floats(const bt_model* m, int rows) {
-    return (m && m->finalized && rows > 0) ? trace_layer_floats(m, rows) * m->cfg.num_layers : 0;
+    return (m && m->finalized && rows > 0) ? trace_layer_floats(m, rows) * (m->lay ? layered_runs(m) : m->cfg.num_layers) : 0;
 }
 extern "C" bt_status bt_model_set_trace(bt_model* m, float* trace_dev, int rows) {
     if (!m || !m->finalized) return set_error(BT_ERR_ARG, "bt_model_set_trace: model not finalized");

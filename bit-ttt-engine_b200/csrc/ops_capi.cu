@@ -104,12 +104,71 @@ extern "C" bt_status bt_kv_create_dense(bt_kv_cache** out, int64_t batch, int64_
     return bt_kv_reset(c);
 }
 
+extern "C" bt_status bt_kv_create_latent(bt_kv_cache** out, int64_t batch, int64_t rank, int64_t rot, int64_t max_seq_len,
+                                         bt_dtype dtype, int device) {
+    if (!out) return set_error(BT_ERR_ARG, "bt_kv_create_latent: null out pointer");
+    *out = nullptr;
+    if (batch < 1 || rank < 1 || rot < 1 || max_seq_len < 1 || rank > latent_max_rank() || rot > latent_max_rot())
+        return set_error(BT_ERR_SHAPE, "bt_kv_create_latent: rank %lld (at most %d), rotated part %lld (at most %d)", (long long)rank, latent_max_rank(), (long long)rot, latent_max_rot());
+    if (dtype != BT_BF16 && dtype != BT_F32) return set_error(BT_ERR_ARG, "bt_kv_create_latent: dtype must be BT_BF16 or BT_F32");
+    if (bt_device_count() <= device || device < 0) return set_error(BT_ERR_DEVICE, "bt_kv_create_latent: no CUDA device %d", device);
+    DeviceGuard guard(device);
+    if (!guard.ok) return set_error(BT_ERR_DEVICE, "cannot select device %d", device);
+    bt_kv_cache* c = new (std::nothrow) bt_kv_cache();
+    if (!c) return set_error(BT_ERR_NOMEM, "host allocation failed");
+    c->device = device;
+    c->batch = batch; c->n_kv = 1; c->head_dim = rank; c->v_dim = rot; c->max_seq = max_seq_len;
+    c->is_dense = c->is_latent = true;
+    LatentView& l = c->latent;
+    l.max_seq = (int)max_seq_len;
+    l.seq_pad = (int)((max_seq_len + 255) / 256 * 256);
+    l.rank = (int)rank; l.rot = (int)rot; l.stride = (int)((rank + rot + 3) / 4 * 4);
+    l.f32 = dtype == BT_F32;
+    cudaError_t e = cudaMalloc(&l.rows, (size_t)(batch * l.seq_bytes()));
+    if (e != cudaSuccess) {
+        bt_kv_destroy(c);
+        return set_error(BT_ERR_NOMEM, "bt_kv_create_latent: %s", cudaGetErrorString(e));
+    }
+    *out = c;
+    return bt_kv_reset(c);
+}
+
 namespace {
+// rows [0, t_len) of sequence b between host f32 [t_len, rank] / [t_len, rot] and a latent cache
+bt_status latent_rows(bt_kv_cache* c, int64_t b, int64_t t_len, float* rank_host, float* rot_host, bool store) {
+    DeviceGuard guard(c->device);
+    BT_CUDA_TRY(cudaDeviceSynchronize());
+    const LatentView& l = c->latent;
+    std::vector<uint8_t> tmp((size_t)l.seq_bytes());
+    uint8_t* dev = reinterpret_cast<uint8_t*>(l.rows) + b * l.seq_bytes();
+    BT_CUDA_TRY(cudaMemcpy(tmp.data(), dev, tmp.size(), cudaMemcpyDeviceToHost));
+    for (int which = 0; which < 2; ++which) {
+        float* host = which ? rot_host : rank_host;
+        const int dim = which ? l.rot : l.rank;
+        if (!host) continue;
+        for (int64_t t = 0; t < t_len; ++t)
+            for (int j = 0; j < dim; ++j) {
+                float& hv = host[t * dim + j];
+                if (l.f32) {
+                    uint8_t* p = tmp.data() + (t * l.stride + (which ? l.rank : 0) + j) * 4;
+                    if (store) memcpy(p, &hv, 4); else memcpy(&hv, p, 4);
+                } else {
+                    uint8_t* p = tmp.data() + dense_off(t, (which ? dense_kpad(l.rank) : 0) + j, l.seq_pad);
+                    __nv_bfloat16 q = __float2bfloat16_rn(hv);
+                    if (store) memcpy(p, &q, 2);
+                    else { memcpy(&q, p, 2); hv = __bfloat162float(q); }
+                }
+            }
+    }
+    if (store) BT_CUDA_TRY(cudaMemcpy(dev, tmp.data(), tmp.size(), cudaMemcpyHostToDevice));
+    return BT_OK;
+}
 // rows [0, t_len) of sequence b between host f32 [n_kv, t_len, dim] and the cache's padded rows
 bt_status dense_rows(bt_kv_cache* c, int64_t b, int64_t t_len, float* k_host, float* v_host, bool store) {
     if (!c || !c->is_dense) return set_error(BT_ERR_ARG, "bt_kv_*_dense: null handle or a quantised cache");
     if (b < 0 || b >= c->batch || t_len < 0 || t_len > c->max_seq)
         return set_error(BT_ERR_SHAPE, "bt_kv_*_dense: sequence %lld / length %lld out of range", (long long)b, (long long)t_len);
+    if (c->is_latent) return latent_rows(c, b, t_len, k_host, v_host, store);
     DeviceGuard guard(c->device);
     BT_CUDA_TRY(cudaDeviceSynchronize());
     for (int which = 0; which < 2; ++which) {
@@ -149,6 +208,10 @@ extern "C" bt_status bt_kv_import_dense(bt_kv_cache* c, int64_t b, int64_t t_len
 extern "C" bt_status bt_kv_reset(bt_kv_cache* c) {
     if (!c) return set_error(BT_ERR_ARG, "bt_kv_reset: null handle");
     DeviceGuard guard(c->device);
+    if (c->is_latent) {
+        BT_CUDA_TRY(cudaMemset(c->latent.rows, 0, (size_t)(c->batch * c->latent.seq_bytes())));
+        return BT_OK;
+    }
     if (c->is_dense) {
         BT_CUDA_TRY(cudaMemset(c->dense.k, 0, c->dense_bytes(c->dense.k_stride)));
         BT_CUDA_TRY(cudaMemset(c->dense.v, 0, c->dense_bytes(c->dense.v_stride)));
@@ -167,7 +230,7 @@ extern "C" bt_status bt_kv_destroy(bt_kv_cache* c) {
     DeviceGuard guard(c->device);
     cudaFree(c->view.k_q); cudaFree(c->view.v_q); cudaFree(c->view.k_s); cudaFree(c->view.v_s);
     cudaFree(c->inv_freq); cudaFree(c->rope_cos); cudaFree(c->rope_sin);
-    cudaFree(c->dense.k); cudaFree(c->dense.v);
+    cudaFree(c->dense.k); cudaFree(c->dense.v); cudaFree(c->latent.rows);
     delete c;
     return BT_OK;
 }

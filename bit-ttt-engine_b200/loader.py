@@ -283,7 +283,7 @@ def load_model(path: str, max_batch: int = 1, device: int = 0, dtype: str | None
     if design is not None:
         if design not in DESIGNS:
             raise CheckpointError(f"config: unknown architecture {design!r} (known: {', '.join(sorted(DESIGNS))})")
-        return build_layered(DESIGNS[design](d), tensors, max_batch=max_batch, device=device, dtype=dtype or "bfloat16",
+        return build_layered(DESIGNS[design](d, tensors), tensors, max_batch=max_batch, device=device, dtype=dtype or "bfloat16",
                              max_seq_len=max_seq_len)
     if dtype == "float32":
         raise CheckpointError("ternary models quantise their activations to 8 bits: there is no 32-bit form of them")

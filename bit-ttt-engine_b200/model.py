@@ -12,11 +12,15 @@ from .layers import _ptr, _stream_ptr, _torch
 
 ARCH_TTT, ARCH_LLAMA = 0, 1
 (W_Q, W_K, W_V, W_O, W_GATE, W_UP, W_DOWN, W_TTT_DOWN, W_TTT_UP) = range(9)
-(T_EMBED, T_LM_HEAD, T_NORM_F, T_NORM1, T_NORM2, T_POS) = range(6)
-MIX_ATTENTION, MIX_SSM = 0, 1
-MLP_NONE, MLP_DENSE_RELU2 = 0, 1
+(T_EMBED, T_LM_HEAD, T_NORM_F, T_NORM1, T_NORM2, T_POS, T_LOOP_IN, T_LOOP_STEP) = range(8)
+MIX_ATTENTION, MIX_SSM, MIX_LATENT, MIX_WKV, MIX_RGLRU = range(5)
+MLP_NONE, MLP_DENSE_RELU2, MLP_MOE_SWIGLU = range(3)
 (LT_NORM1, LT_NORM2, LT_Q, LT_K, LT_V, LT_O, LT_Q_NORM, LT_K_NORM, LT_SINK, LT_VMIX, LT_SSM_IN, LT_SSM_CONV,
- LT_SSM_CONV_B, LT_SSM_DT_BIAS, LT_SSM_A_LOG, LT_SSM_D, LT_SSM_NORM, LT_SSM_O, LT_MLP_UP, LT_MLP_DOWN) = range(20)
+ LT_SSM_CONV_B, LT_SSM_DT_BIAS, LT_SSM_A_LOG, LT_SSM_D, LT_SSM_NORM, LT_SSM_O, LT_MLP_UP, LT_MLP_DOWN, LT_PRE1, LT_PRE2,
+ LT_DKV, LT_DKV_NORM, LT_UK, LT_UV, LT_GATE, LT_MU_R, LT_MU_K, LT_MU_V, LT_MU_G, LT_MU_W, LT_WKV_R, LT_WKV_K, LT_WKV_V,
+ LT_WKV_G, LT_WKV_W1, LT_WKV_W2, LT_WKV_W0, LT_WKV_U, LT_WKV_NORM, LT_RG_Y, LT_RG_Y_B, LT_RG_X, LT_RG_X_B, LT_RG_CONV,
+ LT_RG_CONV_B, LT_RG_RA, LT_RG_RA_B, LT_RG_RI, LT_RG_RI_B, LT_RG_LAM, LT_ROUTER, LT_ROUTER_B, LT_E_GATE, LT_E_UP, LT_E_DOWN,
+ LT_S_GATE, LT_S_UP, LT_S_DOWN) = range(60)
 
 
 class _CModelConfig(C.Structure):
@@ -32,13 +36,16 @@ class _CLayerConfig(C.Structure):
                 ("qk_norm", C.c_int), ("sink", C.c_int), ("v_mix", C.c_int), ("scale", C.c_float),
                 ("softcap", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_double),
                 ("state", C.c_int), ("groups", C.c_int), ("conv_taps", C.c_int), ("norm_groups", C.c_int),
-                ("mlp", C.c_int), ("ff", C.c_int)]
+                ("mlp", C.c_int), ("ff", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("shared_ff", C.c_int),
+                ("rot_dim", C.c_int), ("rot_dims", C.c_int), ("kv_rank", C.c_int), ("out_gate", C.c_int),
+                ("rot_base", C.c_double), ("decay_rank", C.c_int), ("channels", C.c_int), ("blocks", C.c_int)]
 
 
 class _CLayersConfig(C.Structure):
     _fields_ = [("vocab_size", C.c_int), ("width", C.c_int), ("num_layers", C.c_int), ("max_positions", C.c_int),
                 ("max_seq_len", C.c_int), ("max_batch", C.c_int), ("norm_eps", C.c_float),
-                ("norm_one_plus", C.c_int), ("dtype", C.c_int)]
+                ("norm_one_plus", C.c_int), ("dtype", C.c_int), ("pre_norm", C.c_int), ("loop_start", C.c_int),
+                ("loop_stop", C.c_int), ("loop_times", C.c_int), ("logit_softcap", C.c_float)]
 
 
 def _bind():
@@ -84,6 +91,8 @@ def _bind():
     L.bt_kv_import_dense.argtypes = [vp, i64, i64, vp, vp]
     L.bt_model_create_layers.argtypes = [C.POINTER(vp), C.POINTER(_CLayersConfig), C.POINTER(_CLayerConfig), i32]
     L.bt_model_set_layer_tensor.argtypes = [vp, i32, i32, vp, i64]
+    L.bt_model_set_expert_tensor.argtypes = [vp, i32, i32, i32, vp, i64]
+    L.bt_model_layer_runs.argtypes = [vp]
     L.bt_model_enqueue_parts.argtypes = [vp, i32, i32, i32, vp]
     L.bt_model_recurrent_state.restype = vp
     L.bt_model_recurrent_state.argtypes = [vp, i32, C.POINTER(i64)]
@@ -487,37 +496,51 @@ class BitLlama(DeviceModel):
 
 class LayeredLM(DeviceModel):
     """A decoder given as a list of layers (layered.py): dense projections, a mixer per layer, caches and recurrent
-    states per layer behind the same step, prefill and pick as `BitLlama`.  dtype "bfloat16" or "float32"."""
+    states per layer run behind the same step, prefill and pick as `BitLlama`.  dtype "bfloat16" or "float32"."""
+
+    DEFAULT_SEQ_LEN = 4096  # positions the caches hold where neither the caller nor a position table says
 
     def __init__(self, cfg, max_batch: int = 1, device: int = 0, dtype: str = "bfloat16", max_seq_len: int | None = None):
         self._L = _bind()
         self.cfg, self.max_batch, self.device, self.dtype = cfg, max_batch, device, dtype
-        self.max_seq_len = min(max_seq_len or cfg.max_positions, cfg.max_positions)
+        self.max_seq_len = max_seq_len or cfg.max_positions or self.DEFAULT_SEQ_LEN
+        if cfg.max_positions:
+            self.max_seq_len = min(self.max_seq_len, cfg.max_positions)
         if dtype not in ("bfloat16", "float32"):
             raise ValueError(f"dtype {dtype!r} is neither bfloat16 nor float32")
+        start, stop, times = cfg.loop or (0, 0, 0)
         cc = _CLayersConfig(cfg.vocab_size, cfg.width, len(cfg.layers), cfg.max_positions, self.max_seq_len, max_batch,
-                            cfg.norm_eps, int(cfg.norm_one_plus), BT_F32 if dtype == "float32" else BT_BF16)
+                            cfg.norm_eps, int(cfg.norm_one_plus), BT_F32 if dtype == "float32" else BT_BF16,
+                            int(cfg.pre_norm), start, stop, times, cfg.logit_softcap)
         lc = (_CLayerConfig * len(cfg.layers))(*[_CLayerConfig(*[getattr(layer, name) for name, _ in _CLayerConfig._fields_])
                                                  for layer in cfg.layers])
         self._h = C.c_void_p()
         check(self._L.bt_model_create_layers(C.byref(self._h), C.byref(cc), lc, device))
 
+    @property
+    def runs(self) -> list:
+        """The layer of every layer run, in the order they run (a looped layer comes once per pass)."""
+        return self.cfg.runs()
+
     def set_tensor(self, kind: int, data: np.ndarray):
         data = np.ascontiguousarray(data, np.float32)
         check(self._L.bt_model_set_tensor(self._h, kind, 0, data.ctypes.data, data.size))
 
-    def set_layer_tensor(self, layer: int, kind: int, data: np.ndarray):
+    def set_layer_tensor(self, layer: int, kind: int, data: np.ndarray, expert: int | None = None):
         data = np.ascontiguousarray(data, np.float32)
-        check(self._L.bt_model_set_layer_tensor(self._h, layer, kind, data.ctypes.data, data.size))
+        if expert is None:
+            check(self._L.bt_model_set_layer_tensor(self._h, layer, kind, data.ctypes.data, data.size))
+        else:
+            check(self._L.bt_model_set_expert_tensor(self._h, layer, expert, kind, data.ctypes.data, data.size))
 
-    PART_IN, PART_CORE, PART_O, PART_UP, PART_DOWN, PART_ROWS = 1, 2, 4, 8, 16, 32
+    PART_IN, PART_CORE, PART_O, PART_UP, PART_DOWN, PART_ROWS, PART_MID, PART_ROUTE, PART_LOOP = (1 << i for i in range(9))
 
     def enqueue_parts(self, batch: int, n_tokens: int, parts: int) -> None:
         """Measurement aid: some of the launches of a step or of a prefill chunk already run (bt_model_enqueue_parts)."""
         check(self._L.bt_model_enqueue_parts(self._h, batch, n_tokens, parts, _stream_ptr(self.device)))
 
     def set_trace(self, on: bool = True, rows: int = 0) -> None:
-        """Keep the residual stream after every layer of the following steps (rows: see BitLlama.set_trace)."""
+        """Keep the residual stream after every layer run of the following steps (rows: see BitLlama.set_trace)."""
         torch = _torch()
         if on:
             self._trace_rows = max(rows, self.max_batch)
@@ -528,36 +551,46 @@ class LayeredLM(DeviceModel):
             check(self._L.bt_model_set_trace(self._h, None, 0))
 
     def read_trace(self, rows: int) -> np.ndarray:
-        """[layers, rows, width] of the last traced step or prefill (rows ordered [sequence][token])."""
+        """[layer runs, rows, width] of the last traced step or prefill (rows ordered [sequence][token])."""
         torch = _torch()
         torch.cuda.synchronize(self.device)
-        return self._trace.cpu().numpy().reshape(len(self.cfg.layers), self._trace_rows, self.cfg.width)[:, :rows].copy()
+        return self._trace.cpu().numpy().reshape(len(self.runs), self._trace_rows, self.cfg.width)[:, :rows].copy()
 
-    def kv_rows(self, layer: int, b: int, t_len: int):
-        """Cached keys and values of one sequence, f32 [kv_heads, t_len, dim] and [kv_heads, t_len, vdim]."""
-        p = self._L.bt_model_kv_cache(self._h, layer)
-        c = self.cfg.layers[layer]
-        k = np.zeros((c.kv_heads, t_len, c.dim), np.float32)
-        v = np.zeros((c.kv_heads, t_len, c.vdim), np.float32)
+    def _kv_shapes(self, run: int, t_len: int):
+        c = self.cfg.layers[self.runs[run]]
+        if c.mixer == MIX_LATENT:
+            return (t_len, c.kv_rank), (t_len, c.rot_dim)
+        return (c.kv_heads, t_len, c.dim), (c.kv_heads, t_len, c.vdim)
+
+    def kv_rows(self, run: int, b: int, t_len: int):
+        """What a layer run caches of one sequence, f32: keys and values [kv_heads, t_len, dim] and [kv_heads, t_len, vdim],
+        or latents [t_len, kv_rank] and rotated key parts [t_len, rot_dim]."""
+        p = self._L.bt_model_kv_cache(self._h, run)
+        k, v = (np.zeros(shape, np.float32) for shape in self._kv_shapes(run, t_len))
         check(self._L.bt_kv_export_dense(p, b, t_len, k.ctypes.data, v.ctypes.data))
         return k, v
 
-    def load_kv_rows(self, layer: int, b: int, k: np.ndarray, v: np.ndarray) -> None:
+    def load_kv_rows(self, run: int, b: int, k: np.ndarray, v: np.ndarray) -> None:
         k, v = np.ascontiguousarray(k, np.float32), np.ascontiguousarray(v, np.float32)
-        check(self._L.bt_kv_import_dense(self._L.bt_model_kv_cache(self._h, layer), b, k.shape[1], k.ctypes.data, v.ctypes.data))
+        check(self._L.bt_kv_import_dense(self._L.bt_model_kv_cache(self._h, run), b, k.shape[-2], k.ctypes.data, v.ctypes.data))
 
-    def recurrent_state(self, layer: int):
-        """(state, convolution ring) of a recurrent layer as device views, None for attention layers."""
+    def recurrent_state(self, run: int):
+        """(state, last inputs) of a recurrent layer run as device views (bt_model_recurrent_state), None for attention."""
         torch = _torch()
         n, r = C.c_int64(0), C.c_int64(0)
-        p = self._L.bt_model_recurrent_state(self._h, layer, C.byref(n))
-        q = self._L.bt_model_conv_ring(self._h, layer, C.byref(r))
+        p = self._L.bt_model_recurrent_state(self._h, run, C.byref(n))
+        q = self._L.bt_model_conv_ring(self._h, run, C.byref(r))
         if not p:
             return None
-        c = self.cfg.layers[layer]
-        inner = c.heads * c.vdim
-        return (_wrap_dev(p, (self.max_batch, c.heads, c.vdim, n.value // (self.max_batch * inner)), torch.float32, self.device),
-                _wrap_dev(q, (self.max_batch, c.conv_taps, inner + 2 * c.groups * c.state), torch.float32, self.device))
+        c, B = self.cfg.layers[self.runs[run]], self.max_batch
+        if c.mixer == MIX_SSM:
+            inner = c.heads * c.vdim
+            shapes = (B, c.heads, c.vdim, n.value // (B * inner)), (B, c.conv_taps, inner + 2 * c.groups * c.state)
+        elif c.mixer == MIX_WKV:
+            shapes = (B, c.heads, c.dim, c.dim), (2, B, self.cfg.width)
+        else:
+            shapes = (B, c.channels), (B, c.conv_taps, c.channels)
+        return tuple(_wrap_dev(x, shape, torch.float32, self.device) for x, shape in zip((p, q), shapes))
 
     def save_memory(self, path: str) -> None:
         """Caches, recurrent states and the position to a safetensors file, so that the sequences can be resumed without
@@ -566,7 +599,7 @@ class LayeredLM(DeviceModel):
         torch = _torch()
         torch.cuda.synchronize(self.device)
         t_len, tensors = self.current_pos, {"position": np.array([self.current_pos], np.int32)}
-        for li in range(len(self.cfg.layers)):
+        for li in range(len(self.runs)):
             st = self.recurrent_state(li)
             if st is not None:
                 tensors[f"state_{li}"], tensors[f"conv_{li}"] = st[0].cpu().numpy(), st[1].cpu().numpy()
@@ -583,13 +616,13 @@ class LayeredLM(DeviceModel):
         if not 0 <= t_len < self.max_seq_len:
             raise CheckpointError(f"{path}: position {t_len} outside 0..{self.max_seq_len - 1}")
         torch.cuda.synchronize(self.device)
-        for li, c in enumerate(self.cfg.layers):
+        for li in range(len(self.runs)):
             st = self.recurrent_state(li)
             names = (f"state_{li}", f"conv_{li}") if st is not None else (f"kv_{li}.k", f"kv_{li}.v")
             if st is None and t_len == 0:
                 continue
             want = [tuple(x.shape) for x in st] if st is not None else \
-                [(self.max_batch, c.kv_heads, t_len, d) for d in (c.dim, c.vdim)]
+                [(self.max_batch, *shape) for shape in self._kv_shapes(li, t_len)]
             for name, shape in zip(names, want):
                 if name not in tensors or tuple(tensors[name].shape) != shape:
                     raise CheckpointError(f"{path}: {name} is missing or not of shape {shape}")

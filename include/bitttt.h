@@ -210,6 +210,10 @@ bt_status bt_kv_import(bt_kv_cache* cache, int64_t b, int64_t t_len, const uint8
  * (either may be NULL); synchronous. */
 bt_status bt_kv_create_dense(bt_kv_cache** out, int64_t batch, int64_t n_kv_heads, int64_t k_dim, int64_t v_dim,
                              int64_t max_seq_len, bt_dtype dtype, int device);
+/* The cache of latent attention: one latent row of `rank` and one rotated key part of `rot` values per position; export and
+ * import move them as [t_len, rank] (keys) and [t_len, rot] (values). */
+bt_status bt_kv_create_latent(bt_kv_cache** out, int64_t batch, int64_t rank, int64_t rot, int64_t max_seq_len, bt_dtype dtype,
+                              int device);
 bt_status bt_kv_export_dense(bt_kv_cache* cache, int64_t b, int64_t t_len, float* k_host, float* v_host);
 bt_status bt_kv_import_dense(bt_kv_cache* cache, int64_t b, int64_t t_len, const float* k_host, const float* v_host);
 /* QuantizedKVCache::append (RE/layers/kv_cache.rs:50-92) on its own, one new token per sequence:
@@ -263,7 +267,9 @@ typedef enum {
     BT_T_NORM_F,      /* [hidden] */
     BT_T_NORM1,       /* per layer [hidden] */
     BT_T_NORM2,
-    BT_T_POS          /* [max_positions, width], learned positions of a layer-list model */
+    BT_T_POS,         /* [max_positions, width], learned positions of a layer-list model */
+    BT_T_LOOP_IN,     /* [width, 2 width], input product of a loop's passes: stream first, then the embedding */
+    BT_T_LOOP_STEP    /* [loop_times, width], added in front of each pass */
 } bt_tensor_kind;
 
 /* BitLlama::load (RE/model/llama.rs:37-158) split into create / set_* / finalize so that
@@ -376,14 +382,22 @@ bt_status bt_model_prefill_logits(bt_model* m, const int32_t* tokens_host, int b
                                   const int32_t* want_host, int n_want, float* logits_host);
 
 /* ---- models given as a list of layers (no reference counterpart) ---------------------------------------------------
- * A decoder with dense 16-bit projections whose layers each name a mixer (softmax attention or a state-space recurrence)
- * and, optionally, a dense feed-forward.  Every sublayer reads the residual stream x as it is and adds its normed
- * output: x <- x + rmsnorm(sublayer(x)) * norm.  It is a bt_model like the others: set tensors, finalize, then
- * bt_model_prefill / bt_model_forward_one / bt_model_step_dev / bt_model_reset / bt_model_set_trace (the trace then
- * holds [rows, width] per layer, the residual stream after it).  Constants are parameters of the layer, so that one
- * mechanism can be switched off or shared by another design. */
-typedef enum { BT_MIX_ATTENTION = 0, BT_MIX_SSM = 1 } bt_mixer_kind;
-typedef enum { BT_MLP_NONE = 0, BT_MLP_DENSE_RELU2 = 1 } bt_mlp_kind; /* W_down relu(W_up x)^2 */
+ * A decoder with dense 16-bit projections whose layers each name a mixer (softmax attention, latent attention or one of
+ * three recurrences) and, optionally, a feed-forward (dense, or a mixture of experts).  Every sublayer adds its normed
+ * output to the residual stream x: x <- x + rmsnorm(sublayer(x)) * norm; with pre_norm it reads rmsnorm(x) * pre instead of
+ * x itself.  A run of layers may be looped: it runs several times with the same weights, each pass with caches and states of
+ * its own, and in front of every pass x <- W_in [x; embedding] + step[pass].  It is a bt_model like the others: set tensors,
+ * finalize, then bt_model_prefill / bt_model_forward_one / bt_model_step_dev / bt_model_reset / bt_model_set_trace (the trace
+ * then holds [rows, width] per layer run, the residual stream after it).  Layer runs are numbered in the order they run;
+ * functions that name a cache or state take that number.  Constants are parameters of the layer, so that one mechanism can
+ * be switched off or shared by another design. */
+typedef enum { BT_MIX_ATTENTION = 0, BT_MIX_SSM = 1, BT_MIX_LATENT = 2, BT_MIX_WKV = 3, BT_MIX_RGLRU = 4 } bt_mixer_kind;
+typedef enum {
+    BT_MLP_NONE = 0,
+    BT_MLP_DENSE_RELU2 = 1, /* W_down relu(W_up x)^2 */
+    BT_MLP_MOE_SWIGLU = 2   /* the `top` of `experts` with the largest router logits, weighted by a softmax over the chosen
+                               logits, plus a shared one (shared_ff 0: none); each W_down (silu(W_gate x) * (W_up x)) */
+} bt_mlp_kind;
 
 typedef struct {
     int mixer;            /* bt_mixer_kind */
@@ -407,7 +421,26 @@ typedef struct {
     int norm_groups;
     /* feed-forward */
     int mlp;              /* bt_mlp_kind */
-    int ff;
+    int ff;               /* of one expert in a mixture */
+    int experts;
+    int top;
+    int shared_ff;
+    /* latent attention (heads, dim, vdim, scale as above): per head dim unrotated and rot_dim rotated query / key values;
+     * keys and values of all heads are products of one normed latent row per position, the rotated key part is shared.
+     * Pairs (2i, 2i + 1), i < rot_dims / 2, turn by position * rot_base^(-2i / rot_dims). */
+    int rot_dim;
+    int rot_dims;         /* even, <= rot_dim */
+    int kv_rank;
+    int out_gate;         /* a head's output times sigmoid(W_g x)_head */
+    double rot_base;
+    /* BT_MIX_WKV (heads, dim): inputs r, k, v, gate and decay each read x + (x of the token before - x) * mu; the decay is
+     * exp(-exp(W_2 tanh(W_1 .) + w0)) per key channel; o = (S + diag(u) k v^T)^T r, S <- diag(decay) S + k v^T; every head's o
+     * by its root mean square, times norm, times silu(gate) */
+    int decay_rank;
+    /* BT_MIX_RGLRU: y = gelu_tanh(W_y x + b), u = causal convolution (conv_taps) of W_x x + b, gates r and i from square
+     * matrices over `blocks` equal parts of u; S <- a S + sqrt(1 - a^2) i u, a = exp(-8 r softplus(lam)); output S * y */
+    int channels;
+    int blocks;
 } bt_layer_config;
 
 typedef struct {
@@ -420,6 +453,11 @@ typedef struct {
     float norm_eps;
     int norm_one_plus;    /* the layer norms and the final norm multiply by 1 + w */
     int dtype;            /* BT_BF16: bf16 products with f32 accumulation and a bf16 cache; BT_F32: 32-bit throughout */
+    int pre_norm;         /* sublayers read the normed stream */
+    int loop_start;       /* layers loop_start .. loop_stop - 1 run loop_times times; loop_times 0: no loop */
+    int loop_stop;
+    int loop_times;
+    float logit_softcap;  /* logits <- cap * tanh(logits / cap); 0: none */
 } bt_layers_config;
 
 bt_status bt_model_create_layers(bt_model** out, const bt_layers_config* cfg, const bt_layer_config* layers, int device);
@@ -432,17 +470,39 @@ typedef enum {
     BT_LT_SSM_CONV, BT_LT_SSM_CONV_B,                            /* [channels, taps], last column = current token; [channels] */
     BT_LT_SSM_DT_BIAS, BT_LT_SSM_A_LOG, BT_LT_SSM_D,             /* [heads] */
     BT_LT_SSM_NORM, BT_LT_SSM_O,                                 /* [heads vdim]; [width, heads vdim] */
-    BT_LT_MLP_UP, BT_LT_MLP_DOWN                                 /* [ff, width]; [width, ff] */
+    BT_LT_MLP_UP, BT_LT_MLP_DOWN,                                /* [ff, width]; [width, ff] */
+    BT_LT_PRE1, BT_LT_PRE2,                                      /* [width]: norms of the sublayers' inputs */
+    /* latent attention (and BT_LT_Q [heads (dim + rot_dim), width], BT_LT_O): [kv_rank + rot_dim, width], [kv_rank],
+     * [heads dim, kv_rank], [heads vdim, kv_rank], [heads, width] */
+    BT_LT_DKV, BT_LT_DKV_NORM, BT_LT_UK, BT_LT_UV, BT_LT_GATE,
+    /* BT_MIX_WKV (and BT_LT_O): five [width]; four [heads dim, width]; [decay_rank, width], [heads dim, decay_rank],
+     * [heads dim]; [heads, dim]; [heads dim] */
+    BT_LT_MU_R, BT_LT_MU_K, BT_LT_MU_V, BT_LT_MU_G, BT_LT_MU_W, BT_LT_WKV_R, BT_LT_WKV_K, BT_LT_WKV_V, BT_LT_WKV_G,
+    BT_LT_WKV_W1, BT_LT_WKV_W2, BT_LT_WKV_W0, BT_LT_WKV_U, BT_LT_WKV_NORM,
+    /* BT_MIX_RGLRU (and BT_LT_O): [channels, width] and [channels] twice; [channels, taps], [channels];
+     * [blocks, channels / blocks, channels / blocks] and [blocks, channels / blocks] twice; [channels] */
+    BT_LT_RG_Y, BT_LT_RG_Y_B, BT_LT_RG_X, BT_LT_RG_X_B, BT_LT_RG_CONV, BT_LT_RG_CONV_B, BT_LT_RG_RA, BT_LT_RG_RA_B,
+    BT_LT_RG_RI, BT_LT_RG_RI_B, BT_LT_RG_LAM,
+    /* mixture: [experts, width], [experts]; per expert [ff, width] twice and [width, ff]; the shared expert's three */
+    BT_LT_ROUTER, BT_LT_ROUTER_B, BT_LT_E_GATE, BT_LT_E_UP, BT_LT_E_DOWN, BT_LT_S_GATE, BT_LT_S_UP, BT_LT_S_DOWN
 } bt_layer_tensor;
 /* Matrices are kept in bf16 (f32 models compute with exactly those values), vectors in f32. */
 bt_status bt_model_set_layer_tensor(bt_model* m, int layer, bt_layer_tensor kind, const float* data_host, int64_t n_elem);
+/* One expert's matrix (BT_LT_E_GATE, BT_LT_E_UP, BT_LT_E_DOWN). */
+bt_status bt_model_set_expert_tensor(bt_model* m, int layer, int expert, bt_layer_tensor kind, const float* data_host, int64_t n_elem);
+/* Layer runs of one pass over the model: num_layers, plus the loop's repeats. */
+int bt_model_layer_runs(const bt_model* m);
 /* Measurement aid: enqueues some of the launches of a decode step (n_tokens = 1) or of a prefill chunk already run
  * (n_tokens > 1), on whatever the buffers hold: parts is a sum of 1 = mixers' input projections, 2 = attention and
- * recurrence, 4 = their output projections, 8 = feed-forward up, 16 = down, 32 = embedding, norms and residual sums.
+ * recurrence, 4 = their output projections, 8 = feed-forward up, 16 = down, 32 = embedding, norms and residual sums,
+ * 64 = products inside a mixer (latents to keys and values, gates, decays), 128 = router, choice and grouping of experts,
+ * 256 = input product of a loop's passes.
  * Positions stay; recurrent states and the cache rows at the current positions do not. */
 bt_status bt_model_enqueue_parts(bt_model* m, int batch, int n_tokens, int parts, void* stream);
-/* Recurrent state of one layer (NULL for attention layers): f32 [max_batch, heads, vdim, state_pad] and the ring of the
- * convolution's last inputs, f32 [max_batch, taps, channels], slot = position % taps.  Sizes in floats. */
+/* Recurrent state of one layer run (NULL for attention) and the last inputs it keeps, f32, sizes in floats.  BT_MIX_SSM:
+ * [max_batch, heads, vdim, state_pad] and [max_batch, taps, channels], slot = position % taps.  BT_MIX_RGLRU:
+ * [max_batch, channels] and [max_batch, taps, channels].  BT_MIX_WKV: [max_batch, heads, dim (key), dim (value)] and
+ * [2, max_batch, width], the token shift's inputs, slot = position % 2. */
 float* bt_model_recurrent_state(bt_model* m, int layer, int64_t* n_floats);
 float* bt_model_conv_ring(bt_model* m, int layer, int64_t* n_floats);
 
