@@ -402,10 +402,160 @@ def graph_us(torch, fn, reps=10):
     return e0.elapsed_time(e1) * 1e3 / reps
 
 
-def run_layered(bt, device, context):
-    """--layered: the layer-list design beside the ternary model of the same width.  Per size one line for each model:
-    decode rate at batch 1 and 64, prefill rate, and per kind of kernel microseconds, achieved rate and its share of the
-    measured roofline (weights and states larger than L2 rotate through the layers)."""
+def fepapel_bench_config(lay, size):
+    """Layers of the sizes a real model has: a gated linear recurrence, latent attention and a wkv recurrence, then the same
+    three looped twice; a mixture of experts behind each."""
+    w, h, d, rot, rank, wd, experts, top, ff, sh = {"2048": (2048, 16, 128, 64, 512, 64, 32, 4, 896, 1792),
+                                                    "4096": (4096, 32, 128, 64, 512, 64, 32, 4, 1792, 3584)}[size]
+    moe = dict(mlp=lay.MLP_MOE_SWIGLU, ff=ff, experts=experts, top=top, shared_ff=sh)
+    rg = lay.LayerConfig(lay.MIX_RGLRU, channels=w, blocks=16, conv_taps=4, **moe)
+    lat = lay.LayerConfig(lay.MIX_LATENT, h, d, dim=d, rot_dim=rot, rot_dims=rot, rot_base=10000.0, kv_rank=rank, out_gate=1, scale=(d + rot) ** -0.5, **moe)
+    wkv = lay.LayerConfig(lay.MIX_WKV, w // wd, dim=wd, decay_rank=64, **moe)
+    return lay.LayersConfig(32000, w, 0, 1e-5, False, [rg, lat, wkv] * 2, pre_norm=True, loop=(3, 6, 2), logit_softcap=30.0)
+
+
+def fepapel_bench_tensors(lay, cfg):
+    """As layered_bench_tensors; the matrices are views into one block per input size."""
+    rng = np.random.default_rng(6)
+    shapes = lay.tensor_shapes(cfg)
+    most = max(int(np.prod(shape, dtype=np.int64)) for _, shape, _, _ in shapes)
+    block = np.resize(rng.normal(0, 1, 1 << 22).astype(np.float32), most)
+    scaled, out = {}, {}
+    for name, shape, _, _ in shapes:
+        n = int(np.prod(shape, dtype=np.int64))
+        leaf = name.rsplit(".", 1)[-1]
+        if len(shape) >= 2 and leaf not in ("conv", "u", "step", "embed"):
+            k = shape[-1]
+            if k not in scaled:
+                scaled[k] = block / np.float32(np.sqrt(k))
+            out[name] = scaled[k][:n].reshape(shape)
+        elif "norm" in name:
+            out[name] = np.ones(shape, np.float32)
+        elif leaf in ("w0", "lam"):
+            out[name] = rng.uniform(-5, -1, shape).astype(np.float32)
+        elif leaf == "embed":
+            out[name] = block[:n].reshape(shape)
+        else:
+            out[name] = (0.3 * block[:n]).reshape(shape)
+    return out
+
+
+def layer_weights(lay, cfg, c):
+    """Weights per kind of launch that a decode step of one layer reads (a mixture: of the chosen experts)."""
+    W, n = cfg.width, {}
+    if c.mixer == lay.MIX_LATENT:
+        n[1], n[4] = W * (c.heads * (c.dim + c.rot_dim + 1) + c.kv_rank + c.rot_dim), W * c.heads * c.vdim
+        n[64] = c.heads * c.kv_rank * (c.dim + c.vdim)
+    elif c.mixer == lay.MIX_WKV:
+        inner = c.heads * c.dim
+        n[1], n[4], n[64] = W * (4 * inner + c.decay_rank), W * inner, inner * c.decay_rank
+    else:
+        n[1], n[4], n[64] = 2 * W * c.channels, W * c.channels, 2 * c.channels * (c.channels // c.blocks)
+    n[8], n[16], n[128] = 2 * W * c.top * c.ff, W * (c.top * c.ff + c.shared_ff), W * (c.experts + 2 * c.shared_ff)
+    return n
+
+
+def run_fepapel(bt, device, context):
+    """--layered fepapel: the design at two widths beside the lines of `gufotar`."""
+    import torch
+    lay = importlib.import_module("bit-ttt-engine_b200.layered")
+    hbm, bf16_tf, kind = measured_peaks()
+    tm = Timer(torch, None, 1, torch.device(f"cuda:{device}"))
+    rng = np.random.default_rng(3)
+    fma_tf = 148 * 128 * 2 * 1.965e9 / 1e12
+    names = {1: "input projections", 2: "mixers", 4: "output projections", 8: "expert up", 16: "experts and shared down", 32: "norms",
+             64: "products inside mixers", 128: "router, choice, shared up", 256: "loop input"}
+    for size in ("2048", "4096"):
+        cfg = fepapel_bench_config(lay, size)
+        t = fepapel_bench_tensors(lay, cfg)
+        W, runs = cfg.width, [cfg.layers[i] for i in cfg.runs()]
+        sampler = ClockSampler(device)
+        sampler.start()
+        line = {"layered": "fepapel", "width": W, "layer_runs": len(runs), "context": context, "dtype": "bf16", "data": "synthetic", "peak_kind": kind}
+        weights = {part: sum(layer_weights(lay, cfg, c).get(part, 0) for c in runs) for part in names}
+        weights[256] = cfg.loop[2] * 2 * W * W
+        lat, wkv, rg = cfg.layers[1], cfg.layers[2], cfg.layers[0]
+        kv_row = 2 * (lat.kv_rank + lat.rot_dim)
+        for B in (1, 64):
+            m = lay.build_layered(cfg, t, max_batch=B, max_seq_len=context + 256, device=device)
+            prompt = rng.integers(0, cfg.vocab_size, size=(B, context)).astype(np.int32)
+            m.prefill(prompt[:, :2048 // B], want_logits=False)
+            m.reset_kv_cache()
+            m.prefill(prompt, want_logits=False)
+            m.reset_kv_cache()
+            torch.cuda.synchronize()
+            t0 = time.perf_counter()
+            m.prefill(prompt, want_logits=False)
+            dt = time.perf_counter() - t0
+            ms, _ = time_decode(m, cfg, B, 64, 4, context, tm, rng)
+            parts = {}
+            w = dict(weights)
+            if B > 8:  # nearly every expert is read, the shared expert's matrices in the up and down launches
+                for c in runs:
+                    w[8] += 2 * W * ((c.experts - c.top) * c.ff + c.shared_ff)
+                    w[16] += W * (c.experts - c.top) * c.ff
+                    w[128] -= 2 * W * c.shared_ff
+            m.seek(context)
+            for part, name in names.items():
+                us = graph_us(torch, lambda: m.enqueue_parts(B, 1, part))
+                parts[name] = {"us": us, "GBps": 2 * w[part] / us / 1e3, "hbm_frac": 2 * w[part] / us / 1e3 / hbm}
+            line[f"batch{B}"] = {"decode_tokens_per_s": B * 64 / (ms * 1e-3), "ms_per_step": ms / 64, "prefill_tokens_per_s": B * context / dt,
+                                 "weight_GB_read_per_step": 2 * sum(w.values()) / 1e9, "decode_kernels_per_step": parts, "launches_per_step": m.launches_per_step(B)}
+            if B == 1:
+                n = min(2048, context)
+                m.seek(0)
+                pre = {}
+                flops = {part: 2.0 * n * weights[part] for part in names}
+                for c in runs:  # the shared expert's up product is among the up launches
+                    flops[8] += 2.0 * n * 2 * W * c.shared_ff
+                    flops[128] -= 2.0 * n * 2 * W * c.shared_ff
+                for part, name in names.items():
+                    us = graph_us(torch, lambda: m.enqueue_parts(1, n, part), reps=3)
+                    pre[name] = {"us": us, "TFLOPs": flops[part] / us / 1e6, "tensor_frac": flops[part] / us / 1e6 / bf16_tf}
+                line["prefill_chunk_kernels"] = {"tokens": n, **pre}
+            del m
+            # the mixers apart: models of one kind of layer
+            for what, c in (("latent attention", lat), ("wkv recurrence", wkv), ("gated linear recurrence", rg)):
+                c1 = lay.LayerConfig(**{**c.__dict__, "mlp": 0, "ff": 0, "experts": 0, "top": 0, "shared_ff": 0})
+                c2 = lay.LayersConfig(64, W, 0, 1e-5, False, [c1] * 4, pre_norm=True)
+                m = lay.build_layered(c2, fepapel_bench_tensors(lay, c2), max_batch=B, max_seq_len=context + 256, device=device)
+                n = min(2048 // B, context)
+                m.prefill(rng.integers(0, 64, size=(B, n)).astype(np.int32), want_logits=False)
+                d = {}
+                if B == 1:
+                    m.seek(0)
+                    us, mid = (graph_us(torch, lambda: m.enqueue_parts(1, n, p), reps=3) / 4 for p in (2, 64))
+                    d.update(prefill_us_per_layer=us, prefill_inner_products_us_per_layer=mid)
+                    if what == "latent attention":
+                        fl = 2.0 * n * n / 2 * c.heads * (c.dim + c.rot_dim + c.vdim)
+                        d.update(prefill_TFLOPs=fl / us / 1e6, prefill_frac=fl / us / 1e6 / bf16_tf)
+                    elif what == "wkv recurrence":
+                        fl = 5.0 * n * c.heads * c.dim * c.dim
+                        d.update(prefill_TFLOPs=fl / us / 1e6, prefill_frac=fl / us / 1e6 / fma_tf)
+                    else:  # convolution (read 4, write 4 + 4) and recurrence (read 16, write 2) bytes per channel and token
+                        byts = n * c.channels * 30.0
+                        d.update(prefill_GBps=byts / us / 1e3, prefill_frac=byts / us / 1e3 / hbm)
+                m.seek(context)
+                us = graph_us(torch, lambda: m.enqueue_parts(B, 1, 2)) / 4
+                if what == "latent attention":
+                    byts = B * (context + 1) * kv_row
+                elif what == "wkv recurrence":
+                    byts = B * 2 * 4 * c.heads * c.dim * c.dim
+                else:
+                    byts = B * 2 * 4 * c.channels + (2 * layer_weights(lay, cfg, c)[64] if B <= 8 else 0)
+                d.update(decode_us_per_layer=us, decode_frac=byts / us / 1e3 / hbm)
+                line[f"batch{B}"][what] = d
+                del m
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+        del t
+        gufotar_line(bt, device, context, size)
+
+
+def gufotar_line(bt, device, context, size):
+    """The layer-list design with softmax attention and state-space layers: decode rate at batch 1 and 64, prefill rate, and
+    per kind of kernel microseconds, achieved rate and its share of the measured roofline (weights and states larger than
+    L2 rotate through the layers)."""
     import torch
     lay = importlib.import_module("bit-ttt-engine_b200.layered")
     syn = importlib.import_module("bit-ttt-engine_b200.synthetic")
@@ -413,74 +563,92 @@ def run_layered(bt, device, context):
     tm = Timer(torch, None, 1, torch.device(f"cuda:{device}"))
     rng = np.random.default_rng(3)
     fma_tf = 148 * 128 * 2 * 1.965e9 / 1e12  # f32 FMA units at the nominal clock
-    for size in ("2048", "4096"):
-        cfg = layered_bench_config(lay, size)
-        t = layered_bench_tensors(lay, cfg)
-        W = cfg.width
-        sampler = ClockSampler(device)
-        sampler.start()
-        line = {"layered": "gufotar", "width": W, "layers": len(cfg.layers), "context": context, "dtype": "bf16", "data": "synthetic", "peak_kind": kind}
-        att, rec = cfg.layers[1], cfg.layers[0]
-        inner, ch = rec.heads * rec.vdim, rec.heads * rec.vdim + 2 * rec.groups * rec.state
-        n_in = {"att": att.heads * att.dim + att.kv_heads * (att.dim + att.vdim), "rec": inner + ch + rec.heads}
-        params = 4 * W * (n_in["att"] + att.heads * att.vdim + 2 * att.ff + n_in["rec"] + inner)
-        part_params = {1: 4 * W * (n_in["att"] + n_in["rec"]), 4: 4 * W * (att.heads * att.vdim + inner), 8: 4 * W * att.ff, 16: 4 * W * att.ff}
-        names = {1: "input projections", 2: "mixers", 4: "output projections", 8: "up", 16: "down", 32: "norms"}
-        for B in (1, 64):
-            m = lay.build_layered(cfg, t, max_batch=B, max_seq_len=context + 256, device=device)
-            prompt = rng.integers(0, cfg.vocab_size, size=(B, context)).astype(np.int32)
-            m.prefill(prompt[:, :64], want_logits=False)
-            m.reset_kv_cache()
-            m.prefill(prompt[:, :2048 // B], want_logits=False)
-            m.reset_kv_cache()
-            torch.cuda.synchronize()
-            t0 = time.perf_counter()
-            m.prefill(prompt, want_logits=False)
-            dt = time.perf_counter() - t0
-            ms, _ = time_decode(m, cfg, B, 64, 4, context, tm, rng)
-            kv_bytes = 4 * B * 2 * att.kv_heads * (context + 1) * (att.dim + att.vdim)
-            state_bytes = 4 * B * 2 * 4 * inner * rec.state
-            parts = {}
+    cfg = layered_bench_config(lay, size)
+    t = layered_bench_tensors(lay, cfg)
+    W = cfg.width
+    sampler = ClockSampler(device)
+    sampler.start()
+    line = {"layered": "gufotar", "width": W, "layers": len(cfg.layers), "context": context, "dtype": "bf16", "data": "synthetic", "peak_kind": kind}
+    att, rec = cfg.layers[1], cfg.layers[0]
+    inner, ch = rec.heads * rec.vdim, rec.heads * rec.vdim + 2 * rec.groups * rec.state
+    n_in = {"att": att.heads * att.dim + att.kv_heads * (att.dim + att.vdim), "rec": inner + ch + rec.heads}
+    params = 4 * W * (n_in["att"] + att.heads * att.vdim + 2 * att.ff + n_in["rec"] + inner)
+    part_params = {1: 4 * W * (n_in["att"] + n_in["rec"]), 4: 4 * W * (att.heads * att.vdim + inner), 8: 4 * W * att.ff, 16: 4 * W * att.ff}
+    names = {1: "input projections", 2: "mixers", 4: "output projections", 8: "up", 16: "down", 32: "norms"}
+    for B in (1, 64):
+        m = lay.build_layered(cfg, t, max_batch=B, max_seq_len=context + 256, device=device)
+        prompt = rng.integers(0, cfg.vocab_size, size=(B, context)).astype(np.int32)
+        m.prefill(prompt[:, :64], want_logits=False)
+        m.reset_kv_cache()
+        m.prefill(prompt[:, :2048 // B], want_logits=False)
+        m.reset_kv_cache()
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        m.prefill(prompt, want_logits=False)
+        dt = time.perf_counter() - t0
+        ms, _ = time_decode(m, cfg, B, 64, 4, context, tm, rng)
+        kv_bytes = 4 * B * 2 * att.kv_heads * (context + 1) * (att.dim + att.vdim)
+        state_bytes = 4 * B * 2 * 4 * inner * rec.state
+        parts = {}
+        for part, name in names.items():
+            us = graph_us(torch, lambda: m.enqueue_parts(B, 1, part))
+            byts = 2 * part_params[part] if part in part_params else (kv_bytes + state_bytes if part == 2 else 0)
+            parts[name] = {"us": us, "GBps": byts / us / 1e3, "hbm_frac": byts / us / 1e3 / hbm}
+        line[f"batch{B}"] = {"decode_tokens_per_s": B * 64 / (ms * 1e-3), "ms_per_step": ms / 64, "prefill_tokens_per_s": B * context / dt,
+                             "weight_GB": 2 * params / 1e9, "decode_kernels_per_step": parts, "launches_per_step": m.launches_per_step(B)}
+        if B == 1:
+            # a prefill chunk of 2048 tokens: the launches of each kind alone
+            n = min(2048, context)
+            m.seek(0)
+            pre = {}
             for part, name in names.items():
-                us = graph_us(torch, lambda: m.enqueue_parts(B, 1, part))
-                byts = 2 * part_params[part] if part in part_params else (kv_bytes + state_bytes if part == 2 else 0)
-                parts[name] = {"us": us, "GBps": byts / us / 1e3, "hbm_frac": byts / us / 1e3 / hbm}
-            line[f"batch{B}"] = {"decode_tokens_per_s": B * 64 / (ms * 1e-3), "ms_per_step": ms / 64, "prefill_tokens_per_s": B * context / dt,
-                                 "weight_GB": 2 * params / 1e9, "decode_kernels_per_step": parts, "launches_per_step": m.launches_per_step(B)}
+                us = graph_us(torch, lambda: m.enqueue_parts(1, n, part), reps=3)
+                fl = 2.0 * n * part_params[part] if part in part_params else 0
+                pre[name] = {"us": us, "TFLOPs": fl / us / 1e6, "tensor_frac": fl / us / 1e6 / bf16_tf}
+            line["prefill_chunk_kernels"] = {"tokens": n, **pre}
+        del m
+        # the two mixers apart: models of one kind of layer
+        for what, layers in (("attention", [att] * 4), ("recurrence", [rec] * 4)):
+            c2 = lay.LayersConfig(64, W, cfg.max_positions, 1e-5, True, layers)
+            m = lay.build_layered(c2, layered_bench_tensors(lay, c2), max_batch=B, max_seq_len=context + 256, device=device)
+            n = min(2048 // B, context)
+            m.prefill(rng.integers(0, 64, size=(B, n)).astype(np.int32), want_logits=False)
+            pre_us = None
             if B == 1:
-                # a prefill chunk of 2048 tokens: the launches of each kind alone
-                n = min(2048, context)
                 m.seek(0)
-                pre = {}
-                for part, name in names.items():
-                    us = graph_us(torch, lambda: m.enqueue_parts(1, n, part), reps=3)
-                    fl = 2.0 * n * part_params[part] if part in part_params else 0
-                    pre[name] = {"us": us, "TFLOPs": fl / us / 1e6, "tensor_frac": fl / us / 1e6 / bf16_tf}
-                line["prefill_chunk_kernels"] = {"tokens": n, **pre}
+                pre_us = graph_us(torch, lambda: m.enqueue_parts(1, n, 2), reps=3) / 4
+            m.seek(context)
+            us = graph_us(torch, lambda: m.enqueue_parts(B, 1, 2)) / 4
+            byts = (kv_bytes if what == "attention" else state_bytes) / 4
+            d = {"decode_us_per_layer": us, "hbm_frac": byts / us / 1e3 / hbm}
+            if pre_us:
+                fl = 2.0 * n * n / 2 * att.heads * (att.dim + att.vdim) if what == "attention" else 5.0 * n * inner * rec.state
+                d.update(prefill_us_per_layer=pre_us, prefill_TFLOPs=fl / pre_us / 1e6)
+                d["prefill_frac"] = fl / pre_us / 1e6 / (bf16_tf if what == "attention" else fma_tf)
+            line[f"batch{B}"][what] = d
             del m
-            # the two mixers apart: models of one kind of layer
-            for what, layers in (("attention", [att] * 4), ("recurrence", [rec] * 4)):
-                c2 = lay.LayersConfig(64, W, cfg.max_positions, 1e-5, True, layers)
-                m = lay.build_layered(c2, layered_bench_tensors(lay, c2), max_batch=B, max_seq_len=context + 256, device=device)
-                n = min(2048 // B, context)
-                m.prefill(rng.integers(0, 64, size=(B, n)).astype(np.int32), want_logits=False)
-                pre_us = None
-                if B == 1:
-                    m.seek(0)
-                    pre_us = graph_us(torch, lambda: m.enqueue_parts(1, n, 2), reps=3) / 4
-                m.seek(context)
-                us = graph_us(torch, lambda: m.enqueue_parts(B, 1, 2)) / 4
-                byts = (kv_bytes if what == "attention" else state_bytes) / 4
-                d = {"decode_us_per_layer": us, "hbm_frac": byts / us / 1e3 / hbm}
-                if pre_us:
-                    fl = 2.0 * n * n / 2 * att.heads * (att.dim + att.vdim) if what == "attention" else 5.0 * n * inner * rec.state
-                    d.update(prefill_us_per_layer=pre_us, prefill_TFLOPs=fl / pre_us / 1e6)
-                    d["prefill_frac"] = fl / pre_us / 1e6 / (bf16_tf if what == "attention" else fma_tf)
-                line[f"batch{B}"][what] = d
-                del m
-        line["clocks"] = sampler.stop()
-        print(json.dumps(line), flush=True)
-        del t
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line), flush=True)
+    del t
+
+
+def run_layered(bt, device, context, design):
+    """--layered: the layer-list design `gufotar` beside the ternary model of the same width, or `fepapel` beside `gufotar`;
+    per size one line for each model."""
+    if design == "fepapel":
+        run_fepapel(bt, device, context)
+        return
+    import torch
+    lay = importlib.import_module("bit-ttt-engine_b200.layered")
+    syn = importlib.import_module("bit-ttt-engine_b200.synthetic")
+    hbm, bf16_tf, kind = measured_peaks()
+    tm = Timer(torch, None, 1, torch.device(f"cuda:{device}"))
+    rng = np.random.default_rng(4)
+    fma_tf = 148 * 128 * 2 * 1.965e9 / 1e12  # f32 FMA units at the nominal clock
+    for size in ("2048", "4096"):
+        gufotar_line(bt, device, context, size)
+        rec = layered_bench_config(lay, size).layers[0]
+        W, inner = int(size), rec.heads * rec.vdim
         # ---- the ternary model of the same width ----
         line = {"layered": "ternary model beside it", "width": W, "context": context}
         shape = "8b" if size == "4096" else "tinyllama"
@@ -735,8 +903,8 @@ def main():
     ap.add_argument("--sweep", action="store_true",
                     help="BitLinear shape sweep (K,N in {4096x4096, 4096x14336, 14336x4096, 4096x128256}, "
                          "M in {1, 8, 64, 512, 4096}, bf16 activations) plus the TTT update: one JSON line per point")
-    ap.add_argument("--layered", action="store_true",
-                    help="the layer-list design (attention and recurrent layers, bf16) beside the ternary model at two widths: "
+    ap.add_argument("--layered", nargs="?", const="gufotar", default=None, choices=["gufotar", "fepapel"],
+                    help="a layer-list design in bf16 at two widths, gufotar beside the ternary model or fepapel beside gufotar: "
                          "prefill and decode rates and per-kernel roofline shares, one JSON line per model and width")
     ap.add_argument("--profile-case", type=int, default=0, metavar="BATCH",
                     help="small case for a profiler, not a benchmark: --layers blocks of the 8B shape, BATCH sequences, "
@@ -771,7 +939,7 @@ def main():
         run_sweep(bt, local_rank)
         return
     if args.layered:
-        run_layered(bt, local_rank, args.context)
+        run_layered(bt, local_rank, args.context, args.layered)
         return
 
     if args.profile_case:

@@ -80,6 +80,17 @@ pub mod ffi {
         pub norm_groups: c_int,
         pub mlp: c_int,
         pub ff: c_int,
+        pub experts: c_int,
+        pub top: c_int,
+        pub shared_ff: c_int,
+        pub rot_dim: c_int,
+        pub rot_dims: c_int,
+        pub kv_rank: c_int,
+        pub out_gate: c_int,
+        pub rot_base: c_double,
+        pub decay_rank: c_int,
+        pub channels: c_int,
+        pub blocks: c_int,
     }
 
     #[repr(C)]
@@ -94,6 +105,11 @@ pub mod ffi {
         pub norm_eps: c_float,
         pub norm_one_plus: c_int,
         pub dtype: c_int,
+        pub pre_norm: c_int,
+        pub loop_start: c_int,
+        pub loop_stop: c_int,
+        pub loop_times: c_int,
+        pub logit_softcap: c_float,
     }
 
     pub type bt_weight_kind = c_int; // BT_W_Q = 0 .. BT_W_TTT_UP = 8
@@ -140,6 +156,8 @@ pub mod ffi {
                             v_q_host: *const u8, v_s_host: *const c_float) -> bt_status;
         pub fn bt_kv_create_dense(out: *mut *mut bt_kv_cache, batch: i64, n_kv_heads: i64, k_dim: i64, v_dim: i64,
                                   max_seq_len: i64, dtype: bt_dtype, device: c_int) -> bt_status;
+        pub fn bt_kv_create_latent(out: *mut *mut bt_kv_cache, batch: i64, rank: i64, rot: i64, max_seq_len: i64,
+                                   dtype: bt_dtype, device: c_int) -> bt_status;
         pub fn bt_kv_export_dense(cache: *mut bt_kv_cache, b: i64, t_len: i64, k_host: *mut c_float,
                                   v_host: *mut c_float) -> bt_status;
         pub fn bt_kv_import_dense(cache: *mut bt_kv_cache, b: i64, t_len: i64, k_host: *const c_float,
@@ -185,6 +203,9 @@ pub mod ffi {
                                       device: c_int) -> bt_status;
         pub fn bt_model_set_layer_tensor(m: *mut bt_model, layer: c_int, kind: c_int, data_host: *const c_float,
                                          n_elem: i64) -> bt_status;
+        pub fn bt_model_set_expert_tensor(m: *mut bt_model, layer: c_int, expert: c_int, kind: c_int, data_host: *const c_float,
+                                          n_elem: i64) -> bt_status;
+        pub fn bt_model_layer_runs(m: *const bt_model) -> c_int;
         pub fn bt_model_enqueue_parts(m: *mut bt_model, batch: c_int, n_tokens: c_int, parts: c_int,
                                       stream: *mut c_void) -> bt_status;
         pub fn bt_model_recurrent_state(m: *mut bt_model, layer: c_int, n_floats: *mut i64) -> *mut c_float;
