@@ -429,8 +429,8 @@ def fepapel_bench_tensors(lay, cfg):
             if k not in scaled:
                 scaled[k] = block / np.float32(np.sqrt(k))
             out[name] = scaled[k][:n].reshape(shape)
-        elif "norm" in name:
-            out[name] = np.ones(shape, np.float32)
+        elif "norm" in name:  # quiet sublayers: the stream keeps its tokens apart, so that they choose different experts
+            out[name] = np.full(shape, 0.1 if name.endswith(("norm1b", "norm2b")) else 1.0, np.float32)
         elif leaf in ("w0", "lam"):
             out[name] = rng.uniform(-5, -1, shape).astype(np.float32)
         elif leaf == "embed":
@@ -495,6 +495,8 @@ def run_fepapel(bt, device, context):
                     w[8] += 2 * W * ((c.experts - c.top) * c.ff + c.shared_ff)
                     w[16] += W * (c.experts - c.top) * c.ff
                     w[128] -= 2 * W * c.shared_ff
+            m.seek(context)
+            m.forward_one(rng.integers(0, cfg.vocab_size, size=B), want_logits=False)
             m.seek(context)
             for part, name in names.items():
                 us = graph_us(torch, lambda: m.enqueue_parts(B, 1, part))

@@ -46,8 +46,8 @@ struct ActOut {
 inline int64_t dense_mpad(int64_t m) { return m <= 64 ? 64 : (m <= 128 ? 128 : (m + 255) / 256 * 256); }
 
 // SWIGLU: rows 2j and 2j + 1 of the matrix are gate j and up j, the product has n / 2 outputs silu(gate) * up.
-// RGLRU: rows 2j and 2j + 1 are the two gates of channel j (streaming product only, behind DPRO_CONV).
-enum DenseAct : int { DACT_NONE = 0, DACT_RELU2 = 1, DACT_TANH = 2, DACT_SWIGLU = 3, DACT_RGLRU = 4 };
+// RGLRU: rows 2j and 2j + 1 are the two gates of channel j (streaming product only, behind DPRO_CONV).  DECAY: exp(-exp(v)).
+enum DenseAct : int { DACT_NONE = 0, DACT_RELU2 = 1, DACT_TANH = 2, DACT_DECAY = 3, DACT_SWIGLU = 4, DACT_RGLRU = 5 };
 inline int dense_outputs(const DenseLin& lin, int act) { return act >= DACT_SWIGLU ? lin.n / 2 : lin.n; }
 
 // The gated linear recurrence of one token per sequence:
@@ -319,8 +319,8 @@ struct WkvArgs {
     const uint8_t* w2_tiles = nullptr;  // tiled [heads dim, rank], rows padded to w2_pad
     int w2_pad = 0;
     const float* w0 = nullptr;     // [heads dim]
-    // prefill: the decays' exponents, and the token shift's state
-    const float* z = nullptr;      // rows [heads dim]
+    // prefill: the decays, and the token shift's state
+    const float* w = nullptr;      // rows [heads dim]
     const float* hn = nullptr;     // rows [width]
     float* shift = nullptr;        // [2][max_batch][width], slot = parity of the position
     int64_t shift_slot = 0;
@@ -329,7 +329,7 @@ struct WkvArgs {
 };
 int wkv_max_dim();
 cudaError_t launch_wkv_step(const WkvArgs& a, cudaStream_t s, bool pdl);
-cudaError_t launch_wkv_prefill(const WkvArgs& a, bool bf16, cudaStream_t s);
+cudaError_t launch_wkv_prefill(const WkvArgs& a, cudaStream_t s);
 // Token shift of the new rows: x + (x before - x) * mu for the inputs r, k, v, gate (four blocks of tiles or rows) and the
 // decay (tiles: hi | lo).
 struct WkvMix {

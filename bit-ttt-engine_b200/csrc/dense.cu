@@ -28,6 +28,7 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 __device__ __forceinline__ float act_fn(int act, float v) {
     if (act == DACT_RELU2) { v = fmaxf(v, 0.0f); v *= v; }
     else if (act == DACT_TANH) v = tanhf(v);
+    else if (act == DACT_DECAY) v = expf(-expf(v));
     return v;
 }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
@@ -366,7 +367,11 @@ struct TcCfg {
     static constexpr size_t kSmem = (size_t)kStages * kStageBytes + kEpi + 256;
 };
 
-template <int NT>
+// What the epilogue does is a constant of the kernel: f32 rows as they are, f32 rows with bias and activation, tiled bf16
+// (squared relu), gate and up pairs to tiled bf16, bf16 rows.
+enum TcEpi : int { TC_ROWS, TC_ROWS_ACT, TC_TILES, TC_PAIRS, TC_ROWS16 };
+
+template <int NT, int EPI>
 __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a) {
     using Cfg = TcCfg<NT>;
     constexpr int S = Cfg::kStages;
@@ -472,17 +477,15 @@ __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a)
             ptx::tc_fence_after();
             const int f = d.rs * kTcRows + sub * 32 + lane;  // row of the block
             const int64_t tok0 = d.tok0, tok_end = d.tok_end;
-            const float bias = a.bias && f < a.n ? a.bias[(int64_t)d.blk * a.n + f] : 0.0f;
+            const float bias = EPI == TC_ROWS_ACT && a.bias && f < a.n ? a.bias[(int64_t)d.blk * a.n + f] : 0.0f;
+            auto finish = [&](float x) { return EPI == TC_ROWS_ACT ? act_fn(a.act, x + bias) : x; };
 #pragma unroll 1
             for (int q = 0; q < NT; q += 32) {
                 if (tok0 + q >= tok_end) break;
                 uint32_t v[32];
                 ptx::tmem_ld32(tmem_base + ((uint32_t)(sub * 32) << 16) + set * NT + q, v);
                 ptx::tmem_ld_wait();
-                if (a.bias)
-#pragma unroll
-                    for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) + bias);
-                if (a.act == DACT_SWIGLU) {
+                if (EPI == TC_PAIRS) {
                     // neighbouring lanes hold gate and up: the even one finishes the first 16 tokens, the odd one the others;
                     // pieces of (one token, 8 features) through shared memory, [token group][8 features][token]
 #pragma unroll
@@ -503,23 +506,24 @@ __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a)
                                 *reinterpret_cast<const uint4*>(stage + core * 144 + tk * 16);
                     }
                     __syncwarp();
-                } else if (a.out_tiles || a.out_rows16) {
+                } else if (EPI == TC_TILES || EPI == TC_ROWS16) {
                     // through shared memory into 16-byte pieces (one token, 8 features): [token group][8 features][token]
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
-                        const float r = act_fn(a.act, __uint_as_float(v[j]));
+                        float r = __uint_as_float(v[j]);
+                        if (EPI == TC_TILES && a.act == DACT_RELU2) { r = fmaxf(r, 0.0f); r *= r; }
                         *reinterpret_cast<__nv_bfloat16*>(stage + ((j >> 3) * 4 + (lane >> 3)) * 144 + (j & 7) * 16 + (lane & 7) * 2) = __float2bfloat16_rn(r);
                     }
                     __syncwarp();
-                    const int col0 = a.out_tiles ? (int)(d.blk * a.out_block) : 0;
-                    const int limit = a.out_tiles && col0 + a.n_out == a.blocks * a.n_out ? dense_kpad(col0 + a.n_out) - col0 : a.n_out;
+                    const int col0 = EPI == TC_TILES ? (int)(d.blk * a.out_block) : 0;
+                    const int limit = EPI == TC_TILES && col0 + a.n_out == a.blocks * a.n_out ? dense_kpad(col0 + a.n_out) - col0 : a.n_out;
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const int piece = i * 32 + lane, core = piece >> 3, tk = piece & 7;  // core = token group * 4 + feature group
                         const int64_t token = tok0 + q + (core >> 2) * 8 + tk;
                         const int feat = d.rs * kTcRows + sub * 32 + (core & 3) * 8;
                         if (token < tok_end && feat < limit) {
-                            void* dst = a.out_tiles ? (void*)(a.out_tiles + dense_off(token, col0 + feat, a.m_pad))
+                            void* dst = EPI == TC_TILES ? (void*)(a.out_tiles + dense_off(token, col0 + feat, a.m_pad))
                                                     : (void*)(a.out_rows16 + d.blk * a.out_block + token * a.ld + feat);
                             *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(stage + core * 144 + tk * 16);
                         }
@@ -529,11 +533,11 @@ __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a)
                     float* o = a.out + (int64_t)d.sp * a.part_stride + (a.plan ? 0 : d.blk * a.out_block) + (tok0 + q) * a.ld + f;
                     if (tok0 + q + 32 <= tok_end) {
 #pragma unroll
-                        for (int j = 0; j < 32; ++j) o[j * a.ld] = act_fn(a.act, __uint_as_float(v[j]));
+                        for (int j = 0; j < 32; ++j) o[j * a.ld] = finish(__uint_as_float(v[j]));
                     } else {
 #pragma unroll
                         for (int j = 0; j < 32; ++j)
-                            if (tok0 + q + j < tok_end) o[j * a.ld] = act_fn(a.act, __uint_as_float(v[j]));
+                            if (tok0 + q + j < tok_end) o[j * a.ld] = finish(__uint_as_float(v[j]));
                     }
                 }
             }
@@ -576,14 +580,21 @@ __global__ void __launch_bounds__(256) dense_reduce_kernel(const float* __restri
             if (c0 + j < n) out[r * ld + c0 + j] = v[j];
 }
 
-template <int NT>
-cudaError_t tc_launch(const TcArgs& a, int sm_count, cudaStream_t s) {
+template <int NT, int EPI>
+cudaError_t tc_launch_e(const TcArgs& a, int sm_count, cudaStream_t s) {
     static PerDeviceOnce once;
-    cudaError_t e = once.run([] { return cudaFuncSetAttribute(dense_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcCfg<NT>::kSmem); });
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(dense_tc_kernel<NT, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcCfg<NT>::kSmem); });
     if (e != cudaSuccess) return e;
     const int64_t tiles = (int64_t)(a.n_pad / kTcRows) * ((a.m + NT - 1) / NT) * a.splits * a.blocks;  // a.m: the plan's upper bound
-    dense_tc_kernel<NT><<<(unsigned)(tiles < sm_count ? tiles : sm_count), kTcThreads, TcCfg<NT>::kSmem, s>>>(a);
+    dense_tc_kernel<NT, EPI><<<(unsigned)(tiles < sm_count ? tiles : sm_count), kTcThreads, TcCfg<NT>::kSmem, s>>>(a);
     return cudaGetLastError();
+}
+template <int NT>
+cudaError_t tc_launch(const TcArgs& a, int sm_count, cudaStream_t s) {
+    if (a.act == DACT_SWIGLU) return tc_launch_e<NT, TC_PAIRS>(a, sm_count, s);
+    if (a.out_tiles) return tc_launch_e<NT, TC_TILES>(a, sm_count, s);
+    if (a.out_rows16) return tc_launch_e<NT, TC_ROWS16>(a, sm_count, s);
+    return a.bias || a.act != DACT_NONE ? tc_launch_e<NT, TC_ROWS_ACT>(a, sm_count, s) : tc_launch_e<NT, TC_ROWS>(a, sm_count, s);
 }
 
 // token rows per tile: 64 and 128 while one block covers them; above, 256 unless that leaves SMs idle
@@ -973,7 +984,8 @@ cudaError_t launch_dense_tc(const DenseLin& lin, const uint8_t* x_tiles, int64_t
     const bool whole = o.act == DACT_SWIGLU || o.out_rows16 || o.plan || blocks > 1;  // never cut
     const int sp = whole ? 1 : tc_splits(lin, m, sm_count);
     const int nt = o.plan ? o.plan->tile : tc_tokens(lin, m, sm_count, blocks);
-    if ((o.act == DACT_SWIGLU && (!o.out_tiles || lin.n % 2)) || o.act == DACT_RGLRU || o.halves < 1 || o.halves > 2 ||
+    if ((o.act == DACT_SWIGLU && (!o.out_tiles || lin.n % 2 || o.bias)) || o.act == DACT_RGLRU ||
+        (sp == 1 && o.out_tiles && (o.bias || (o.act != DACT_NONE && o.act != DACT_RELU2 && o.act != DACT_SWIGLU))) || (o.out_rows16 && (o.bias || o.act != DACT_NONE)) || o.halves < 1 || o.halves > 2 ||
         (o.out_rows16 && (o.ld % 8 || o.out_block % 8 || n_out % 8)) || (o.out_tiles && blocks > 1 && !o.plan && (o.out_block % 8 || n_out % 8)))
         return cudaErrorInvalidValue;
     TcArgs a;

@@ -12,7 +12,7 @@ namespace bt {
 
 namespace {
 
-constexpr int kMaxRank = 512, kMaxRot = 128;
+constexpr int kMaxRank = 512, kMaxRot = 128, kMaxSplits = 16;
 constexpr unsigned kErrLatentTimeout = 0x4c41544eu;  // 'LATN'
 
 __device__ __forceinline__ float warp_sum(float v) {
@@ -113,9 +113,9 @@ __device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, flo
     const int i1 = (int)((int64_t)total * (split + 1) / splits);
     for (int i = (int)((int64_t)total * split / splits) + threadIdx.x; i < i1; i += blockDim.x) {
         const int h = i / a.rank, c = i - h * a.rank, head = head0 + h;
-        float ms[8], ls[8], os[8], m = -INFINITY;
+        float ms[kMaxSplits], ls[kMaxSplits], os[kMaxSplits], m = -INFINITY;
 #pragma unroll
-        for (int s = 0; s < 8; ++s) {  // all remote reads in flight together
+        for (int s = 0; s < kMaxSplits; ++s) {  // all remote reads in flight together
             ms[s] = -INFINITY; ls[s] = os[s] = 0.0f;
             if (s < splits) {
                 ms[s] = *(splits > 1 ? cluster.map_shared_rank(m_s, s) + h : m_s + h);
@@ -126,7 +126,7 @@ __device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, flo
         }
         float den = 0.0f, num = 0.0f;
 #pragma unroll
-        for (int s = 0; s < 8; ++s) {
+        for (int s = 0; s < kMaxSplits; ++s) {
             const float f = LOG2 ? ex2(ms[s] - m) : expf(ms[s] - m);  // an empty span: 0
             den = fmaf(ls[s], f, den);
             num = fmaf(os[s], f, num);
@@ -140,41 +140,43 @@ __device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, flo
 }
 
 // ---------------------------------------------------------------------------------------
-// one query position, 16 heads, on the tensor cores (bf16 cache)
+// one query position, 16 MT heads, on the tensor cores (bf16 cache)
 // ---------------------------------------------------------------------------------------
-// The cache is laid out in core matrices (8 positions x 16 bytes), so blocks of 64 positions arrive as one bulk copy per 64
-// columns and every ldmatrix reads 128 consecutive bytes.  Per block: eight warps make the scores of 8 positions each, then
-// the softmax of two heads each, then 8 NT latent columns each.  Queries and softmax weights enter as bf16 hi + lo.
-constexpr int kSpanThreads = 256, kKeys = 64, kHeads = 16;
+// The cache is laid out in core matrices (8 positions x 16 bytes), so blocks of 32 positions arrive as one bulk copy per 64
+// columns and every ldmatrix reads 128 consecutive bytes.  Per block: sixteen warps share the scores' product, eight parts of
+// the columns (each warp has its part of the queries in registers) x 16 positions, and leave partial scores; then each makes
+// the softmax of MT heads and multiplies its 8 NT latent columns.  Softmax weights enter their product as bf16 hi + lo.
+constexpr int kSpanThreads = 512, kSpanWarps = kSpanThreads / 32, kKeys = 32, kMaxSteps = (kMaxRank + kMaxRot) / 16 / 8;
+constexpr int kScoreLd = 40;  // floats per row of partial scores
 
-struct SpanShape {
-    int chunks, kc, kr;  // 64-column blocks; 16-column steps of the latent part and of all columns in use
-    int stages;
+template <int MT>
+struct SpanCfg {
+    static constexpr int H = 16 * MT;
+    static constexpr size_t kPart = (size_t)8 * H * kScoreLd * 4;  // partial scores; first the queries
+    static size_t part(int chunks) { const size_t q = (size_t)chunks * MT * 2048; return q > kPart ? q : kPart; }
+    static size_t fixed(int chunks) { return part(chunks) + (size_t)MT * 2 * 1024 + 3 * H * 4 + 32 * 4 + (size_t)chunks * 128 + 64; }
 };
-__host__ __device__ inline size_t span_fixed_bytes(int chunks) {
-    return (size_t)2 * chunks * 2048 + 2 * 2048 + (size_t)kHeads * kKeys * 4 + 3 * kHeads * 4 + 32 * 4 + (size_t)chunks * 128 + 64;
-}
 
-template <int NT>
-__global__ void __launch_bounds__(kSpanThreads) latent_span_mma_kernel(const LatentAttn a, bool prepared, int splits, int stages,
-                                                                       unsigned int* err, const ActOut out) {
+template <int NT, int MT>
+__global__ void __launch_bounds__(kSpanThreads, 1) latent_span_mma_kernel(const LatentAttn a, bool prepared, int splits, int stages,
+                                                                       int part_bytes, unsigned int* err, const ActOut out) {
+    constexpr int NH = 16 * MT, NS = MT;  // heads of the CTA; of a warp in the softmax
     extern __shared__ __align__(128) uint8_t sm[];
     const int kcl = dense_kpad(a.rank) / 64, chunks = kcl + dense_kpad(a.rot) / 64;
     const int stage_bytes = chunks * kKeys * 128;
-    uint8_t* q_hi = sm + (size_t)stages * stage_bytes;   // [chunk][2 groups of 8 heads][8 pieces][8 heads][16 bytes]
-    uint8_t* q_lo = q_hi + chunks * 2048;
-    uint8_t* p_hi = q_lo + chunks * 2048;                // softmax weights [16 heads][64 positions], core matrices
-    uint8_t* p_lo = p_hi + 2048;
-    float* s_s = reinterpret_cast<float*>(p_lo + 2048);  // scores [16][64]
-    float* m_s = s_s + kHeads * kKeys;
-    float* l_s = m_s + kHeads;
-    float* al_s = l_s + kHeads;
-    float* red = al_s + kHeads;
+    uint8_t* q_s = sm + (size_t)stages * stage_bytes;    // [chunk][MT][2 groups of 8 heads][8 pieces][8 heads][16 bytes]
+    float* s_s = reinterpret_cast<float*>(q_s);          // [8 warps][heads][kScoreLd]
+    uint8_t* p_hi = q_s + part_bytes;                    // softmax weights [MT][16 heads][32 positions], core matrices
+    uint8_t* p_lo = p_hi + MT * 1024;
+    float* m_s = reinterpret_cast<float*>(p_lo + MT * 1024);
+    float* l_s = m_s + NH;
+    float* al_s = l_s + NH;
+    float* red = al_s + NH;
     __nv_bfloat16* new_s = reinterpret_cast<__nv_bfloat16*>(red + 32);  // the new token's row [chunks * 64]
-    uint64_t* full = reinterpret_cast<uint64_t*>(new_s + chunks * 64);
+    uint64_t* full = reinterpret_cast<uint64_t*>(new_s + chunks * 64);  // up to eight
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int H = a.heads, hd = a.dim + a.rot;
-    const int head0 = blockIdx.y * kHeads, nh = min(kHeads, H - head0);
+    const int head0 = blockIdx.y * NH, nh = min(NH, H - head0);
     const int64_t r = blockIdx.z;
     const int b = (int)(r / a.q_rows), split = blockIdx.x;
     const int p = a.pos[b] + (int)(r % a.q_rows);
@@ -190,33 +192,32 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_mma_kernel(const Lat
         ptx::mbar_fence_init();
     }
     __syncthreads();
-    auto load = [&](int i) {  // thread 0: the i-th block of the span
+    auto load = [&](int i, int slot) {  // warp 0: the i-th block of the span, a lane per 64 columns
         if (i >= blocks) return;
-        uint8_t* st = sm + (size_t)(i % stages) * stage_bytes;
-        ptx::mbar_arrive_expect_tx(&full[i % stages], stage_bytes);
-        for (int c = 0; c < chunks; ++c)
-            ptx::bulk_g2s(st + c * kKeys * 128, seq + ((int64_t)c * a.kv.seq_pad + t0 + i * kKeys) * 128, kKeys * 128, &full[i % stages]);
+        if (lane == 0) ptx::mbar_arrive_expect_tx(&full[slot], stage_bytes);
+        __syncwarp();
+        if (lane < chunks)
+            ptx::bulk_g2s(sm + (size_t)slot * stage_bytes + lane * kKeys * 128, seq + ((int64_t)lane * a.kv.seq_pad + t0 + i * kKeys) * 128, kKeys * 128, &full[slot]);
     };
     if (prepared) ptx::pdl_wait();  // the cache rows come from the kernel in front
-    if (threadIdx.x == 0)
-        for (int i = 0; i < stages - 1; ++i) load(i);
+    if (warp == 0)
+        for (int i = 0; i < stages - 1; ++i) load(i, i);
     if (!prepared) ptx::pdl_wait();
     ptx::pdl_launch_dependents();
 
-    // ---- queries: [absorbed | rotated] as hi and lo ----
+    // ---- queries: [absorbed | rotated] ----
     const float* row = a.proj + r * a.ld;
     const int kl = kcl * 64;
-    for (int i = threadIdx.x; i < kHeads * chunks * 64; i += kSpanThreads) {
-        const int h = i / (chunks * 64), c = i - h * chunks * 64;
-        float v = 0.0f;
-        if (h < nh) {
-            if (c < kl) { if (c < a.rank) v = a.q_abs[(r * H + head0 + h) * a.rank + c]; }
-            else if (c - kl < a.rot) v = prepared ? a.q_rot[(r * H + head0 + h) * a.rot + c - kl] : rotated(a, row + (head0 + h) * hd + a.dim, c - kl, p);
-        }
-        const int o = (c >> 6) * 2048 + (h >> 3) * 1024 + ((c & 63) >> 3) * 128 + (h & 7) * 16 + (c & 7) * 2;
-        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-        *reinterpret_cast<__nv_bfloat16*>(q_hi + o) = hi;
-        *reinterpret_cast<__nv_bfloat16*>(q_lo + o) = __float2bfloat16_rn(v - __bfloat162float(hi));
+    for (int i = threadIdx.x; i < NH * chunks * 32; i += kSpanThreads) {  // two columns at a time
+        const int h = i / (chunks * 32), c = (i - h * chunks * 32) * 2;
+        float v[2] = {0.0f, 0.0f};
+        if (h < nh)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                if (c < kl) { if (c + j < a.rank) v[j] = a.q_abs[(r * H + head0 + h) * a.rank + c + j]; }
+                else if (c + j - kl < a.rot) v[j] = prepared ? a.q_rot[(r * H + head0 + h) * a.rot + c + j - kl] : rotated(a, row + (head0 + h) * hd + a.dim, c + j - kl, p);
+            }
+        *reinterpret_cast<uint32_t*>(q_s + (c >> 6) * MT * 2048 + (h >> 3) * 1024 + ((c & 63) >> 3) * 128 + (h & 7) * 16 + (c & 7) * 2) = ptx::pack2(v[0], v[1]);
     }
     if (owner) {
         const float* c = row + H * hd;
@@ -230,24 +231,43 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_mma_kernel(const Lat
             if (blockIdx.y == 0) *reinterpret_cast<__nv_bfloat16*>(seq + dense_off(p, i, a.kv.seq_pad)) = w;
         }
     }
-    if (threadIdx.x < kHeads) { m_s[threadIdx.x] = -INFINITY; l_s[threadIdx.x] = 0.0f; }
     __syncthreads();
+    // this warp's 16-column steps: part, part + 8, ... of the latent part's and the rotated part's
+    const int part = warp & 7, half = warp >> 3;
+    const int steps_l = (a.rank + 15) / 16, steps = steps_l + (a.rot + 15) / 16;
+    uint32_t qf[kMaxSteps][MT][4];
+    uint32_t k_off[kMaxSteps];
+#pragma unroll
+    for (int i = 0; i < kMaxSteps; ++i) {
+        const int ks = part + 8 * i, kk = ks < steps_l ? ks : ks - steps_l + kcl * 4;
+        k_off[i] = (uint32_t)((kk >> 2) * kKeys * 128 + (kk & 3) * 256 + half * 2048);
+        if (ks < steps)
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+                ptx::ldsm4(qf[i][m], ptx::smem_u32(q_s) + ((kk >> 2) * MT + m) * 2048 + (kk & 3) * 256 + ((lane >> 3) & 1) * 1024 + (lane >> 4) * 128 + (lane & 7) * 16);
+    }
+    __syncthreads();  // the partial scores take the queries' place
 
-    float acc[NT][4];
+    float acc[MT][NT][4];
 #pragma unroll
-    for (int i = 0; i < NT; ++i)
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
+        for (int i = 0; i < NT; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[m][i][j] = 0.0f;
+    float m_run[NS], l_run[NS];  // heads NS warp ..: maximum; this lane's share of the sum
+#pragma unroll
+    for (int j = 0; j < NS; ++j) { m_run[j] = -INFINITY; l_run[j] = 0.0f; }
     const float unit = a.scale * 1.4426950408889634f;
-    const int steps_l = (a.rank + 15) / 16, steps_r = (a.rot + 15) / 16;
-    const uint32_t q_off = ((lane >> 3) & 1) * 1024 + (lane >> 4) * 128 + (lane & 7) * 16;
-    const uint32_t qh = ptx::smem_u32(q_hi) + q_off, ql = ptx::smem_u32(q_lo) + q_off;
-    const uint32_t ph = ptx::smem_u32(p_hi) + q_off, pl = ptx::smem_u32(p_lo) + q_off;
-    const uint32_t core = (lane >> 3) * 128 + (lane & 7) * 16;  // four pieces of eight positions
+    const uint32_t p_off = ((lane >> 3) & 1) * 512 + (lane >> 4) * 128 + (lane & 7) * 16;
+    const uint32_t ph = ptx::smem_u32(p_hi) + p_off, pl = ptx::smem_u32(p_lo) + p_off;
+    const uint32_t k_core = (lane >> 4) * 1024 + ((lane >> 3) & 1) * 128 + (lane & 7) * 16;  // two groups of positions x two pieces
 
+    int slot = 0, before = stages - 1;  // ring slots of this block and of the one before it
+    uint32_t parity = 0;
     for (int i = 0; i < blocks; ++i) {
-        uint8_t* st = sm + (size_t)(i % stages) * stage_bytes;
-        ok &= ptx::mbar_wait_bounded(&full[i % stages], (uint32_t)((i / stages) & 1));
+        uint8_t* st = sm + (size_t)slot * stage_bytes;
+        ok &= ptx::mbar_wait_bounded(&full[slot], parity);
         const int base = t0 + i * kKeys;
         if (owner && i == blocks - 1) {  // the new row has not been in the copy
             const int at = p - base;
@@ -256,83 +276,107 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_mma_kernel(const Lat
             __syncthreads();
         }
         const uint32_t kv = ptx::smem_u32(st);
-        float s[4][4] = {};  // hi and lo, even and odd steps
-        auto score_steps = [&](int chunk0, int steps) {
-            for (int k = 0; k < steps; k += 2) {
-                const uint32_t q0 = (uint32_t)((chunk0 + (k >> 2)) * 2048 + (k & 3) * 256);
-                uint32_t kf[4], qa[4];
-                ptx::ldsm4(kf, kv + (chunk0 + (k >> 2)) * kKeys * 128 + warp * 1024 + (k & 3) * 256 + core);
-                ptx::ldsm4(qa, qh + q0);
-                ptx::mma_bf16(s[0], qa, kf[0], kf[1]);
-                ptx::ldsm4(qa, ql + q0);
-                ptx::mma_bf16(s[1], qa, kf[0], kf[1]);
-                ptx::ldsm4(qa, qh + q0 + 256);
-                ptx::mma_bf16(s[2], qa, kf[2], kf[3]);
-                ptx::ldsm4(qa, ql + q0 + 256);
-                ptx::mma_bf16(s[3], qa, kf[2], kf[3]);
-            }
-        };
-        score_steps(0, steps_l);     // an odd last step meets zeros of the padding
-        score_steps(kcl, steps_r);
         {
-            const int k0 = warp * 8 + (lane & 3) * 2;
+            float s[MT][2][4] = {};
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int key = k0 + (j & 1), h = (lane >> 2) + (j >> 1) * 8;
-                s_s[h * kKeys + key] = base + key < t1 ? (s[0][j] + s[1][j] + s[2][j] + s[3][j]) * unit : -INFINITY;
+            for (int k = 0; k < kMaxSteps; ++k)
+                if (part + 8 * k < steps) {
+                    uint32_t kf[4];
+                    ptx::ldsm4(kf, kv + k_off[k] + k_core);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        ptx::mma_bf16(s[m][0], qf[k][m], kf[0], kf[1]);
+                        ptx::mma_bf16(s[m][1], qf[k][m], kf[2], kf[3]);
+                    }
+                }
+            float* sp = s_s + (part * NH + (lane >> 2)) * kScoreLd + half * 16 + (lane & 3) * 2;
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int g = 0; g < 2; ++g) {
+                    *reinterpret_cast<float2*>(sp + m * 16 * kScoreLd + g * 8) = make_float2(s[m][g][0], s[m][g][1]);
+                    *reinterpret_cast<float2*>(sp + (m * 16 + 8) * kScoreLd + g * 8) = make_float2(s[m][g][2], s[m][g][3]);
+                }
+        }
+        __syncthreads();
+        if (warp == 0) load(i + stages - 1, before);  // into the slot of the block before this one
+        {
+            float x[NS], mx[NS];
+#pragma unroll
+            for (int j = 0; j < NS; ++j) {
+                const float* sp = s_s + (warp * NS + j) * kScoreLd + lane;
+                float v = 0.0f;
+#pragma unroll
+                for (int w = 0; w < 8; ++w) v += sp[w * NH * kScoreLd];
+                x[j] = base + lane < t1 ? v * unit : -INFINITY;
+                mx[j] = x[j];
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int j = 0; j < NS; ++j) mx[j] = fmaxf(mx[j], __shfl_xor_sync(0xffffffffu, mx[j], o));
+#pragma unroll
+            for (int j = 0; j < NS; ++j) {
+                const int h = warp * NS + j;
+                const float m_new = fmaxf(m_run[j], mx[j]), al = ex2(m_run[j] - m_new), e = ex2(x[j] - m_new);  // al: 0 for the first block
+                m_run[j] = m_new;
+                l_run[j] = fmaf(l_run[j], al, e);
+                const __nv_bfloat16 hi = __float2bfloat16_rn(e);
+                const int o = (h >> 4) * 1024 + ((h >> 3) & 1) * 512 + (lane >> 3) * 128 + (h & 7) * 16 + (lane & 7) * 2;
+                *reinterpret_cast<__nv_bfloat16*>(p_hi + o) = hi;
+                *reinterpret_cast<__nv_bfloat16*>(p_lo + o) = __float2bfloat16_rn(e - __bfloat162float(hi));
+                if (lane == 0) al_s[h] = al;
             }
         }
         __syncthreads();
-        if (threadIdx.x == 0) load(i + stages - 1);  // into the slot of the block before this one
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-            const int h = warp * 2 + j;
-            const float2 x = *reinterpret_cast<const float2*>(s_s + h * kKeys + lane * 2);
-            const float m_old = m_s[h], m_new = fmaxf(m_old, warp_max(fmaxf(x.x, x.y)));
-            const float e0 = ex2(x.x - m_new), e1 = ex2(x.y - m_new);
-            const float sum = warp_sum(e0 + e1);
-            const uint32_t hi = ptx::pack2(e0, e1);
-            const int o = (h >> 3) * 1024 + (lane >> 2) * 128 + (h & 7) * 16 + (lane & 3) * 4;
-            *reinterpret_cast<uint32_t*>(p_hi + o) = hi;
-            *reinterpret_cast<uint32_t*>(p_lo + o) = ptx::pack2(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
-            __syncwarp();
-            if (lane == 0) {
-                const float al = ex2(m_old - m_new);  // 0 for the first block
-                al_s[h] = al;
-                m_s[h] = m_new;
-                l_s[h] = l_s[h] * al + sum;
-            }
+        for (int m = 0; m < MT; ++m) {
+            const float al0 = al_s[m * 16 + (lane >> 2)], al1 = al_s[m * 16 + (lane >> 2) + 8];
+            if (__any_sync(0xffffffffu, al0 != 1.0f || al1 != 1.0f))
+#pragma unroll
+                for (int n = 0; n < NT; ++n) { acc[m][n][0] *= al0; acc[m][n][1] *= al0; acc[m][n][2] *= al1; acc[m][n][3] *= al1; }
         }
-        __syncthreads();
-        const float al0 = al_s[lane >> 2], al1 = al_s[(lane >> 2) + 8];
+        const int col0 = warp * NT * 8;
+        if (col0 < a.rank) {
+            uint32_t hi[2][MT][4], lo[2][MT][4];
 #pragma unroll
-        for (int n = 0; n < NT; ++n) { acc[n][0] *= al0; acc[n][1] *= al0; acc[n][2] *= al1; acc[n][3] *= al1; }
+            for (int k = 0; k < 2; ++k)
 #pragma unroll
-        for (int k = 0; k < kKeys / 16; ++k) {
-            uint32_t hi[4], lo[4];
-            ptx::ldsm4(hi, ph + k * 256);
-            ptx::ldsm4(lo, pl + k * 256);
+                for (int m = 0; m < MT; ++m) {
+                    ptx::ldsm4(hi[k][m], ph + m * 1024 + k * 256);
+                    ptx::ldsm4(lo[k][m], pl + m * 1024 + k * 256);
+                }
 #pragma unroll
-            for (int n = 0; n < NT; n += 2) {
-                const int col = (warp * NT + n) * 8;
-                if (col < a.rank) {
-                    uint32_t vf[4];  // (positions 0-7, 8-15) x (columns 0-7, 8-15)
-                    ptx::ldsm4t(vf, kv + (col >> 6) * kKeys * 128 + (2 * k + ((lane >> 3) & 1)) * 1024 + (((col & 63) >> 3) + (lane >> 4)) * 128 + (lane & 7) * 16);
-                    ptx::mma_bf16(acc[n], hi, vf[0], vf[1]);
-                    ptx::mma_bf16(acc[n + 1], hi, vf[2], vf[3]);
-                    ptx::mma_bf16(acc[n], lo, vf[0], vf[1]);
-                    ptx::mma_bf16(acc[n + 1], lo, vf[2], vf[3]);
+            for (int n = 0; n < NT; ++n) {
+                const int col = col0 + n * 8;
+                uint32_t vf[4];  // 8 columns of the four groups of positions
+                ptx::ldsm4t(vf, kv + (col >> 6) * kKeys * 128 + ((col & 63) >> 3) * 128 + (lane >> 3) * 1024 + (lane & 7) * 16);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    ptx::mma_bf16(acc[m][n], hi[0][m], vf[0], vf[1]);
+                    ptx::mma_bf16(acc[m][n], lo[0][m], vf[0], vf[1]);
+                    ptx::mma_bf16(acc[m][n], hi[1][m], vf[2], vf[3]);
+                    ptx::mma_bf16(acc[m][n], lo[1][m], vf[2], vf[3]);
                 }
             }
         }
+        before = slot;
+        if (++slot == stages) { slot = 0; parity ^= 1; }
+    }
+#pragma unroll
+    for (int j = 0; j < NS; ++j) {
+        const float l = warp_sum(l_run[j]);
+        if (lane == 0) { m_s[warp * NS + j] = m_run[j]; l_s[warp * NS + j] = l; }
     }
     __syncthreads();  // the ring is free
-    constexpr int W = 64 * NT;
-    float* o_s = reinterpret_cast<float*>(sm);  // [16][W], in the ring's place
+    constexpr int W = 8 * kSpanWarps * NT;
+    float* o_s = reinterpret_cast<float*>(sm);  // [heads][W], in the ring's place
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) o_s[((lane >> 2) + (j >> 1) * 8) * W + (warp * NT + n) * 8 + (lane & 3) * 2 + (j & 1)] = acc[n][j];
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) o_s[(m * 16 + (lane >> 2) + (j >> 1) * 8) * W + (warp * NT + n) * 8 + (lane & 3) * 2 + (j & 1)] = acc[m][n][j];
     if (!ok) atomicExch(err, kErrLatentTimeout);
     merge_spans<true>(a, m_s, l_s, o_s, W, nh, head0, r, split, splits, out);
 }
@@ -340,8 +384,8 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_mma_kernel(const Lat
 // ---------------------------------------------------------------------------------------
 // the same in f32 on the FMA units (32-bit models): 8 heads per CTA, tiles of 32 positions
 // ---------------------------------------------------------------------------------------
-constexpr int kF32Heads = 8, kF32Keys = 32;
-__global__ void __launch_bounds__(kSpanThreads) latent_span_f32_kernel(const LatentAttn a, bool prepared, int splits, const ActOut out) {
+constexpr int kF32Heads = 8, kF32Keys = 32, kF32Threads = 256;
+__global__ void __launch_bounds__(kF32Threads) latent_span_f32_kernel(const LatentAttn a, bool prepared, int splits, const ActOut out) {
     extern __shared__ __align__(16) float fs[];
     const int D = a.rank + a.rot, W = a.rank;
     float* q_s = fs;                          // [8][D]
@@ -364,7 +408,7 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_f32_kernel(const Lat
     const int t0 = min(split * span, total), t1 = min(t0 + span, total);
     float* cache = reinterpret_cast<float*>(a.kv.rows) + (int64_t)b * a.kv.max_seq * a.kv.stride;
     const float* row = a.proj + r * a.ld;
-    for (int i = threadIdx.x; i < kF32Heads * D; i += kSpanThreads) {
+    for (int i = threadIdx.x; i < kF32Heads * D; i += kF32Threads) {
         const int h = i / D, c = i - h * D;
         float v = 0.0f;
         if (h < nh)
@@ -376,11 +420,11 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_f32_kernel(const Lat
         const float* c = row + H * hd;
         const float inv = latent_inv(a, c, red);
         float* dst = cache + (int64_t)p * a.kv.stride;
-        for (int i = threadIdx.x; i < D; i += kSpanThreads) dst[i] = i < a.rank ? c[i] * inv * a.c_norm[i] : rotated(a, c + a.rank, i - a.rank, p);
+        for (int i = threadIdx.x; i < D; i += kF32Threads) dst[i] = i < a.rank ? c[i] * inv * a.c_norm[i] : rotated(a, c + a.rank, i - a.rank, p);
     }
     if (threadIdx.x < kF32Heads) { m_s[threadIdx.x] = -INFINITY; l_s[threadIdx.x] = 0.0f; }
     __syncthreads();
-    float acc[kF32Heads][kMaxRank / kSpanThreads] = {};
+    float acc[kF32Heads][kMaxRank / kF32Threads] = {};
     for (int base = t0; base < t1; base += kF32Keys) {
         for (int k = warp; k < kF32Keys; k += 8) {
             const int t = base + k;
@@ -414,12 +458,12 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_f32_kernel(const Lat
 #pragma unroll
         for (int h = 0; h < kF32Heads; ++h)
 #pragma unroll
-            for (int j = 0; j < kMaxRank / kSpanThreads; ++j) acc[h][j] *= al_s[h];
+            for (int j = 0; j < kMaxRank / kF32Threads; ++j) acc[h][j] *= al_s[h];
         const int n = min(kF32Keys, t1 - base);
         for (int k = 0; k < n; ++k)
 #pragma unroll
-            for (int j = 0; j < kMaxRank / kSpanThreads; ++j) {
-                const int c = threadIdx.x + j * kSpanThreads;
+            for (int j = 0; j < kMaxRank / kF32Threads; ++j) {
+                const int c = threadIdx.x + j * kF32Threads;
                 if (c < a.rank) {
                     const float x = cache[(int64_t)(base + k) * a.kv.stride + c];
 #pragma unroll
@@ -431,8 +475,8 @@ __global__ void __launch_bounds__(kSpanThreads) latent_span_f32_kernel(const Lat
 #pragma unroll
     for (int h = 0; h < kF32Heads; ++h)
 #pragma unroll
-        for (int j = 0; j < kMaxRank / kSpanThreads; ++j) {
-            const int c = threadIdx.x + j * kSpanThreads;
+        for (int j = 0; j < kMaxRank / kF32Threads; ++j) {
+            const int c = threadIdx.x + j * kF32Threads;
             if (c < a.rank) o_s[h * W + c] = acc[h][j];
         }
     merge_spans<false>(a, m_s, l_s, o_s, W, nh, head0, r, split, splits, out);
@@ -456,31 +500,36 @@ cudaError_t launch_cluster(void (*kernel)(KArgs...), dim3 grid, int threads, siz
 }
 int span_splits(const LatentAttn& a, int64_t groups) {
     int splits = 1;
-    while (splits < 8 && groups * splits * 2 <= a.sm_count && splits * 64 < a.kv.max_seq) splits *= 2;
+    while (splits < kMaxSplits && groups * splits * 2 <= a.sm_count && splits * 64 < a.kv.max_seq) splits *= 2;
     return splits;
 }
 
 constexpr size_t kSpanSmem = 220 * 1024;
-template <int NT>
+template <int NT, int MT>
 cudaError_t span_launch(const LatentAttn& a, bool prepared, const ActOut& out, unsigned int* err, cudaStream_t s, bool pdl) {
     static PerDeviceOnce once;
-    cudaError_t e = once.run([] { return cudaFuncSetAttribute(latent_span_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSpanSmem); });
+    cudaError_t e = once.run([] {
+        cudaError_t x = cudaFuncSetAttribute(latent_span_mma_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSpanSmem);
+        return x != cudaSuccess ? x : cudaFuncSetAttribute(latent_span_mma_kernel<NT, MT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    });
     if (e != cudaSuccess) return e;
-    const int chunks = (dense_kpad(a.rank) + dense_kpad(a.rot)) / 64, hg = (a.heads + kHeads - 1) / kHeads;
-    const size_t stage = (size_t)chunks * kKeys * 128, fixed = span_fixed_bytes(chunks);
-    int stages = (int)((kSpanSmem - fixed) / stage);
-    if (stages < 2) return cudaErrorInvalidConfiguration;
-    // up to 110 KB: two CTAs share an SM; the ring must also take the outputs
-    const int small = (int)((110 * 1024 - fixed) / stage);
-    stages = small >= 2 && 110 * 1024 > fixed ? small : stages;
-    if (stages > 4) stages = 4;
-    size_t ring = stages * stage;
-    const size_t outs = (size_t)kHeads * 64 * NT * sizeof(float);
-    while (ring < outs) { ++stages; ring += stage; }
+    const int chunks = (dense_kpad(a.rank) + dense_kpad(a.rot)) / 64, hg = (a.heads + 16 * MT - 1) / (16 * MT);
+    const size_t stage = (size_t)chunks * kKeys * 128, fixed = SpanCfg<MT>::fixed(chunks), outs = (size_t)16 * MT * 8 * kSpanWarps * NT * sizeof(float);
+    // six blocks in flight where two CTAs then share an SM, else as many as fit; the ring must also take the outputs
+    int stages = 6;
+    if (stages * stage + fixed > 110 * 1024) stages = (int)((kSpanSmem - fixed) / stage) < 6 ? (int)((kSpanSmem - fixed) / stage) : 6;
+    while (stages * stage < outs) ++stages;
+    if (stages < 2 || stages > 8 || stages * stage + fixed > kSpanSmem) return cudaErrorInvalidConfiguration;
     const int64_t rows = (int64_t)a.batch * a.q_rows;
     const int splits = span_splits(a, rows * hg);
-    return launch_cluster(latent_span_mma_kernel<NT>, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, ring + fixed, s, pdl,
-                          a, prepared, splits, stages, err, out);
+    return launch_cluster(latent_span_mma_kernel<NT, MT>, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, stages * stage + fixed, s, pdl,
+                          a, prepared, splits, stages, (int)SpanCfg<MT>::part(chunks), err, out);
+}
+template <int NT>
+cudaError_t span_launch_m(const LatentAttn& a, bool prepared, const ActOut& out, unsigned int* err, cudaStream_t s, bool pdl) {
+    // 32 heads share the cache rows once that leaves no SM idle
+    const bool wide = a.heads > 16 && (int64_t)a.batch * a.q_rows * ((a.heads + 31) / 32) * 4 >= a.sm_count;
+    return wide ? span_launch<NT, 2>(a, prepared, out, err, s, pdl) : span_launch<NT, 1>(a, prepared, out, err, s, pdl);
 }
 
 }  // namespace
@@ -497,21 +546,24 @@ cudaError_t launch_latent_span(const LatentAttn& a, bool prepared, const ActOut&
     if (a.rank > kMaxRank || a.rot > kMaxRot || (!prepared && a.q_rows != 1)) return cudaErrorInvalidValue;
     if (a.kv.f32) {
         static PerDeviceOnce once;
-        cudaError_t e = once.run([] { return cudaFuncSetAttribute(latent_span_f32_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024); });
+        cudaError_t e = once.run([] {
+            cudaError_t x = cudaFuncSetAttribute(latent_span_f32_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
+            return x != cudaSuccess ? x : cudaFuncSetAttribute(latent_span_f32_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        });
         if (e != cudaSuccess) return e;
         const int hg = (a.heads + kF32Heads - 1) / kF32Heads;
         const int64_t rows = (int64_t)a.batch * a.q_rows;
         const int splits = span_splits(a, rows * hg);
         const size_t smem = ((size_t)kF32Heads * (2 * a.rank + a.rot) + kF32Heads * kF32Keys + 3 * kF32Heads + 32) * sizeof(float);
-        return launch_cluster(latent_span_f32_kernel, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, smem, s, pdl, a, prepared, splits, out);
+        return launch_cluster(latent_span_f32_kernel, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kF32Threads, smem, s, pdl, a, prepared, splits, out);
     }
     int dev = 0;
     cudaError_t e = cudaGetDevice(&dev);
     if (e != cudaSuccess) return e;
     unsigned int* err = device_error_word(dev);
-    if (a.rank <= 128) return span_launch<2>(a, prepared, out, err, s, pdl);
-    if (a.rank <= 256) return span_launch<4>(a, prepared, out, err, s, pdl);
-    return span_launch<8>(a, prepared, out, err, s, pdl);
+    if (a.rank <= 128) return span_launch_m<1>(a, prepared, out, err, s, pdl);
+    if (a.rank <= 256) return span_launch_m<2>(a, prepared, out, err, s, pdl);
+    return span_launch_m<4>(a, prepared, out, err, s, pdl);
 }
 
 }  // namespace bt

@@ -43,7 +43,7 @@ struct RowBuffers {
     float* hn = nullptr;       // a sublayer's normed input, f32 rows
     float* cat = nullptr;      // loops: stream and embedding side by side (fused step: the embedding)
     float* a = nullptr;        // latent: absorbed queries; rglru: convolution outputs; wkv: low-rank decay inputs
-    float* b = nullptr;        // latent: weighted latents; rglru: gates; wkv: decay exponents
+    float* b = nullptr;        // latent: weighted latents; rglru: gates; wkv: decays
     float* c = nullptr;        // latent: rotated queries; wkv: mixed inputs, finished rows
     void* q = nullptr;         // prepared queries
     uint8_t* xt = nullptr;     // bf16 models: tiled activations (sublayer input, mixer output, feed-forward, inside a mixer)
@@ -349,7 +349,7 @@ WkvArgs wkv_args(const bt_model* m, const LayLayer& l, const LayRun& run, const 
     a.heads = c.heads; a.dim = c.dim; a.s = run.state; a.pos = m->pos; a.batch = batch; a.q_rows = n;
     a.y = r.mix;
     a.low = r.a; a.rank = c.decay_rank;
-    a.z = r.b; a.hn = r.hn; a.shift = run.ring; a.shift_slot = (int64_t)m->cfg.max_batch * m->lay->c.width; a.width = m->lay->c.width;
+    a.w = r.b; a.hn = r.hn; a.shift = run.ring; a.shift_slot = (int64_t)m->cfg.max_batch * m->lay->c.width; a.width = m->lay->c.width;
     a.sm_count = m->sm_count;
     return a;
 }
@@ -668,10 +668,10 @@ struct RowPass {
         low.halves = 2;
         BT_CUDA_TRY(product(PART_MID, l.mid, r.t2, r.c + 4ll * W, 5ll * W, low));
         if (!f32 && (parts & PART_MID)) BT_CUDA_TRY(launch_rows_tile(r.a, rank, 0, 1, rank, 2, DACT_TANH, M, r.t2, mp, s));
-        DenseOut z = rows_out(r.b, HD, DACT_NONE, l.vec[BT_LT_WKV_W0]);
+        DenseOut z = rows_out(r.b, HD, DACT_DECAY, l.vec[BT_LT_WKV_W0]);
         z.halves = 2;
         BT_CUDA_TRY(product(PART_MID, l.mid2, r.t2, r.a, rank, z));
-        if (parts & PART_CORE) BT_CUDA_TRY(launch_wkv_prefill(wkv_args(m, l, run, r, batch, n), !f32, s));
+        if (parts & PART_CORE) BT_CUDA_TRY(launch_wkv_prefill(wkv_args(m, l, run, r, batch, n), s));
         RowArgs g;
         g.op = ROW_GROUPNORM; g.y = r.mix; g.ld = HD; g.w = l.vec[BT_LT_WKV_NORM]; g.eps = eps; g.groups = l.c.heads; g.rows = M; g.k = HD;
         g.gate = r.proj + 3ll * HD; g.gate_ld = 4ll * HD;

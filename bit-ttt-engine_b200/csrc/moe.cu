@@ -325,10 +325,10 @@ cudaError_t launch_moe_down(const MoeStep& a, cudaStream_t s, bool pdl) {
     return stream_launch<true>(m, a.sm_count, s, pdl);
 }
 
-// rows per tile of the grouped products: about what an expert gets
+// rows per tile of the grouped products: an expert's last tile is half empty on average
 int moe_tile_rows(int64_t rows, int top, int experts) {
     const int64_t each = rows * top / experts;
-    return each <= 64 ? 64 : (each <= 160 ? 128 : 256);
+    return each <= 48 ? 64 : (each <= 640 ? 128 : 256);
 }
 int moe_max_tiles(int64_t rows, int top, int experts, int tile) {
     const int64_t all = rows * top, busy = all < experts ? all : experts;

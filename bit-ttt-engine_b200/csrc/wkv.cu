@@ -58,9 +58,10 @@ __global__ void __launch_bounds__(256) wkv_mix_kernel(const WkvMix a) {
 }
 
 // ---------------------------------------------------------------------------------------
-// one token per sequence: decays, recurrence, norm of the head's output and gate in one launch
+// one token per sequence: decays, recurrence, norm of the head's output and gate in one launch; or, with the decays given,
+// the recurrence alone
 // ---------------------------------------------------------------------------------------
-// A CTA per (head, sequence); threads as key groups x value columns, 32 KEYS state rows per thread group and turn.
+// A CTA per (head, sequence); threads as key groups x value columns.
 constexpr int kStepThreads = 512, kMaxRank = 512;
 
 template <int CW>  // columns: 32, 64, 128, 256
@@ -84,7 +85,8 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
     ptx::pdl_wait();
     ptx::pdl_launch_dependents();
     const float* row = a.proj + b * a.ld + head * D;
-    for (int i = threadIdx.x; i < a.rank; i += kStepThreads) low_s[i] = a.low[(int64_t)b * a.rank + i];
+    if (!a.w)
+        for (int i = threadIdx.x; i < a.rank; i += kStepThreads) low_s[i] = a.low[(int64_t)b * a.rank + i];
     if (threadIdx.x < CW) {
         const bool live = threadIdx.x < D;
         const float rv = live ? row[threadIdx.x] : 0.0f, kv = live ? row[HD + threadIdx.x] : 0.0f;
@@ -94,7 +96,7 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
     }
     const float v = col < D ? row[2 * HD + col] : 0.0f;
     __syncthreads();
-    {   // decays of the head's key channels: G threads share a channel
+    if (!a.w) {  // decays of the head's key channels: G threads share a channel
         float z = 0.0f;
         if (col < D)
             for (int c0 = g * 8; c0 < a.rank; c0 += G * 8) {
@@ -111,9 +113,14 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
     __syncthreads();
     if (threadIdx.x < CW) {
         float z = 0.0f;
+        if (a.w) {
+            if (threadIdx.x < D) z = a.w[(int64_t)b * HD + head * D + threadIdx.x];
+        } else {
 #pragma unroll
-        for (int i = 0; i < G; ++i) z += part[i * CW + threadIdx.x];
-        w_s[threadIdx.x] = threadIdx.x < D ? expf(-expf(z + a.w0[head * D + threadIdx.x])) : 0.0f;
+            for (int i = 0; i < G; ++i) z += part[i * CW + threadIdx.x];
+            z = threadIdx.x < D ? expf(-expf(z + a.w0[head * D + threadIdx.x])) : 0.0f;
+        }
+        w_s[threadIdx.x] = z;
     }
     __syncthreads();
     float o = 0.0f;
@@ -130,8 +137,16 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
         o = 0.0f;
 #pragma unroll
         for (int i = 0; i < G; ++i) o += part[i * CW + threadIdx.x];
+        if (a.w && threadIdx.x < D) a.y[(int64_t)b * HD + head * D + threadIdx.x] = o;
         const float ss = warp_sum(o * o);
         if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    }
+    if (a.w) {
+        if (head == 0) {  // the token shift's state
+            float* keep = a.shift + (int64_t)(p & 1) * a.shift_slot + (int64_t)b * a.width;
+            for (int c = threadIdx.x; c < a.width; c += kStepThreads) keep[c] = a.hn[(int64_t)b * a.width + c];
+        }
+        return;
     }
     __syncthreads();
     if (threadIdx.x < D) {
@@ -146,109 +161,194 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
 // ---------------------------------------------------------------------------------------
 // many tokens, one after the other
 // ---------------------------------------------------------------------------------------
-// A CTA owns 32 value columns of one head: eight lanes share a column, each with 4 NJ state elements in registers (key
-// channels 32 j + 4 lane .. + 3).  r, k, the decays and v of a tile of tokens are staged in shared memory, the next tile's
-// values wait in registers.
+// A CTA owns 16 value columns of one head, a warp 8: eight lanes share two columns, each with 4 NJ of their state elements in
+// registers (key channels 32 j + 4 lane .. + 3).  r, k, the decays and v of a tile of tokens arrive in shared memory by
+// asynchronous copies, one tile ahead; tokens go by eights, whose sums over the lanes are folded together.
+constexpr int kScanThreads = 64, kScanCols = 16;
 template <int NJ>
-__global__ void __launch_bounds__(256) wkv_scan_kernel(const WkvArgs a) {
-    constexpr int DP = 32 * NJ, TT = NJ <= 4 ? 16 : 8, NL = TT * DP / 256;
-    __shared__ __align__(16) float r_s[TT * DP], k_s[TT * DP], w_s[TT * DP];
-    __shared__ float v_s[TT * 32], bonus_s[TT];
-    const int head = blockIdx.x, v0 = blockIdx.y * 32, b = blockIdx.z;
-    const int D = a.dim, HD = a.heads * D, vc = min(32, D - v0);
+struct ScanCfg {
+    static constexpr int DP = 32 * NJ, TT = NJ <= 4 ? 16 : 8;
+    static constexpr int kTile = TT * (3 * DP + kScanCols);  // floats
+    static constexpr size_t kSmem = (size_t)(2 * kTile + TT) * sizeof(float);
+};
+
+template <int NJ>
+__global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a) {
+    using Cfg = ScanCfg<NJ>;
+    constexpr int DP = Cfg::DP, TT = Cfg::TT;
+    extern __shared__ __align__(16) float sm[];  // two tiles of r, k, w [TT][DP] and v [TT][16]; bonus [TT]
+    float* bonus_s = sm + 2 * Cfg::kTile;
+    const int head = blockIdx.x, v0 = blockIdx.y * kScanCols, b = blockIdx.z;
+    const int D = a.dim, HD = a.heads * D, vc = min(kScanCols, D - v0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int col = warp * 4 + (lane >> 3), kg = lane & 7;
-    const bool live = col < vc;
+    const int col = warp * 8 + (lane >> 3) * 2, kg = lane & 7;
     const int p0 = a.pos[b];
-    float* state = a.s + ((int64_t)b * a.heads + head) * D * D + v0 + (live ? col : 0);
-    float s[4 * NJ];
+    float* state = a.s + ((int64_t)b * a.heads + head) * D * D + v0 + col;
+    float s[4 * NJ][2];
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int k = 32 * j + 4 * kg + e;
-            s[4 * j + e] = live && k < D && p0 > 0 ? state[(int64_t)k * D] : 0.0f;
-        }
-    const float* base = a.proj + (int64_t)b * a.q_rows * a.ld + head * D;
-    const float* zb = a.z + (int64_t)b * a.q_rows * HD + head * D;
-    float rr[NL], kr[NL], zr[NL], vr[TT * 32 / 256];
-    auto fetch = [&](int i0) {
+        for (int e = 0; e < 4; ++e)
 #pragma unroll
-        for (int i = 0; i < NL; ++i) {
-            const int e = threadIdx.x + i * 256, t = i0 + e / DP, c = e % DP;
-            const bool ok = t < a.q_rows && c < D;
-            rr[i] = ok ? base[(int64_t)t * a.ld + c] : 0.0f;
-            kr[i] = ok ? base[(int64_t)t * a.ld + HD + c] : 0.0f;
-            zr[i] = ok ? zb[(int64_t)t * HD + c] : 0.0f;
+            for (int c = 0; c < 2; ++c) {
+                const int k = 32 * j + 4 * kg + e;
+                s[4 * j + e][c] = col + c < vc && k < D && p0 > 0 ? state[(int64_t)k * D + c] : 0.0f;
+            }
+    const float* rows = a.proj + (int64_t)b * a.q_rows * a.ld + head * D;
+    const float* wrows = a.w + (int64_t)b * a.q_rows * HD + head * D;
+    for (int i = threadIdx.x; i < 2 * Cfg::kTile; i += kScanThreads) sm[i] = 0.0f;  // columns beyond the head's stay zero
+    __syncthreads();
+    const bool vec = (D & 3) == 0 && (a.ld & 3) == 0;
+    auto fetch = [&](int i0, int buf) {  // tokens i0 .. of the tile
+        float* t = sm + buf * Cfg::kTile;
+        const int n = min(TT, a.q_rows - i0);
+        if (n <= 0) return;
+        if (vec) {
+            const int q = D >> 2;
+            for (int e = threadIdx.x; e < n * q; e += kScanThreads) {
+                const int i = e / q, c = (e - i * q) * 4;
+                const float* src = rows + (int64_t)(i0 + i) * a.ld + c;
+                const uint32_t dst = ptx::smem_u32(t + i * DP + c);
+                ptx::cp16(dst, src, true);
+                ptx::cp16(dst + TT * DP * 4, src + HD, true);
+                ptx::cp16(dst + 2 * TT * DP * 4, wrows + (int64_t)(i0 + i) * HD + c, true);
+            }
+            const int vq = vc >> 2;
+            for (int e = threadIdx.x; e < n * vq; e += kScanThreads) {
+                const int i = e / vq, c = (e - i * vq) * 4;
+                ptx::cp16(ptx::smem_u32(t + 3 * TT * DP + i * kScanCols + c), rows + (int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c, true);
+            }
+        } else {
+            for (int e = threadIdx.x; e < n * D; e += kScanThreads) {
+                const int i = e / D, c = e - i * D;
+                const float* src = rows + (int64_t)(i0 + i) * a.ld + c;
+                t[i * DP + c] = src[0];
+                t[TT * DP + i * DP + c] = src[HD];
+                t[2 * TT * DP + i * DP + c] = wrows[(int64_t)(i0 + i) * HD + c];
+            }
+            for (int e = threadIdx.x; e < n * vc; e += kScanThreads) {
+                const int i = e / vc, c = e - i * vc;
+                t[3 * TT * DP + i * kScanCols + c] = rows[(int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c];
+            }
         }
-#pragma unroll
-        for (int i = 0; i < TT * 32 / 256; ++i) {
-            const int e = threadIdx.x + i * 256, t = i0 + e / 32, c = e % 32;
-            vr[i] = t < a.q_rows && c < vc ? base[(int64_t)t * a.ld + 2 * HD + v0 + c] : 0.0f;
+        for (int e = threadIdx.x; e < (TT - n) * DP; e += kScanThreads) {  // behind the last token: nothing is added, nothing decays
+            const int o = n * DP + e;
+            t[o] = 0.0f;
+            t[TT * DP + o] = 0.0f;
+            t[2 * TT * DP + o] = 1.0f;
         }
     };
-    fetch(0);
-    for (int i0 = 0; i0 < a.q_rows; i0 += TT) {
-        const int n = min(TT, a.q_rows - i0);
-        __syncthreads();
+    auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+    fetch(0, 0);
+    commit();
+    float uu[(DP + 31) / 32];
 #pragma unroll
-        for (int i = 0; i < NL; ++i) {
-            const int e = threadIdx.x + i * 256;
-            r_s[e] = rr[i];
-            k_s[e] = kr[i];
-            w_s[e] = expf(-expf(zr[i]));
-        }
-#pragma unroll
-        for (int i = 0; i < TT * 32 / 256; ++i) v_s[threadIdx.x + i * 256] = vr[i];
-        fetch(i0 + TT);
+    for (int j = 0; j < (DP + 31) / 32; ++j) uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f;
+    int buf = 0;
+    for (int i0 = 0; i0 < a.q_rows; i0 += TT, buf ^= 1) {
+        fetch(i0 + TT, buf ^ 1);
+        commit();
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
-        for (int t = warp; t < n; t += 8) {
-            float x = 0.0f;
-            for (int c = lane; c < D; c += 32) x = fmaf(r_s[t * DP + c] * a.u[head * D + c], k_s[t * DP + c], x);
-            x = warp_sum(x);
-            if (lane == 0) bonus_s[t] = x;
-        }
-        __syncthreads();
-        for (int t = 0; t < n; ++t) {
-            const float v = v_s[t * 32 + col];
-            float o0 = 0.0f, o1 = 0.0f;
+        const float* t = sm + buf * Cfg::kTile;
+        const float* rs = t;
+        const float* ks = t + TT * DP;
+        const float* ws = t + 2 * TT * DP;
+        const float* vs = t + 3 * TT * DP;
+        {   // the current token's own weight, sum of r u k
+            float x[TT / 2];
 #pragma unroll
-            for (int j = 0; j < NJ; ++j) {
-                const int at = t * DP + 32 * j + 4 * kg;
-                const float4 r = *reinterpret_cast<const float4*>(r_s + at), k = *reinterpret_cast<const float4*>(k_s + at), w = *reinterpret_cast<const float4*>(w_s + at);
-                o0 = fmaf(r.x, s[4 * j], o0); o1 = fmaf(r.y, s[4 * j + 1], o1);
-                o0 = fmaf(r.z, s[4 * j + 2], o0); o1 = fmaf(r.w, s[4 * j + 3], o1);
-                s[4 * j] = fmaf(w.x, s[4 * j], k.x * v);
-                s[4 * j + 1] = fmaf(w.y, s[4 * j + 1], k.y * v);
-                s[4 * j + 2] = fmaf(w.z, s[4 * j + 2], k.z * v);
-                s[4 * j + 3] = fmaf(w.w, s[4 * j + 3], k.w * v);
+            for (int i = 0; i < TT / 2; ++i) {
+                x[i] = 0.0f;
+#pragma unroll
+                for (int j = 0; j < DP / 32; ++j) x[i] = fmaf(rs[(warp * (TT / 2) + i) * DP + j * 32 + lane] * uu[j], ks[(warp * (TT / 2) + i) * DP + j * 32 + lane], x[i]);
             }
-            float o = o0 + o1;
-            o += __shfl_xor_sync(0xffffffffu, o, 1);
-            o += __shfl_xor_sync(0xffffffffu, o, 2);
-            o += __shfl_xor_sync(0xffffffffu, o, 4);
-            if (live && kg == (t & 7)) a.y[((int64_t)b * a.q_rows + i0 + t) * HD + head * D + v0 + col] = fmaf(bonus_s[t], v, o);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int i = 0; i < TT / 2; ++i) x[i] += __shfl_xor_sync(0xffffffffu, x[i], o);
+            if (lane == 0)
+#pragma unroll
+                for (int i = 0; i < TT / 2; ++i) bonus_s[warp * (TT / 2) + i] = x[i];
         }
+        __syncthreads();
+#pragma unroll 1
+        for (int g = 0; g < TT && i0 + g < a.q_rows; g += 8) {
+            float o[8][2];
+#pragma unroll
+            for (int q = 0; q < 8; ++q) {
+                const int tk = g + q;
+                const float2 v = *reinterpret_cast<const float2*>(vs + tk * kScanCols + col);
+                float o0 = 0.0f, o1 = 0.0f;
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    const int at = tk * DP + 32 * j + 4 * kg;
+                    const float4 r4 = *reinterpret_cast<const float4*>(rs + at), k4 = *reinterpret_cast<const float4*>(ks + at), w4 = *reinterpret_cast<const float4*>(ws + at);
+                    const float r[4] = {r4.x, r4.y, r4.z, r4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, w[4] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        o0 = fmaf(r[e], s[4 * j + e][0], o0);
+                        o1 = fmaf(r[e], s[4 * j + e][1], o1);
+                        s[4 * j + e][0] = fmaf(w[e], s[4 * j + e][0], k[e] * v.x);
+                        s[4 * j + e][1] = fmaf(w[e], s[4 * j + e][1], k[e] * v.y);
+                    }
+                }
+                o[q][0] = o0;
+                o[q][1] = o1;
+            }
+            // fold over the eight lanes of a column pair: lane kg ends with token g + kg
+#pragma unroll
+            for (int st = 4; st > 0; st >>= 1) {
+                const bool hi = kg & st;
+#pragma unroll
+                for (int q = 0; q < st; ++q)
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        const float give = hi ? o[q][c] : o[q + st][c], keep = hi ? o[q + st][c] : o[q][c];
+                        o[q][c] = keep + __shfl_xor_sync(0xffffffffu, give, st);
+                    }
+            }
+            const int tk = g + kg;
+            if (i0 + tk < a.q_rows) {
+                float* y = a.y + ((int64_t)b * a.q_rows + i0 + tk) * HD + head * D + v0 + col;
+                const float bonus = bonus_s[tk];
+#pragma unroll
+                for (int c = 0; c < 2; ++c)
+                    if (col + c < vc) y[c] = fmaf(bonus, vs[tk * kScanCols + col + c], o[0][c]);
+            }
+        }
+        __syncthreads();  // before the tile is refilled
     }
-    if (live)
 #pragma unroll
-        for (int j = 0; j < NJ; ++j)
+    for (int j = 0; j < NJ; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
                 const int k = 32 * j + 4 * kg + e;
-                if (k < D) state[(int64_t)k * D] = s[4 * j + e];
+                if (col + c < vc && k < D) state[(int64_t)k * D + c] = s[4 * j + e][c];
             }
     if (blockIdx.x == 0 && blockIdx.y == 0) {  // the token shift's state
         const int64_t last = (int64_t)b * a.q_rows + a.q_rows - 1;
         float* keep = a.shift + (int64_t)((p0 + a.q_rows - 1) & 1) * a.shift_slot + (int64_t)b * a.width;
-        for (int c = threadIdx.x; c < a.width; c += 256) keep[c] = a.hn[last * a.width + c];
+        for (int c = threadIdx.x; c < a.width; c += kScanThreads) keep[c] = a.hn[last * a.width + c];
     }
 }
 
 template <int NJ>
 cudaError_t scan_launch(const WkvArgs& a, cudaStream_t s) {
-    wkv_scan_kernel<NJ><<<dim3((unsigned)a.heads, (unsigned)((a.dim + 31) / 32), (unsigned)a.batch), 256, 0, s>>>(a);
+    static PerDeviceOnce once;
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(wkv_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ScanCfg<NJ>::kSmem); });
+    if (e != cudaSuccess) return e;
+    wkv_scan_kernel<NJ><<<dim3((unsigned)a.heads, (unsigned)((a.dim + kScanCols - 1) / kScanCols), (unsigned)a.batch), kScanThreads, ScanCfg<NJ>::kSmem, s>>>(a);
     return cudaGetLastError();
+}
+cudaError_t step_launch(const WkvArgs& a, cudaStream_t s, bool pdl) {
+    const dim3 grid((unsigned)a.heads, (unsigned)a.batch), block(kStepThreads);
+    if (a.dim <= 32) return launch_pdl(wkv_step_kernel<32>, grid, block, 0, s, pdl, a);
+    if (a.dim <= 64) return launch_pdl(wkv_step_kernel<64>, grid, block, 0, s, pdl, a);
+    if (a.dim <= 128) return launch_pdl(wkv_step_kernel<128>, grid, block, 0, s, pdl, a);
+    return launch_pdl(wkv_step_kernel<256>, grid, block, 0, s, pdl, a);
 }
 
 }  // namespace
@@ -262,19 +362,18 @@ cudaError_t launch_wkv_mix(const WkvMix& a, cudaStream_t s) {
 
 cudaError_t launch_wkv_step(const WkvArgs& a, cudaStream_t s, bool pdl) {
     if (a.dim > wkv_max_dim() || a.rank > kMaxRank || a.q_rows != 1) return cudaErrorInvalidValue;
-    const dim3 grid((unsigned)a.heads, (unsigned)a.batch), block(kStepThreads);
-    if (a.dim <= 32) return launch_pdl(wkv_step_kernel<32>, grid, block, 0, s, pdl, a);
-    if (a.dim <= 64) return launch_pdl(wkv_step_kernel<64>, grid, block, 0, s, pdl, a);
-    if (a.dim <= 128) return launch_pdl(wkv_step_kernel<128>, grid, block, 0, s, pdl, a);
-    return launch_pdl(wkv_step_kernel<256>, grid, block, 0, s, pdl, a);
+    WkvArgs x = a;
+    x.w = nullptr;
+    return step_launch(x, s, pdl);
 }
 
-cudaError_t launch_wkv_prefill(const WkvArgs& a, bool bf16, cudaStream_t s) {
-    (void)bf16;
+cudaError_t launch_wkv_prefill(const WkvArgs& a, cudaStream_t s) {
+    if (a.dim > wkv_max_dim() || !a.w) return cudaErrorInvalidValue;
+    if (a.q_rows == 1) return step_launch(a, s, false);
     if (a.dim <= 32) return scan_launch<1>(a, s);
     if (a.dim <= 64) return scan_launch<2>(a, s);
     if (a.dim <= 128) return scan_launch<4>(a, s);
-    return a.dim <= wkv_max_dim() ? scan_launch<8>(a, s) : cudaErrorInvalidValue;
+    return scan_launch<8>(a, s);
 }
 
 }  // namespace bt
