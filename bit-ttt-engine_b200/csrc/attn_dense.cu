@@ -697,9 +697,8 @@ struct LatentTile {
     const __nv_bfloat16* kv = nullptr;  // [sequence][kv_rows][heads k_main | heads v_stride]
     int64_t kv_ld = 0, kv_seq = 0;      // elements between positions and between sequences
     int k_main = 0;                     // columns of a head's own key part
-    const uint8_t* rot = nullptr;       // tiled latent cache
-    int64_t rot_seq = 0;
-    int rot_col = 0, seq_pad = 0, b0 = 0;
+    LatentView latent;
+    int b0 = 0;
     const float* gate = nullptr;        // output gates of the rows
     int64_t gate_ld = 0;
 };
@@ -736,7 +735,7 @@ __global__ void __launch_bounds__(kTileThreads) attn_tile_kernel(const DenseAttn
             const int r = i / qpieces, c = i - r * qpieces;
             const bool live = base + r <= last && c * 8 < ks;
             const void* src = kg + (int64_t)(base + r) * k_ld + c * 8;
-            if (LATENT && c * 8 >= lt.k_main) src = lt.rot + b * lt.rot_seq + dense_off(base + r, lt.rot_col + c * 8 - lt.k_main, lt.seq_pad);
+            if (LATENT && c * 8 >= lt.k_main) src = reinterpret_cast<const uint8_t*>(lt.latent.rows) + b * lt.latent.seq_bytes() + lt.latent.off(base + r, lt.latent.rot_col() + c * 8 - lt.k_main);
             ptx::cp16(k_sm + (bufi * kTileKeys + r) * KS + c * 16, live ? src : kg, live);
         }
         for (int i = threadIdx.x; i < kTileKeys * vpieces; i += kTileThreads) {
@@ -938,7 +937,7 @@ cudaError_t launch_latent_tile(const LatentAttn& l, const __nv_bfloat16* kv16, i
     a.dk = a.kv.k_stride; a.dv = l.vdim;
     LatentTile t;
     t.kv = kv16; t.k_main = pad8(l.dim); t.kv_ld = (int64_t)l.heads * (t.k_main + a.kv.v_stride); t.kv_seq = kv_rows * t.kv_ld;
-    t.rot = reinterpret_cast<const uint8_t*>(l.kv.rows); t.rot_seq = l.kv.seq_bytes(); t.rot_col = dense_kpad(l.rank); t.seq_pad = l.kv.seq_pad; t.b0 = b0;
+    t.latent = l.kv; t.b0 = b0;
     t.gate = l.gate ? l.proj + l.heads * (l.dim + l.rot) + l.rank + l.rot : nullptr;
     t.gate_ld = l.ld;
     return tile_launch_k<true>(a, t, out, s);

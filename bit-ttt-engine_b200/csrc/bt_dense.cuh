@@ -232,11 +232,16 @@ int attn_max_dim();  // of query/key and of value heads
 // Latent attention: keys and values of all heads are products of one latent row per position, one rotated key part is
 // shared by the heads
 // ---------------------------------------------------------------------------------------
+// f32 models: rows of `stride` floats.  bf16: groups of 8 positions, inside a group core matrices of 8 positions x 16 bytes over
+// the columns, latent [rank padded to 16] | rotated part [rot padded to 16]; a run of groups is contiguous.
 struct LatentView {
-    void* rows = nullptr;  // bf16: tiled [batch][(kpad(rank) + kpad(rot)) / 64][seq_pad][64]; f32: [batch, max_seq, stride]
+    void* rows = nullptr;
     int max_seq = 0, seq_pad = 0, rank = 0, rot = 0, stride = 0;
     bool f32 = false;
-    __host__ __device__ int64_t seq_bytes() const { return f32 ? (int64_t)max_seq * stride * 4 : (int64_t)seq_pad * (dense_kpad(rank) + dense_kpad(rot)) * 2; }
+    __host__ __device__ int rot_col() const { return (rank + 15) / 16 * 16; }
+    __host__ __device__ int cols() const { return rot_col() + (rot + 15) / 16 * 16; }
+    __host__ __device__ int64_t seq_bytes() const { return f32 ? (int64_t)max_seq * stride * 4 : (int64_t)seq_pad * cols() * 2; }
+    __host__ __device__ int64_t off(int64_t pos, int c) const { return (pos >> 3) * cols() * 16 + (c >> 3) * 128 + (pos & 7) * 16 + (c & 7) * 2; }  // bytes
 };
 struct LatentAttn {
     const float* proj = nullptr;   // rows q [heads][dim | rot] | latent [rank] | rotated key part [rot] | output gates [heads]
@@ -257,6 +262,8 @@ struct LatentAttn {
     __nv_bfloat16* q_buf = nullptr;  // tile kernel: [rows][heads][pad8(dim) + pad8(rot)]
     int64_t m_pad = 0;
 };
+// latents of positions [0, n) of `nb` sequences -> tiled activations [nb][kpad(rank) / 64][m_pad][64]
+cudaError_t launch_latent_tiles(const LatentView& v, int b0, int nb, int64_t n, uint8_t* tiles, int64_t m_pad, cudaStream_t s);
 // New tokens: latents normed, key parts rotated, both into the cache; queries to q_buf, or to q_rot and q_tiles / q_rows32
 cudaError_t launch_latent_prep(const LatentAttn& a, cudaStream_t s);
 // Attention over the latents (absorbed queries), one query position per CTA group; output rows [heads][rank], weighted by

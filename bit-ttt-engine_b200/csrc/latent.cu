@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentAttn a) {
     const int64_t r = blockIdx.x;
     const int b = (int)(r / a.q_rows), p = a.pos[b] + (int)(r % a.q_rows);
     const float* row = a.proj + r * a.ld;
-    const int H = a.heads, hd = a.dim + a.rot, kr = dense_kpad(a.rank);
+    const int H = a.heads, hd = a.dim + a.rot, kr = a.kv.rot_col();
     const float* c = row + H * hd;
     const float inv = latent_inv(a, c, red);
     if (p < 0 || p >= a.kv.max_seq) return;
@@ -70,9 +70,9 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentAttn a) {
         for (int i = threadIdx.x; i < a.rot; i += 256) dst[a.rank + i] = rotated(a, c + a.rank, i, p);
     } else {
         for (int i = threadIdx.x; i < a.rank; i += 256)
-            *reinterpret_cast<__nv_bfloat16*>(seq + dense_off(p, i, a.kv.seq_pad)) = __float2bfloat16_rn(c[i] * inv * a.c_norm[i]);
+            *reinterpret_cast<__nv_bfloat16*>(seq + a.kv.off(p, i)) = __float2bfloat16_rn(c[i] * inv * a.c_norm[i]);
         for (int i = threadIdx.x; i < a.rot; i += 256)
-            *reinterpret_cast<__nv_bfloat16*>(seq + dense_off(p, kr + i, a.kv.seq_pad)) = __float2bfloat16_rn(rotated(a, c + a.rank, i, p));
+            *reinterpret_cast<__nv_bfloat16*>(seq + a.kv.off(p, kr + i)) = __float2bfloat16_rn(rotated(a, c + a.rank, i, p));
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (a.q_buf) {  // the sizes padded to whole 16-byte pieces
@@ -101,215 +101,264 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentAttn a) {
     }
 }
 
+__global__ void __launch_bounds__(256) latent_tiles_kernel(const LatentView v, int b0, int64_t n, uint8_t* __restrict__ tiles, int64_t m_pad) {
+    const int per = dense_kpad(v.rank) / 8;  // pieces per position
+    const int64_t groups = (n + 7) / 8, total = groups * per * 8;
+    const uint8_t* src = reinterpret_cast<const uint8_t*>(v.rows) + (b0 + (int64_t)blockIdx.y) * v.seq_bytes();
+    uint8_t* dst = tiles + blockIdx.y * m_pad * per * 16;
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t pos = i / (per * 8) * 8 + (i & 7);
+        const int c = (int)(i / 8 % per) * 8;
+        *reinterpret_cast<uint4*>(dst + dense_off(pos, c, m_pad)) = c < v.rot_col() ? *reinterpret_cast<const uint4*>(src + v.off(pos, c)) : make_uint4(0, 0, 0, 0);
+    }
+}
+
 // The end of a span kernel: every CTA of the cluster holds maxima, sums and un-normed outputs [head][W] of its span; each
-// finishes an equal share of the outputs.  LOG2: the maxima are in units of ln 2.
+// finishes an equal share of the outputs.  LOG2: the maxima are in units of ln 2.  fac: [heads][kMaxSplits] floats.
 template <bool LOG2>
-__device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, float* l_s, float* o_s, int W, int nh, int head0,
+__device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, float* l_s, float* o_s, float* fac, int W, int nh, int head0,
                                             int64_t r, int split, int splits, const ActOut& out) {
     cg::cluster_group cluster = cg::this_cluster();
     if (splits > 1) cluster.sync(); else __syncthreads();
     const float* gates = a.gate ? a.proj + r * a.ld + a.heads * (a.dim + a.rot) + a.rank + a.rot : nullptr;
-    const int kr = dense_kpad(a.rank), total = nh * a.rank;
-    const int i1 = (int)((int64_t)total * (split + 1) / splits);
-    for (int i = (int)((int64_t)total * split / splits) + threadIdx.x; i < i1; i += blockDim.x) {
-        const int h = i / a.rank, c = i - h * a.rank, head = head0 + h;
-        float ms[kMaxSplits], ls[kMaxSplits], os[kMaxSplits], m = -INFINITY;
+    // a span's factor per head: its share of the softmax over all spans, times the output gate
+    for (int h = threadIdx.x; h < nh; h += blockDim.x) {
+        float ms[kMaxSplits], m = -INFINITY, den = 0.0f;
 #pragma unroll
         for (int s = 0; s < kMaxSplits; ++s) {  // all remote reads in flight together
-            ms[s] = -INFINITY; ls[s] = os[s] = 0.0f;
-            if (s < splits) {
-                ms[s] = *(splits > 1 ? cluster.map_shared_rank(m_s, s) + h : m_s + h);
-                ls[s] = *(splits > 1 ? cluster.map_shared_rank(l_s, s) + h : l_s + h);
-                os[s] = *(splits > 1 ? cluster.map_shared_rank(o_s, s) + h * W + c : o_s + h * W + c);
-            }
+            ms[s] = s < splits ? *(splits > 1 ? cluster.map_shared_rank(m_s, s) + h : m_s + h) : -INFINITY;
             m = fmaxf(m, ms[s]);
         }
-        float den = 0.0f, num = 0.0f;
 #pragma unroll
-        for (int s = 0; s < kMaxSplits; ++s) {
-            const float f = LOG2 ? ex2(ms[s] - m) : expf(ms[s] - m);  // an empty span: 0
-            den = fmaf(ls[s], f, den);
-            num = fmaf(os[s], f, num);
+        for (int s = 0; s < kMaxSplits; ++s)
+            if (s < splits) {
+                ms[s] = LOG2 ? ex2(ms[s] - m) : expf(ms[s] - m);  // an empty span: 0
+                den = fmaf(*(splits > 1 ? cluster.map_shared_rank(l_s, s) + h : l_s + h), ms[s], den);
+            }
+        const float f = (gates ? sigmoid_f(gates[head0 + h]) : 1.0f) / den;
+#pragma unroll
+        for (int s = 0; s < kMaxSplits; ++s)
+            if (s < splits) fac[h * kMaxSplits + s] = ms[s] * f;
+    }
+    __syncthreads();
+    const int kr = dense_kpad(a.rank), quads = (a.rank + 3) / 4, total = nh * quads;  // W is a multiple of 4
+    const int i1 = (int)((int64_t)total * (split + 1) / splits);
+    for (int i = (int)((int64_t)total * split / splits) + threadIdx.x; i < i1; i += blockDim.x) {
+        const int h = i / quads, c = (i - h * quads) * 4, head = head0 + h;
+        float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll 4
+        for (int s = 0; s < splits; ++s) {
+            const float4 o = *reinterpret_cast<const float4*>((splits > 1 ? cluster.map_shared_rank(o_s, s) : o_s) + h * W + c);
+            const float f = fac[h * kMaxSplits + s];
+            v[0] = fmaf(o.x, f, v[0]); v[1] = fmaf(o.y, f, v[1]); v[2] = fmaf(o.z, f, v[2]); v[3] = fmaf(o.w, f, v[3]);
         }
-        float v = num / den;
-        if (gates) v *= sigmoid_f(gates[head]);
-        if (out.tiles) *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, head * kr + c, out.m_pad)) = __float2bfloat16_rn(v);
-        else out.rows[r * out.ld + head * a.rank + c] = v;
+        if (out.tiles && c + 4 <= a.rank) {
+            *reinterpret_cast<uint2*>(out.tiles + dense_off(r, head * kr + c, out.m_pad)) = make_uint2(ptx::pack2(v[0], v[1]), ptx::pack2(v[2], v[3]));
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (c + j >= a.rank) break;
+                if (out.tiles) *reinterpret_cast<__nv_bfloat16*>(out.tiles + dense_off(r, head * kr + c + j, out.m_pad)) = __float2bfloat16_rn(v[j]);
+                else out.rows[r * out.ld + head * a.rank + c + j] = v[j];
+            }
+        }
     }
     if (splits > 1) cluster.sync();  // no CTA leaves while its sums are being read
 }
 
 // ---------------------------------------------------------------------------------------
-// one query position, 16 MT heads, on the tensor cores (bf16 cache)
+// one query position, HG heads, on the tensor cores (bf16 cache)
 // ---------------------------------------------------------------------------------------
-// The cache is laid out in core matrices (8 positions x 16 bytes), so blocks of 32 positions arrive as one bulk copy per 64
-// columns and every ldmatrix reads 128 consecutive bytes.  Per block: sixteen warps share the scores' product, eight parts of
-// the columns (each warp has its part of the queries in registers) x 16 positions, and leave partial scores; then each makes
-// the softmax of MT heads and multiplies its 8 NT latent columns.  Softmax weights enter their product as bf16 hi + lo.
-constexpr int kSpanThreads = 512, kSpanWarps = kSpanThreads / 32, kKeys = 32, kMaxSteps = (kMaxRank + kMaxRot) / 16 / 8;
-constexpr int kScoreLd = 40;  // floats per row of partial scores
+// The cache is laid out in core matrices (8 positions x 16 bytes), per group of 8 positions all columns one after the other, so
+// that a block of 128 positions is a few bulk copies.  In shared memory it is the K-major A operand of the scores (positions x
+// columns) and, read the other way, the MN-major A operand of the values (latent columns x positions).
+//   scores^T [128 positions][HG]  = block . queries^T            (tcgen05, accumulators in TMEM)
+//   softmax: scores through shared memory, a warp per HG / 16 heads; weights leave as bf16 hi and lo
+//   outputs^T [rank][HG]         += block^T . (hi + lo)^T        (tiles of 128 latent columns, accumulators in TMEM)
+// The outputs are rescaled only when a maximum has grown by more than 2^8.
+constexpr int kSpanThreads = 512, kSpanWarps = kSpanThreads / 32, kKeys = 128, kMaxStages = 3;
+constexpr float kLazy = 8.0f;
 
-template <int MT>
+template <int HG>
 struct SpanCfg {
-    static constexpr int H = 16 * MT;
-    static constexpr size_t kPart = (size_t)8 * H * kScoreLd * 4;  // partial scores; first the queries
-    static size_t part(int chunks) { const size_t q = (size_t)chunks * MT * 2048; return q > kPart ? q : kPart; }
-    static size_t fixed(int chunks) { return part(chunks) + (size_t)MT * 2 * 1024 + 3 * H * 4 + 32 * 4 + (size_t)chunks * 128 + 64; }
+    static constexpr int kP = HG * kKeys * 2;                                   // bytes of the weights' hi (lo) part
+    static constexpr size_t kFixed = (size_t)2 * kP + HG * kKeys * 4 + (3 + kMaxSplits) * HG * 4 + 32 * 4 + 128;
+    __host__ __device__ static size_t q(int cols) { return (size_t)HG * cols * 2; }
+    static size_t fixed(int cols) { return q(cols) + kFixed + (size_t)cols * 2; }
 };
+__device__ __forceinline__ uint32_t span_idesc(int n, bool a_mn) {  // f32 += bf16 . bf16, M = 128
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((a_mn ? 1u : 0u) << 15) | ((uint32_t)(n >> 3) << 17) | (8u << 24);
+}
 
-template <int NT, int MT>
-__global__ void __launch_bounds__(kSpanThreads, 1) latent_span_mma_kernel(const LatentAttn a, bool prepared, int splits, int stages,
-                                                                       int part_bytes, unsigned int* err, const ActOut out) {
-    constexpr int NH = 16 * MT, NS = MT;  // heads of the CTA; of a warp in the softmax
+template <int HG>
+__global__ void __launch_bounds__(kSpanThreads, 1) latent_span_tc_kernel(const LatentAttn a, bool prepared, int splits, int stages,
+                                                                         unsigned int* err, const ActOut out) {
+    using Cfg = SpanCfg<HG>;
+    constexpr int NS = HG / kSpanWarps;  // heads of a warp in the softmax
     extern __shared__ __align__(128) uint8_t sm[];
-    const int kcl = dense_kpad(a.rank) / 64, chunks = kcl + dense_kpad(a.rot) / 64;
-    const int stage_bytes = chunks * kKeys * 128;
-    uint8_t* q_s = sm + (size_t)stages * stage_bytes;    // [chunk][MT][2 groups of 8 heads][8 pieces][8 heads][16 bytes]
-    float* s_s = reinterpret_cast<float*>(q_s);          // [8 warps][heads][kScoreLd]
-    uint8_t* p_hi = q_s + part_bytes;                    // softmax weights [MT][16 heads][32 positions], core matrices
-    uint8_t* p_lo = p_hi + MT * 1024;
-    float* m_s = reinterpret_cast<float*>(p_lo + MT * 1024);
-    float* l_s = m_s + NH;
-    float* al_s = l_s + NH;
-    float* red = al_s + NH;
-    __nv_bfloat16* new_s = reinterpret_cast<__nv_bfloat16*>(red + 32);  // the new token's row [chunks * 64]
-    uint64_t* full = reinterpret_cast<uint64_t*>(new_s + chunks * 64);  // up to eight
+    const int kl = a.kv.rot_col(), cols = a.kv.cols(), pieces = cols / 8;
+    const uint32_t group = (uint32_t)cols * 16;          // bytes of 8 positions (heads)
+    const uint32_t stage_bytes = group * (kKeys / 8);
+    uint8_t* q_s = sm + (size_t)stages * stage_bytes;    // queries [HG / 8][pieces][8 heads][16 bytes]
+    uint8_t* p_hi = q_s + Cfg::q(cols);                // softmax weights [HG / 8][16 pieces][8 heads][16 bytes]
+    uint8_t* p_lo = p_hi + Cfg::kP;
+    float* s_s = reinterpret_cast<float*>(p_lo + Cfg::kP);  // scores [HG][128]
+    float* m_s = s_s + HG * kKeys;
+    float* l_s = m_s + HG;
+    float* al_s = l_s + HG;
+    float* fac = al_s + HG;                              // [HG][kMaxSplits]
+    float* red = fac + HG * kMaxSplits;
+    uint64_t* full = reinterpret_cast<uint64_t*>(red + 32);
+    uint64_t* s_done = full + kMaxStages;
+    uint64_t* o_done = s_done + 1;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_done + 1);
+    __nv_bfloat16* new_s = reinterpret_cast<__nv_bfloat16*>(full + 16);  // the new token's row [cols]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int H = a.heads, hd = a.dim + a.rot;
-    const int head0 = blockIdx.y * NH, nh = min(NH, H - head0);
+    const int head0 = blockIdx.y * HG, nh = min(HG, H - head0);
     const int64_t r = blockIdx.z;
     const int b = (int)(r / a.q_rows), split = blockIdx.x;
     const int p = a.pos[b] + (int)(r % a.q_rows);
     const int total = min(p + 1, a.kv.max_seq);
-    const int span = ((total + splits - 1) / splits + kKeys - 1) / kKeys * kKeys;
+    const int span = ((total + splits - 1) / splits + 7) / 8 * 8;
     const int t0 = min(split * span, total), t1 = min(t0 + span, total);
     const int blocks = (t1 - t0 + kKeys - 1) / kKeys;
     const bool owner = !prepared && t1 == p + 1 && t0 < t1;
     uint8_t* seq = reinterpret_cast<uint8_t*>(a.kv.rows) + b * a.kv.seq_bytes();
     bool ok = true;
     if (threadIdx.x == 0) {
-        for (int s = 0; s < stages; ++s) ptx::mbar_init(&full[s], 1);
+        for (int s = 0; s < kMaxStages; ++s) ptx::mbar_init(&full[s], 1);
+        ptx::mbar_init(s_done, 1);
+        ptx::mbar_init(o_done, 1);
         ptx::mbar_fence_init();
     }
+    if (warp == 1) { ptx::tmem_alloc(tmem_slot, 256); ptx::tmem_relinquish(); }
+    ptx::tc_fence_before();
     __syncthreads();
-    auto load = [&](int i, int slot) {  // warp 0: the i-th block of the span, a lane per 64 columns
+    ptx::tc_fence_after();
+    const uint32_t tmem = *tmem_slot, tmem_o = tmem + HG;
+    auto load = [&](int i) {  // warp 0: the i-th block of the span
         if (i >= blocks) return;
-        if (lane == 0) ptx::mbar_arrive_expect_tx(&full[slot], stage_bytes);
+        const int slot = i % stages, live = (min(kKeys, t1 - t0 - i * kKeys) + 7) / 8;  // groups with a position of the span
+        if (lane == 0) ptx::mbar_arrive_expect_tx(&full[slot], live * group);
         __syncwarp();
-        if (lane < chunks)
-            ptx::bulk_g2s(sm + (size_t)slot * stage_bytes + lane * kKeys * 128, seq + ((int64_t)lane * a.kv.seq_pad + t0 + i * kKeys) * 128, kKeys * 128, &full[slot]);
+        const int g0 = lane * 2, n = min(2, live - g0);  // two groups a lane
+        if (n > 0) ptx::bulk_g2s(sm + (size_t)slot * stage_bytes + g0 * group, seq + ((int64_t)t0 / 8 + i * (kKeys / 8) + g0) * group, n * group, &full[slot]);
     };
     if (prepared) ptx::pdl_wait();  // the cache rows come from the kernel in front
+    if (blocks > 0 && blocks <= stages) {  // groups of the last block that no copy fills
+        uint8_t* st = sm + (size_t)(blocks - 1) * stage_bytes;
+        const uint32_t o = (uint32_t)((t1 - t0 - (blocks - 1) * kKeys + 7) / 8) * group;
+        for (uint32_t e = o + threadIdx.x * 16; e < stage_bytes; e += kSpanThreads * 16) *reinterpret_cast<uint4*>(st + e) = make_uint4(0, 0, 0, 0);
+    }
     if (warp == 0)
-        for (int i = 0; i < stages - 1; ++i) load(i, i);
+        for (int i = 0; i < stages; ++i) load(i);
     if (!prepared) ptx::pdl_wait();
     ptx::pdl_launch_dependents();
 
     // ---- queries: [absorbed | rotated] ----
     const float* row = a.proj + r * a.ld;
-    const int kl = kcl * 64;
-    for (int i = threadIdx.x; i < NH * chunks * 32; i += kSpanThreads) {  // two columns at a time
-        const int h = i / (chunks * 32), c = (i - h * chunks * 32) * 2;
-        float v[2] = {0.0f, 0.0f};
-        if (h < nh)
+    for (int i = threadIdx.x; i < HG * pieces; i += kSpanThreads) {  // eight columns at a time
+        const int h = i / pieces, piece = i - h * pieces, c = piece * 8;
+        float v[8];
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                if (c < kl) { if (c + j < a.rank) v[j] = a.q_abs[(r * H + head0 + h) * a.rank + c + j]; }
-                else if (c + j - kl < a.rot) v[j] = prepared ? a.q_rot[(r * H + head0 + h) * a.rot + c + j - kl] : rotated(a, row + (head0 + h) * hd + a.dim, c + j - kl, p);
+        for (int j = 0; j < 8; ++j) v[j] = 0.0f;
+        if (h < nh) {
+            if (c < kl) {
+                const float* src = a.q_abs + (r * H + head0 + h) * a.rank + c;
+                if (c + 8 <= a.rank && (a.rank & 3) == 0) {
+                    const float4 x = *reinterpret_cast<const float4*>(src), y = *reinterpret_cast<const float4*>(src + 4);
+                    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) if (c + j < a.rank) v[j] = src[j];
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    if (c + j - kl < a.rot)
+                        v[j] = prepared ? a.q_rot[(r * H + head0 + h) * a.rot + c + j - kl] : rotated(a, row + (head0 + h) * hd + a.dim, c + j - kl, p);
             }
-        *reinterpret_cast<uint32_t*>(q_s + (c >> 6) * MT * 2048 + (h >> 3) * 1024 + ((c & 63) >> 3) * 128 + (h & 7) * 16 + (c & 7) * 2) = ptx::pack2(v[0], v[1]);
+        }
+        *reinterpret_cast<uint4*>(q_s + (h >> 3) * group + piece * 128 + (h & 7) * 16) =
+            make_uint4(ptx::pack2(v[0], v[1]), ptx::pack2(v[2], v[3]), ptx::pack2(v[4], v[5]), ptx::pack2(v[6], v[7]));
     }
     if (owner) {
         const float* c = row + H * hd;
         const float inv = latent_inv(a, c, red);
-        for (int i = threadIdx.x; i < chunks * 64; i += kSpanThreads) {
+        for (int i = threadIdx.x; i < cols; i += kSpanThreads) {
             float v = 0.0f;
             if (i < kl) { if (i < a.rank) v = c[i] * inv * a.c_norm[i]; }
             else if (i - kl < a.rot) v = rotated(a, c + a.rank, i - kl, p);
             const __nv_bfloat16 w = __float2bfloat16_rn(v);
             new_s[i] = w;
-            if (blockIdx.y == 0) *reinterpret_cast<__nv_bfloat16*>(seq + dense_off(p, i, a.kv.seq_pad)) = w;
+            if (blockIdx.y == 0) *reinterpret_cast<__nv_bfloat16*>(seq + a.kv.off(p, i)) = w;
         }
     }
+    ptx::fence_async_smem();
     __syncthreads();
-    // this warp's 16-column steps: part, part + 8, ... of the latent part's and the rotated part's
-    const int part = warp & 7, half = warp >> 3;
-    const int steps_l = (a.rank + 15) / 16, steps = steps_l + (a.rot + 15) / 16;
-    uint32_t qf[kMaxSteps][MT][4];
-    uint32_t k_off[kMaxSteps];
-#pragma unroll
-    for (int i = 0; i < kMaxSteps; ++i) {
-        const int ks = part + 8 * i, kk = ks < steps_l ? ks : ks - steps_l + kcl * 4;
-        k_off[i] = (uint32_t)((kk >> 2) * kKeys * 128 + (kk & 3) * 256 + half * 2048);
-        if (ks < steps)
-#pragma unroll
-            for (int m = 0; m < MT; ++m)
-                ptx::ldsm4(qf[i][m], ptx::smem_u32(q_s) + ((kk >> 2) * MT + m) * 2048 + (kk & 3) * 256 + ((lane >> 3) & 1) * 1024 + (lane >> 4) * 128 + (lane & 7) * 16);
-    }
-    __syncthreads();  // the partial scores take the queries' place
 
-    float acc[MT][NT][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int i = 0; i < NT; ++i)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) acc[m][i][j] = 0.0f;
-    float m_run[NS], l_run[NS];  // heads NS warp ..: maximum; this lane's share of the sum
+    float m_run[NS], l_run[NS];  // heads NS warp ..: reference maximum; this lane's share of the sum
 #pragma unroll
     for (int j = 0; j < NS; ++j) { m_run[j] = -INFINITY; l_run[j] = 0.0f; }
     const float unit = a.scale * 1.4426950408889634f;
-    const uint32_t p_off = ((lane >> 3) & 1) * 512 + (lane >> 4) * 128 + (lane & 7) * 16;
-    const uint32_t ph = ptx::smem_u32(p_hi) + p_off, pl = ptx::smem_u32(p_lo) + p_off;
-    const uint32_t k_core = (lane >> 4) * 1024 + ((lane >> 3) & 1) * 128 + (lane & 7) * 16;  // two groups of positions x two pieces
-
-    int slot = 0, before = stages - 1;  // ring slots of this block and of the one before it
-    uint32_t parity = 0;
+    const int steps = cols / 16, m_tiles = (a.rank + 127) / 128;
     for (int i = 0; i < blocks; ++i) {
+        const int slot = i % stages;
         uint8_t* st = sm + (size_t)slot * stage_bytes;
-        ok &= ptx::mbar_wait_bounded(&full[slot], parity);
+        const uint32_t kv = ptx::smem_u32(st);
         const int base = t0 + i * kKeys;
+        if (warp == 0 && i > 0) {  // the block before this one is used up: its slot takes the next one to come
+            ok &= ptx::mbar_wait_bounded(o_done, (uint32_t)((i - 1) & 1));
+            load(i + stages - 1);
+        }
         if (owner && i == blocks - 1) {  // the new row has not been in the copy
+            ok &= ptx::mbar_wait_bounded(&full[slot], (uint32_t)((i / stages) & 1));
             const int at = p - base;
-            for (int c = threadIdx.x; c < chunks * 8; c += kSpanThreads)
-                *reinterpret_cast<uint4*>(st + (c >> 3) * kKeys * 128 + (at >> 3) * 1024 + (c & 7) * 128 + (at & 7) * 16) = *reinterpret_cast<const uint4*>(new_s + c * 8);
+            for (int c = threadIdx.x; c < pieces; c += kSpanThreads)
+                *reinterpret_cast<uint4*>(st + (at >> 3) * group + c * 128 + (at & 7) * 16) = *reinterpret_cast<const uint4*>(new_s + c * 8);
+            ptx::fence_async_smem();
             __syncthreads();
         }
-        const uint32_t kv = ptx::smem_u32(st);
-        {
-            float s[MT][2][4] = {};
+        if (warp == 1 && lane == 0) {
+            ok &= ptx::mbar_wait_bounded(&full[slot], (uint32_t)((i / stages) & 1));
+            ptx::tc_fence_after();
+            const uint32_t q_addr = ptx::smem_u32(q_s);
+            for (int k = 0; k < steps; ++k) {
+                const uint32_t o = (uint32_t)k * 256;
+                ptx::umma_f16(tmem, ptx::smem_desc(kv + o, 128, group), ptx::smem_desc(q_addr + o, 128, group), span_idesc(HG, false), k > 0 ? 1u : 0u);
+            }
+            ptx::umma_commit(s_done);
+        }
+        __syncwarp();
+        if (warp < 4) {  // lane = position
+            ok &= ptx::mbar_wait_bounded(s_done, (uint32_t)(i & 1));
+            ptx::tc_fence_after();
+            const int key = warp * 32 + lane;
+            const bool live = base + key < t1;
 #pragma unroll
-            for (int k = 0; k < kMaxSteps; ++k)
-                if (part + 8 * k < steps) {
-                    uint32_t kf[4];
-                    ptx::ldsm4(kf, kv + k_off[k] + k_core);
+            for (int c = 0; c < HG; c += 16) {
+                uint32_t v[16];
+                ptx::tmem_ld16(tmem + ((uint32_t)(warp * 32) << 16) + c, v);
+                ptx::tmem_ld_wait();
 #pragma unroll
-                    for (int m = 0; m < MT; ++m) {
-                        ptx::mma_bf16(s[m][0], qf[k][m], kf[0], kf[1]);
-                        ptx::mma_bf16(s[m][1], qf[k][m], kf[2], kf[3]);
-                    }
-                }
-            float* sp = s_s + (part * NH + (lane >> 2)) * kScoreLd + half * 16 + (lane & 3) * 2;
-#pragma unroll
-            for (int m = 0; m < MT; ++m)
-#pragma unroll
-                for (int g = 0; g < 2; ++g) {
-                    *reinterpret_cast<float2*>(sp + m * 16 * kScoreLd + g * 8) = make_float2(s[m][g][0], s[m][g][1]);
-                    *reinterpret_cast<float2*>(sp + (m * 16 + 8) * kScoreLd + g * 8) = make_float2(s[m][g][2], s[m][g][3]);
-                }
+                for (int j = 0; j < 16; ++j) s_s[(c + j) * kKeys + key] = live ? __uint_as_float(v[j]) * unit : -INFINITY;
+            }
+            ptx::tc_fence_before();
         }
         __syncthreads();
-        if (warp == 0) load(i + stages - 1, before);  // into the slot of the block before this one
+        if (i > 0) {  // the weights' buffers and the outputs are free
+            ok &= ptx::mbar_wait_bounded(o_done, (uint32_t)((i - 1) & 1));
+            ptx::tc_fence_after();
+        }
+        bool grown = false;
         {
-            float x[NS], mx[NS];
+            float4 x[NS];
+            float mx[NS];
 #pragma unroll
             for (int j = 0; j < NS; ++j) {
-                const float* sp = s_s + (warp * NS + j) * kScoreLd + lane;
-                float v = 0.0f;
-#pragma unroll
-                for (int w = 0; w < 8; ++w) v += sp[w * NH * kScoreLd];
-                x[j] = base + lane < t1 ? v * unit : -INFINITY;
-                mx[j] = x[j];
+                x[j] = *reinterpret_cast<const float4*>(s_s + (warp * NS + j) * kKeys + lane * 4);
+                mx[j] = fmaxf(fmaxf(x[j].x, x[j].y), fmaxf(x[j].z, x[j].w));
             }
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1)
@@ -318,67 +367,80 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_mma_kernel(const 
 #pragma unroll
             for (int j = 0; j < NS; ++j) {
                 const int h = warp * NS + j;
-                const float m_new = fmaxf(m_run[j], mx[j]), al = ex2(m_run[j] - m_new), e = ex2(x[j] - m_new);  // al: 0 for the first block
-                m_run[j] = m_new;
-                l_run[j] = fmaf(l_run[j], al, e);
-                const __nv_bfloat16 hi = __float2bfloat16_rn(e);
-                const int o = (h >> 4) * 1024 + ((h >> 3) & 1) * 512 + (lane >> 3) * 128 + (h & 7) * 16 + (lane & 7) * 2;
-                *reinterpret_cast<__nv_bfloat16*>(p_hi + o) = hi;
-                *reinterpret_cast<__nv_bfloat16*>(p_lo + o) = __float2bfloat16_rn(e - __bfloat162float(hi));
+                float al = 1.0f;
+                if (mx[j] > m_run[j] + kLazy) {  // the first block always
+                    al = ex2(m_run[j] - mx[j]);
+                    m_run[j] = mx[j];
+                    grown = true;
+                }
+                const float e0 = ex2(x[j].x - m_run[j]), e1 = ex2(x[j].y - m_run[j]), e2 = ex2(x[j].z - m_run[j]), e3 = ex2(x[j].w - m_run[j]);
+                l_run[j] = fmaf(l_run[j], al, (e0 + e1) + (e2 + e3));
+                const uint32_t h0 = ptx::pack2(e0, e1), h1 = ptx::pack2(e2, e3);
+                const int o = (h >> 3) * 2048 + (lane >> 1) * 128 + (h & 7) * 16 + (lane & 1) * 8;
+                *reinterpret_cast<uint2*>(p_hi + o) = make_uint2(h0, h1);
+                *reinterpret_cast<uint2*>(p_lo + o) = make_uint2(ptx::pack2(e0 - __uint_as_float(h0 << 16), e1 - __uint_as_float(h0 & 0xffff0000u)),
+                                                                 ptx::pack2(e2 - __uint_as_float(h1 << 16), e3 - __uint_as_float(h1 & 0xffff0000u)));
                 if (lane == 0) al_s[h] = al;
             }
         }
-        __syncthreads();
+        ptx::fence_async_smem();
+        const int rescale = __syncthreads_or(grown && i > 0);
+        if (rescale) {  // warps w, w + 4, ... take the same lanes and different tiles
+            for (int mt = warp >> 2; mt < m_tiles; mt += 4) {
+                const uint32_t at = tmem_o + mt * HG + ((uint32_t)((warp & 3) * 32) << 16);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-            const float al0 = al_s[m * 16 + (lane >> 2)], al1 = al_s[m * 16 + (lane >> 2) + 8];
-            if (__any_sync(0xffffffffu, al0 != 1.0f || al1 != 1.0f))
+                for (int c = 0; c < HG; c += 16) {
+                    uint32_t v[16];
+                    ptx::tmem_ld16(at + c, v);
+                    ptx::tmem_ld_wait();
 #pragma unroll
-                for (int n = 0; n < NT; ++n) { acc[m][n][0] *= al0; acc[m][n][1] *= al0; acc[m][n][2] *= al1; acc[m][n][3] *= al1; }
-        }
-        const int col0 = warp * NT * 8;
-        if (col0 < a.rank) {
-            uint32_t hi[2][MT][4], lo[2][MT][4];
-#pragma unroll
-            for (int k = 0; k < 2; ++k)
-#pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    ptx::ldsm4(hi[k][m], ph + m * 1024 + k * 256);
-                    ptx::ldsm4(lo[k][m], pl + m * 1024 + k * 256);
-                }
-#pragma unroll
-            for (int n = 0; n < NT; ++n) {
-                const int col = col0 + n * 8;
-                uint32_t vf[4];  // 8 columns of the four groups of positions
-                ptx::ldsm4t(vf, kv + (col >> 6) * kKeys * 128 + ((col & 63) >> 3) * 128 + (lane >> 3) * 1024 + (lane & 7) * 16);
-#pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    ptx::mma_bf16(acc[m][n], hi[0][m], vf[0], vf[1]);
-                    ptx::mma_bf16(acc[m][n], lo[0][m], vf[0], vf[1]);
-                    ptx::mma_bf16(acc[m][n], hi[1][m], vf[2], vf[3]);
-                    ptx::mma_bf16(acc[m][n], lo[1][m], vf[2], vf[3]);
+                    for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) * al_s[c + j]);
+                    ptx::tmem_st16(at + c, v);
                 }
             }
+            ptx::tmem_st_wait();
+            ptx::tc_fence_before();
+            __syncthreads();
         }
-        before = slot;
-        if (++slot == stages) { slot = 0; parity ^= 1; }
+        if (warp == 1 && lane == 0) {
+            ptx::tc_fence_after();
+            const uint32_t ph = ptx::smem_u32(p_hi), pl = ptx::smem_u32(p_lo);
+            for (int mt = 0; mt < m_tiles; ++mt)
+#pragma unroll
+                for (int k = 0; k < kKeys / 16; ++k) {
+                    const uint64_t ad = ptx::smem_desc(kv + mt * 2048 + k * 2 * group, group, 128);
+                    ptx::umma_f16(tmem_o + mt * HG, ad, ptx::smem_desc(ph + k * 256, 128, 2048), span_idesc(HG, true), i > 0 || k > 0 ? 1u : 0u);
+                    ptx::umma_f16(tmem_o + mt * HG, ad, ptx::smem_desc(pl + k * 256, 128, 2048), span_idesc(HG, true), 1u);
+                }
+            ptx::umma_commit(o_done);
+        }
     }
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
         const float l = warp_sum(l_run[j]);
         if (lane == 0) { m_s[warp * NS + j] = m_run[j]; l_s[warp * NS + j] = l; }
     }
-    __syncthreads();  // the ring is free
-    constexpr int W = 8 * kSpanWarps * NT;
+    const int W = m_tiles * 128;
     float* o_s = reinterpret_cast<float*>(sm);  // [heads][W], in the ring's place
+    if (blocks > 0) {
+        ok &= ptx::mbar_wait_bounded(o_done, (uint32_t)((blocks - 1) & 1));
+        ptx::tc_fence_after();
+    }
+    __syncthreads();
+    for (int mt = warp >> 2; mt < m_tiles; mt += 4)
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+        for (int c = 0; c < HG; c += 16) {
+            uint32_t v[16];
+            ptx::tmem_ld16(tmem_o + mt * HG + c + ((uint32_t)((warp & 3) * 32) << 16), v);
+            ptx::tmem_ld_wait();
 #pragma unroll
-        for (int n = 0; n < NT; ++n)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) o_s[(m * 16 + (lane >> 2) + (j >> 1) * 8) * W + (warp * NT + n) * 8 + (lane & 3) * 2 + (j & 1)] = acc[m][n][j];
+            for (int j = 0; j < 16; ++j) o_s[(c + j) * W + mt * 128 + (warp & 3) * 32 + lane] = blocks > 0 ? __uint_as_float(v[j]) : 0.0f;
+        }
     if (!ok) atomicExch(err, kErrLatentTimeout);
-    merge_spans<true>(a, m_s, l_s, o_s, W, nh, head0, r, split, splits, out);
+    ptx::tc_fence_before();
+    __syncthreads();
+    if (warp == 1) ptx::tmem_dealloc(tmem, 256);
+    merge_spans<true>(a, m_s, l_s, o_s, fac, W, nh, head0, r, split, splits, out);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -387,14 +449,15 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_mma_kernel(const 
 constexpr int kF32Heads = 8, kF32Keys = 32, kF32Threads = 256;
 __global__ void __launch_bounds__(kF32Threads) latent_span_f32_kernel(const LatentAttn a, bool prepared, int splits, const ActOut out) {
     extern __shared__ __align__(16) float fs[];
-    const int D = a.rank + a.rot, W = a.rank;
-    float* q_s = fs;                          // [8][D]
-    float* o_s = q_s + kF32Heads * D;         // [8][rank]
-    float* p_s = o_s + kF32Heads * W;         // [8][32]
+    const int D = a.rank + a.rot, W = (a.rank + 3) / 4 * 4;
+    float* o_s = fs;                          // [8][W]
+    float* q_s = o_s + kF32Heads * W;         // [8][D]
+    float* p_s = q_s + kF32Heads * D;         // [8][32]
     float* m_s = p_s + kF32Heads * kF32Keys;
     float* l_s = m_s + kF32Heads;
     float* al_s = l_s + kF32Heads;
-    float* red = al_s + kF32Heads;            // 32
+    float* fac = al_s + kF32Heads;            // [8][kMaxSplits]
+    float* red = fac + kF32Heads * kMaxSplits;  // 32
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int H = a.heads, hd = a.dim + a.rot;
     const int head0 = blockIdx.y * kF32Heads, nh = min(kF32Heads, H - head0);
@@ -479,7 +542,7 @@ __global__ void __launch_bounds__(kF32Threads) latent_span_f32_kernel(const Late
             const int c = threadIdx.x + j * kF32Threads;
             if (c < a.rank) o_s[h * W + c] = acc[h][j];
         }
-    merge_spans<false>(a, m_s, l_s, o_s, W, nh, head0, r, split, splits, out);
+    merge_spans<false>(a, m_s, l_s, o_s, fac, W, nh, head0, r, split, splits, out);
 }
 
 template <typename... KArgs, typename... Args>
@@ -500,42 +563,42 @@ cudaError_t launch_cluster(void (*kernel)(KArgs...), dim3 grid, int threads, siz
 }
 int span_splits(const LatentAttn& a, int64_t groups) {
     int splits = 1;
-    while (splits < kMaxSplits && groups * splits * 2 <= a.sm_count && splits * 64 < a.kv.max_seq) splits *= 2;
+    while (splits < kMaxSplits && groups * splits * 2 <= a.sm_count && splits * kKeys < a.kv.max_seq) splits *= 2;
     return splits;
 }
 
-constexpr size_t kSpanSmem = 220 * 1024;
-template <int NT, int MT>
+constexpr size_t kSpanSmem = 224 * 1024;
+template <int HG>
 cudaError_t span_launch(const LatentAttn& a, bool prepared, const ActOut& out, unsigned int* err, cudaStream_t s, bool pdl) {
     static PerDeviceOnce once;
     cudaError_t e = once.run([] {
-        cudaError_t x = cudaFuncSetAttribute(latent_span_mma_kernel<NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSpanSmem);
-        return x != cudaSuccess ? x : cudaFuncSetAttribute(latent_span_mma_kernel<NT, MT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaError_t x = cudaFuncSetAttribute(latent_span_tc_kernel<HG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSpanSmem);
+        return x != cudaSuccess ? x : cudaFuncSetAttribute(latent_span_tc_kernel<HG>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     });
     if (e != cudaSuccess) return e;
-    const int chunks = (dense_kpad(a.rank) + dense_kpad(a.rot)) / 64, hg = (a.heads + 16 * MT - 1) / (16 * MT);
-    const size_t stage = (size_t)chunks * kKeys * 128, fixed = SpanCfg<MT>::fixed(chunks), outs = (size_t)16 * MT * 8 * kSpanWarps * NT * sizeof(float);
-    // six blocks in flight where two CTAs then share an SM, else as many as fit; the ring must also take the outputs
-    int stages = 6;
-    if (stages * stage + fixed > 110 * 1024) stages = (int)((kSpanSmem - fixed) / stage) < 6 ? (int)((kSpanSmem - fixed) / stage) : 6;
-    while (stages * stage < outs) ++stages;
-    if (stages < 2 || stages > 8 || stages * stage + fixed > kSpanSmem) return cudaErrorInvalidConfiguration;
+    const int cols = a.kv.cols(), hg = (a.heads + HG - 1) / HG;
+    const size_t stage = (size_t)cols * kKeys * 2, fixed = SpanCfg<HG>::fixed(cols), outs = (size_t)HG * ((a.rank + 127) / 128 * 128) * sizeof(float);
+    // (the values are read in whole tiles of 128 latent columns: up to 2 KB behind a stage, which is shared memory in use)
+    int stages = (int)((kSpanSmem - fixed) / stage);
+    stages = stages > kMaxStages ? kMaxStages : stages;
+    if (stages < 1 || stages * stage < outs) return cudaErrorInvalidConfiguration;
     const int64_t rows = (int64_t)a.batch * a.q_rows;
     const int splits = span_splits(a, rows * hg);
-    return launch_cluster(latent_span_mma_kernel<NT, MT>, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, stages * stage + fixed, s, pdl,
-                          a, prepared, splits, stages, (int)SpanCfg<MT>::part(chunks), err, out);
-}
-template <int NT>
-cudaError_t span_launch_m(const LatentAttn& a, bool prepared, const ActOut& out, unsigned int* err, cudaStream_t s, bool pdl) {
-    // 32 heads share the cache rows once that leaves no SM idle
-    const bool wide = a.heads > 16 && (int64_t)a.batch * a.q_rows * ((a.heads + 31) / 32) * 4 >= a.sm_count;
-    return wide ? span_launch<NT, 2>(a, prepared, out, err, s, pdl) : span_launch<NT, 1>(a, prepared, out, err, s, pdl);
+    return launch_cluster(latent_span_tc_kernel<HG>, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, stages * stage + fixed, s, pdl,
+                          a, prepared, splits, stages, err, out);
 }
 
 }  // namespace
 
 int latent_max_rank() { return kMaxRank; }
 int latent_max_rot() { return kMaxRot; }
+
+cudaError_t launch_latent_tiles(const LatentView& v, int b0, int nb, int64_t n, uint8_t* tiles, int64_t m_pad, cudaStream_t s) {
+    if (v.f32) return cudaErrorInvalidValue;
+    const int64_t total = (n + 7) / 8 * dense_kpad(v.rank);
+    latent_tiles_kernel<<<dim3((unsigned)((total + 255) / 256 < 592 ? (total + 255) / 256 : 592), (unsigned)nb), 256, 0, s>>>(v, b0, n, tiles, m_pad);
+    return cudaGetLastError();
+}
 
 cudaError_t launch_latent_prep(const LatentAttn& a, cudaStream_t s) {
     latent_prep_kernel<<<(unsigned)(a.batch * a.q_rows), 256, 0, s>>>(a);
@@ -554,16 +617,18 @@ cudaError_t launch_latent_span(const LatentAttn& a, bool prepared, const ActOut&
         const int hg = (a.heads + kF32Heads - 1) / kF32Heads;
         const int64_t rows = (int64_t)a.batch * a.q_rows;
         const int splits = span_splits(a, rows * hg);
-        const size_t smem = ((size_t)kF32Heads * (2 * a.rank + a.rot) + kF32Heads * kF32Keys + 3 * kF32Heads + 32) * sizeof(float);
+        const size_t smem = ((size_t)kF32Heads * (2 * a.rank + 3 + a.rot) + kF32Heads * kF32Keys + (3 + kMaxSplits) * kF32Heads + 32) * sizeof(float);
         return launch_cluster(latent_span_f32_kernel, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kF32Threads, smem, s, pdl, a, prepared, splits, out);
     }
     int dev = 0;
     cudaError_t e = cudaGetDevice(&dev);
     if (e != cudaSuccess) return e;
     unsigned int* err = device_error_word(dev);
-    if (a.rank <= 128) return span_launch_m<1>(a, prepared, out, err, s, pdl);
-    if (a.rank <= 256) return span_launch_m<2>(a, prepared, out, err, s, pdl);
-    return span_launch_m<4>(a, prepared, out, err, s, pdl);
+    // 32 heads share the cache rows once that leaves no SM idle
+    const int cols = a.kv.cols();
+    const bool wide = a.heads > 16 && (int64_t)a.batch * a.q_rows * ((a.heads + 31) / 32) * 4 >= a.sm_count &&
+                      (size_t)cols * kKeys * 2 + SpanCfg<32>::fixed(cols) <= kSpanSmem;
+    return wide ? span_launch<32>(a, prepared, out, err, s, pdl) : span_launch<16>(a, prepared, out, err, s, pdl);
 }
 
 }  // namespace bt

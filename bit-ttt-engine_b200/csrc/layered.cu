@@ -625,16 +625,20 @@ struct RowPass {
             // keys and values of every position so far, a group of sequences at a time
             a.q_buf = reinterpret_cast<__nv_bfloat16*>(r.q);
             if (parts & PART_CORE) BT_CUDA_TRY(launch_latent_prep(a, s));
-            const int64_t rows = ((int64_t)past + n + 63) / 64 * 64, seq = rows * l.expand.n;
+            const int64_t rows = ((int64_t)past + n + 63) / 64 * 64, tile_rows = dense_mpad(past + n), tile_bytes = tile_rows * l.expand.k_pad * 2;
+            const int64_t seq = rows * l.expand.n;
             const int group = (int)std::max<int64_t>(1, std::min<int64_t>(batch, (int64_t)kExpandElems / seq));
-            bt_status st = expand_room(L, (size_t)(group * seq));
+            bt_status st = expand_room(L, (size_t)(group * (seq + tile_bytes / 2)));
+            uint8_t* tiles = reinterpret_cast<uint8_t*>(L->kv16 + group * seq);  // the latents as the product reads them
             if (st != BT_OK) return st;
             for (int b0 = 0; b0 < batch; b0 += group) {
                 const int nb = std::min(group, batch - b0);
                 DenseOut o;
-                o.out_rows16 = L->kv16; o.ld = l.expand.n; o.out_block = seq; o.shared_weights = true; o.blocks = nb; o.x_block = a.kv.seq_bytes(); o.m_pad = a.kv.seq_pad;
-                if (parts & PART_MID)
-                    BT_CUDA_TRY(launch_dense_tc(l.expand, reinterpret_cast<const uint8_t*>(a.kv.rows) + b0 * a.kv.seq_bytes(), past + n, o, nullptr, err, sm, s));
+                o.out_rows16 = L->kv16; o.ld = l.expand.n; o.out_block = seq; o.shared_weights = true; o.blocks = nb; o.x_block = tile_bytes; o.m_pad = tile_rows;
+                if (parts & PART_MID) {
+                    BT_CUDA_TRY(launch_latent_tiles(a.kv, b0, nb, past + n, tiles, tile_rows, s));
+                    BT_CUDA_TRY(launch_dense_tc(l.expand, tiles, past + n, o, nullptr, err, sm, s));
+                }
                 if (parts & PART_CORE) BT_CUDA_TRY(launch_latent_tile(a, L->kv16, rows, b0, nb, tiled(r.mt), s));
             }
             return BT_OK;

@@ -153,7 +153,7 @@ bt_status latent_rows(bt_kv_cache* c, int64_t b, int64_t t_len, float* rank_host
                     uint8_t* p = tmp.data() + (t * l.stride + (which ? l.rank : 0) + j) * 4;
                     if (store) memcpy(p, &hv, 4); else memcpy(&hv, p, 4);
                 } else {
-                    uint8_t* p = tmp.data() + dense_off(t, (which ? dense_kpad(l.rank) : 0) + j, l.seq_pad);
+                    uint8_t* p = tmp.data() + l.off(t, (which ? l.rot_col() : 0) + j);
                     __nv_bfloat16 q = __float2bfloat16_rn(hv);
                     if (store) memcpy(p, &q, 2);
                     else { memcpy(&q, p, 2); hv = __bfloat162float(q); }

@@ -161,107 +161,111 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
 // ---------------------------------------------------------------------------------------
 // many tokens, one after the other
 // ---------------------------------------------------------------------------------------
-// A CTA owns 16 value columns of one head, a warp 8: eight lanes share two columns, each with 4 NJ of their state elements in
-// registers (key channels 32 j + 4 lane .. + 3).  r, k, the decays and v of a tile of tokens arrive in shared memory by
-// asynchronous copies, one tile ahead; tokens go by eights, whose sums over the lanes are folded together.
-constexpr int kScanThreads = 64, kScanCols = 16;
+// A CTA owns 16 value columns of one head.  Two warps compute, 8 columns each: eight lanes share two columns, each with 4 NJ
+// of their state elements in registers as pairs (key channels 32 j + 4 lane .. + 3); tokens go by eights, whose sums over the
+// lanes are folded together.  Two more warps bring r, k, the decays and v of a tile of tokens into shared memory, two tiles
+// ahead, and make the current token's own weight, sum of r u k, one tile ahead.
+constexpr int kScanThreads = 128, kScanCols = 16, kScanBufs = 3;
 template <int NJ>
 struct ScanCfg {
     static constexpr int DP = 32 * NJ, TT = NJ <= 4 ? 16 : 8;
-    static constexpr int kTile = TT * (3 * DP + kScanCols);  // floats
-    static constexpr size_t kSmem = (size_t)(2 * kTile + TT) * sizeof(float);
+    static constexpr int kTile = TT * (3 * DP + kScanCols + 1);  // floats: r, k, w, v, bonus
+    static constexpr size_t kSmem = (size_t)kScanBufs * kTile * sizeof(float);
 };
+// two f32 values side by side
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+    f2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+    f2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f2 pair2(float x, float y) {
+    f2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+    return d;
+}
+__device__ __forceinline__ float2 split2(f2 a) {
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(a));
+    return d;
+}
 
 template <int NJ>
 __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a) {
     using Cfg = ScanCfg<NJ>;
-    constexpr int DP = Cfg::DP, TT = Cfg::TT;
-    extern __shared__ __align__(16) float sm[];  // two tiles of r, k, w [TT][DP] and v [TT][16]; bonus [TT]
-    float* bonus_s = sm + 2 * Cfg::kTile;
+    constexpr int DP = Cfg::DP, TT = Cfg::TT, Q = DP / 4;  // Q: 16-byte pieces per row
+    extern __shared__ __align__(16) float sm[];
     const int head = blockIdx.x, v0 = blockIdx.y * kScanCols, b = blockIdx.z;
     const int D = a.dim, HD = a.heads * D, vc = min(kScanCols, D - v0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int col = warp * 8 + (lane >> 3) * 2, kg = lane & 7;
-    const int p0 = a.pos[b];
-    float* state = a.s + ((int64_t)b * a.heads + head) * D * D + v0 + col;
-    float s[4 * NJ][2];
-#pragma unroll
-    for (int j = 0; j < NJ; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-#pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const int k = 32 * j + 4 * kg + e;
-                s[4 * j + e][c] = col + c < vc && k < D && p0 > 0 ? state[(int64_t)k * D + c] : 0.0f;
-            }
-    const float* rows = a.proj + (int64_t)b * a.q_rows * a.ld + head * D;
-    const float* wrows = a.w + (int64_t)b * a.q_rows * HD + head * D;
-    for (int i = threadIdx.x; i < 2 * Cfg::kTile; i += kScanThreads) sm[i] = 0.0f;  // columns beyond the head's stay zero
+    const int p0 = a.pos[b], tiles = (a.q_rows + TT - 1) / TT;
+    for (int i = threadIdx.x; i < kScanBufs * Cfg::kTile; i += kScanThreads) sm[i] = 0.0f;  // columns beyond the head's stay zero
     __syncthreads();
-    const bool vec = (D & 3) == 0 && (a.ld & 3) == 0;
-    auto fetch = [&](int i0, int buf) {  // tokens i0 .. of the tile
-        float* t = sm + buf * Cfg::kTile;
-        const int n = min(TT, a.q_rows - i0);
-        if (n <= 0) return;
-        if (vec) {
-            const int q = D >> 2;
-            for (int e = threadIdx.x; e < n * q; e += kScanThreads) {
-                const int i = e / q, c = (e - i * q) * 4;
-                const float* src = rows + (int64_t)(i0 + i) * a.ld + c;
-                const uint32_t dst = ptx::smem_u32(t + i * DP + c);
-                ptx::cp16(dst, src, true);
-                ptx::cp16(dst + TT * DP * 4, src + HD, true);
-                ptx::cp16(dst + 2 * TT * DP * 4, wrows + (int64_t)(i0 + i) * HD + c, true);
-            }
-            const int vq = vc >> 2;
-            for (int e = threadIdx.x; e < n * vq; e += kScanThreads) {
-                const int i = e / vq, c = (e - i * vq) * 4;
-                ptx::cp16(ptx::smem_u32(t + 3 * TT * DP + i * kScanCols + c), rows + (int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c, true);
-            }
-        } else {
-            for (int e = threadIdx.x; e < n * D; e += kScanThreads) {
-                const int i = e / D, c = e - i * D;
-                const float* src = rows + (int64_t)(i0 + i) * a.ld + c;
-                t[i * DP + c] = src[0];
-                t[TT * DP + i * DP + c] = src[HD];
-                t[2 * TT * DP + i * DP + c] = wrows[(int64_t)(i0 + i) * HD + c];
-            }
-            for (int e = threadIdx.x; e < n * vc; e += kScanThreads) {
-                const int i = e / vc, c = e - i * vc;
-                t[3 * TT * DP + i * kScanCols + c] = rows[(int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c];
-            }
-        }
-        for (int e = threadIdx.x; e < (TT - n) * DP; e += kScanThreads) {  // behind the last token: nothing is added, nothing decays
-            const int o = n * DP + e;
-            t[o] = 0.0f;
-            t[TT * DP + o] = 0.0f;
-            t[2 * TT * DP + o] = 1.0f;
-        }
-    };
     auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
-    fetch(0, 0);
-    commit();
-    float uu[(DP + 31) / 32];
+    if (warp >= 2) {
+        const int tid = threadIdx.x - 64;
+        const float* rows = a.proj + (int64_t)b * a.q_rows * a.ld + head * D;
+        const float* wrows = a.w + (int64_t)b * a.q_rows * HD + head * D;
+        const bool vec = (D & 3) == 0 && (a.ld & 3) == 0;
+        auto fetch = [&](int ti) {
+            if (ti >= tiles) return;
+            float* t = sm + (ti % kScanBufs) * Cfg::kTile;
+            const int i0 = ti * TT, n = min(TT, a.q_rows - i0);
+            if (vec) {
+#pragma unroll 4
+                for (int e = tid; e < TT * Q; e += 64) {
+                    const int i = e / Q, c = e % Q * 4;
+                    if (i < n && c < D) {
+                        const float* src = rows + (int64_t)(i0 + i) * a.ld + c;
+                        const uint32_t dst = ptx::smem_u32(t + i * DP + c);
+                        ptx::cp16(dst, src, true);
+                        ptx::cp16(dst + TT * DP * 4, src + HD, true);
+                        ptx::cp16(dst + 2 * TT * DP * 4, wrows + (int64_t)(i0 + i) * HD + c, true);
+                    }
+                }
+                if (tid < TT * (kScanCols / 4)) {
+                    const int i = tid / (kScanCols / 4), c = tid % (kScanCols / 4) * 4;
+                    if (i < n && c < vc) ptx::cp16(ptx::smem_u32(t + 3 * TT * DP + i * kScanCols + c), rows + (int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c, true);
+                }
+            } else {
+                for (int e = tid; e < n * DP; e += 64) {
+                    const int i = e / DP, c = e % DP;
+                    if (c >= D) continue;
+                    const float* src = rows + (int64_t)(i0 + i) * a.ld + c;
+                    t[i * DP + c] = src[0];
+                    t[TT * DP + i * DP + c] = src[HD];
+                    t[2 * TT * DP + i * DP + c] = wrows[(int64_t)(i0 + i) * HD + c];
+                }
+                for (int e = tid; e < n * kScanCols; e += 64) {
+                    const int i = e / kScanCols, c = e % kScanCols;
+                    if (c < vc) t[3 * TT * DP + i * kScanCols + c] = rows[(int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c];
+                }
+            }
+            for (int e = tid; e < (TT - n) * DP; e += 64) {  // behind the last token: nothing is added, nothing decays
+                const int o = n * DP + e;
+                t[o] = 0.0f;
+                t[TT * DP + o] = 0.0f;
+                t[2 * TT * DP + o] = 1.0f;
+            }
+        };
+        float uu[NJ];
 #pragma unroll
-    for (int j = 0; j < (DP + 31) / 32; ++j) uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f;
-    int buf = 0;
-    for (int i0 = 0; i0 < a.q_rows; i0 += TT, buf ^= 1) {
-        fetch(i0 + TT, buf ^ 1);
-        commit();
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();
-        const float* t = sm + buf * Cfg::kTile;
-        const float* rs = t;
-        const float* ks = t + TT * DP;
-        const float* ws = t + 2 * TT * DP;
-        const float* vs = t + 3 * TT * DP;
-        {   // the current token's own weight, sum of r u k
+        for (int j = 0; j < NJ; ++j) uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f;
+        auto bonus = [&](int ti) {  // each of the two warps half of the tile's tokens
+            if (ti >= tiles) return;
+            float* t = sm + (ti % kScanBufs) * Cfg::kTile;
+            const int first = (warp - 2) * (TT / 2);
             float x[TT / 2];
 #pragma unroll
             for (int i = 0; i < TT / 2; ++i) {
                 x[i] = 0.0f;
 #pragma unroll
-                for (int j = 0; j < DP / 32; ++j) x[i] = fmaf(rs[(warp * (TT / 2) + i) * DP + j * 32 + lane] * uu[j], ks[(warp * (TT / 2) + i) * DP + j * 32 + lane], x[i]);
+                for (int j = 0; j < NJ; ++j) x[i] = fmaf(t[(first + i) * DP + j * 32 + lane] * uu[j], t[TT * DP + (first + i) * DP + j * 32 + lane], x[i]);
             }
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1)
@@ -269,32 +273,93 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
                 for (int i = 0; i < TT / 2; ++i) x[i] += __shfl_xor_sync(0xffffffffu, x[i], o);
             if (lane == 0)
 #pragma unroll
-                for (int i = 0; i < TT / 2; ++i) bonus_s[warp * (TT / 2) + i] = x[i];
-        }
+                for (int i = 0; i < TT / 2; ++i) t[TT * (3 * DP + kScanCols) + first + i] = x[i];
+        };
+        auto landed = [&] {  // the copies of both warps, all but the last tile asked for
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+            asm volatile("bar.sync 1, 64;" ::: "memory");
+        };
+        fetch(0);
+        commit();
+        fetch(1);
+        commit();
+        landed();
+        bonus(0);
         __syncthreads();
+        for (int ti = 0; ti < tiles; ++ti) {
+            fetch(ti + 2);
+            commit();
+            landed();
+            bonus(ti + 1);
+            __syncthreads();
+        }
+        if (blockIdx.x == 0 && blockIdx.y == 0) {  // the token shift's state
+            const int64_t last = (int64_t)b * a.q_rows + a.q_rows - 1;
+            float* keep = a.shift + (int64_t)((p0 + a.q_rows - 1) & 1) * a.shift_slot + (int64_t)b * a.width;
+            for (int c = tid; c < a.width; c += 64) keep[c] = a.hn[last * a.width + c];
+        }
+        return;
+    }
+    const int col = warp * 8 + (lane >> 3) * 2, kg = lane & 7;
+    float* state = a.s + ((int64_t)b * a.heads + head) * D * D + v0 + col;
+    f2 s[2 * NJ][2];  // pairs of key channels x two columns
+#pragma unroll
+    for (int j = 0; j < 2 * NJ; ++j)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+            float x[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int k = 32 * (j >> 1) + 4 * kg + 2 * (j & 1) + e;
+                x[e] = col + c < vc && k < D && p0 > 0 ? state[(int64_t)k * D + c] : 0.0f;
+            }
+            s[j][c] = pair2(x[0], x[1]);
+        }
+    __syncthreads();
+    for (int ti = 0; ti < tiles; ++ti) {
+        const float* rs = sm + (ti % kScanBufs) * Cfg::kTile;
+        const float* ks = rs + TT * DP;
+        const float* ws = ks + TT * DP;
+        const float* vs = ws + TT * DP;
+        const float* bonus_s = vs + TT * kScanCols;
+        const int i0 = ti * TT;
 #pragma unroll 1
         for (int g = 0; g < TT && i0 + g < a.q_rows; g += 8) {
             float o[8][2];
-#pragma unroll
-            for (int q = 0; q < 8; ++q) {
-                const int tk = g + q;
-                const float2 v = *reinterpret_cast<const float2*>(vs + tk * kScanCols + col);
-                float o0 = 0.0f, o1 = 0.0f;
+            // a token's values are loaded while the one before it is worked on
+            ulonglong2 r4[2][NJ], k4[2][NJ], w4[2][NJ];
+            float2 v2[2];
+            auto take = [&](int which, int tk) {
+                v2[which] = *reinterpret_cast<const float2*>(vs + tk * kScanCols + col);
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
                     const int at = tk * DP + 32 * j + 4 * kg;
-                    const float4 r4 = *reinterpret_cast<const float4*>(rs + at), k4 = *reinterpret_cast<const float4*>(ks + at), w4 = *reinterpret_cast<const float4*>(ws + at);
-                    const float r[4] = {r4.x, r4.y, r4.z, r4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, w[4] = {w4.x, w4.y, w4.z, w4.w};
+                    r4[which][j] = *reinterpret_cast<const ulonglong2*>(rs + at);
+                    k4[which][j] = *reinterpret_cast<const ulonglong2*>(ks + at);
+                    w4[which][j] = *reinterpret_cast<const ulonglong2*>(ws + at);
+                }
+            };
+            take(0, g);
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        o0 = fmaf(r[e], s[4 * j + e][0], o0);
-                        o1 = fmaf(r[e], s[4 * j + e][1], o1);
-                        s[4 * j + e][0] = fmaf(w[e], s[4 * j + e][0], k[e] * v.x);
-                        s[4 * j + e][1] = fmaf(w[e], s[4 * j + e][1], k[e] * v.y);
+            for (int q = 0; q < 8; ++q) {
+                if (q < 7) take((q + 1) & 1, g + q + 1);
+                const f2 vv[2] = {pair2(v2[q & 1].x, v2[q & 1].x), pair2(v2[q & 1].y, v2[q & 1].y)};
+                f2 sum[2][2];
+#pragma unroll
+                for (int j = 0; j < 2 * NJ; ++j) {
+                    const ulonglong2 x = r4[q & 1][j >> 1], y = k4[q & 1][j >> 1], z = w4[q & 1][j >> 1];
+                    const f2 r = j & 1 ? x.y : x.x, k = j & 1 ? y.y : y.x, w = j & 1 ? z.y : z.x;
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        sum[j & 1][c] = j < 2 ? mul2(r, s[j][c]) : fma2(r, s[j][c], sum[j & 1][c]);
+                        s[j][c] = fma2(w, s[j][c], mul2(k, vv[c]));
                     }
                 }
-                o[q][0] = o0;
-                o[q][1] = o1;
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    const float2 x = split2(sum[0][c]), y = split2(sum[1][c]);
+                    o[q][c] = (x.x + y.x) + (x.y + y.y);
+                }
             }
             // fold over the eight lanes of a column pair: lane kg ends with token g + kg
 #pragma unroll
@@ -317,22 +382,19 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
                     if (col + c < vc) y[c] = fmaf(bonus, vs[tk * kScanCols + col + c], o[0][c]);
             }
         }
-        __syncthreads();  // before the tile is refilled
+        __syncthreads();  // the tile may be refilled, the next one is there
     }
 #pragma unroll
-    for (int j = 0; j < NJ; ++j)
+    for (int j = 0; j < 2 * NJ; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-#pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const int k = 32 * j + 4 * kg + e;
-                if (col + c < vc && k < D) state[(int64_t)k * D + c] = s[4 * j + e][c];
+        for (int c = 0; c < 2; ++c) {
+            const float2 x = split2(s[j][c]);
+            const int k = 32 * (j >> 1) + 4 * kg + 2 * (j & 1);
+            if (col + c < vc) {
+                if (k < D) state[(int64_t)k * D + c] = x.x;
+                if (k + 1 < D) state[(int64_t)(k + 1) * D + c] = x.y;
             }
-    if (blockIdx.x == 0 && blockIdx.y == 0) {  // the token shift's state
-        const int64_t last = (int64_t)b * a.q_rows + a.q_rows - 1;
-        float* keep = a.shift + (int64_t)((p0 + a.q_rows - 1) & 1) * a.shift_slot + (int64_t)b * a.width;
-        for (int c = threadIdx.x; c < a.width; c += kScanThreads) keep[c] = a.hn[last * a.width + c];
-    }
+        }
 }
 
 template <int NJ>
