@@ -333,7 +333,12 @@ struct WkvArgs {
     int64_t shift_slot = 0;
     int width = 0;
     int sm_count = 0;
+    // prefill in segments of the tokens, side by side (null: one after the other)
+    float* seg_s = nullptr;        // wkv_segment_floats per sequence: states and decays of the segments
+    float* seg_w = nullptr;        // wkv_prefix_floats: decays up to each block of 64 tokens
 };
+int64_t wkv_segment_floats(int heads, int dim);  // 0: the head size has no such form
+int64_t wkv_prefix_floats(int heads, int dim, int64_t rows, int batch);
 int wkv_max_dim();
 cudaError_t launch_wkv_step(const WkvArgs& a, cudaStream_t s, bool pdl);
 cudaError_t launch_wkv_prefill(const WkvArgs& a, cudaStream_t s);

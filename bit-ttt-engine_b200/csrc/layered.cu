@@ -45,6 +45,7 @@ struct RowBuffers {
     float* a = nullptr;        // latent: absorbed queries; rglru: convolution outputs; wkv: low-rank decay inputs
     float* b = nullptr;        // latent: weighted latents; rglru: gates; wkv: decays
     float* c = nullptr;        // latent: rotated queries; wkv: mixed inputs, finished rows
+    float* wkv_pre = nullptr;  // wkv: decays up to each block of tokens
     void* q = nullptr;         // prepared queries
     uint8_t* xt = nullptr;     // bf16 models: tiled activations (sublayer input, mixer output, feed-forward, inside a mixer)
     uint8_t* mt = nullptr;
@@ -61,7 +62,7 @@ struct RowBuffers {
     float* ye = nullptr;
     int64_t grouped = 0;
     void release() {
-        for (void* p : {(void*)proj, (void*)mix, (void*)y, (void*)ff, (void*)conv, (void*)v_first, (void*)hn, (void*)cat, (void*)a, (void*)b, (void*)c, q,
+        for (void* p : {(void*)proj, (void*)mix, (void*)y, (void*)ff, (void*)conv, (void*)v_first, (void*)hn, (void*)cat, (void*)a, (void*)b, (void*)c, (void*)wkv_pre, q,
                         (void*)xt, (void*)mt, (void*)ft, (void*)t1, (void*)t2, (void*)scratch, (void*)logits, (void*)choice, (void*)wt, (void*)xe, (void*)fe, (void*)ye})
             cudaFree(p);
         *this = RowBuffers();
@@ -144,6 +145,7 @@ struct Layered {
     int fused_rows = 0;
     __nv_bfloat16* kv16 = nullptr;  // prefill: keys and values expanded from latents
     size_t kv16_elems = 0;
+    float* wkv_seg = nullptr;       // prefill: states of the segments of a wkv recurrence
     bool loops() const { return c.loop_times > 0; }
 };
 
@@ -248,6 +250,10 @@ bt_status alloc_rows(const bt_model* m, RowBuffers& r, int rows, bool wide) {
         BT_CUDA_TRY(dev_alloc(&r.c, n * q.c));
         BT_CUDA_TRY(cudaMalloc(&r.q, std::max<size_t>(16, n * q.q * sizeof(float))));
         if (!L->f32) {
+            int64_t pre = 0;
+            for (const LayLayer& l : L->layers)
+                if (l.c.mixer == BT_MIX_WKV) pre = std::max(pre, wkv_prefix_floats(l.c.heads, l.c.dim, rows, L->c.max_batch));
+            BT_CUDA_TRY(dev_alloc(&r.wkv_pre, (size_t)pre));
             size_t scratch = 0;
             for (const LayLayer& l : L->layers) {
                 size_t count;
@@ -351,6 +357,8 @@ WkvArgs wkv_args(const bt_model* m, const LayLayer& l, const LayRun& run, const 
     a.low = r.a; a.rank = c.decay_rank;
     a.w = r.b; a.hn = r.hn; a.shift = run.ring; a.shift_slot = (int64_t)m->cfg.max_batch * m->lay->c.width; a.width = m->lay->c.width;
     a.sm_count = m->sm_count;
+    a.seg_s = m->lay->f32 ? nullptr : m->lay->wkv_seg;
+    a.seg_w = r.wkv_pre;
     return a;
 }
 RgluArgs rglru_args(const bt_model* m, const LayLayer& l, const LayRun& run, const RowBuffers& r, int batch, int n) {
@@ -981,6 +989,12 @@ bt_status layered_finalize(bt_model* m) {
             BT_CUDA_TRY(dev_alloc(&run.ring, (size_t)(B * l.ring_floats(W))));
         }
     }
+    if (!L->f32) {
+        int64_t most = 0;
+        for (const LayLayer& l : L->layers)
+            if (l.c.mixer == BT_MIX_WKV) most = std::max(most, wkv_segment_floats(l.c.heads, l.c.dim));
+        if (most) BT_CUDA_TRY(dev_alloc(&L->wkv_seg, (size_t)(most * B)));
+    }
     m->rms_eps = L->c.norm_eps;
     m->logit_cap = L->c.logit_softcap;
     m->head_rows = std::max(B, 64);
@@ -1024,7 +1038,7 @@ void layered_destroy(bt_model* m) {
     for (RotTable& t : L->tables) { cudaFree(t.cos_t); cudaFree(t.sin_t); }
     L->dec.release();
     L->pf.release();
-    cudaFree(L->pos_table); cudaFree(L->h2); cudaFree(L->loop_in.tiles); cudaFree(L->loop_step); cudaFree(L->kv16);
+    cudaFree(L->pos_table); cudaFree(L->h2); cudaFree(L->loop_in.tiles); cudaFree(L->loop_step); cudaFree(L->kv16); cudaFree(L->wkv_seg);
     delete L;
     m->lay = nullptr;
 }

@@ -20,33 +20,48 @@ __device__ __forceinline__ float warp_sum(float v) {
 // ---------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) wkv_mix_kernel(const WkvMix a) {
     const int64_t r = blockIdx.x;
+    const int b = (int)(r / a.q_rows), i = (int)(r % a.q_rows), W = a.width;
+    const int p0 = a.pos[b];
+    const float* h = a.hn + r * W;
+    const float* before = i > 0 ? h - W : (p0 > 0 ? a.shift + (int64_t)((p0 + 1) & 1) * a.shift_slot + (int64_t)b * W : nullptr);
+    for (int c = threadIdx.x; c < W; c += 256) {
+        const float v = h[c], d = (before ? before[c] : 0.0f) - v;
+#pragma unroll
+        for (int s = 0; s < 5; ++s) a.rows5[(r * 5 + s) * W + c] = fmaf(d, a.mu[s][c], v);
+    }
+}
+// the same into tiles: a CTA per 8 rows, eight lanes per piece of 8 columns, so that a piece of the rows is one run of 128 bytes
+__global__ void __launch_bounds__(256) wkv_mix_tiles_kernel(const WkvMix a) {
+    const int64_t r = (int64_t)blockIdx.x * 8 + (threadIdx.x & 7);
+    if (r >= (int64_t)a.batch * a.q_rows) return;
     const int b = (int)(r / a.q_rows), i = (int)(r % a.q_rows), W = a.width, kp = dense_kpad(W);
     const int p0 = a.pos[b];
     const float* h = a.hn + r * W;
     const float* before = i > 0 ? h - W : (p0 > 0 ? a.shift + (int64_t)((p0 + 1) & 1) * a.shift_slot + (int64_t)b * W : nullptr);
-    if (a.rows5) {
-        for (int c = threadIdx.x; c < W; c += 256) {
-            const float v = h[c], d = (before ? before[c] : 0.0f) - v;
+    const bool vec = (W & 3) == 0;
+    auto get = [&](const float* p, int c0, float (&v)[8]) {
+        if (p && vec && c0 + 8 <= W) {
+            const float4 x = *reinterpret_cast<const float4*>(p + c0), y = *reinterpret_cast<const float4*>(p + c0 + 4);
+            v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+        } else {
 #pragma unroll
-            for (int s = 0; s < 5; ++s) a.rows5[(r * 5 + s) * W + c] = fmaf(d, a.mu[s][c], v);
+            for (int j = 0; j < 8; ++j) v[j] = p && c0 + j < W ? p[c0 + j] : 0.0f;
         }
-        return;
-    }
-    for (int c0 = threadIdx.x * 8; c0 < kp; c0 += 256 * 8) {
+    };
+    for (int c0 = (threadIdx.x >> 3) * 8; c0 < kp; c0 += 32 * 8) {
         float v[8], d[8];
+        get(h, c0, v);
+        get(before, c0, d);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const bool live = c0 + j < W;
-            v[j] = live ? h[c0 + j] : 0.0f;
-            d[j] = (live && before ? before[c0 + j] : 0.0f) - v[j];
-        }
+        for (int j = 0; j < 8; ++j) d[j] -= v[j];
 #pragma unroll
         for (int s = 0; s < 5; ++s) {
+            float m[8];
+            get(a.mu[s], c0, m);
             uint32_t hi[4], lo[4];
 #pragma unroll
             for (int j = 0; j < 8; j += 2) {
-                const float x = c0 + j < W ? fmaf(d[j], a.mu[s][c0 + j], v[j]) : 0.0f;
-                const float y = c0 + j + 1 < W ? fmaf(d[j + 1], a.mu[s][c0 + j + 1], v[j + 1]) : 0.0f;
+                const float x = fmaf(d[j], m[j], v[j]), y = fmaf(d[j + 1], m[j + 1], v[j + 1]);
                 hi[j / 2] = ptx::pack2(x, y);
                 lo[j / 2] = ptx::pack2(x - __uint_as_float(hi[j / 2] << 16), y - __uint_as_float(hi[j / 2] & 0xffff0000u));
             }
@@ -159,63 +174,47 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
 }
 
 // ---------------------------------------------------------------------------------------
-// many tokens, one after the other
+// many tokens
 // ---------------------------------------------------------------------------------------
-// A CTA owns 16 value columns of one head.  Two warps compute, 8 columns each: eight lanes share two columns, each with 4 NJ
-// of their state elements in registers as pairs (key channels 32 j + 4 lane .. + 3); tokens go by eights, whose sums over the
-// lanes are folded together.  Two more warps bring r, k, the decays and v of a tile of tokens into shared memory, two tiles
-// ahead, and make the current token's own weight, sum of r u k, one tile ahead.
-constexpr int kScanThreads = 128, kScanCols = 16, kScanBufs = 3;
+// A CTA owns 64 value columns of one head and a segment of the tokens.  Four warps compute, 16 columns each: eight lanes share
+// four columns, each with 4 NJ of their state elements in registers (key channels 32 j + 4 lane .. + 3); tokens go by
+// fours, whose sums over the lanes are folded together.  Two more warps bring r, k, the decays and v of a tile of tokens into
+// shared memory, two tiles ahead, and make the current token's own weight, sum of r u k, one tile ahead.
+// Several segments: each but the first starts from zero; wkv_join_kernel carries the states over the segments, wkv_carry_kernel
+// adds what a segment's incoming state means for its tokens.
+constexpr int kScanCompute = 4, kScanThreads = 32 * kScanCompute + 64, kScanCols = 64, kScanBufs = 3, kSegments = 16, kBlock = 64;
 template <int NJ>
 struct ScanCfg {
     static constexpr int DP = 32 * NJ, TT = NJ <= 4 ? 16 : 8;
     static constexpr int kTile = TT * (3 * DP + kScanCols + 1);  // floats: r, k, w, v, bonus
     static constexpr size_t kSmem = (size_t)kScanBufs * kTile * sizeof(float);
 };
-// two f32 values side by side
-typedef unsigned long long f2;
-__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
-    f2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
-    f2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-__device__ __forceinline__ f2 pair2(float x, float y) {
-    f2 d;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
-    return d;
-}
-__device__ __forceinline__ float2 split2(f2 a) {
-    float2 d;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(a));
-    return d;
-}
-
 template <int NJ>
-__global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a) {
+__global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel(const WkvArgs a, int segs, int seg_tokens) {
     using Cfg = ScanCfg<NJ>;
     constexpr int DP = Cfg::DP, TT = Cfg::TT, Q = DP / 4;  // Q: 16-byte pieces per row
     extern __shared__ __align__(16) float sm[];
-    const int head = blockIdx.x, v0 = blockIdx.y * kScanCols, b = blockIdx.z;
+    const int head = blockIdx.x, v0 = blockIdx.y * kScanCols, b = blockIdx.z / segs, seg = blockIdx.z - b * segs;
     const int D = a.dim, HD = a.heads * D, vc = min(kScanCols, D - v0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int p0 = a.pos[b], tiles = (a.q_rows + TT - 1) / TT;
+    const int first = seg * seg_tokens, count = min(seg_tokens, a.q_rows - first);  // this segment's tokens
+    const int p0 = a.pos[b], tiles = (count + TT - 1) / TT;
+    const int64_t row0 = (int64_t)b * a.q_rows + first;
+    // where the segment's last state goes: the sequence's state, or its place among the segments
+    float* state = a.s + ((int64_t)b * a.heads + head) * D * D;
+    float* result = segs > 1 ? a.seg_s + (((int64_t)b * a.heads + head) * kSegments + seg) * (D * D + D) : state;
     for (int i = threadIdx.x; i < kScanBufs * Cfg::kTile; i += kScanThreads) sm[i] = 0.0f;  // columns beyond the head's stay zero
     __syncthreads();
     auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
-    if (warp >= 2) {
-        const int tid = threadIdx.x - 64;
-        const float* rows = a.proj + (int64_t)b * a.q_rows * a.ld + head * D;
-        const float* wrows = a.w + (int64_t)b * a.q_rows * HD + head * D;
+    if (warp >= kScanCompute) {
+        const int tid = threadIdx.x - 32 * kScanCompute;
+        const float* rows = a.proj + row0 * a.ld + head * D;
+        const float* wrows = a.w + row0 * HD + head * D;
         const bool vec = (D & 3) == 0 && (a.ld & 3) == 0;
         auto fetch = [&](int ti) {
             if (ti >= tiles) return;
             float* t = sm + (ti % kScanBufs) * Cfg::kTile;
-            const int i0 = ti * TT, n = min(TT, a.q_rows - i0);
+            const int i0 = ti * TT, n = min(TT, count - i0);
             if (vec) {
 #pragma unroll 4
                 for (int e = tid; e < TT * Q; e += 64) {
@@ -228,8 +227,8 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
                         ptx::cp16(dst + 2 * TT * DP * 4, wrows + (int64_t)(i0 + i) * HD + c, true);
                     }
                 }
-                if (tid < TT * (kScanCols / 4)) {
-                    const int i = tid / (kScanCols / 4), c = tid % (kScanCols / 4) * 4;
+                for (int e = tid; e < TT * (kScanCols / 4); e += 64) {
+                    const int i = e / (kScanCols / 4), c = e % (kScanCols / 4) * 4;
                     if (i < n && c < vc) ptx::cp16(ptx::smem_u32(t + 3 * TT * DP + i * kScanCols + c), rows + (int64_t)(i0 + i) * a.ld + 2 * HD + v0 + c, true);
                 }
             } else {
@@ -253,19 +252,28 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
                 t[2 * TT * DP + o] = 1.0f;
             }
         };
-        float uu[NJ];
+        float uu[NJ], whole[NJ];  // the bonus; half of the tokens' decays multiplied up
 #pragma unroll
-        for (int j = 0; j < NJ; ++j) uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f;
+        for (int j = 0; j < NJ; ++j) { uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f; whole[j] = 1.0f; }
         auto bonus = [&](int ti) {  // each of the two warps half of the tile's tokens
             if (ti >= tiles) return;
             float* t = sm + (ti % kScanBufs) * Cfg::kTile;
-            const int first = (warp - 2) * (TT / 2);
+            if (segs > 1 && seg > 0 && blockIdx.y == 0 && ti * TT % kBlock == 0)  // the decays up to this block of tokens, this warp's share
+#pragma unroll
+                for (int j = 0; j < NJ; ++j)
+                    if (j * 32 + lane < D)
+                        a.seg_w[((((int64_t)b * ((a.q_rows + kBlock - 1) / kBlock) + (first + ti * TT) / kBlock) * 2 + warp - kScanCompute) * a.heads + head) * D + j * 32 + lane] = whole[j];
+            const int from = (warp - kScanCompute) * (TT / 2);
             float x[TT / 2];
 #pragma unroll
             for (int i = 0; i < TT / 2; ++i) {
                 x[i] = 0.0f;
 #pragma unroll
-                for (int j = 0; j < NJ; ++j) x[i] = fmaf(t[(first + i) * DP + j * 32 + lane] * uu[j], t[TT * DP + (first + i) * DP + j * 32 + lane], x[i]);
+                for (int j = 0; j < NJ; ++j) {
+                    const int at = (from + i) * DP + j * 32 + lane;
+                    x[i] = fmaf(t[at] * uu[j], t[TT * DP + at], x[i]);
+                    if (segs > 1) whole[j] *= t[2 * TT * DP + at];
+                }
             }
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1)
@@ -273,7 +281,7 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
                 for (int i = 0; i < TT / 2; ++i) x[i] += __shfl_xor_sync(0xffffffffu, x[i], o);
             if (lane == 0)
 #pragma unroll
-                for (int i = 0; i < TT / 2; ++i) t[TT * (3 * DP + kScanCols) + first + i] = x[i];
+                for (int i = 0; i < TT / 2; ++i) t[TT * (3 * DP + kScanCols) + from + i] = x[i];
         };
         auto landed = [&] {  // the copies of both warps, all but the last tile asked for
             asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -293,27 +301,30 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
             bonus(ti + 1);
             __syncthreads();
         }
-        if (blockIdx.x == 0 && blockIdx.y == 0) {  // the token shift's state
-            const int64_t last = (int64_t)b * a.q_rows + a.q_rows - 1;
+        if (segs > 1 && blockIdx.y == 0) {  // the segment's whole decay per channel
+            if (warp == kScanCompute)
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) sm[j * 32 + lane] = whole[j];
+            asm volatile("bar.sync 1, 64;" ::: "memory");
+            if (warp != kScanCompute)
+#pragma unroll
+                for (int j = 0; j < NJ; ++j)
+                    if (j * 32 + lane < D) result[D * D + j * 32 + lane] = sm[j * 32 + lane] * whole[j];
+        }
+        if (blockIdx.x == 0 && blockIdx.y == 0 && seg == segs - 1) {  // the token shift's state
             float* keep = a.shift + (int64_t)((p0 + a.q_rows - 1) & 1) * a.shift_slot + (int64_t)b * a.width;
-            for (int c = tid; c < a.width; c += 64) keep[c] = a.hn[last * a.width + c];
+            for (int c = tid; c < a.width; c += 64) keep[c] = a.hn[(row0 + count - 1) * a.width + c];
         }
         return;
     }
-    const int col = warp * 8 + (lane >> 3) * 2, kg = lane & 7;
-    float* state = a.s + ((int64_t)b * a.heads + head) * D * D + v0 + col;
-    f2 s[2 * NJ][2];  // pairs of key channels x two columns
+    const int col = warp * 16 + (lane >> 3) * 4, kg = lane & 7;
+    float s[4 * NJ][4];  // key channels x columns
 #pragma unroll
-    for (int j = 0; j < 2 * NJ; ++j)
+    for (int j = 0; j < 4 * NJ; ++j)
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-            float x[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int k = 32 * (j >> 1) + 4 * kg + 2 * (j & 1) + e;
-                x[e] = col + c < vc && k < D && p0 > 0 ? state[(int64_t)k * D + c] : 0.0f;
-            }
-            s[j][c] = pair2(x[0], x[1]);
+        for (int c = 0; c < 4; ++c) {
+            const int k = 32 * (j >> 2) + 4 * kg + (j & 3);
+            s[j][c] = col + c < vc && k < D && p0 > 0 && seg == 0 ? state[(int64_t)k * D + v0 + col + c] : 0.0f;
         }
     __syncthreads();
     for (int ti = 0; ti < tiles; ++ti) {
@@ -324,85 +335,206 @@ __global__ void __launch_bounds__(kScanThreads) wkv_scan_kernel(const WkvArgs a)
         const float* bonus_s = vs + TT * kScanCols;
         const int i0 = ti * TT;
 #pragma unroll 1
-        for (int g = 0; g < TT && i0 + g < a.q_rows; g += 8) {
-            float o[8][2];
-            // a token's values are loaded while the one before it is worked on
-            ulonglong2 r4[2][NJ], k4[2][NJ], w4[2][NJ];
-            float2 v2[2];
-            auto take = [&](int which, int tk) {
-                v2[which] = *reinterpret_cast<const float2*>(vs + tk * kScanCols + col);
+        for (int g = 0; g < TT && i0 + g < count; g += 4) {
+            float o[4][4];
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                const float4 v = *reinterpret_cast<const float4*>(vs + (g + q) * kScanCols + col);
+                const float vv[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int c = 0; c < 4; ++c) o[q][c] = 0.0f;
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
-                    const int at = tk * DP + 32 * j + 4 * kg;
-                    r4[which][j] = *reinterpret_cast<const ulonglong2*>(rs + at);
-                    k4[which][j] = *reinterpret_cast<const ulonglong2*>(ks + at);
-                    w4[which][j] = *reinterpret_cast<const ulonglong2*>(ws + at);
-                }
-            };
-            take(0, g);
+                    const int at = (g + q) * DP + 32 * j + 4 * kg;
+                    const float4 x = *reinterpret_cast<const float4*>(rs + at), y = *reinterpret_cast<const float4*>(ks + at), z = *reinterpret_cast<const float4*>(ws + at);
+                    const float r[4] = {x.x, x.y, x.z, x.w}, k[4] = {y.x, y.y, y.z, y.w}, w[4] = {z.x, z.y, z.z, z.w};
 #pragma unroll
-            for (int q = 0; q < 8; ++q) {
-                if (q < 7) take((q + 1) & 1, g + q + 1);
-                const f2 vv[2] = {pair2(v2[q & 1].x, v2[q & 1].x), pair2(v2[q & 1].y, v2[q & 1].y)};
-                f2 sum[2][2];
+                    for (int e = 0; e < 4; ++e)
 #pragma unroll
-                for (int j = 0; j < 2 * NJ; ++j) {
-                    const ulonglong2 x = r4[q & 1][j >> 1], y = k4[q & 1][j >> 1], z = w4[q & 1][j >> 1];
-                    const f2 r = j & 1 ? x.y : x.x, k = j & 1 ? y.y : y.x, w = j & 1 ? z.y : z.x;
-#pragma unroll
-                    for (int c = 0; c < 2; ++c) {
-                        sum[j & 1][c] = j < 2 ? mul2(r, s[j][c]) : fma2(r, s[j][c], sum[j & 1][c]);
-                        s[j][c] = fma2(w, s[j][c], mul2(k, vv[c]));
-                    }
-                }
-#pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    const float2 x = split2(sum[0][c]), y = split2(sum[1][c]);
-                    o[q][c] = (x.x + y.x) + (x.y + y.y);
+                        for (int c = 0; c < 4; ++c) {
+                            o[q][c] = fmaf(r[e], s[4 * j + e][c], o[q][c]);
+                            s[4 * j + e][c] = fmaf(w[e], s[4 * j + e][c], k[e] * vv[c]);
+                        }
                 }
             }
-            // fold over the eight lanes of a column pair: lane kg ends with token g + kg
+            // fold over the eight lanes of the columns: lane kg ends with two columns of token g + kg / 2
 #pragma unroll
-            for (int st = 4; st > 0; st >>= 1) {
-                const bool hi = kg & st;
+            for (int st = 2; st > 0; st >>= 1) {
+                const bool hi = kg & (2 * st);
 #pragma unroll
                 for (int q = 0; q < st; ++q)
 #pragma unroll
-                    for (int c = 0; c < 2; ++c) {
+                    for (int c = 0; c < 4; ++c) {
                         const float give = hi ? o[q][c] : o[q + st][c], keep = hi ? o[q + st][c] : o[q][c];
-                        o[q][c] = keep + __shfl_xor_sync(0xffffffffu, give, st);
+                        o[q][c] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * st);
                     }
             }
-            const int tk = g + kg;
-            if (i0 + tk < a.q_rows) {
-                float* y = a.y + ((int64_t)b * a.q_rows + i0 + tk) * HD + head * D + v0 + col;
+            const int c0 = (kg & 1) * 2, tk = g + (kg >> 1);
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const float give = c0 ? o[0][c] : o[0][c + 2], keep = c0 ? o[0][c + 2] : o[0][c];
+                o[0][c] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+            }
+            if (i0 + tk < count) {
+                float* y = a.y + (row0 + i0 + tk) * HD + head * D + v0 + col + c0;
                 const float bonus = bonus_s[tk];
 #pragma unroll
                 for (int c = 0; c < 2; ++c)
-                    if (col + c < vc) y[c] = fmaf(bonus, vs[tk * kScanCols + col + c], o[0][c]);
+                    if (col + c0 + c < vc) y[c] = fmaf(bonus, vs[tk * kScanCols + col + c0 + c], o[0][c]);
             }
         }
         __syncthreads();  // the tile may be refilled, the next one is there
     }
 #pragma unroll
-    for (int j = 0; j < 2 * NJ; ++j)
+    for (int j = 0; j < 4 * NJ; ++j)
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-            const float2 x = split2(s[j][c]);
-            const int k = 32 * (j >> 1) + 4 * kg + 2 * (j & 1);
-            if (col + c < vc) {
-                if (k < D) state[(int64_t)k * D + c] = x.x;
-                if (k + 1 < D) state[(int64_t)(k + 1) * D + c] = x.y;
+        for (int c = 0; c < 4; ++c) {
+            const int k = 32 * (j >> 2) + 4 * kg + (j & 3);
+            if (col + c < vc && k < D) result[(int64_t)k * D + v0 + col + c] = s[j][c];
+        }
+}
+
+// The states over the segments: a segment's place gets its incoming state, the sequence the last one.
+__global__ void __launch_bounds__(256) wkv_join_kernel(const WkvArgs a, int segs) {
+    const int D = a.dim, e = blockIdx.x * 256 + threadIdx.x;
+    if (e >= D * D) return;
+    const int64_t head = blockIdx.y;  // of all sequences
+    float* seg = a.seg_s + head * kSegments * (D * D + D);
+    float own[kSegments], decay[kSegments];
+#pragma unroll
+    for (int i = 0; i < kSegments; ++i) {
+        own[i] = i < segs ? seg[(int64_t)i * (D * D + D) + e] : 0.0f;
+        decay[i] = i < segs ? seg[(int64_t)i * (D * D + D) + D * D + e / D] : 0.0f;
+    }
+    float s = own[0];
+#pragma unroll
+    for (int i = 1; i < kSegments; ++i)
+        if (i < segs) {
+            seg[(int64_t)i * (D * D + D) + e] = s;
+            s = fmaf(decay[i], s, own[i]);
+        }
+    a.s[head * D * D + e] = s;
+}
+
+// o_t += (r_t times the decays since the segment's start)^T S for the segments behind the first: a CTA per head and 64 tokens,
+// on the tensor cores, both factors as bf16 hi + lo (16 significand bits).  Head size 64.
+constexpr int kCarryDim = 64, kCarryLd = 72;  // bf16 elements per shared-memory row
+__global__ void __launch_bounds__(256) wkv_carry_kernel(const WkvArgs a, int seg_tokens) {
+    __shared__ __align__(16) __nv_bfloat16 rh[64][kCarryLd], rl[64][kCarryLd], sh[64][kCarryLd], sl[64][kCarryLd];
+    __shared__ float part[4][64];
+    __shared__ int any;
+    const int D = kCarryDim, HD = a.heads * D;
+    const int per = seg_tokens / kBlock;
+    const int head = blockIdx.x, seg = blockIdx.y / per + 1, b = blockIdx.z, t0 = (blockIdx.y % per) * kBlock;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int first = seg * seg_tokens, count = min(seg_tokens, a.q_rows - first);
+    if (t0 >= count) return;
+    const int64_t row0 = (int64_t)b * a.q_rows + first;
+    const float* S = a.seg_s + (((int64_t)b * a.heads + head) * kSegments + seg) * (D * D + D);
+    const int ch = threadIdx.x & 63, quarter = threadIdx.x >> 6;  // a channel, 16 of the 64 tokens
+    float r[16], w[16], p = 1.0f, run;                              // run: the decays before the token
+    {
+        const float* up = a.seg_w + (((int64_t)b * ((a.q_rows + kBlock - 1) / kBlock) + (first + t0) / kBlock) * 2 * a.heads + head) * D + ch;
+        run = up[0] * up[(int64_t)a.heads * D];
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int t = t0 + quarter * 16 + i;
+        const bool ok = t < count;
+        r[i] = ok ? a.proj[(row0 + t) * a.ld + head * D + ch] : 0.0f;
+        w[i] = ok ? a.w[(row0 + t) * HD + head * D + ch] : 1.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) p *= w[i];
+    part[quarter][ch] = p;
+    if (threadIdx.x == 0) any = 0;
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 3; ++i)
+        if (i < quarter) run *= part[i][ch];
+    bool live = false;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const float v = r[i] * run;
+        live |= v != 0.0f;
+        run *= w[i];
+        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+        rh[quarter * 16 + i][ch] = hi;
+        rl[quarter * 16 + i][ch] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+    if (live) any = 1;
+    __syncthreads();
+    if (any == 0) return;  // everything has decayed away
+    for (int i = threadIdx.x; i < D * D; i += 256) {  // [key][value]
+        const float v = S[i];
+        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+        sh[i >> 6][i & 63] = hi;
+        sl[i >> 6][i & 63] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+    __syncthreads();
+    // warps as 4 (16 tokens) x 2 (32 values)
+    const int tt = warp >> 1, vv = (warp & 1) * 32;
+    float o[4][4] = {};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        uint32_t ah[4], al[4];
+        const uint32_t a_off = ((tt * 16 + (lane & 15)) * kCarryLd + k * 16 + (lane >> 4) * 8) * 2;
+        ptx::ldsm4(ah, ptx::smem_u32(rh) + a_off);
+        ptx::ldsm4(al, ptx::smem_u32(rl) + a_off);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            uint32_t bh[4], bl[4];
+            const uint32_t b_off = ((k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kCarryLd + vv + n * 16 + (lane >> 4) * 8) * 2;
+            ptx::ldsm4t(bh, ptx::smem_u32(sh) + b_off);
+            ptx::ldsm4t(bl, ptx::smem_u32(sl) + b_off);
+#pragma unroll
+            for (int q = 0; q < 2; ++q) {
+                ptx::mma_bf16(o[2 * n + q], ah, bh[2 * q], bh[2 * q + 1]);
+                ptx::mma_bf16(o[2 * n + q], al, bh[2 * q], bh[2 * q + 1]);
+                ptx::mma_bf16(o[2 * n + q], ah, bl[2 * q], bl[2 * q + 1]);
+            }
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int t = t0 + tt * 16 + (lane >> 2) + half * 8;
+            if (t < count) {
+                float2* y = reinterpret_cast<float2*>(a.y + (row0 + t) * HD + head * D + vv + n * 8 + (lane & 3) * 2);
+                float2 x = *y;
+                x.x += o[n][2 * half];
+                x.y += o[n][2 * half + 1];
+                *y = x;
             }
         }
 }
 
+// segments of the tokens: the fewest rounds of CTAs (three share an SM) times tokens, no segment below 128 tokens
+int scan_segments(const WkvArgs& a) {
+    if (!a.seg_s || !a.seg_w || a.dim != kCarryDim) return 1;
+    const int64_t ctas = (int64_t)a.heads * ((a.dim + kScanCols - 1) / kScanCols) * a.batch, slots = 3ll * a.sm_count;
+    int best = 1;
+    int64_t least = 0;
+    for (int segs = 1; segs <= kSegments && (segs == 1 || a.q_rows / segs >= 128); ++segs) {
+        const int64_t cost = (ctas * segs + slots - 1) / slots * (((a.q_rows + segs - 1) / segs + kBlock - 1) / kBlock);
+        if (segs == 1 || cost < least) { best = segs; least = cost; }
+    }
+    return best;
+}
 template <int NJ>
 cudaError_t scan_launch(const WkvArgs& a, cudaStream_t s) {
     static PerDeviceOnce once;
     cudaError_t e = once.run([] { return cudaFuncSetAttribute(wkv_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ScanCfg<NJ>::kSmem); });
     if (e != cudaSuccess) return e;
-    wkv_scan_kernel<NJ><<<dim3((unsigned)a.heads, (unsigned)((a.dim + kScanCols - 1) / kScanCols), (unsigned)a.batch), kScanThreads, ScanCfg<NJ>::kSmem, s>>>(a);
+    int segs = scan_segments(a);
+    const int tokens = ((a.q_rows + segs - 1) / segs + kBlock - 1) / kBlock * kBlock;
+    segs = (a.q_rows + tokens - 1) / tokens;
+    wkv_scan_kernel<NJ><<<dim3((unsigned)a.heads, (unsigned)((a.dim + kScanCols - 1) / kScanCols), (unsigned)(a.batch * segs)), kScanThreads, ScanCfg<NJ>::kSmem, s>>>(a, segs, tokens);
+    if (segs > 1) {
+        wkv_join_kernel<<<dim3((unsigned)((a.dim * a.dim + 255) / 256), (unsigned)(a.heads * a.batch)), 256, 0, s>>>(a, segs);
+        wkv_carry_kernel<<<dim3((unsigned)a.heads, (unsigned)((segs - 1) * (tokens / kBlock)), (unsigned)a.batch), 256, 0, s>>>(a, tokens);
+    }
     return cudaGetLastError();
 }
 cudaError_t step_launch(const WkvArgs& a, cudaStream_t s, bool pdl) {
@@ -416,9 +548,13 @@ cudaError_t step_launch(const WkvArgs& a, cudaStream_t s, bool pdl) {
 }  // namespace
 
 int wkv_max_dim() { return 256; }
+int64_t wkv_segment_floats(int heads, int dim) { return dim == kCarryDim ? (int64_t)heads * kSegments * (dim * dim + dim) : 0; }
+int64_t wkv_prefix_floats(int heads, int dim, int64_t rows, int batch) { return dim == kCarryDim ? (rows / kBlock + batch) * 2 * heads * dim : 0; }
 
 cudaError_t launch_wkv_mix(const WkvMix& a, cudaStream_t s) {
-    wkv_mix_kernel<<<(unsigned)(a.batch * a.q_rows), 256, 0, s>>>(a);
+    const unsigned rows = (unsigned)(a.batch * a.q_rows);
+    if (a.rows5) wkv_mix_kernel<<<rows, 256, 0, s>>>(a);
+    else wkv_mix_tiles_kernel<<<(rows + 7) / 8, 256, 0, s>>>(a);
     return cudaGetLastError();
 }
 

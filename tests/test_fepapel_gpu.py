@@ -158,13 +158,14 @@ def test_mechanisms_alone(bt, what):
         m.set_trace(False)
 
 
-@pytest.mark.parametrize("mixer", ["wkv", "rglru"])
+@pytest.mark.parametrize("mixer", ["wkv", "wkv_in_segments", "rglru"])
 def test_recurrence_carries_a_far_token(bt, mixer):
     """A first token of weight far behind still shows: with slow decays the state carries it over hundreds of positions."""
-    cfg = config(40, 48, [wkv(2, 32, 4) if mixer == "wkv" else rglru(64, 2, 4)])
+    dim = {"wkv": 32, "wkv_in_segments": 64}.get(mixer)
+    cfg = config(40, 48, [wkv(2, dim, 4) if dim else rglru(64, 2, 4)])
     t = make_tensors(cfg, seed=4)
-    if mixer == "wkv":
-        t["l0.mix.w0"] = bf16(np.full(64, -8.0))
+    if dim:
+        t["l0.mix.w0"] = bf16(np.full(2 * dim, -8.0))
         t["l0.mix.w2"] = bf16(0.01 * t["l0.mix.w2"])
     else:
         t["l0.mix.lam"] = bf16(np.full(64, -9.0))
@@ -172,7 +173,7 @@ def test_recurrence_carries_a_far_token(bt, mixer):
     rng = np.random.default_rng(4)
     tokens = rng.integers(1, 40, 600).astype(np.int32)
     tokens[0] = 0
-    key = "l0.mix.k" if mixer == "wkv" else "l0.mix.x"
+    key = "l0.mix.k" if dim else "l0.mix.x"
     e0 = ref.unit_rms(np.asarray(t["embed"], np.float64)[0], 1e-5) * np.asarray(t["l0.norm1"], np.float64)
     gain = np.asarray(t[key], np.float64)
     t[key] = bf16((gain + 12.0 * np.outer(np.sign(gain @ e0), e0 / (e0 @ e0))).astype(np.float32))  # token 0 enters with weight
@@ -182,7 +183,7 @@ def test_recurrence_carries_a_far_token(bt, mixer):
     assert row_errors(oracle(cfg, t, other)[0], logits)[-1] > 100 * TOL["float32"][0]
     for dtype in ("float32", "bfloat16"):
         m = lay.build_layered(cfg, t, dtype=dtype, max_seq_len=600)
-        for sizes in ([600], [250, 1, 2, 37], [500] + [1] * 100, [63, 65], [256, 16, 8]):
+        for sizes in ([600], [250, 1, 2, 37], [500] + [1] * 100, [63, 65], [256, 16, 8], [2, 598], [300]):
             m.reset_kv_cache()
             assert_close(feed(m, tokens, sizes), logits, dtype, sizes)
 
