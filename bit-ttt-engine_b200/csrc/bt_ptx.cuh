@@ -120,6 +120,11 @@ __device__ __forceinline__ void bulk_g2s(void* dst_smem, const void* src_gmem, u
         : "memory");
 }
 
+// asks for `bytes` (a multiple of 16, 16-byte aligned) of global memory to be brought into L2
+__device__ __forceinline__ void prefetch_l2(const void* src_gmem, uint32_t bytes) {
+    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(src_gmem), "r"(bytes) : "memory");
+}
+
 // Programmatic dependent launch: let the next kernel of the stream start its prologue /
 // wait until everything this kernel depends on has completed and is visible.
 __device__ __forceinline__ void pdl_launch_dependents() {

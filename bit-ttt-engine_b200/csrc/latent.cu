@@ -123,18 +123,19 @@ __device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, flo
     const float* gates = a.gate ? a.proj + r * a.ld + a.heads * (a.dim + a.rot) + a.rank + a.rot : nullptr;
     // a span's factor per head: its share of the softmax over all spans, times the output gate
     for (int h = threadIdx.x; h < nh; h += blockDim.x) {
-        float ms[kMaxSplits], m = -INFINITY, den = 0.0f;
+        float ms[kMaxSplits], ls[kMaxSplits], m = -INFINITY, den = 0.0f;
 #pragma unroll
         for (int s = 0; s < kMaxSplits; ++s) {  // all remote reads in flight together
             ms[s] = s < splits ? *(splits > 1 ? cluster.map_shared_rank(m_s, s) + h : m_s + h) : -INFINITY;
-            m = fmaxf(m, ms[s]);
+            ls[s] = s < splits ? *(splits > 1 ? cluster.map_shared_rank(l_s, s) + h : l_s + h) : 0.0f;
         }
 #pragma unroll
-        for (int s = 0; s < kMaxSplits; ++s)
-            if (s < splits) {
-                ms[s] = LOG2 ? ex2(ms[s] - m) : expf(ms[s] - m);  // an empty span: 0
-                den = fmaf(*(splits > 1 ? cluster.map_shared_rank(l_s, s) + h : l_s + h), ms[s], den);
-            }
+        for (int s = 0; s < kMaxSplits; ++s) m = fmaxf(m, ms[s]);
+#pragma unroll
+        for (int s = 0; s < kMaxSplits; ++s) {
+            ms[s] = LOG2 ? ex2(ms[s] - m) : expf(ms[s] - m);  // an empty span: 0
+            den = fmaf(ls[s], ms[s], den);
+        }
         const float f = (gates ? sigmoid_f(gates[head0 + h]) : 1.0f) / den;
 #pragma unroll
         for (int s = 0; s < kMaxSplits; ++s)
@@ -146,7 +147,7 @@ __device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, flo
     for (int i = (int)((int64_t)total * split / splits) + threadIdx.x; i < i1; i += blockDim.x) {
         const int h = i / quads, c = (i - h * quads) * 4, head = head0 + h;
         float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll 4
+#pragma unroll 8
         for (int s = 0; s < splits; ++s) {
             const float4 o = *reinterpret_cast<const float4*>((splits > 1 ? cluster.map_shared_rank(o_s, s) : o_s) + h * W + c);
             const float f = fac[h * kMaxSplits + s];
@@ -174,7 +175,7 @@ __device__ __forceinline__ void merge_spans(const LatentAttn& a, float* m_s, flo
 // columns) and, read the other way, the MN-major A operand of the values (latent columns x positions).
 //   scores^T [128 positions][HG]  = block . queries^T            (tcgen05, accumulators in TMEM)
 //   softmax: scores through shared memory, a warp per HG / 16 heads; weights leave as bf16 hi and lo
-//   outputs^T [rank][HG]         += block^T . (hi + lo)^T        (tiles of 128 latent columns, accumulators in TMEM)
+//   outputs^T [rank][2 HG]       += block^T . [hi | lo]^T        (tiles of 128 latent columns, accumulators in TMEM)
 // The outputs are rescaled only when a maximum has grown by more than 2^8.
 constexpr int kSpanThreads = 512, kSpanWarps = kSpanThreads / 32, kKeys = 128, kMaxStages = 3;
 constexpr float kLazy = 8.0f;
@@ -182,6 +183,7 @@ constexpr float kLazy = 8.0f;
 template <int HG>
 struct SpanCfg {
     static constexpr int kP = HG * kKeys * 2;                                   // bytes of the weights' hi (lo) part
+    static constexpr int kTmem = HG == 32 ? 512 : 256;                           // columns: scores, outputs of up to four tiles
     static constexpr size_t kFixed = (size_t)2 * kP + HG * kKeys * 4 + (3 + kMaxSplits) * HG * 4 + 32 * 4 + 128;
     __host__ __device__ static size_t q(int cols) { return (size_t)HG * cols * 2; }
     static size_t fixed(int cols) { return q(cols) + kFixed + (size_t)cols * 2; }
@@ -232,7 +234,7 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_tc_kernel(const L
         ptx::mbar_init(o_done, 1);
         ptx::mbar_fence_init();
     }
-    if (warp == 1) { ptx::tmem_alloc(tmem_slot, 256); ptx::tmem_relinquish(); }
+    if (warp == 1) { ptx::tmem_alloc(tmem_slot, Cfg::kTmem); ptx::tmem_relinquish(); }
     ptx::tc_fence_before();
     __syncthreads();
     ptx::tc_fence_after();
@@ -323,14 +325,21 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_tc_kernel(const L
         if (warp == 1 && lane == 0) {
             ok &= ptx::mbar_wait_bounded(&full[slot], (uint32_t)((i / stages) & 1));
             ptx::tc_fence_after();
-            const uint32_t q_addr = ptx::smem_u32(q_s);
-            for (int k = 0; k < steps; ++k) {
-                const uint32_t o = (uint32_t)k * 256;
-                ptx::umma_f16(tmem, ptx::smem_desc(kv + o, 128, group), ptx::smem_desc(q_addr + o, 128, group), span_idesc(HG, false), k > 0 ? 1u : 0u);
+            uint64_t ad = ptx::smem_desc(kv, 128, group), qd = ptx::smem_desc(ptx::smem_u32(q_s), 128, group);
+            ptx::umma_f16(tmem, ad, qd, span_idesc(HG, false), 0u);
+#pragma unroll 4
+            for (int k = 1; k < steps; ++k) {  // 256 bytes further in units of 16
+                ad += 16;
+                qd += 16;
+                ptx::umma_f16(tmem, ad, qd, span_idesc(HG, false), 1u);
             }
             ptx::umma_commit(s_done);
         }
         __syncwarp();
+        if (warp == 15 && i + stages < blocks && lane < 8) {  // the block that will take this one's slot comes into L2 meanwhile
+            const int g0 = lane * 2, n = min(2, (min(kKeys, t1 - t0 - (i + stages) * kKeys) + 7) / 8 - g0);
+            if (n > 0) ptx::prefetch_l2(seq + ((int64_t)t0 / 8 + (i + stages) * (kKeys / 8) + g0) * group, n * group);
+        }
         if (warp < 4) {  // lane = position
             ok &= ptx::mbar_wait_bounded(s_done, (uint32_t)(i & 1));
             ptx::tc_fence_after();
@@ -387,14 +396,14 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_tc_kernel(const L
         const int rescale = __syncthreads_or(grown && i > 0);
         if (rescale) {  // warps w, w + 4, ... take the same lanes and different tiles
             for (int mt = warp >> 2; mt < m_tiles; mt += 4) {
-                const uint32_t at = tmem_o + mt * HG + ((uint32_t)((warp & 3) * 32) << 16);
+                const uint32_t at = tmem_o + mt * 2 * HG + ((uint32_t)((warp & 3) * 32) << 16);
 #pragma unroll
-                for (int c = 0; c < HG; c += 16) {
+                for (int c = 0; c < 2 * HG; c += 16) {
                     uint32_t v[16];
                     ptx::tmem_ld16(at + c, v);
                     ptx::tmem_ld_wait();
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) * al_s[c + j]);
+                    for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) * al_s[(c + j) % HG]);
                     ptx::tmem_st16(at + c, v);
                 }
             }
@@ -404,14 +413,14 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_tc_kernel(const L
         }
         if (warp == 1 && lane == 0) {
             ptx::tc_fence_after();
-            const uint32_t ph = ptx::smem_u32(p_hi), pl = ptx::smem_u32(p_lo);
-            for (int mt = 0; mt < m_tiles; ++mt)
+            const uint64_t pd = ptx::smem_desc(ptx::smem_u32(p_hi), 128, 2048);  // hi and lo rows behind one another
+            uint64_t at = ptx::smem_desc(kv, group, 128);
+            for (int mt = 0; mt < m_tiles; ++mt, at += 2048 / 16) {
+                uint64_t ad = at;
 #pragma unroll
-                for (int k = 0; k < kKeys / 16; ++k) {
-                    const uint64_t ad = ptx::smem_desc(kv + mt * 2048 + k * 2 * group, group, 128);
-                    ptx::umma_f16(tmem_o + mt * HG, ad, ptx::smem_desc(ph + k * 256, 128, 2048), span_idesc(HG, true), i > 0 || k > 0 ? 1u : 0u);
-                    ptx::umma_f16(tmem_o + mt * HG, ad, ptx::smem_desc(pl + k * 256, 128, 2048), span_idesc(HG, true), 1u);
-                }
+                for (int k = 0; k < kKeys / 16; ++k, ad += group / 8)  // two groups of positions further
+                    ptx::umma_f16(tmem_o + mt * 2 * HG, ad, pd + k * 16, span_idesc(2 * HG, true), i > 0 || k > 0 ? 1u : 0u);
+            }
             ptx::umma_commit(o_done);
         }
     }
@@ -430,16 +439,19 @@ __global__ void __launch_bounds__(kSpanThreads, 1) latent_span_tc_kernel(const L
     for (int mt = warp >> 2; mt < m_tiles; mt += 4)
 #pragma unroll
         for (int c = 0; c < HG; c += 16) {
-            uint32_t v[16];
-            ptx::tmem_ld16(tmem_o + mt * HG + c + ((uint32_t)((warp & 3) * 32) << 16), v);
+            uint32_t v[16], l[16];
+            const uint32_t at = tmem_o + mt * 2 * HG + c + ((uint32_t)((warp & 3) * 32) << 16);
+            ptx::tmem_ld16(at, v);
+            ptx::tmem_ld16(at + HG, l);
             ptx::tmem_ld_wait();
 #pragma unroll
-            for (int j = 0; j < 16; ++j) o_s[(c + j) * W + mt * 128 + (warp & 3) * 32 + lane] = blocks > 0 ? __uint_as_float(v[j]) : 0.0f;
+            for (int j = 0; j < 16; ++j)
+                o_s[(c + j) * W + mt * 128 + (warp & 3) * 32 + lane] = blocks > 0 ? __uint_as_float(v[j]) + __uint_as_float(l[j]) : 0.0f;
         }
     if (!ok) atomicExch(err, kErrLatentTimeout);
     ptx::tc_fence_before();
     __syncthreads();
-    if (warp == 1) ptx::tmem_dealloc(tmem, 256);
+    if (warp == 1) ptx::tmem_dealloc(tmem, Cfg::kTmem);
     merge_spans<true>(a, m_s, l_s, o_s, fac, W, nh, head0, r, split, splits, out);
 }
 
