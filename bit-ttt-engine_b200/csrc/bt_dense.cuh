@@ -333,6 +333,7 @@ struct WkvArgs {
     int64_t shift_slot = 0;
     int width = 0;
     int sm_count = 0;
+    bool split16 = false;          // prefill: the factors of the products with states and values as bf16 hi + lo
     // prefill in segments of the tokens, side by side (null: one after the other)
     float* seg_s = nullptr;        // wkv_segment_floats per sequence: states and decays of the segments
     float* seg_w = nullptr;        // wkv_prefix_floats: decays up to each block of 64 tokens

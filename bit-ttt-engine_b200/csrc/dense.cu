@@ -417,6 +417,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a)
         d.tok_end = a.m;
         return d;
     };
+    // an expert's tile is as wide as its rows need
+    auto tile_rows = [&](const Tile& d) -> uint32_t { return a.plan ? (uint32_t)((d.tok_end - d.tok0 + 15) / 16 * 16) : (uint32_t)NT; };
 
     if (warp == 0) {
         if (lane == 0) {
@@ -425,13 +427,14 @@ __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a)
                 const Tile d = decode(t);
                 const uint8_t* wp = a.w + (int64_t)d.blk * a.w_block + (int64_t)d.rs * kTcRows * 128;
                 const uint8_t* xp = a.x + (a.plan ? 0 : (int64_t)d.blk * a.x_block) + d.tok0 * 128;
+                const uint32_t x_bytes = tile_rows(d) * 128;
                 for (int kc = d.c0; kc < d.c1; ++kc) {
                     const int wc = kc >= a.w_chunks ? kc - a.w_chunks : kc;  // hi and lo halves meet the same weights
                     if (!first) { if (!ptx::mbar_wait_bounded(&empty[slot], par)) { ok = false; break; } }
                     uint8_t* st = smem + (size_t)slot * Cfg::kStageBytes;
-                    ptx::mbar_arrive_expect_tx(&full[slot], Cfg::kStageBytes);
+                    ptx::mbar_arrive_expect_tx(&full[slot], kTcRows * 128 + x_bytes);
                     ptx::bulk_g2s(st, wp + (int64_t)wc * a.n_pad * 128, kTcRows * 128, &full[slot]);
-                    ptx::bulk_g2s(st + kTcRows * 128, xp + (int64_t)kc * a.m_pad * 128, NT * 128, &full[slot]);
+                    ptx::bulk_g2s(st + kTcRows * 128, xp + (int64_t)kc * a.m_pad * 128, x_bytes, &full[slot]);
                     ++issued;
                     if (++slot == S) { slot = 0; first = false; par ^= 1; }
                 }
@@ -444,10 +447,10 @@ __global__ void __launch_bounds__(kTcThreads, 1) dense_tc_kernel(const TcArgs a)
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            const uint32_t idesc = tc_idesc(NT);
             int slot = 0, set = 0; uint32_t par = 0, acc_par = 1; int done = 0;
             for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x, ++done) {
                 const Tile d = decode(t);
+                const uint32_t idesc = tc_idesc((int)tile_rows(d));
                 if (done >= 2) ok &= ptx::mbar_spin_relaxed(&acc_empty[set], acc_par);
                 ptx::tc_fence_after();
                 for (int kc = d.c0; kc < d.c1 && ok; ++kc) {

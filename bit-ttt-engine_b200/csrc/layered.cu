@@ -357,6 +357,7 @@ WkvArgs wkv_args(const bt_model* m, const LayLayer& l, const LayRun& run, const 
     a.low = r.a; a.rank = c.decay_rank;
     a.w = r.b; a.hn = r.hn; a.shift = run.ring; a.shift_slot = (int64_t)m->cfg.max_batch * m->lay->c.width; a.width = m->lay->c.width;
     a.sm_count = m->sm_count;
+    a.split16 = !m->lay->f32;
     a.seg_s = m->lay->f32 ? nullptr : m->lay->wkv_seg;
     a.seg_w = r.wkv_pre;
     return a;

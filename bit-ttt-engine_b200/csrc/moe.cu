@@ -227,7 +227,8 @@ __global__ void __launch_bounds__(256) moe_choose_kernel(const MoeRoute a) {
     }
 }
 
-// one CTA: the experts' rows behind one another, each at a multiple of 8; tiles of `tile` rows; the counts start over
+// one CTA: the experts' rows behind one another, each at a multiple of 8, in tiles of about equal size, at
+// most `tile` rows; the counts start over
 __global__ void __launch_bounds__(kMaxExperts) moe_plan_kernel(const MoeRoute a) {
     __shared__ int rows_s[32], tiles_s[32];
     const int e = threadIdx.x, lane = e & 31, warp = e >> 5;
@@ -257,9 +258,10 @@ __global__ void __launch_bounds__(kMaxExperts) moe_plan_kernel(const MoeRoute a)
         a.row_start[e] = r0;
         a.counts_done[e] = n;
         a.counts[e] = 0;
+        const int each = nt ? ((n + nt - 1) / nt + 15) / 16 * 16 : 0;
         for (int i = 0; i < nt && t0 + i < a.max_tiles; ++i) {
             ExpertTile t;
-            t.expert = e; t.row0 = r0 + i * a.tile; t.row_end = r0 + n; t.pad = 0;
+            t.expert = e; t.row0 = r0 + i * each; t.row_end = r0 + min(n, (i + 1) * each); t.pad = 0;
             a.tiles[t0 + i] = t;
         }
     }
@@ -325,10 +327,10 @@ cudaError_t launch_moe_down(const MoeStep& a, cudaStream_t s, bool pdl) {
     return stream_launch<true>(m, a.sm_count, s, pdl);
 }
 
-// rows per tile of the grouped products: an expert's last tile is half empty on average
+// most rows per tile of the grouped products
 int moe_tile_rows(int64_t rows, int top, int experts) {
     const int64_t each = rows * top / experts;
-    return each <= 48 ? 64 : (each <= 640 ? 128 : 256);
+    return each <= 48 ? 64 : (each <= 112 ? 128 : 256);
 }
 int moe_max_tiles(int64_t rows, int top, int experts, int tile) {
     const int64_t all = rows * top, busy = all < experts ? all : experts;

@@ -176,13 +176,11 @@ __global__ void __launch_bounds__(kStepThreads) wkv_step_kernel(const WkvArgs a)
 // ---------------------------------------------------------------------------------------
 // many tokens
 // ---------------------------------------------------------------------------------------
-// A CTA owns 64 value columns of one head and a segment of the tokens.  Four warps compute, 16 columns each: eight lanes share
+// A CTA owns 64 value columns of one head.  Four warps compute, 16 columns each: eight lanes share
 // four columns, each with 4 NJ of their state elements in registers (key channels 32 j + 4 lane .. + 3); tokens go by
 // fours, whose sums over the lanes are folded together.  Two more warps bring r, k, the decays and v of a tile of tokens into
 // shared memory, two tiles ahead, and make the current token's own weight, sum of r u k, one tile ahead.
-// Several segments: each but the first starts from zero; wkv_join_kernel carries the states over the segments, wkv_carry_kernel
-// adds what a segment's incoming state means for its tokens.
-constexpr int kScanCompute = 4, kScanThreads = 32 * kScanCompute + 64, kScanCols = 64, kScanBufs = 3, kSegments = 16, kBlock = 64;
+constexpr int kScanCompute = 4, kScanThreads = 32 * kScanCompute + 64, kScanCols = 64, kScanBufs = 3;
 template <int NJ>
 struct ScanCfg {
     static constexpr int DP = 32 * NJ, TT = NJ <= 4 ? 16 : 8;
@@ -190,19 +188,16 @@ struct ScanCfg {
     static constexpr size_t kSmem = (size_t)kScanBufs * kTile * sizeof(float);
 };
 template <int NJ>
-__global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel(const WkvArgs a, int segs, int seg_tokens) {
+__global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 2 : 1) wkv_scan_kernel(const WkvArgs a) {
     using Cfg = ScanCfg<NJ>;
     constexpr int DP = Cfg::DP, TT = Cfg::TT, Q = DP / 4;  // Q: 16-byte pieces per row
     extern __shared__ __align__(16) float sm[];
-    const int head = blockIdx.x, v0 = blockIdx.y * kScanCols, b = blockIdx.z / segs, seg = blockIdx.z - b * segs;
+    const int head = blockIdx.x, v0 = blockIdx.y * kScanCols, b = blockIdx.z;
     const int D = a.dim, HD = a.heads * D, vc = min(kScanCols, D - v0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int first = seg * seg_tokens, count = min(seg_tokens, a.q_rows - first);  // this segment's tokens
-    const int p0 = a.pos[b], tiles = (count + TT - 1) / TT;
-    const int64_t row0 = (int64_t)b * a.q_rows + first;
-    // where the segment's last state goes: the sequence's state, or its place among the segments
+    const int p0 = a.pos[b], count = a.q_rows, tiles = (count + TT - 1) / TT;
+    const int64_t row0 = (int64_t)b * count;
     float* state = a.s + ((int64_t)b * a.heads + head) * D * D;
-    float* result = segs > 1 ? a.seg_s + (((int64_t)b * a.heads + head) * kSegments + seg) * (D * D + D) : state;
     for (int i = threadIdx.x; i < kScanBufs * Cfg::kTile; i += kScanThreads) sm[i] = 0.0f;  // columns beyond the head's stay zero
     __syncthreads();
     auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
@@ -252,17 +247,12 @@ __global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel
                 t[2 * TT * DP + o] = 1.0f;
             }
         };
-        float uu[NJ], whole[NJ];  // the bonus; half of the tokens' decays multiplied up
+        float uu[NJ];  // the bonus
 #pragma unroll
-        for (int j = 0; j < NJ; ++j) { uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f; whole[j] = 1.0f; }
+        for (int j = 0; j < NJ; ++j) uu[j] = j * 32 + lane < D ? a.u[head * D + j * 32 + lane] : 0.0f;
         auto bonus = [&](int ti) {  // each of the two warps half of the tile's tokens
             if (ti >= tiles) return;
             float* t = sm + (ti % kScanBufs) * Cfg::kTile;
-            if (segs > 1 && seg > 0 && blockIdx.y == 0 && ti * TT % kBlock == 0)  // the decays up to this block of tokens, this warp's share
-#pragma unroll
-                for (int j = 0; j < NJ; ++j)
-                    if (j * 32 + lane < D)
-                        a.seg_w[((((int64_t)b * ((a.q_rows + kBlock - 1) / kBlock) + (first + ti * TT) / kBlock) * 2 + warp - kScanCompute) * a.heads + head) * D + j * 32 + lane] = whole[j];
             const int from = (warp - kScanCompute) * (TT / 2);
             float x[TT / 2];
 #pragma unroll
@@ -272,7 +262,6 @@ __global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel
                 for (int j = 0; j < NJ; ++j) {
                     const int at = (from + i) * DP + j * 32 + lane;
                     x[i] = fmaf(t[at] * uu[j], t[TT * DP + at], x[i]);
-                    if (segs > 1) whole[j] *= t[2 * TT * DP + at];
                 }
             }
 #pragma unroll
@@ -301,17 +290,7 @@ __global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel
             bonus(ti + 1);
             __syncthreads();
         }
-        if (segs > 1 && blockIdx.y == 0) {  // the segment's whole decay per channel
-            if (warp == kScanCompute)
-#pragma unroll
-                for (int j = 0; j < NJ; ++j) sm[j * 32 + lane] = whole[j];
-            asm volatile("bar.sync 1, 64;" ::: "memory");
-            if (warp != kScanCompute)
-#pragma unroll
-                for (int j = 0; j < NJ; ++j)
-                    if (j * 32 + lane < D) result[D * D + j * 32 + lane] = sm[j * 32 + lane] * whole[j];
-        }
-        if (blockIdx.x == 0 && blockIdx.y == 0 && seg == segs - 1) {  // the token shift's state
+        if (blockIdx.x == 0 && blockIdx.y == 0) {  // the token shift's state
             float* keep = a.shift + (int64_t)((p0 + a.q_rows - 1) & 1) * a.shift_slot + (int64_t)b * a.width;
             for (int c = tid; c < a.width; c += 64) keep[c] = a.hn[(row0 + count - 1) * a.width + c];
         }
@@ -324,7 +303,7 @@ __global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             const int k = 32 * (j >> 2) + 4 * kg + (j & 3);
-            s[j][c] = col + c < vc && k < D && p0 > 0 && seg == 0 ? state[(int64_t)k * D + v0 + col + c] : 0.0f;
+            s[j][c] = col + c < vc && k < D && p0 > 0 ? state[(int64_t)k * D + v0 + col + c] : 0.0f;
         }
     __syncthreads();
     for (int ti = 0; ti < tiles; ++ti) {
@@ -390,8 +369,221 @@ __global__ void __launch_bounds__(kScanThreads, NJ <= 2 ? 3 : 1) wkv_scan_kernel
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             const int k = 32 * (j >> 2) + 4 * kg + (j & 3);
-            if (col + c < vc && k < D) result[(int64_t)k * D + v0 + col + c] = s[j][c];
+            if (col + c < vc && k < D) state[(int64_t)k * D + v0 + col + c] = s[j][c];
         }
+}
+
+// ---------------------------------------------------------------------------------------
+// many tokens of a 16-bit model, heads of at most 64: sixteen tokens at a time on the tensor cores
+// ---------------------------------------------------------------------------------------
+// With P_t the product of the block's decays before token t and Q_t of those behind it, a block of tokens is
+//   o_t = (r_t P_t)^T S + sum over s <= t of A_ts v_s,    S <- diag(all decays) S + sum over s of (k_s Q_s) v_s^T,
+//   A_ts = sum over channels of r_t k_s (the decays between s and t) for s < t,    A_tt = sum of r_t u k_t.
+// No quotient of decays appears, so nothing overflows.  A, P and Q are made in f32; the factors of the products go in as bf16
+// hi + lo (16 significand bits), sums and the state stay f32.  A CTA owns a head and a segment of the tokens, a warp 16 value
+// columns of it, whose state S^T stays in the warp's accumulators.
+// Several segments: each but the first starts from zero; wkv_join_kernel carries the states over the segments, wkv_carry_kernel
+// adds what a segment's incoming state means for its tokens.
+constexpr int kSegments = 16, kBlock = 64;  // most segments; their length is a multiple of kBlock
+constexpr int kTok = 16, kHead = 64, kLd = 72, kLdA = 24;  // tokens per step, padded head, bf16 elements per shared-memory row
+struct BlockSmem {
+    float raw[2][4][kTok][kHead];  // r, k, decays, v as they come
+    float decay[2][kHead];         // a step's whole decay per channel
+    __nv_bfloat16 rows[2][6][kTok][kLd];  // hi and lo of r P, k Q and v
+    __nv_bfloat16 tri[2][2][kTok][kLdA];  // hi and lo of A
+};
+__device__ __forceinline__ void split16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
+    hi = __float2bfloat16_rn(v);
+    lo = __float2bfloat16_rn(v - __bfloat162float(hi));
+}
+// two values into bf16 pairs: hi parts and lo parts
+__device__ __forceinline__ void split16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = ptx::pack2(x, y);
+    lo = ptx::pack2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+}
+__global__ void __launch_bounds__(128, 3) wkv_block_kernel(const WkvArgs a, int segs, int seg_tokens) {
+    extern __shared__ __align__(16) uint8_t block_smem[];
+    BlockSmem& m = *reinterpret_cast<BlockSmem*>(block_smem);
+    const int D = a.dim, HD = a.heads * D;
+    const int head = blockIdx.x, seg = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int first = seg * seg_tokens, count = min(seg_tokens, a.q_rows - first), steps = (count + kTok - 1) / kTok;
+    const int p0 = a.pos[b];
+    const int64_t row0 = (int64_t)b * a.q_rows + first;
+    // where the segment's last state goes: the sequence's state, or its place among the segments
+    float* state = a.s + ((int64_t)b * a.heads + head) * D * D;
+    float* result = segs > 1 ? a.seg_s + (((int64_t)b * a.heads + head) * kSegments + seg) * (D * D + D) : state;
+    const float* proj = a.proj + row0 * a.ld + head * D;
+    const float* wrow = a.w + row0 * HD + head * D;
+    auto fetch = [&](int i) {
+        if (i < steps) {
+#pragma unroll
+            for (int e = tid; e < kTok * kHead / 4; e += 128) {
+                const int t = e >> 4, c = (e & 15) * 4, at = i * kTok + t;
+                const bool ok = at < count && c < D;
+                const float* src = proj + (int64_t)(ok ? at : 0) * a.ld + (ok ? c : 0);
+                ptx::cp16(ptx::smem_u32(&m.raw[i & 1][0][t][c]), src, ok);
+                ptx::cp16(ptx::smem_u32(&m.raw[i & 1][1][t][c]), src + HD, ok);
+                ptx::cp16(ptx::smem_u32(&m.raw[i & 1][3][t][c]), src + 2 * HD, ok);
+                if (at < count) ptx::cp16(ptx::smem_u32(&m.raw[i & 1][2][t][c]), wrow + (int64_t)at * HD + (ok ? c : 0), ok);
+                else *reinterpret_cast<float4*>(&m.raw[i & 1][2][t][c]) = make_float4(1.f, 1.f, 1.f, 1.f);  // behind the last token nothing decays
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0);
+    fetch(1);
+    for (int i = tid; i < (int)sizeof(m.tri) / 4; i += 128) reinterpret_cast<uint32_t*>(m.tri)[i] = 0;  // above A's diagonal
+    float st[8][4];  // S^T: tiles of 8 key channels; this lane's rows (values) and columns (keys) as in an accumulator
+    const int vr = warp * 16 + (lane >> 2), kc = (lane & 3) * 2;
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int v = vr + (e >> 1) * 8, k = n * 8 + kc + (e & 1);
+            st[n][e] = v < D && k < D && p0 > 0 && seg == 0 ? state[k * D + v] : 0.0f;
+        }
+    const int c4 = (lane & 15) * 4, s0 = 2 * warp + (lane >> 4), s1 = kTok - 1 - s0;  // A's columns of this lane's group
+    float u[4], whole = 1.0f;  // whole: the decays of the segment so far, channel tid
+#pragma unroll
+    for (int e = 0; e < 4; ++e) u[e] = c4 + e < D ? a.u[head * D + c4 + e] : 0.0f;
+    for (int i = 0; i < steps; ++i) {
+        const int buf = i & 1;
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const float(*rs)[kHead] = m.raw[buf][0], (*ks)[kHead] = m.raw[buf][1], (*ws)[kHead] = m.raw[buf][2], (*vs)[kHead] = m.raw[buf][3];
+        {   // r with the decays before it (threads 0-63), k with those behind it
+            const int c = tid & 63;
+            float run = 1.0f;
+            if (tid < 64) {
+#pragma unroll
+                for (int t = 0; t < kTok; ++t) {
+                    split16(rs[t][c] * run, m.rows[buf][0][t][c], m.rows[buf][1][t][c]);
+                    run *= ws[t][c];
+                }
+                m.decay[buf][c] = run;
+                if (segs > 1 && c < D) {
+                    if (seg > 0 && i * kTok % kBlock == 0)
+                        a.seg_w[(((int64_t)b * ((a.q_rows + kBlock - 1) / kBlock) + (first + i * kTok) / kBlock) * a.heads + head) * D + c] = whole;
+                    whole *= run;
+                }
+            } else {
+#pragma unroll
+                for (int t = kTok - 1; t >= 0; --t) {
+                    split16(ks[t][c] * run, m.rows[buf][2][t][c], m.rows[buf][3][t][c]);
+                    run *= ws[t][c];
+                }
+            }
+        }
+        {   // v
+            const int t = tid >> 3, c = (tid & 7) * 8;
+            const float4 x = *reinterpret_cast<const float4*>(&vs[t][c]), y = *reinterpret_cast<const float4*>(&vs[t][c + 4]);
+            uint4 hi, lo;
+            split16x2(x.x, x.y, hi.x, lo.x);
+            split16x2(x.z, x.w, hi.y, lo.y);
+            split16x2(y.x, y.y, hi.z, lo.z);
+            split16x2(y.z, y.w, hi.w, lo.w);
+            *reinterpret_cast<uint4*>(&m.rows[buf][4][t][c]) = hi;
+            *reinterpret_cast<uint4*>(&m.rows[buf][5][t][c]) = lo;
+        }
+        {   // A: sixteen lanes share columns s0 and 15 - s0, fifteen elements below the diagonal and two on it
+            float x[16], last = 0.0f, kd[4];
+            const int n0 = kTok - 1 - s0;  // elements of column s0
+            const float4 ka = *reinterpret_cast<const float4*>(&ks[s0][c4]), kb = *reinterpret_cast<const float4*>(&ks[s1][c4]);
+            const float4 ra = *reinterpret_cast<const float4*>(&rs[s0][c4]), rb = *reinterpret_cast<const float4*>(&rs[s1][c4]);
+            x[15] = ra.x * u[0] * ka.x + ra.y * u[1] * ka.y + ra.z * u[2] * ka.z + ra.w * u[3] * ka.w;
+            last = rb.x * u[0] * kb.x + rb.y * u[1] * kb.y + rb.z * u[2] * kb.z + rb.w * u[3] * kb.w;
+            kd[0] = ka.x; kd[1] = ka.y; kd[2] = ka.z; kd[3] = ka.w;
+#pragma unroll
+            for (int j = 0; j < kTok - 1; ++j) {
+                if (j == n0) { kd[0] = kb.x; kd[1] = kb.y; kd[2] = kb.z; kd[3] = kb.w; }
+                const int t = j < n0 ? s0 + 1 + j : j + 1;
+                const float4 r = *reinterpret_cast<const float4*>(&rs[t][c4]), w = *reinterpret_cast<const float4*>(&ws[t][c4]);
+                x[j] = fmaf(r.x, kd[0], fmaf(r.y, kd[1], fmaf(r.z, kd[2], r.w * kd[3])));
+                kd[0] *= w.x; kd[1] *= w.y; kd[2] *= w.z; kd[3] *= w.w;
+            }
+#pragma unroll
+            for (int h = 8; h > 0; h >>= 1) {
+                const bool up = lane & h;
+#pragma unroll
+                for (int q = 0; q < h; ++q) {
+                    const float give = up ? x[q] : x[q + h], keep = up ? x[q + h] : x[q];
+                    x[q] = keep + __shfl_xor_sync(0xffffffffu, give, h);
+                }
+                last += __shfl_xor_sync(0xffffffffu, last, h);
+            }
+            const int l = lane & 15, s = l < n0 || l == 15 ? s0 : s1, t = l == 15 ? s0 : (l < n0 ? s0 + 1 + l : l + 1);
+            split16(x[0], m.tri[buf][0][t][s], m.tri[buf][1][t][s]);
+            if (l == 0) split16(last, m.tri[buf][0][s1][s1], m.tri[buf][1][s1][s1]);
+        }
+        __syncthreads();
+        fetch(i + 2);
+        float o[2][4] = {};  // o^T: tiles of 8 tokens
+        uint32_t vh[4], vl[4];
+        {
+            const uint32_t at = (((lane & 7) + (lane >> 4) * 8) * kLd + warp * 16 + ((lane >> 3) & 1) * 8) * 2;
+            ptx::ldsm4t(vh, ptx::smem_u32(m.rows[buf][4]) + at);
+            ptx::ldsm4t(vl, ptx::smem_u32(m.rows[buf][5]) + at);
+            uint32_t th[4], tl[4];
+            const uint32_t ta = (((lane & 7) + (lane >> 4) * 8) * kLdA + ((lane >> 3) & 1) * 8) * 2;
+            ptx::ldsm4(th, ptx::smem_u32(m.tri[buf][0]) + ta);
+            ptx::ldsm4(tl, ptx::smem_u32(m.tri[buf][1]) + ta);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                ptx::mma_bf16(o[n], vh, th[2 * n], th[2 * n + 1]);
+                ptx::mma_bf16(o[n], vl, th[2 * n], th[2 * n + 1]);
+                ptx::mma_bf16(o[n], vh, tl[2 * n], tl[2 * n + 1]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {  // sixteen key channels
+            uint32_t sh[4], sl[4], bh[4], bl[4];
+            split16x2(st[2 * k][0], st[2 * k][1], sh[0], sl[0]);
+            split16x2(st[2 * k][2], st[2 * k][3], sh[1], sl[1]);
+            split16x2(st[2 * k + 1][0], st[2 * k + 1][1], sh[2], sl[2]);
+            split16x2(st[2 * k + 1][2], st[2 * k + 1][3], sh[3], sl[3]);
+            const uint32_t ra = (((lane & 7) + (lane >> 4) * 8) * kLd + k * 16 + ((lane >> 3) & 1) * 8) * 2;
+            ptx::ldsm4(bh, ptx::smem_u32(m.rows[buf][0]) + ra);
+            ptx::ldsm4(bl, ptx::smem_u32(m.rows[buf][1]) + ra);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                ptx::mma_bf16(o[n], sh, bh[2 * n], bh[2 * n + 1]);
+                ptx::mma_bf16(o[n], sl, bh[2 * n], bh[2 * n + 1]);
+                ptx::mma_bf16(o[n], sh, bl[2 * n], bl[2 * n + 1]);
+            }
+            const uint32_t ka = (((lane & 7) + ((lane >> 3) & 1) * 8) * kLd + k * 16 + (lane >> 4) * 8) * 2;
+            ptx::ldsm4t(bh, ptx::smem_u32(m.rows[buf][2]) + ka);
+            ptx::ldsm4t(bl, ptx::smem_u32(m.rows[buf][3]) + ka);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                float(&x)[4] = st[2 * k + n];
+                const float2 d = *reinterpret_cast<const float2*>(&m.decay[buf][k * 16 + n * 8 + kc]);
+                x[0] *= d.x; x[1] *= d.y; x[2] *= d.x; x[3] *= d.y;
+                ptx::mma_bf16(x, vh, bh[2 * n], bh[2 * n + 1]);
+                ptx::mma_bf16(x, vl, bh[2 * n], bh[2 * n + 1]);
+                ptx::mma_bf16(x, vh, bl[2 * n], bl[2 * n + 1]);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int t = i * kTok + n * 8 + kc + (e & 1), v = vr + (e >> 1) * 8;
+                if (t < count && v < D) a.y[(row0 + t) * HD + head * D + v] = o[n][e];
+            }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int v = vr + (e >> 1) * 8, k = n * 8 + kc + (e & 1);
+            if (v < D && k < D) result[k * D + v] = st[n][e];
+        }
+    if (segs > 1 && tid < D) result[D * D + tid] = whole;  // heads of 64: threads 0-63
+    if (head == 0 && seg == segs - 1) {  // the token shift's state
+        float* keep = a.shift + (int64_t)((p0 + a.q_rows - 1) & 1) * a.shift_slot + (int64_t)b * a.width;
+        for (int c = tid; c < a.width; c += 128) keep[c] = a.hn[(row0 + count - 1) * a.width + c];
+    }
 }
 
 // The states over the segments: a segment's place gets its incoming state, the sequence the last one.
@@ -418,7 +610,7 @@ __global__ void __launch_bounds__(256) wkv_join_kernel(const WkvArgs a, int segs
 
 // o_t += (r_t times the decays since the segment's start)^T S for the segments behind the first: a CTA per head and 64 tokens,
 // on the tensor cores, both factors as bf16 hi + lo (16 significand bits).  Head size 64.
-constexpr int kCarryDim = 64, kCarryLd = 72;  // bf16 elements per shared-memory row
+constexpr int kCarryDim = 64, kCarryLd = 72;
 __global__ void __launch_bounds__(256) wkv_carry_kernel(const WkvArgs a, int seg_tokens) {
     __shared__ __align__(16) __nv_bfloat16 rh[64][kCarryLd], rl[64][kCarryLd], sh[64][kCarryLd], sl[64][kCarryLd];
     __shared__ float part[4][64];
@@ -434,8 +626,7 @@ __global__ void __launch_bounds__(256) wkv_carry_kernel(const WkvArgs a, int seg
     const int ch = threadIdx.x & 63, quarter = threadIdx.x >> 6;  // a channel, 16 of the 64 tokens
     float r[16], w[16], p = 1.0f, run;                              // run: the decays before the token
     {
-        const float* up = a.seg_w + (((int64_t)b * ((a.q_rows + kBlock - 1) / kBlock) + (first + t0) / kBlock) * 2 * a.heads + head) * D + ch;
-        run = up[0] * up[(int64_t)a.heads * D];
+        run = a.seg_w[(((int64_t)b * ((a.q_rows + kBlock - 1) / kBlock) + (first + t0) / kBlock) * a.heads + head) * D + ch];
     }
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
@@ -511,9 +702,9 @@ __global__ void __launch_bounds__(256) wkv_carry_kernel(const WkvArgs a, int seg
 }
 
 // segments of the tokens: the fewest rounds of CTAs (three share an SM) times tokens, no segment below 128 tokens
-int scan_segments(const WkvArgs& a) {
+int segments(const WkvArgs& a) {
     if (!a.seg_s || !a.seg_w || a.dim != kCarryDim) return 1;
-    const int64_t ctas = (int64_t)a.heads * ((a.dim + kScanCols - 1) / kScanCols) * a.batch, slots = 3ll * a.sm_count;
+    const int64_t ctas = (int64_t)a.heads * a.batch, slots = 3ll * a.sm_count;
     int best = 1;
     int64_t least = 0;
     for (int segs = 1; segs <= kSegments && (segs == 1 || a.q_rows / segs >= 128); ++segs) {
@@ -527,10 +718,18 @@ cudaError_t scan_launch(const WkvArgs& a, cudaStream_t s) {
     static PerDeviceOnce once;
     cudaError_t e = once.run([] { return cudaFuncSetAttribute(wkv_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ScanCfg<NJ>::kSmem); });
     if (e != cudaSuccess) return e;
-    int segs = scan_segments(a);
+    wkv_scan_kernel<NJ><<<dim3((unsigned)a.heads, (unsigned)((a.dim + kScanCols - 1) / kScanCols), (unsigned)a.batch), kScanThreads, ScanCfg<NJ>::kSmem, s>>>(a);
+    return cudaGetLastError();
+}
+bool takes_blocks(const WkvArgs& a) { return a.split16 && a.dim <= kHead && a.dim % 4 == 0 && a.ld % 4 == 0 && a.q_rows >= kTok; }
+cudaError_t block_launch(const WkvArgs& a, cudaStream_t s) {
+    static PerDeviceOnce once;
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(wkv_block_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(BlockSmem)); });
+    if (e != cudaSuccess) return e;
+    int segs = segments(a);
     const int tokens = ((a.q_rows + segs - 1) / segs + kBlock - 1) / kBlock * kBlock;
     segs = (a.q_rows + tokens - 1) / tokens;
-    wkv_scan_kernel<NJ><<<dim3((unsigned)a.heads, (unsigned)((a.dim + kScanCols - 1) / kScanCols), (unsigned)(a.batch * segs)), kScanThreads, ScanCfg<NJ>::kSmem, s>>>(a, segs, tokens);
+    wkv_block_kernel<<<dim3((unsigned)a.heads, (unsigned)segs, (unsigned)a.batch), 128, sizeof(BlockSmem), s>>>(a, segs, tokens);
     if (segs > 1) {
         wkv_join_kernel<<<dim3((unsigned)((a.dim * a.dim + 255) / 256), (unsigned)(a.heads * a.batch)), 256, 0, s>>>(a, segs);
         wkv_carry_kernel<<<dim3((unsigned)a.heads, (unsigned)((segs - 1) * (tokens / kBlock)), (unsigned)a.batch), 256, 0, s>>>(a, tokens);
@@ -549,7 +748,7 @@ cudaError_t step_launch(const WkvArgs& a, cudaStream_t s, bool pdl) {
 
 int wkv_max_dim() { return 256; }
 int64_t wkv_segment_floats(int heads, int dim) { return dim == kCarryDim ? (int64_t)heads * kSegments * (dim * dim + dim) : 0; }
-int64_t wkv_prefix_floats(int heads, int dim, int64_t rows, int batch) { return dim == kCarryDim ? (rows / kBlock + batch) * 2 * heads * dim : 0; }
+int64_t wkv_prefix_floats(int heads, int dim, int64_t rows, int batch) { return dim == kCarryDim ? (rows / kBlock + batch) * heads * dim : 0; }
 
 cudaError_t launch_wkv_mix(const WkvMix& a, cudaStream_t s) {
     const unsigned rows = (unsigned)(a.batch * a.q_rows);
@@ -568,6 +767,7 @@ cudaError_t launch_wkv_step(const WkvArgs& a, cudaStream_t s, bool pdl) {
 cudaError_t launch_wkv_prefill(const WkvArgs& a, cudaStream_t s) {
     if (a.dim > wkv_max_dim() || !a.w) return cudaErrorInvalidValue;
     if (a.q_rows == 1) return step_launch(a, s, false);
+    if (takes_blocks(a)) return block_launch(a, s);
     if (a.dim <= 32) return scan_launch<1>(a, s);
     if (a.dim <= 64) return scan_launch<2>(a, s);
     if (a.dim <= 128) return scan_launch<4>(a, s);
