@@ -284,6 +284,39 @@ def test_long_decoding(bt):
         assert np.sqrt((row_errors(again, got) ** 2).mean()) <= TOL[dtype][1] * (1 if dtype == "float32" else 1.5)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_prompt_longer_than_one_pass(bt, dtype):
+    """The host cuts a long prompt: positions on both sides of the cut, portions that cross it, decoding behind it."""
+    cfg = config(48, 64, [wkv(1, 64, 8, **moe(24, 4, 4, 16)), latent(2, 32, 16, 24, 40), rglru(48, 2, 4)], loop=(1, 2, 2))
+    t = make_tensors(cfg, seed=12)
+    tokens = np.random.default_rng(12).integers(0, 48, 2301).astype(np.int32)
+    logits, _ = oracle(cfg, t, tokens)
+    at = np.array([0, 1, 1023, 2046, 2047, 2048, 2049, 2050, 2111, 2112, 2298, 2299])
+    m = lay.build_layered(cfg, t, dtype=dtype, max_seq_len=2304)
+    assert_close(m.prefill_logits(tokens[:2300], at), logits[at], dtype)
+    assert_close(m.forward_one(tokens[2300:])[0], logits[2300:], dtype)
+    m.reset_kv_cache()
+    m.prefill(tokens[:1900], want_logits=False)
+    assert_close(m.prefill_logits(tokens[1900:], np.arange(401)), logits[1900:], dtype)
+
+
+@pytest.mark.parametrize("dim", [16, 64])
+def test_decays_from_none_to_all(bt, dim):
+    """Channels that keep everything beside channels that forget everything: nothing overflows, nothing is lost."""
+    cfg = config(50, 64, [wkv(2, dim, 4)], cap=0.0)
+    t = make_tensors(cfg, seed=13)
+    t["l0.mix.w0"] = bf16(np.where(np.arange(2 * dim) % 2 == 0, -14.0, np.linspace(0.0, 6.0, 2 * dim)).astype(np.float32))
+    tokens = np.random.default_rng(13).integers(0, 50, 300).astype(np.int32)
+    _, stream = ref.forward({**lay.fepapel_dict(cfg), "logit_softcap": 1e9}, t, tokens)
+    for dtype in ("float32", "bfloat16"):
+        m = lay.build_layered(cfg, t, dtype=dtype, max_seq_len=300)
+        m.set_trace(True, rows=300)
+        m.prefill(tokens)
+        e = row_errors(m.read_trace(300)[0], stream[0])
+        m.set_trace(False)
+        assert e.max() <= (5e-5 if dtype == "float32" else 0.15), (dtype, e.max())
+
+
 def test_greedy_generation(bt):
     cfg, t, tokens, _, _ = case("wide")
     m = lay.build_layered(cfg, t, max_batch=2, dtype="float32", max_seq_len=64)
