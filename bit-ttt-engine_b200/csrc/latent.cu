@@ -573,9 +573,10 @@ cudaError_t launch_cluster(void (*kernel)(KArgs...), dim3 grid, int threads, siz
     cfg.numAttrs = pdl ? 2 : 1;
     return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
 }
-int span_splits(const LatentAttn& a, int64_t groups) {
+// active: for 1, 2, 4, ... CTAs the clusters that can be resident at once (a cluster sits in one GPC); null: as many as there are SMs
+int span_splits(const LatentAttn& a, int64_t groups, const int* active = nullptr) {
     int splits = 1;
-    while (splits < kMaxSplits && groups * splits * 2 <= a.sm_count && splits * kKeys < a.kv.max_seq) splits *= 2;
+    for (int i = 1; splits < kMaxSplits && groups * splits * 2 <= a.sm_count && splits * kKeys < a.kv.max_seq && (!active || groups <= active[i]); ++i) splits *= 2;
     return splits;
 }
 
@@ -583,9 +584,19 @@ constexpr size_t kSpanSmem = 224 * 1024;
 template <int HG>
 cudaError_t span_launch(const LatentAttn& a, bool prepared, const ActOut& out, unsigned int* err, cudaStream_t s, bool pdl) {
     static PerDeviceOnce once;
+    static int active[5];  // every device of a process is the same GPU model
     cudaError_t e = once.run([] {
         cudaError_t x = cudaFuncSetAttribute(latent_span_tc_kernel<HG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSpanSmem);
-        return x != cudaSuccess ? x : cudaFuncSetAttribute(latent_span_tc_kernel<HG>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        if (x == cudaSuccess) x = cudaFuncSetAttribute(latent_span_tc_kernel<HG>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        for (int i = 0; i < 5 && x == cudaSuccess; ++i) {
+            cudaLaunchConfig_t cfg = {};
+            cudaLaunchAttribute attr;
+            attr.id = cudaLaunchAttributeClusterDimension;
+            attr.val.clusterDim.x = 1u << i; attr.val.clusterDim.y = 1; attr.val.clusterDim.z = 1;
+            cfg.gridDim = dim3(1u << i); cfg.blockDim = dim3(kSpanThreads); cfg.dynamicSmemBytes = kSpanSmem; cfg.attrs = &attr; cfg.numAttrs = 1;
+            x = cudaOccupancyMaxActiveClusters(&active[i], latent_span_tc_kernel<HG>, &cfg);
+        }
+        return x;
     });
     if (e != cudaSuccess) return e;
     const int cols = a.kv.cols(), hg = (a.heads + HG - 1) / HG;
@@ -595,8 +606,10 @@ cudaError_t span_launch(const LatentAttn& a, bool prepared, const ActOut& out, u
     stages = stages > kMaxStages ? kMaxStages : stages;
     if (stages < 1 || stages * stage < outs) return cudaErrorInvalidConfiguration;
     const int64_t rows = (int64_t)a.batch * a.q_rows;
-    const int splits = span_splits(a, rows * hg);
-    return launch_cluster(latent_span_tc_kernel<HG>, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, stages * stage + fixed, s, pdl,
+    const int splits = span_splits(a, rows * hg, active);
+    // one CTA per SM, whatever its registers: none waits for tensor memory while its cluster holds some elsewhere
+    const size_t smem = stages * stage + fixed, least = (size_t)116 * 1024;
+    return launch_cluster(latent_span_tc_kernel<HG>, dim3((unsigned)splits, (unsigned)hg, (unsigned)rows), kSpanThreads, smem > least ? smem : least, s, pdl,
                           a, prepared, splits, stages, err, out);
 }
 
